@@ -14,7 +14,7 @@ import torch
 from ..cache.paged import PAGE  # cache positions per page; the library's MLL_PAGE is checked against it on load
 from .build import KernelBuildError, load_library
 
-ABI_VERSION = 33
+ABI_VERSION = 34
 MAX_TOP_K = 1024
 
 
@@ -596,6 +596,47 @@ def add_layernorm(x: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.
     _check(lib().mll_add_layernorm(_ptr(x), _ptr(delta), _ptr(weight), _ptr(bias), _ptr(out), _ptr(rows),
                                    dtype_code(delta_dtype), dtype_code(out.dtype), ctypes.c_int(n_rows),
                                    ctypes.c_int(width), ctypes.c_float(eps), _stream()), "layernorm")
+
+
+class TanhNorm(NamedTuple):
+    """out = tanh(alpha * x) * weight + bias: alpha float32 [1], weight and bias float32 [D], out [rows, D]."""
+    alpha: torch.Tensor
+    weight: torch.Tensor
+    bias: torch.Tensor
+    out: torch.Tensor
+
+
+def add_dynamic_tanh(x: torch.Tensor, deltas, norms, rows: Optional[torch.Tensor] = None) -> None:
+    """x += sum of scale * delta over `deltas` (up to three (tensor, scale); float32 residual, in place), then every
+    `TanhNorm` of `norms` (up to two) of the sum.  `rows` (int32 [n]): only those rows, x unchanged."""
+    _need(x, "tanh norm x", torch.float32, 2)
+    width = x.shape[1]
+    n_rows = x.shape[0] if rows is None else rows.shape[0]
+    if rows is not None:
+        _need(rows, "tanh norm rows", torch.int32, 1)
+    if len(deltas) > 3 or len(norms) > 2:
+        raise KernelError(f"tanh norm: {len(deltas)} deltas and {len(norms)} norms")
+    for d, _ in deltas:
+        _need(d, "tanh norm delta", deltas[0][0].dtype, 2)
+        if d.shape != x.shape:
+            raise KernelError(f"tanh norm: delta {tuple(d.shape)} differs from x {tuple(x.shape)}")
+    for n in norms:
+        _need(n.alpha, "tanh norm alpha", torch.float32, 1)
+        _need(n.weight, "tanh norm weight", torch.float32, 1)
+        _need(n.bias, "tanh norm bias", torch.float32, 1)
+        _need(n.out, "tanh norm out", norms[0].out.dtype, 2)
+        if n.weight.shape[0] != width or n.bias.shape[0] != width or tuple(n.out.shape) != (n_rows, width) or n.alpha.shape[0] != 1:
+            raise KernelError(f"tanh norm: weight {tuple(n.weight.shape)}, bias {tuple(n.bias.shape)}, out {tuple(n.out.shape)} "
+                              f"for {n_rows} rows of {width}")
+    if not deltas and not norms:
+        return
+    out_dtype = norms[0].out.dtype if norms else deltas[0][0].dtype
+    delta_dtype = deltas[0][0].dtype if deltas else out_dtype
+    d = [(_ptr(t), ctypes.c_float(f)) for t, f in deltas] + [(_ptr(None), ctypes.c_float(0.0))] * (3 - len(deltas))
+    n = [(_ptr(v.alpha), _ptr(v.weight), _ptr(v.bias), _ptr(v.out)) for v in norms] + [(_ptr(None),) * 4] * (2 - len(norms))
+    _check(lib().mll_add_tanh_norm(_ptr(x), *(p for p, _ in d), *(f for _, f in d), *n[0], *n[1], _ptr(rows),
+                                   dtype_code(delta_dtype), dtype_code(out_dtype), ctypes.c_int(n_rows),
+                                   ctypes.c_int(width), _stream()), "tanh_norm")
 
 
 def stream_concat(x: torch.Tensor, delta: Optional[torch.Tensor], x0: torch.Tensor, out: torch.Tensor) -> None:
@@ -1408,16 +1449,140 @@ def head_norm_gate(o, weight, gate, out, n_heads: int, dv: int, eps: float, act:
 
 
 # --------------------------------------------------------------------------- #
+# gated linear recurrent unit
+# --------------------------------------------------------------------------- #
+USE_TENSOR_CORE_LRU = True  # tests switch it off to reach the float32 gate products in bfloat16 runs
+
+
+def lru_mma_supported(dtype: torch.dtype, block: int) -> bool:
+    """Whether the gates' block-diagonal products run on tensor cores (bfloat16 matrices, see `lru_gates`)."""
+    return USE_TENSOR_CORE_LRU and dtype == torch.bfloat16 and bool(lib().mll_lru_mma_supported(dtype_code(dtype), block))
+
+
+def lru_gates(proj, x_col: int, y_col: int, x_bias, y_bias, conv_w, conv_b, conv_state, gate_w, gate_b, lam, state,
+              tok_pos, tok_seq, seq_slot, seq_qstart, blocks: int, rate: float, decay=None, write=None, out=None) -> None:
+    """The inputs of a gated linear recurrent unit from a step's projection rows (csrc/rglru.cu): u = short causal
+    convolution of proj's columns x_col .. + width (+ x_bias) over conv_w float32 [width, taps] (+ conv_b), earlier
+    inputs from conv_state [slots, taps - 1, width]; r, i = sigmoid of block-diagonal products of u (gate_w: bfloat16
+    [n, 2, bs, bs] with rows as outputs, or float32 [n, bs, 2 bs] with columns as outputs; gate_b float32 [2, width]);
+    decay = exp(-rate r softplus(lam)) and write = sqrt(1 - decay^2) i u to float32 [T, width].  With `out` instead of
+    `decay` and `write` every sequence brings one token: `state` float32 [slots, width] advances and out [T, width] =
+    state * gelu(proj's columns y_col .. + y_bias)."""
+    _need(proj, "lru proj", None, 2)
+    n, ld = proj.shape
+    width, taps = conv_w.shape
+    single = out is not None
+    for name, t, shape in (("x bias", x_bias, (width,)), ("y bias", y_bias, (width,)), ("conv weights", conv_w, (width, taps)),
+                           ("conv bias", conv_b, (width,)), ("gate bias", gate_b, (2, width)), ("lam", lam, (width,))):
+        _need(t, f"lru {name}", torch.float32)
+        if tuple(t.shape) != shape:
+            raise KernelError(f"lru: {name} {tuple(t.shape)}, expected {shape}")
+    if blocks < 1 or width % blocks:
+        raise KernelError(f"lru: {width} channels in {blocks} blocks")
+    bs = width // blocks
+    mma = gate_w.dtype == torch.bfloat16
+    _need(gate_w, "lru gate matrices", torch.bfloat16 if mma else torch.float32)
+    if tuple(gate_w.shape) != ((blocks, 2, bs, bs) if mma else (blocks, bs, 2 * bs)):
+        raise KernelError(f"lru: gate matrices {tuple(gate_w.shape)} for {blocks} blocks of {bs}")
+    _need(conv_state, "lru conv state", torch.float32, 3)
+    _need(state, "lru state", torch.float32, 2)
+    if tuple(conv_state.shape[1:]) != (taps - 1, width) or state.shape[1] != width:
+        raise KernelError(f"lru: conv state {tuple(conv_state.shape)} / state {tuple(state.shape)} for {width} channels of {taps} taps")
+    for name, t, dtype in ((("out", out, proj.dtype),) if single else (("decay", decay, torch.float32), ("write", write, torch.float32))):
+        _need(t, f"lru {name}", dtype, 2)
+        if tuple(t.shape) != (n, width):
+            raise KernelError(f"lru: {name} {tuple(t.shape)}, expected {(n, width)}")
+    for name, t in (("tok_pos", tok_pos), ("tok_seq", tok_seq), ("seq_slot", seq_slot), ("seq_qstart", seq_qstart)):
+        _need(t, f"lru {name}", torch.int32, 1)
+    _check(lib().mll_lru_gates(
+        _ptr(proj), _ptr(x_bias), _ptr(y_bias), _ptr(conv_w), _ptr(conv_b), _ptr(conv_state), _ptr(gate_w), _ptr(gate_b),
+        _ptr(lam), _ptr(state), _ptr(decay), _ptr(write), _ptr(out), _ptr(tok_pos), _ptr(tok_seq), _ptr(seq_slot),
+        _ptr(seq_qstart), dtype_code(proj.dtype), ctypes.c_int(n), ctypes.c_int(ld), ctypes.c_int(x_col),
+        ctypes.c_int(y_col), ctypes.c_int(width), ctypes.c_int(blocks), ctypes.c_int(taps), ctypes.c_float(rate),
+        ctypes.c_int(int(mma)), ctypes.c_int(int(single)), _stream()), "lru_gates (single tokens)" if single else "lru_gates")
+
+
+def lru_scan(decay, write, proj, y_col: int, y_bias, state, out, seq_slot, seq_qstart, seq_qlen, n_seqs: int,
+             longest: int) -> None:
+    """state <- decay * state + write over each sequence's tokens of the step (float32 [slots, width], one number per
+    channel); out [T, width] = state * gelu_tanh(proj's columns y_col .. + y_bias).  `longest`: the most tokens a
+    sequence brings."""
+    _need(decay, "lru scan decay", torch.float32, 2)
+    n, width = decay.shape
+    _need(write, "lru scan write", torch.float32, 2)
+    _need(proj, "lru scan proj", None, 2)
+    _need(out, "lru scan out", proj.dtype, 2)
+    _need(state, "lru scan state", torch.float32, 2)
+    _need(y_bias, "lru scan bias", torch.float32, 1)
+    if (write.shape != decay.shape or out.shape != decay.shape or proj.shape[0] != n or state.shape[1] != width
+            or y_bias.shape[0] != width):
+        raise KernelError(f"lru scan: decay {tuple(decay.shape)}, out {tuple(out.shape)}, state {tuple(state.shape)}")
+    _check(lib().mll_lru_scan(_ptr(decay), _ptr(write), _ptr(proj), _ptr(y_bias), _ptr(state), _ptr(out), _ptr(seq_slot),
+                              _ptr(seq_qstart), _ptr(seq_qlen), dtype_code(proj.dtype), ctypes.c_int(n_seqs),
+                              ctypes.c_int(proj.shape[1]), ctypes.c_int(y_col), ctypes.c_int(width), ctypes.c_int(longest),
+                              _stream()), "lru_scan")
+
+
+# --------------------------------------------------------------------------- #
+# attention with mixed scores and sigmoid weights
+# --------------------------------------------------------------------------- #
+def _check_mixed(q, k_cache, v_cache, out, mix, bias, n_heads: int, n_kv_heads: int, d: int, dv: int) -> int:
+    _need(q, "mixed attention q", None, 2)
+    _need(out, "mixed attention out", q.dtype, 2)
+    _need(k_cache, "mixed attention k cache", q.dtype, 4)
+    _need(v_cache, "mixed attention v cache", q.dtype, 4)
+    n = q.shape[0]
+    if tuple(q.shape) != (n, n_heads * d) or tuple(out.shape) != (n, n_heads * dv):
+        raise KernelError(f"mixed attention: q {tuple(q.shape)} / out {tuple(out.shape)} for {n_heads} heads of {d} / {dv}")
+    _check_local_caches(k_cache, v_cache, n_kv_heads, d, dv, False)
+    if mix is not None:
+        _need(mix, "mixed attention mixing matrix", torch.float32, 2)
+        if tuple(mix.shape) != (n_heads, n_heads):
+            raise KernelError(f"mixed attention: mixing matrix {tuple(mix.shape)} for {n_heads} heads")
+    if bias is not None:
+        _need(bias, "mixed attention bias", torch.float32, 1)
+        if bias.shape[0] != n_heads:
+            raise KernelError(f"mixed attention: {bias.shape[0]} biases for {n_heads} heads")
+    return n
+
+
+def mixed_attention(q, k_cache, v_cache, tok_pos, tok_seq, seq_slot, block_table, mix, bias, out, n_heads: int,
+                    n_kv_heads: int, d: int, dv: int, window: int, scale: float) -> None:
+    """out [T, H * dv]: head h sums sigmoid(sum_g mix[h, g] scale q_g . k_j + bias_h) v_j over the keys j <= i of the
+    window (j > i - window; 0: all), not normalised.  mix float32 [H, H] or None (no mixing), bias float32 [H] or None;
+    the step's own keys are in the cache already.  Any dtype and size."""
+    n = _check_mixed(q, k_cache, v_cache, out, mix, bias, n_heads, n_kv_heads, d, dv)
+    for name, t in (("tok_pos", tok_pos), ("tok_seq", tok_seq), ("seq_slot", seq_slot)):
+        _need(t, f"mixed attention {name}", torch.int32, 1)
+    _need(block_table, "mixed attention block table", torch.int32, 2)
+    _check(lib().mll_mixed_attention(
+        _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(tok_pos), _ptr(tok_seq), _ptr(seq_slot), _ptr(block_table), _ptr(mix),
+        _ptr(bias), _ptr(out), dtype_code(q.dtype), ctypes.c_int(n), ctypes.c_int(n_heads), ctypes.c_int(n_kv_heads),
+        ctypes.c_int(d), ctypes.c_int(dv), ctypes.c_int(window), ctypes.c_int(block_table.shape[1]), ctypes.c_float(scale),
+        _stream()), "mixed_attention")
+
+
+# --------------------------------------------------------------------------- #
 # attention over a shared low-rank latent
 # --------------------------------------------------------------------------- #
 def latent_prepare(proj, c_weight, cos, sin, tok_pos, tok_seq, seq_slot, block_table, q_out, kv_cache, n_heads: int,
-                   d: int, rot: int, rank: int, interleaved: bool, eps: float) -> None:
+                   d: int, rot: int, rank: int, interleaved: bool, eps: float, cq_weight: Optional[torch.Tensor] = None,
+                   cq_out: Optional[torch.Tensor] = None) -> None:
     """proj [T, ld]: H heads of (d plain + rot rotated) query columns, then the down projection's rank + rot columns.
     Writes the cache row [c | k_r] of every token (c = the first rank columns divided by their root mean square and
     multiplied by `c_weight`, k_r = the last rot columns rotated by position) into its page of `kv_cache`
     [pages, 1, PAGE, rank + rot], and the rotated part of every head's query into the last rot columns of that head
-    in `q_out` [T, H * (rank + rot)]."""
+    in `q_out` [T, H * (rank + rot)].  `cq_weight` (float32 [q_rank]) and `cq_out` [T, q_rank]: the row starts with the
+    queries' own latent of q_rank columns instead of the heads' queries (rot is 0 then); it is normalised like the keys'
+    latent and goes to `cq_out`."""
     _need(proj, "latent prepare proj", None, 2)
+    q_rank = 0
+    if cq_weight is not None:
+        _need(cq_weight, "latent prepare query norm weight", torch.float32, 1)
+        _need(cq_out, "latent prepare query latent", proj.dtype, 2)
+        q_rank = cq_weight.shape[0]
+        if tuple(cq_out.shape) != (proj.shape[0], q_rank):
+            raise KernelError(f"latent prepare: query latent {tuple(cq_out.shape)}, expected {(proj.shape[0], q_rank)}")
     _need(q_out, "latent prepare q", proj.dtype, 2)
     _need(kv_cache, "latent prepare cache", proj.dtype, 4)
     _need(c_weight, "latent prepare norm weight", torch.float32, 1)
@@ -1438,8 +1603,8 @@ def latent_prepare(proj, c_weight, cos, sin, tok_pos, tok_seq, seq_slot, block_t
         _ptr(proj), _ptr(c_weight), _ptr(cos if rot else None), _ptr(sin if rot else None), _ptr(tok_pos), _ptr(tok_seq),
         _ptr(seq_slot), _ptr(block_table), _ptr(q_out), _ptr(kv_cache), dtype_code(proj.dtype), ctypes.c_int(n),
         ctypes.c_int(proj.shape[1]), ctypes.c_int(n_heads), ctypes.c_int(d), ctypes.c_int(rot), ctypes.c_int(rank),
-        ctypes.c_int(int(interleaved)), ctypes.c_int(block_table.shape[1]), ctypes.c_float(eps), _stream()),
-        "latent_prepare")
+        ctypes.c_int(q_rank), _ptr(cq_weight), _ptr(cq_out), ctypes.c_int(int(interleaved)),
+        ctypes.c_int(block_table.shape[1]), ctypes.c_float(eps), _stream()), "latent_prepare")
 
 
 # --------------------------------------------------------------------------- #

@@ -11,13 +11,19 @@
 //   k_r = the last `rot` columns of it, pairs (2i, 2i + 1) (or (i, i + rot/2)) rotated by position * f_i
 //   the cache row [c | k_r] is written into the token's page;
 //   q_r of every head rotated the same way and written behind the head's q~ columns of the query buffer.
+// Where the queries come from a latent of their own (`q_rank`), the row starts with that latent instead of the heads'
+// queries; it is normalised the same way, c_q = c_q' / sqrt(mean(c_q'^2) + eps) * w_q, and written out for the product
+// that makes the heads' queries of it.
 #include "common.cuh"
 
 namespace mll {
 
 struct LatentPrepArgs {
-  const void* proj;        // [T, ld]: H heads of (d plain + rot rotated) query columns, then rank + rot down-projection columns
+  const void* proj;        // [T, ld]: H heads of (d plain + rot rotated) query columns (or the q_rank columns of the
+                           // queries' latent), then rank + rot down-projection columns
   const float* c_weight;   // [rank]
+  const float* cq_weight;  // [q_rank]
+  void* cq_out;            // [T, q_rank]
   const float* cos_table;  // [max_pos, rot / 2]
   const float* sin_table;
   const int* tok_pos;
@@ -26,7 +32,7 @@ struct LatentPrepArgs {
   const int* block_table;
   void* q_out;             // [T, H, rank + rot]: only the last rot columns of every head are written here
   void* kv_cache;          // [pages, 1, PAGE, rank + rot]
-  int ld, n_heads, d, rot, rank, interleaved, max_blocks;
+  int ld, n_heads, d, rot, rank, q_rank, interleaved, max_blocks;  // q_rank 0: the row holds the queries themselves
   float eps;
 };
 
@@ -48,7 +54,7 @@ template <typename T>
 __global__ void __launch_bounds__(256) latent_prepare_kernel(LatentPrepArgs a) {
   __shared__ float scratch[32];
   const int t = blockIdx.x;
-  const int nq = a.n_heads * (a.d + a.rot), row_w = a.rank + a.rot;
+  const int nq = a.q_rank > 0 ? a.q_rank : a.n_heads * (a.d + a.rot), row_w = a.rank + a.rot;
   const T* row = (const T*)a.proj + (size_t)t * a.ld;
   const T* down = row + nq;
   float ss = 0.f;
@@ -58,6 +64,17 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(LatentPrepArgs a) {
   }
   ss = block_sum(ss, scratch);
   const float f = 1.f / sqrtf(ss / (float)a.rank + a.eps);
+  if (a.q_rank > 0) {
+    float sq = 0.f;
+    for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) {
+      const float v = to_float(row[i]);
+      sq += v * v;
+    }
+    sq = block_sum(sq, scratch);
+    const float fq = 1.f / sqrtf(sq / (float)a.q_rank + a.eps);
+    T* cq = (T*)a.cq_out + (size_t)t * a.q_rank;
+    for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) cq[i] = from_float<T>(to_float(row[i]) * fq * a.cq_weight[i]);
+  }
   const int pos = a.tok_pos[t];
   const int slot = a.seq_slot[a.tok_seq[t]];
   const int page = a.block_table[(size_t)slot * a.max_blocks + pos / MLL_PAGE];
@@ -80,14 +97,17 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(LatentPrepArgs a) {
 MLL_API int mll_latent_prepare(const void* proj, const float* c_weight, const float* cos_table, const float* sin_table,
                                const int* tok_pos, const int* tok_seq, const int* seq_slot, const int* block_table,
                                void* q_out, void* kv_cache, int dtype, int n_tokens, int ld, int n_heads, int d, int rot,
-                               int rank, int interleaved, int max_blocks, float eps, cudaStream_t stream) {
+                               int rank, int q_rank, const float* cq_weight, void* cq_out, int interleaved, int max_blocks,
+                               float eps, cudaStream_t stream) {
   MLL_REQUIRE(n_tokens >= 0 && n_heads > 0 && d > 0 && rank > 0, "latent prepare: bad sizes");
   MLL_REQUIRE(rot >= 0 && rot % 2 == 0, "latent prepare: %d rotated dimensions", rot);
-  MLL_REQUIRE(ld >= n_heads * (d + rot) + rank + rot, "latent prepare: row stride %d too short", ld);
+  MLL_REQUIRE(q_rank >= 0 && (q_rank == 0 || (rot == 0 && cq_weight && cq_out)),
+              "latent prepare: queries from a latent go without rotated dimensions and need a weight and an output");
+  MLL_REQUIRE(ld >= (q_rank > 0 ? q_rank : n_heads * (d + rot)) + rank + rot, "latent prepare: row stride %d too short", ld);
   MLL_REQUIRE(rot == 0 || (cos_table && sin_table), "latent prepare: rotated dimensions without tables");
   if (n_tokens == 0) return 0;
-  mll::LatentPrepArgs a{proj, c_weight, cos_table, sin_table, tok_pos, tok_seq, seq_slot, block_table, q_out, kv_cache,
-                        ld, n_heads, d, rot, rank, interleaved, max_blocks, eps};
+  mll::LatentPrepArgs a{proj, c_weight, cq_weight, cq_out, cos_table, sin_table, tok_pos, tok_seq, seq_slot, block_table,
+                        q_out, kv_cache, ld, n_heads, d, rot, rank, q_rank, interleaved, max_blocks, eps};
   if (dtype == MLL_F32)
     MLL_LAUNCH((mll::latent_prepare_kernel<float>), n_tokens, 256, 0, stream, a);
   else if (dtype == MLL_BF16)

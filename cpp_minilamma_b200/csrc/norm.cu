@@ -336,6 +336,91 @@ int launch_add_layernorm(float* x, const void* delta, const float* weight, const
   return 0;
 }
 
+// A norm without statistics, fused with the residual add:
+//   x[t, :] += scale_0 delta_0[t, :] (+ scale_1 delta_1 + scale_2 delta_2)
+//   out_n[t, i] = tanh(alpha_n * x[t, i]) * w_n[i] + b_n[i]        for none, one or two norms n of the same stream
+// Every column by itself, so a thread owns four neighbouring columns (or one, where the width is no multiple of four)
+// and nothing is exchanged.  `rows` gathers as above (the stream is then left alone).  Float32 throughout.
+struct TanhNormArgs {
+  float* x;
+  const void* delta[3];
+  float scale[3];
+  const float* alpha[2];   // one number on the device each
+  const float* weight[2];
+  const float* bias[2];
+  void* out[2];
+  const int* rows;
+  int n_rows, width, n_deltas, n_norms;
+};
+
+template <typename DeltaT, typename OutT>
+__global__ void __launch_bounds__(256) add_tanh_norm_vec_kernel(TanhNormArgs a) {
+  const int groups = a.width >> 2;
+  const long long at = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (at >= (long long)a.n_rows * groups) return;
+  const int r = (int)(at / groups), g = (int)(at % groups);
+  const size_t src = (size_t)(a.rows ? a.rows[r] : r) * a.width + 4 * g;
+  float4 v = load4<float>(a.x + src);
+  if (a.n_deltas > 0) {
+    float4 d[3];
+#pragma unroll
+    for (int i = 0; i < 3; ++i)
+      if (i < a.n_deltas) d[i] = load4<DeltaT>((const DeltaT*)a.delta[i] + src);
+    float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < 3; ++i)
+      if (i < a.n_deltas) {
+        sum.x = fmaf(a.scale[i], d[i].x, sum.x); sum.y = fmaf(a.scale[i], d[i].y, sum.y);
+        sum.z = fmaf(a.scale[i], d[i].z, sum.z); sum.w = fmaf(a.scale[i], d[i].w, sum.w);
+      }
+    v.x += sum.x; v.y += sum.y; v.z += sum.z; v.w += sum.w;
+    if (!a.rows) store4(a.x + src, v);
+  }
+#pragma unroll
+  for (int n = 0; n < 2; ++n)
+    if (n < a.n_norms) {
+      const float al = *a.alpha[n];
+      const float4 w = load4<float>(a.weight[n] + 4 * g), b = load4<float>(a.bias[n] + 4 * g);
+      store4((OutT*)a.out[n] + (size_t)r * a.width + 4 * g,
+             make_float4(fmaf(tanhf(al * v.x), w.x, b.x), fmaf(tanhf(al * v.y), w.y, b.y), fmaf(tanhf(al * v.z), w.z, b.z),
+                         fmaf(tanhf(al * v.w), w.w, b.w)));
+    }
+}
+
+template <typename DeltaT, typename OutT>
+__global__ void __launch_bounds__(256) add_tanh_norm_kernel(TanhNormArgs a) {
+  const long long at = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (at >= (long long)a.n_rows * a.width) return;
+  const int r = (int)(at / a.width), c = (int)(at % a.width);
+  const size_t src = (size_t)(a.rows ? a.rows[r] : r) * a.width + c;
+  float v = a.x[src];
+  if (a.n_deltas > 0) {
+    float sum = 0.f;
+    for (int i = 0; i < a.n_deltas; ++i) sum = fmaf(a.scale[i], to_float(((const DeltaT*)a.delta[i])[src]), sum);
+    v += sum;
+    if (!a.rows) a.x[src] = v;
+  }
+  for (int n = 0; n < a.n_norms; ++n)
+    ((OutT*)a.out[n])[(size_t)r * a.width + c] = from_float<OutT>(fmaf(tanhf(*a.alpha[n] * v), a.weight[n][c], a.bias[n][c]));
+}
+
+template <typename DeltaT, typename OutT>
+int launch_add_tanh_norm(const TanhNormArgs& a, cudaStream_t stream) {
+  bool vec = a.width % 4 == 0 && (uintptr_t)a.x % 16 == 0;
+  for (int i = 0; i < a.n_deltas; ++i) vec = vec && (uintptr_t)a.delta[i] % 16 == 0;
+  for (int n = 0; n < a.n_norms; ++n)
+    vec = vec && (uintptr_t)a.weight[n] % 16 == 0 && (uintptr_t)a.bias[n] % 16 == 0 && (uintptr_t)a.out[n] % 16 == 0;
+  const long long items = (long long)a.n_rows * (vec ? a.width / 4 : a.width);
+  MLL_REQUIRE((items + 255) / 256 <= 0x7fffffffLL, "tanh norm: too many elements");
+  const unsigned blocks = (unsigned)((items + 255) / 256);
+  if (vec)
+    MLL_LAUNCH((add_tanh_norm_vec_kernel<DeltaT, OutT>), blocks, 256, 0, stream, a);
+  else
+    MLL_LAUNCH((add_tanh_norm_kernel<DeltaT, OutT>), blocks, 256, 0, stream, a);
+  MLL_LAUNCH_CHECK();
+  return 0;
+}
+
 // Finishes a norm whose rows were left without their factor (RowNormIn), for a product that cannot do
 // it itself: out[m, i] = values[m, i] * factor(m).  One block per row.
 __global__ void apply_row_norm_kernel(const __nv_bfloat16* __restrict__ values, RowNormIn in,
@@ -434,5 +519,28 @@ MLL_API int mll_add_layernorm(float* x, const void* delta, const float* weight, 
     return mll::launch_add_layernorm<__nv_bfloat16, float>(x, delta, weight, bias, out, rows, n_rows, width, eps,
                                                            stream);
   MLL_REQUIRE(false, "layernorm: dtypes %d / %d", delta_dtype, out_dtype);
+  return -1;
+}
+
+// x: float32 [*, width]; up to three deltas [*, width] of `delta_dtype` with a factor each (null: not there, packed from
+// the front); up to two norms (null alpha: not there) with their outputs [n_rows, width] of `out_dtype`; rows: optional
+// int32 [n_rows] gather list.  See add_tanh_norm_vec_kernel.
+MLL_API int mll_add_tanh_norm(float* x, const void* delta0, const void* delta1, const void* delta2, float scale0,
+                              float scale1, float scale2, const float* alpha0, const float* weight0, const float* bias0,
+                              void* out0, const float* alpha1, const float* weight1, const float* bias1, void* out1,
+                              const int* rows, int delta_dtype, int out_dtype, int n_rows, int width,
+                              cudaStream_t stream) {
+  MLL_REQUIRE(n_rows >= 0 && width > 0, "tanh norm: bad sizes rows=%d width=%d", n_rows, width);
+  MLL_REQUIRE((delta0 || !delta1) && (delta1 || !delta2), "tanh norm: a later delta without an earlier one");
+  MLL_REQUIRE(alpha0 || !alpha1, "tanh norm: a second norm without a first");
+  if (n_rows == 0) return 0;
+  mll::TanhNormArgs a{x, {delta0, delta1, delta2}, {scale0, scale1, scale2}, {alpha0, alpha1}, {weight0, weight1},
+                      {bias0, bias1}, {out0, out1}, rows, n_rows, width,
+                      delta2 ? 3 : (delta1 ? 2 : (delta0 ? 1 : 0)), alpha1 ? 2 : (alpha0 ? 1 : 0)};
+  if (delta_dtype == MLL_F32 && out_dtype == MLL_F32) return mll::launch_add_tanh_norm<float, float>(a, stream);
+  if (delta_dtype == MLL_BF16 && out_dtype == MLL_BF16)
+    return mll::launch_add_tanh_norm<__nv_bfloat16, __nv_bfloat16>(a, stream);
+  if (delta_dtype == MLL_BF16 && out_dtype == MLL_F32) return mll::launch_add_tanh_norm<__nv_bfloat16, float>(a, stream);
+  MLL_REQUIRE(false, "tanh norm: dtypes %d / %d", delta_dtype, out_dtype);
   return -1;
 }

@@ -1,0 +1,360 @@
+// A gated linear recurrent unit behind a short convolution:
+//
+//   u_t = conv(x_t + b_x) + b_c         causal, `taps` inputs per channel, nothing before a sequence's first token
+//   r_t = sigmoid(A u_t + a),  i_t = sigmoid(I u_t + c)       A, I block-diagonal: n square blocks of `bs` channels
+//   decay_t = exp(-rate * r_t * softplus(lam))
+//   S_t = decay_t S_(t-1) + sqrt(1 - decay_t^2) i_t u_t       one number per channel, float32, zero at the start
+//   out_t = S_t * gelu(y_t + b_y)       (the tanh form)
+//
+// x and y are columns of one projection row.  u, the gates, the decays and the state are float32.
+//
+// Kernels (each for prompts and single tokens alike; a step's tokens of one sequence are consecutive rows):
+//   * lru_gates       decay and write (sqrt(1 - decay^2) i u) of every token and channel.  A block owns a tile of tokens
+//                     and 64 channels of one diagonal block; it forms u for the tile's tokens and the whole diagonal
+//                     block in shared memory and multiplies.  Two versions: float32 FMAs (any block size, either dtype),
+//                     and mma.sync for bfloat16 matrices: u is cut into three bfloat16 terms that add up to all 24 bits
+//                     of its float32 value, so the products are those of the float32 u, accumulated in float32.
+//                     In steps of single tokens the same blocks also advance the state and write the output.
+//   * lru_scan        the recurrence over a prompt's tokens: a warp per run of tokens, a lane per channel.  Every run is
+//                     summarised (product of decays, state from zero), the runs' carries are chained through shared
+//                     memory, and a second pass over the run applies the carry, multiplies by gelu(y) and writes.
+#include "attention_decode.cuh"
+#include "common.cuh"
+
+namespace mll {
+
+__device__ __forceinline__ float lru_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float lru_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+__device__ __forceinline__ float lru_gelu(float z) {
+  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+
+struct LruArgs {
+  const void* proj;         // [T, ld]: y in columns y_col .. + width, x in columns x_col .. + width
+  const float* x_bias;      // [width]
+  const float* y_bias;      // [width]
+  const float* conv_w;      // [width, taps]
+  const float* conv_b;      // [width]
+  const float* conv_state;  // [slots, taps - 1, width]: the last inputs of every sequence, without x_bias
+  const void* gate_w;       // mma: bfloat16 [n, 2, bs(out), bs(in)]; FMA: float32 [n, bs(in), 2 bs(out)]
+  const float* gate_b;      // [2, width]: r's, then i's
+  const float* lam;         // [width]
+  float* state;             // [slots, width]
+  float* decay;             // [T, width]
+  float* write;             // [T, width]
+  void* out;                // [T, width] in the run's dtype
+  const int* tok_pos;
+  const int* tok_seq;
+  const int* seq_slot;
+  const int* seq_qstart;
+  const int* seq_qlen;
+  int n_tokens, ld, x_col, y_col, width, blocks, taps, single;
+  float rate;
+};
+
+// u of token t, channel c (see above): inputs of this step come from the projection, earlier ones from the state.
+template <typename T>
+__device__ __forceinline__ float lru_conv(const LruArgs& a, int t, int c, int pos, int local, const float* state) {
+  float u = a.conv_b[c];
+  const float xb = a.x_bias[c];
+  for (int back = 0; back < a.taps; ++back) {  // the input `back` tokens ago meets tap taps - 1 - back
+    if (pos - back < 0) break;                  // before the sequence: nothing, not even the bias
+    const float x = back <= local ? to_float(((const T*)a.proj)[(size_t)(t - back) * a.ld + a.x_col + c])
+                                  : state[(size_t)(local - back + a.taps - 1) * a.width + c];
+    u = fmaf(a.conv_w[(size_t)c * a.taps + (a.taps - 1 - back)], x + xb, u);
+  }
+  return u;
+}
+
+// From the two gates' pre-activations to the recurrence's inputs; with `single` also the step itself.
+template <typename T>
+__device__ __forceinline__ void lru_finish(const LruArgs& a, int t, int c, float zr, float zi, float u) {
+  const float r = lru_sigmoid(zr + a.gate_b[c]), i = lru_sigmoid(zi + a.gate_b[a.width + c]);
+  const float log_decay = -a.rate * r * lru_softplus(a.lam[c]);
+  const float decay = expf(log_decay);
+  const float write = sqrtf(-expm1f(2.f * log_decay)) * i * u;  // 1 - decay^2 without cancellation
+  if (a.single) {
+    float* S = a.state + (size_t)a.seq_slot[a.tok_seq[t]] * a.width + c;
+    const float s = fmaf(decay, *S, write);
+    *S = s;
+    const float y = to_float(((const T*)a.proj)[(size_t)t * a.ld + a.y_col + c]) + a.y_bias[c];
+    ((T*)a.out)[(size_t)t * a.width + c] = from_float<T>(s * lru_gelu(y));
+  } else {
+    a.decay[(size_t)t * a.width + c] = decay;
+    a.write[(size_t)t * a.width + c] = write;
+  }
+}
+
+// grid (ceil(tokens / 16), n * ceil(bs / 64)), 256 threads: a thread owns one channel and four tokens.
+template <typename T>
+__global__ void __launch_bounds__(256) lru_gates_kernel(LruArgs a) {
+  extern __shared__ float u_s[];  // [16][bs]
+  const int bs = a.width / a.blocks, tiles = (bs + 63) / 64;
+  const int block = blockIdx.y / tiles, col = (blockIdx.y % tiles) * 64 + (threadIdx.x & 63);
+  const int t0 = blockIdx.x * 16, n = min(16, a.n_tokens - t0);
+  for (int i = threadIdx.x; i < n * bs; i += 256) {
+    const int t = t0 + i / bs, seq = a.tok_seq[t];
+    u_s[i] = lru_conv<T>(a, t, block * bs + i % bs, a.tok_pos[t], t - a.seq_qstart[seq],
+                         a.conv_state + (size_t)a.seq_slot[seq] * (a.taps - 1) * a.width);
+  }
+  __syncthreads();
+  if (col >= bs) return;
+  const float* w = (const float*)a.gate_w + (size_t)block * bs * 2 * bs;
+  const int q0 = (threadIdx.x >> 6) * 4;
+  float r[4] = {0.f, 0.f, 0.f, 0.f}, z[4] = {0.f, 0.f, 0.f, 0.f};
+  for (int k = 0; k < bs; ++k) {
+    const float wr = w[(size_t)k * 2 * bs + col], wi = w[(size_t)k * 2 * bs + bs + col];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float u = q0 + i < n ? u_s[(q0 + i) * bs + k] : 0.f;
+      r[i] = fmaf(wr, u, r[i]);
+      z[i] = fmaf(wi, u, z[i]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+    if (q0 + i < n) lru_finish<T>(a, t0 + q0 + i, block * bs + col, r[i], z[i], u_s[(q0 + i) * bs + col]);
+}
+
+// grid (ceil(tokens / (16 MT)), n * ceil(bs / 64)), 256 threads.  Warp w owns channels 8w .. 8w + 7 of the 64 and both
+// gates of them, so that a thread ends with r and i of the same four (token, channel) pairs per 16 tokens.
+// Shared memory: three bfloat16 planes [3][16 MT][row] of u (high, middle, low term).  The k-order inside a product is
+// free as long as both operands agree: a thread's 16 bytes (eight neighbouring inputs) serve two k-steps.
+template <int MT>
+__global__ void __launch_bounds__(256) lru_gates_mma_kernel(LruArgs a, int row) {
+  extern __shared__ __align__(16) __nv_bfloat16 planes[];
+  constexpr int M = 16 * MT;
+  const int bs = a.width / a.blocks, tiles = (bs + 63) / 64;
+  const int block = blockIdx.y / tiles, c0 = (blockIdx.y % tiles) * 64;
+  const int t0 = blockIdx.x * M, n = min(M, a.n_tokens - t0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3;
+  const int k_pad = (bs + 31) & ~31;
+  for (int i = threadIdx.x; i < M * k_pad; i += 256) {
+    const int m = i / k_pad, k = i % k_pad;
+    float u = 0.f;
+    if (m < n && k < bs) {
+      const int t = t0 + m, seq = a.tok_seq[t];
+      u = lru_conv<__nv_bfloat16>(a, t, block * bs + k, a.tok_pos[t], t - a.seq_qstart[seq],
+                                  a.conv_state + (size_t)a.seq_slot[seq] * (a.taps - 1) * a.width);
+    }
+    const __nv_bfloat16 hi = __float2bfloat16_rn(u);
+    const float rest = u - __bfloat162float(hi);          // exact
+    const __nv_bfloat16 mid = __float2bfloat16_rn(rest);
+    planes[(size_t)m * row + k] = hi;
+    planes[(size_t)(M + m) * row + k] = mid;
+    planes[(size_t)(2 * M + m) * row + k] = __float2bfloat16_rn(rest - __bfloat162float(mid));
+  }
+  __syncthreads();
+  float acc[2][MT][4];
+#pragma unroll
+  for (int e = 0; e < 2; ++e)
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[e][m][i] = 0.f;
+  const int col = c0 + warp * 8 + g;  // this thread's row of the two matrices
+  const __nv_bfloat16* w = (const __nv_bfloat16*)a.gate_w + (size_t)block * 2 * bs * bs;
+  const uint4* wr = reinterpret_cast<const uint4*>(w + (size_t)min(col, bs - 1) * bs);
+  const uint4* wi = reinterpret_cast<const uint4*>(w + (size_t)(bs + min(col, bs - 1)) * bs);
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+#pragma unroll 2
+  for (int k = 0; k < k_pad; k += 32) {
+    const bool in = k + 8 * q < bs && col < bs;  // bs is a multiple of 8: eight inputs are inside or outside together
+    const uint4 b[2] = {in ? wr[(k >> 3) + q] : zero, in ? wi[(k >> 3) + q] : zero};
+#pragma unroll
+    for (int p = 0; p < 3; ++p) {
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        const uint4 lo = *reinterpret_cast<const uint4*>(planes + (size_t)(p * M + m * 16 + g) * row + k + 8 * q);
+        const uint4 up = *reinterpret_cast<const uint4*>(planes + (size_t)(p * M + m * 16 + g + 8) * row + k + 8 * q);
+        const unsigned a0[4] = {lo.x, up.x, lo.y, up.y}, a1[4] = {lo.z, up.z, lo.w, up.w};
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          mma_16816(acc[e][m], a0, b[e].x, b[e].y);
+          mma_16816(acc[e][m], a1, b[e].z, b[e].w);
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int tok = m * 16 + g + 8 * (i >> 1), c = c0 + warp * 8 + 2 * q + (i & 1);
+      if (tok < n && c < bs) {
+        const float u = __bfloat162float(planes[(size_t)tok * row + c]) + __bfloat162float(planes[(size_t)(M + tok) * row + c]) +
+                        __bfloat162float(planes[(size_t)(2 * M + tok) * row + c]);
+        lru_finish<__nv_bfloat16>(a, t0 + tok, block * bs + c, acc[0][m][i], acc[1][m][i], u);
+      }
+    }
+}
+
+// grid (ceil(width / 32), sequences), (32, runs) threads: lane = channel, warp = run of tokens.
+template <typename T>
+__global__ void __launch_bounds__(1024) lru_scan_kernel(LruArgs a) {
+  __shared__ float prod_s[32][33], end_s[32][33];
+  const int lane = threadIdx.x, run = threadIdx.y, runs = blockDim.y;
+  const int seq = blockIdx.y, c = blockIdx.x * 32 + lane;
+  const int row0 = a.seq_qstart[seq], n = a.seq_qlen[seq];
+  const int per = (n + runs - 1) / runs;
+  const int lo = row0 + min(n, run * per), hi = row0 + min(n, (run + 1) * per);
+  const bool live = c < a.width;
+  const float* dec = a.decay + c;
+  const float* wri = a.write + c;
+  float* S = a.state + (size_t)a.seq_slot[seq] * a.width + c;
+  float carry = live ? *S : 0.f;
+  if (runs > 1) {
+    float prod = 1.f, s = 0.f;
+    if (live) {
+      int t = lo;
+      for (; t + 8 <= hi; t += 8) {
+        float d[8], w[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          d[i] = dec[(size_t)(t + i) * a.width];
+          w[i] = wri[(size_t)(t + i) * a.width];
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          s = fmaf(d[i], s, w[i]);
+          prod *= d[i];
+        }
+      }
+      for (; t < hi; ++t) {
+        const float d = dec[(size_t)t * a.width];
+        s = fmaf(d, s, wri[(size_t)t * a.width]);
+        prod *= d;
+      }
+    }
+    prod_s[run][lane] = prod;
+    end_s[run][lane] = s;
+    __syncthreads();  // every run has read the old state too: the last one may write it below
+    for (int e = 0; e < run; ++e) carry = fmaf(prod_s[e][lane], carry, end_s[e][lane]);
+  }
+  if (!live) return;
+  const float yb = a.y_bias[c];
+  const T* y = (const T*)a.proj + a.y_col + c;
+  T* out = (T*)a.out + c;
+  int t = lo;
+  for (; t + 8 <= hi; t += 8) {
+    float d[8], w[8], v[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      d[i] = dec[(size_t)(t + i) * a.width];
+      w[i] = wri[(size_t)(t + i) * a.width];
+      v[i] = to_float(y[(size_t)(t + i) * a.ld]);
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      carry = fmaf(d[i], carry, w[i]);
+      out[(size_t)(t + i) * a.width] = from_float<T>(carry * lru_gelu(v[i] + yb));
+    }
+  }
+  for (; t < hi; ++t) {
+    carry = fmaf(dec[(size_t)t * a.width], carry, wri[(size_t)t * a.width]);
+    out[(size_t)t * a.width] = from_float<T>(carry * lru_gelu(to_float(y[(size_t)t * a.ld]) + yb));
+  }
+  if (hi == row0 + n && lo < hi) *S = carry;  // exactly one run ends with the sequence's last token
+}
+
+// Bytes of shared memory and elements between rows of a plane: 16-byte words of neighbouring rows in different banks.
+inline int lru_plane_row(int bs) { return ((bs + 31) / 32) * 32 + (((bs + 31) / 32) % 2 ? 0 : 32); }
+
+template <int MT>
+int launch_lru_gates_mma(const LruArgs& a, cudaStream_t stream) {
+  const int bs = a.width / a.blocks, row = lru_plane_row(bs);
+  const size_t smem = (size_t)3 * 16 * MT * row * 2;
+  auto kernel = lru_gates_mma_kernel<MT>;
+  if (smem > 48 * 1024) {
+    cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (err != cudaSuccess) {
+      mll_set_error("linear recurrent unit: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(err));
+      return (int)err;
+    }
+  }
+  const dim3 grid((a.n_tokens + 16 * MT - 1) / (16 * MT), a.blocks * ((bs + 63) / 64));
+  MLL_LAUNCH((kernel), grid, 256, smem, stream, a, row);
+  MLL_LAUNCH_CHECK();
+  return 0;
+}
+
+template <typename T>
+int launch_lru_gates(const LruArgs& a, cudaStream_t stream) {
+  const int bs = a.width / a.blocks;
+  const size_t smem = (size_t)16 * bs * sizeof(float);
+  auto kernel = lru_gates_kernel<T>;
+  if (smem > 48 * 1024) {
+    cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (err != cudaSuccess) {
+      mll_set_error("linear recurrent unit: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(err));
+      return (int)err;
+    }
+  }
+  const dim3 grid((a.n_tokens + 15) / 16, a.blocks * ((bs + 63) / 64));
+  MLL_LAUNCH((kernel), grid, 256, smem, stream, a);
+  MLL_LAUNCH_CHECK();
+  return 0;
+}
+
+}  // namespace mll
+
+// Whether the tensor-core version takes diagonal blocks of this size (bfloat16 matrices).
+MLL_API int mll_lru_mma_supported(int dtype, int bs) {
+  return dtype == MLL_BF16 && bs % 8 == 0 && bs >= 8 && (size_t)3 * 16 * mll::lru_plane_row(bs) * 2 <= 200 * 1024;
+}
+
+// `mma`: gate_w is bfloat16 [n, 2, bs, bs] (rows are outputs), else float32 [n, bs(in), 2 bs(out)].
+// `single`: every sequence brings one token; the state advances and `out` is written here (decay, write may be null).
+MLL_API int mll_lru_gates(const void* proj, const float* x_bias, const float* y_bias, const float* conv_w,
+                          const float* conv_b, const float* conv_state, const void* gate_w, const float* gate_b,
+                          const float* lam, float* state, float* decay, float* write, void* out, const int* tok_pos,
+                          const int* tok_seq, const int* seq_slot, const int* seq_qstart, int dtype, int n_tokens, int ld,
+                          int x_col, int y_col, int width, int blocks, int taps, float rate, int mma, int single,
+                          cudaStream_t stream) {
+  MLL_REQUIRE(n_tokens >= 0 && width > 0 && blocks > 0 && width % blocks == 0 && taps > 0, "linear recurrent unit: bad sizes");
+  MLL_REQUIRE(x_col >= 0 && y_col >= 0 && x_col + width <= ld && y_col + width <= ld,
+              "linear recurrent unit: columns outside rows of %d", ld);
+  MLL_REQUIRE(single ? (state && out) : (decay && write), "linear recurrent unit: an output is missing");
+  const int bs = width / blocks;
+  MLL_REQUIRE((size_t)16 * bs * 4 <= 200 * 1024, "linear recurrent unit: blocks of %d exceed the 3200 the kernel takes", bs);
+  MLL_REQUIRE((long long)blocks * ((bs + 63) / 64) <= 65535, "linear recurrent unit: too many blocks for one launch");
+  if (n_tokens == 0) return 0;
+  mll::LruArgs a{proj, x_bias, y_bias, conv_w, conv_b, conv_state, gate_w, gate_b, lam, state, decay, write, out, tok_pos,
+                 tok_seq, seq_slot, seq_qstart, nullptr, n_tokens, ld, x_col, y_col, width, blocks, taps, single, rate};
+  if (mma) {
+    MLL_REQUIRE(mll_lru_mma_supported(dtype, bs), "linear recurrent unit: blocks of %d on tensor cores", bs);
+    const size_t per16 = (size_t)3 * 16 * mll::lru_plane_row(bs) * 2;
+    // a tall tile reads the matrices less often, a low one gives more blocks
+    if (n_tokens > 256 && 4 * per16 <= 110 * 1024) return mll::launch_lru_gates_mma<4>(a, stream);
+    if (n_tokens > 16 && 2 * per16 <= 110 * 1024) return mll::launch_lru_gates_mma<2>(a, stream);
+    return mll::launch_lru_gates_mma<1>(a, stream);
+  }
+  if (dtype == MLL_F32) return mll::launch_lru_gates<float>(a, stream);
+  if (dtype == MLL_BF16) return mll::launch_lru_gates<__nv_bfloat16>(a, stream);
+  MLL_REQUIRE(false, "linear recurrent unit: unknown dtype %d", dtype);
+  return -1;
+}
+
+// `longest`: the most tokens any sequence of the step brings (how many warps share a sequence follows from it).
+MLL_API int mll_lru_scan(const float* decay, const float* write, const void* proj, const float* y_bias, float* state,
+                         void* out, const int* seq_slot, const int* seq_qstart, const int* seq_qlen, int dtype, int n_seqs,
+                         int ld, int y_col, int width, int longest, cudaStream_t stream) {
+  MLL_REQUIRE(n_seqs >= 0 && n_seqs <= 65535 && width > 0 && longest >= 0 && y_col >= 0 && y_col + width <= ld,
+              "linear recurrent scan: bad sizes");
+  if (n_seqs == 0 || longest == 0) return 0;
+  mll::LruArgs a{};
+  a.decay = const_cast<float*>(decay); a.write = const_cast<float*>(write);
+  a.proj = proj; a.y_bias = y_bias; a.state = state; a.out = out;
+  a.seq_slot = seq_slot; a.seq_qstart = seq_qstart; a.seq_qlen = seq_qlen;
+  a.ld = ld; a.y_col = y_col; a.width = width;
+  const int runs = min(32, max(1, (longest + 15) / 16));
+  const dim3 grid((width + 31) / 32, n_seqs), block(32, runs);
+  if (dtype == MLL_F32)
+    MLL_LAUNCH((mll::lru_scan_kernel<float>), grid, block, 0, stream, a);
+  else if (dtype == MLL_BF16)
+    MLL_LAUNCH((mll::lru_scan_kernel<__nv_bfloat16>), grid, block, 0, stream, a);
+  else
+    MLL_REQUIRE(false, "linear recurrent scan: unknown dtype %d", dtype);
+  MLL_LAUNCH_CHECK();
+  return 0;
+}

@@ -158,12 +158,14 @@ class PendingSum:
     """The outputs of two parts that read the same norm (a block whose mixer and feed-forward run side by
     side), both still to be added to the residual stream: the next norm adds `first + second` to it in
     float32 in the same kernel that normalises.  `scale_first`, `scale_second`: factors on the two (a mixer made of
-    two mixers side by side, each with a weight of its own)."""
+    two mixers side by side, each with a weight of its own).  `third`: one more output (a feed-forward that runs
+    beside such a mixer), without a factor."""
 
     first: torch.Tensor
     second: torch.Tensor
     scale_first: float = 1.0
     scale_second: float = 1.0
+    third: Optional[torch.Tensor] = None
 
 
 @dataclass
@@ -310,6 +312,12 @@ class Norm(Part):
         `rows` only those rows, x unchanged.  A `PreNormed` made for this norm is handed on as it is;
         a `PendingSum` adds both of its tensors."""
         raise NotImplementedError
+
+    def forward_pair(self, step, x: torch.Tensor, delta, other: "Norm", out_names: Tuple[str, str] = ("h", "h2")):
+        """(norm(x), other(x)) after x += delta: two norms of one stream (a block whose sub-layers both read x).
+        A norm with a kernel for the pair overrides this."""
+        return (self.forward(step, x, delta, out_name=out_names[0]),
+                other.forward(step, x, None, out_name=out_names[1]))
 
     def prenorm_weight(self):
         """(weight float32 [D], eps) if the norm is x * weight / sqrt(mean(x^2) + eps) and may be folded

@@ -6,6 +6,8 @@ With `residual_mult` m (not in the reference) both outputs join the stream times
 x' = r + m feed_forward(..); a layer without a feed-forward ends at r.
 `parallel` (not in the reference) lets mixer and feed-forward read one norm:
     h = norm(x);   x' = x + mixer(h) + feed_forward(h)
+`parallel_two_norms` (not in the reference) gives each of the two a norm of its own, both of the same stream:
+    x' = x + mixer(norm_m(x)) + feed_forward(norm_f(x))
 `sandwich` (not in the reference) puts a norm behind each sub-layer as well as in front of it:
     r = x + norm_mo(mixer(norm_in(x)));   x' = r + norm_fo(feed_forward(norm_pf(r)))
 The residual adds are not separate kernels: a part's output stays "pending" until the
@@ -15,6 +17,7 @@ itself and hands on a `PreNormed`, which the part behind reads (small decode bat
 """
 from __future__ import annotations
 
+from dataclasses import replace
 from typing import List
 
 from .mlp import NoFeedForward
@@ -78,6 +81,26 @@ class ParallelBlock(Block):
         return mixed if fed is None else PendingSum(mixed, fed)
 
 
+class ParallelTwoNormsBlock(Block):
+    """Two norms of one stream:   x' = x + mixer(norm_m(x)) + feed_forward(norm_f(x)), norms "mixer" and "feed_forward".
+    The norms run together where their kind has a kernel for the pair (`Norm.forward_pair`); all outputs - the mixer's
+    may be a `PendingSum` itself - stay pending until the next norm."""
+
+    capturable = True
+
+    def norm_names(self) -> List[str]:
+        return ["mixer", "feed_forward"]
+
+    def forward(self, step, x, pending, layer, cache):
+        norm = layer.norms["mixer"]
+        if isinstance(layer.feed_forward, NoFeedForward):
+            return layer.mixer.forward(step, norm.forward(step, x, pending), cache)
+        h, h_ff = norm.forward_pair(step, x, pending, layer.norms["feed_forward"])
+        mixed = layer.mixer.forward(step, h, cache)
+        fed = layer.feed_forward.forward(step, h_ff)
+        return replace(mixed, third=fed) if isinstance(mixed, PendingSum) else PendingSum(mixed, fed)
+
+
 class SandwichBlock(Block):
     """Norms "input" and "mixer_out" around the mixer, "pre_ff" and "ff_out" around the feed-forward.  A sub-layer's
     output stays pending together with the norm behind it (`NormedDelta`): the norm that reads the stream next
@@ -98,6 +121,7 @@ class SandwichBlock(Block):
         return NormedDelta(layer.feed_forward.forward(step, h), layer.norms["ff_out"])
 
 
+register_part("block", "parallel_two_norms", ParallelTwoNormsBlock)
 register_part("block", "sandwich", SandwichBlock)
 register_part("block", "pre_norm", PreNormBlock)
 register_part("block", "parallel", ParallelBlock)

@@ -12,9 +12,13 @@ stream normalised again in the one kernel.
 `layer_norm` (not in the reference): y_i = (x_i - mean) / sqrt(var + eps) * w_i + b_i with var the mean of the
 squared deviations; weight and bias are tensors of their own.  It has no factor that the products around it could
 apply, so it is never folded away (`prenorm_weight` stays None).
+
+`dynamic_tanh` (not in the reference): y_i = tanh(alpha * x_i) * w_i + b_i with one number alpha per norm: no mean, no
+variance, every column by itself.  Two such norms of one stream are one kernel (`forward_pair`).
 """
 from __future__ import annotations
 
+from dataclasses import replace
 from typing import List, Optional
 
 import torch
@@ -35,10 +39,20 @@ def _delta_parts(delta):
     if isinstance(delta, ScaledDelta):
         first, s1 = delta.delta, delta.scale
     elif isinstance(delta, PendingSum):
+        if delta.third is not None and norm is not None:
+            raise RuntimeError("a sum of three outputs cannot pass a norm on its way into the stream")
         first, second, s1, s2 = delta.first, delta.second, delta.scale_first, delta.scale_second
     if norm is None and s1 == 1.0 and s2 == 1.0:
         return first, second, None
     return first, second, K.DeltaNorm(norm.weight if norm is not None else None, norm.eps if norm is not None else 0.0, s1, s2)
+
+
+def _add_third(x, delta):
+    """The norms below take two outputs: a third one joins the stream in a kernel of its own first."""
+    if isinstance(delta, PendingSum) and delta.third is not None:
+        K.add_dynamic_tanh(x, [(delta.third, 1.0)], [])
+        return replace(delta, third=None)
+    return delta
 
 
 class RMSNorm(Norm):
@@ -79,6 +93,7 @@ class RMSNorm(Norm):
             return delta  # x is up to date; the product that reads the rows applies the factor
         n = x.shape[0] if rows is None else rows.shape[0]
         out = step.ws.buffer(out_name, (n, self.width), self.ctx.act_dtype)
+        delta = _add_third(x, delta)
         first, second, delta_norm = _delta_parts(delta)
         K.add_rmsnorm(x, first, self.weight, out, self.eps, rows, delta2=second, delta_norm=delta_norm)
         return out
@@ -122,6 +137,7 @@ class LayerNorm(Norm):
             raise RuntimeError(f"{self.name}: a layer norm cannot finish rows that were prepared for another norm")
         n = x.shape[0] if rows is None else rows.shape[0]
         out = step.ws.buffer(out_name, (n, self.width), self.ctx.act_dtype)
+        delta = _add_third(x, delta)
         if isinstance(delta, (NormedDelta, ScaledDelta)) or (isinstance(delta, PendingSum) and (delta.scale_first != 1.0 or delta.scale_second != 1.0)):
             raise RuntimeError(f"{self.name}: a layer norm adds its delta as it is (no norm or factor on the way in)")
         if isinstance(delta, PendingSum):
@@ -134,5 +150,66 @@ class LayerNorm(Norm):
         return out
 
 
+class DynamicTanh(Norm):
+    """y = tanh(alpha * x) * weight + bias.  params: width, name (tensor name of the weight), alpha and bias (tensor names;
+    alpha is a scalar), optional (True: a folder may leave the tensors out)."""
+
+    capturable = True
+
+    def __init__(self, params, ctx: BuildContext):
+        super().__init__(params, ctx)
+        self.width = int(params["width"])
+        self.name = params["name"]
+        self.alpha_name = params["alpha"]
+        self.bias_name = params["bias"]
+        self.optional = bool(params.get("optional", False))
+        self.weight: Optional[torch.Tensor] = None
+        self.alpha: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
+
+    def weight_specs(self) -> List[WeightSpec]:
+        return [WeightSpec(self.name, (self.width,), kind="vector", init="norm", optional=self.optional),
+                WeightSpec(self.bias_name, (self.width,), kind="vector", init="normal", optional=self.optional),
+                WeightSpec(self.alpha_name, (), kind="vector", init="norm", optional=self.optional)]
+
+    def bind(self, store) -> None:
+        self.weight = store.take(self.name)
+        self.bias = store.take(self.bias_name)
+        self.alpha = store.take(self.alpha_name).reshape(1).contiguous()
+
+    def parameter_bytes(self) -> int:
+        return self.width * 8 + 4
+
+    def _form(self, out):
+        return K.TanhNorm(self.alpha, self.weight, self.bias, out)
+
+    @staticmethod
+    def _deltas(delta):
+        if delta is None:
+            return []
+        if isinstance(delta, (PreNormed, NormedDelta)):
+            raise RuntimeError("a dynamic tanh cannot finish rows prepared for another norm, nor normalise a delta")
+        if isinstance(delta, ScaledDelta):
+            return [(delta.delta, delta.scale)]
+        if isinstance(delta, PendingSum):
+            out = [(delta.first, delta.scale_first), (delta.second, delta.scale_second)]
+            return out + ([(delta.third, 1.0)] if delta.third is not None else [])
+        return [(delta, 1.0)]
+
+    def forward(self, step, x, delta, rows=None, out_name: str = "h"):
+        n = x.shape[0] if rows is None else rows.shape[0]
+        out = step.ws.buffer(out_name, (n, self.width), self.ctx.act_dtype)
+        K.add_dynamic_tanh(x, self._deltas(delta), [self._form(out)], rows)
+        return out
+
+    def forward_pair(self, step, x, delta, other, out_names=("h", "h2")):
+        if not isinstance(other, DynamicTanh):
+            return super().forward_pair(step, x, delta, other, out_names)
+        first, second = (step.ws.buffer(name, (x.shape[0], self.width), self.ctx.act_dtype) for name in out_names)
+        K.add_dynamic_tanh(x, self._deltas(delta), [self._form(first), other._form(second)])
+        return first, second
+
+
+register_part("norm", "dynamic_tanh", DynamicTanh)
 register_part("norm", "rms_norm", RMSNorm)
 register_part("norm", "layer_norm", LayerNorm)
