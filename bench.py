@@ -607,6 +607,53 @@ def badolix_rooflines(size, tokens, batch, context, peaks):
     return out
 
 
+def mefolorn_config(size):
+    """Six layers: latent attention (queries through a latent of 3/8 of the width, 256 latent columns per position), mixed
+    scores beside a linear recurrent unit (as wide as the model, in blocks of 256, 4 taps), the pair again, latent
+    attention, the pair, latent attention; every attention under a window of 1,024 positions, a dense feed-forward
+    beside every mixer."""
+    import cpp_minilamma_b200 as ml
+    s = DESIGN_SIZES[size]
+    mlp = {"kind": "dense", "ff": s["ff"]}
+    latent = {"type": "latent_attention", "mlp": mlp,
+              "mixer": {"heads": s["heads"], "dim": 128, "vdim": 128, "q_rank": 3 * s["width"] // 8, "kv_rank": 256,
+                        "scale": 128 ** -0.5, "mask": {"size": 1024}}}
+    pair = {"type": "parallel", "mlp": mlp,
+            "mixer": {"left": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                               "mask": {"size": 1024}, "rot": {"base": 500000.0, "dims": 128}},
+                      "right": {"width": s["width"], "blocks": s["width"] // 256, "conv": 4},
+                      "left_scale": 0.8, "right_scale": 1.2}}
+    return ml.config_from_dict({"architecture": "Mefolorn", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5},
+                                "embedding": {"scale": 2.0}, "layers": [latent, pair, pair, latent, pair, latent],
+                                "torch_dtype": "bfloat16"})
+
+
+def mefolorn_rooflines(size, tokens, batch, context, peaks):
+    """As `design_rooflines`, for the kernels of the Mefolorn decoder and their like in the Badolix decoder."""
+    s = DESIGN_SIZES[size]
+    H, G, d, D, ff = s["heads"], s["kv_heads"], 128, s["width"], s["ff"]
+    rank, q_rank, W, bs, taps = 256, 3 * D // 8, D, 256, 4
+    out = {k: v for k, v in badolix_rooflines(size, tokens, batch, context, peaks).items() if k[0] == "badolix"}
+    seen = sum(min(i + 1, 1024) for i in range(tokens))
+    visible = min(context, 1024)
+    out["mefolorn", "prefill", "mixed_attention_mma"] = ("tensor", 2.0 * seen * (H * 2 * d + H * H))
+    out["mefolorn", "decode", "mixed_attention_single"] = ("hbm", batch * visible * G * 2 * d * 2)
+    out["mefolorn", "prefill", "local_attention_mma"] = ("tensor", 2.0 * H * seen * 2 * rank)
+    out["mefolorn", "decode", "local_attention_heads"] = ("hbm", batch * visible * rank * 2)
+    qkv = (H * d + 2 * G * d) * 2
+    for kind, n, seqs in (("prefill", tokens, 1), ("decode", batch, batch)):
+        out["mefolorn", kind, "tanh_norm"] = ("hbm", n * D * (4 + 4 + 2.5 * 2 + 2 * 2))  # half of them add three outputs
+        out["mefolorn", kind, "local_attention_prepare"] = ("hbm", n * 2 * qkv)
+        out["mefolorn", kind, "latent_prepare"] = ("hbm", n * (q_rank + rank) * 4)
+        out["mefolorn", kind, "heads_gate"] = ("hbm", n * H * d * 4)
+        out["mefolorn", kind, "swiglu"] = ("hbm", n * ff * (4 + 2))
+        out["mefolorn", kind, "conv_state_update"] = ("hbm", seqs * (taps - 1) * W * (2 + 4))
+    out["mefolorn", "prefill", "lru_gates"] = ("hbm", tokens * W * (2 + 8) + 2 * W * bs * 2)
+    out["mefolorn", "prefill", "lru_scan"] = ("hbm", tokens * W * (8 + 2 + 2))
+    out["mefolorn", "decode", "lru_gates (single tokens)"] = ("hbm", batch * W * (4 + 2 + 8 + 4 * (taps - 1)) + 2 * W * bs * 2)
+    return out
+
+
 def llama_like_config(size):
     import cpp_minilamma_b200 as ml
     s = DESIGN_SIZES[size]
@@ -673,8 +720,8 @@ def design_rooflines(size, tokens, batch, context, peaks):
 
 
 def bench_design(args):
-    """Prompt and decode throughput of the Kupirax or Malulorn decoder and of the Llama decoder (of the Sopanex decoder
-    and of the Malulorn decoder, the closest to it) at equal width,
+    """Prompt and decode throughput of the Kupirax or Malulorn decoder and of the Llama decoder (of the Sopanex or Badolix
+    decoder and of the Malulorn decoder, the closest to them; of the Mefolorn decoder and of the Badolix decoder) at equal width,
     feed-forward, heads and layer count (random bfloat16 weights), and the device time of each of this library's kernels in one
     prompt step and one decode step of either, with the fraction of the measured peak it reaches."""
     import numpy as np
@@ -686,10 +733,11 @@ def bench_design(args):
     tokens, batch, context = PREFILL_TOKENS, 64, 1024
     design = args.design
     make_config = {"kupirax": kupirax_config, "malulorn": malulorn_config, "sopanex": sopanex_config,
-                   "badolix": badolix_config}[design]
+                   "badolix": badolix_config, "mefolorn": mefolorn_config}[design]
     rooflines = {"kupirax": design_rooflines, "malulorn": malulorn_rooflines, "sopanex": sopanex_rooflines,
-                 "badolix": badolix_rooflines}[design]
-    beside, beside_config = ("malulorn", malulorn_config) if design in ("sopanex", "badolix") else ("llama", llama_like_config)
+                 "badolix": badolix_rooflines, "mefolorn": mefolorn_rooflines}[design]
+    beside, beside_config = {"sopanex": ("malulorn", malulorn_config), "badolix": ("malulorn", malulorn_config),
+                             "mefolorn": ("badolix", badolix_config)}.get(design, ("llama", llama_like_config))
     result = {"design": design, "beside": beside, "dtype": "bf16", "data": "synthetic token ids, random-init weights",
               "prefill_tokens": tokens, "decode_prompts": "uniform[128,1024)", "steps": steps, "warmup": warmup,
               "peaks": {"hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"], "source": peaks["source"]},
@@ -761,9 +809,9 @@ def main():
     parser.add_argument("--shape", choices=sorted(SHAPES), default="llama31_8b", help="model shape of the --profile step")
     parser.add_argument("--batch", type=int, default=BATCH, help="batch of the --profile decode step")
     parser.add_argument("--context", type=int, default=1024, help="prompt length of the --profile decode step")
-    parser.add_argument("--design", choices=["kupirax", "malulorn", "sopanex", "badolix"], default=None,
+    parser.add_argument("--design", choices=["kupirax", "malulorn", "sopanex", "badolix", "mefolorn"], default=None,
                         help="instead of the default workload: prompt and decode throughput and kernel times of that "
-                             "decoder beside the Llama decoder (sopanex, badolix: beside the Malulorn decoder) at equal sizes")
+                             "decoder beside the Llama decoder (sopanex, badolix: beside the Malulorn decoder; mefolorn: beside the Badolix decoder) at equal sizes")
     parser.add_argument("--size", choices=sorted(DESIGN_SIZES), default=None, help="one size of --design (default: all)")
     args = parser.parse_args()
 

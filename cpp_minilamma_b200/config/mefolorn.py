@@ -51,7 +51,9 @@ class MixedHeadsSide:
                    scale=take_float(raw, "scale"), window=_window(raw, what))
         if raw.get("rot") is not None:
             rot = _object(raw["rot"], what + ".rot")
-            side.rot_base, side.rot_dims = take_float(rot, "base"), take_int(rot, "dims", minimum=0)
+            side.rot_dims = take_int(rot, "dims", minimum=0)
+            if side.rot_dims:
+                side.rot_base = take_float(rot, "base")
         if side.heads % side.kv_heads:
             raise ConfigError(f"config.json: {what}: {side.heads} heads are not a multiple of {side.kv_heads} kv_heads")
         if side.rot_dims % 2 or side.rot_dims > side.dim or side.rot_base <= 0:

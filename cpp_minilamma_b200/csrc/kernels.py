@@ -1562,6 +1562,64 @@ def mixed_attention(q, k_cache, v_cache, tok_pos, tok_seq, seq_slot, block_table
         _stream()), "mixed_attention")
 
 
+USE_TENSOR_CORE_MIXED = True  # tests switch it off to reach the general kernel in bfloat16
+
+
+def mixed_attention_mma_supported(dtype: torch.dtype, single: bool, n_heads: int, n_kv_heads: int, d: int, dv: int) -> bool:
+    """Whether `mixed_attention_tiles` (single False) or `mixed_attention_single` takes the sizes."""
+    return USE_TENSOR_CORE_MIXED and dtype == torch.bfloat16 and bool(lib().mll_mixed_attention_mma_supported(
+        dtype_code(dtype), ctypes.c_int(int(single)), ctypes.c_int(n_heads), ctypes.c_int(n_kv_heads), ctypes.c_int(d),
+        ctypes.c_int(dv)))
+
+
+def _mixed_mma(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_qlen, tile_seq, tile_row0, block_table, mix, bias,
+               out, scratch, n_tiles, n_heads, n_kv_heads, d, dv, window, n_splits, scale, what) -> None:
+    _need(q, "mixed attention q", torch.bfloat16)
+    _check_mixed(q, k_cache, v_cache, out, mix, bias, n_heads, n_kv_heads, d, dv)
+    for name, t in (("seq_slot", seq_slot), ("seq_ctx", seq_ctx), ("seq_qstart", seq_qstart), ("seq_qlen", seq_qlen)):
+        _need(t, f"mixed attention {name}", torch.int32, 1)
+    _need(block_table, "mixed attention block table", torch.int32, 2)
+    _check(lib().mll_mixed_attention_mma(
+        _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(seq_slot), _ptr(seq_ctx), _ptr(seq_qstart), _ptr(seq_qlen),
+        _ptr(tile_seq), _ptr(tile_row0), _ptr(block_table), _ptr(mix), _ptr(bias), _ptr(out), _ptr(scratch),
+        ctypes.c_int(n_tiles), ctypes.c_int(n_heads), ctypes.c_int(n_kv_heads), ctypes.c_int(d), ctypes.c_int(dv),
+        ctypes.c_int(window), ctypes.c_int(block_table.shape[1]), ctypes.c_int(n_splits), ctypes.c_float(scale),
+        _stream()), what, kernels=2 if n_splits > 1 else 1)
+
+
+def mixed_attention_tiles(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_qlen, tile_seq, tile_row0, block_table,
+                          mix, bias, out, n_heads: int, n_kv_heads: int, d: int, dv: int, window: int, scale: float) -> None:
+    """`mixed_attention` for prompt steps in bfloat16 on tensor cores: the work is a list of tiles of up to PREFILL_TILE
+    query rows, (sequence, first row among the sequence's new tokens)."""
+    for name, t in (("tile_seq", tile_seq), ("tile_row0", tile_row0)):
+        _need(t, f"mixed attention {name}", torch.int32, 1)
+    if tile_seq.shape != tile_row0.shape:
+        raise KernelError("mixed attention: the tile lists differ in length")
+    _mixed_mma(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_qlen, tile_seq, tile_row0, block_table, mix, bias, out,
+               None, tile_seq.shape[0], n_heads, n_kv_heads, d, dv, window, 1, scale, "mixed_attention_mma")
+
+
+def mixed_attention_single_scratch(n_seqs: int, n_heads: int, dv: int, n_splits: int) -> int:
+    return n_seqs * n_splits * n_heads * dv
+
+
+def mixed_attention_single(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_qlen, block_table, mix, bias, out,
+                           n_seqs: int, n_heads: int, n_kv_heads: int, d: int, dv: int, window: int, scale: float,
+                           n_splits: int = 1, scratch: Optional[torch.Tensor] = None) -> None:
+    """`mixed_attention` for steps in which every sequence brings one token, bfloat16, on tensor cores.  `n_splits` > 1:
+    that many blocks along every context, whose results are added up; `scratch` float32 of
+    `mixed_attention_single_scratch` floats."""
+    if q.shape[0] != n_seqs:
+        raise KernelError(f"mixed attention: {q.shape[0]} rows for {n_seqs} single tokens")
+    if n_splits > 1:
+        _need(scratch, "mixed attention scratch", torch.float32)
+        if scratch.numel() < mixed_attention_single_scratch(n_seqs, n_heads, dv, n_splits):
+            raise KernelError("mixed attention: scratch too small for the split count")
+    _mixed_mma(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_qlen, None, None, block_table, mix, bias, out,
+               scratch if n_splits > 1 else None, n_seqs, n_heads, n_kv_heads, d, dv, window, n_splits, scale,
+               "mixed_attention_single")
+
+
 # --------------------------------------------------------------------------- #
 # attention over a shared low-rank latent
 # --------------------------------------------------------------------------- #

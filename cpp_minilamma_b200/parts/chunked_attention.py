@@ -34,6 +34,27 @@ from .linear import Linear
 from .rope import shared_position_encoding
 
 
+def prompt_tiles(shape):
+    """The index arrays of a prompt step's attention on tensor cores: tiles of up to PREFILL_TILE query rows as
+    (sequence, first row among the sequence's new tokens), the sequences with the most rows first, and the same rows in
+    tiles of twice as many.  Steps of single tokens need no list."""
+    if shape.all_decode:
+        return {}
+    lists = {"tile_seq": [], "tile_row0": []}
+    wide = []
+    for i in sorted(range(shape.n_seqs), key=lambda i: -shape.lens[i]):
+        for row0 in range(0, shape.lens[i], K.PREFILL_TILE):
+            lists["tile_seq"].append(i)
+            lists["tile_row0"].append(row0)
+        for row0 in range(0, shape.lens[i], 2 * K.PREFILL_TILE):
+            wide.append((shape.starts[i] + min(shape.lens[i], row0 + 2 * K.PREFILL_TILE), i, row0))
+    # the same rows in tiles of twice as many, for the tcgen05 kernel, which walks its list from the back
+    wide.sort()
+    lists["wide_seq"] = [i for _, i, _ in wide]
+    lists["wide_row0"] = [row0 for _, _, row0 in wide]
+    return lists
+
+
 class ChunkedAttention(Mixer):
     """params:
       n_heads, n_kv_heads, head_dim, v_head_dim     sizes
@@ -170,23 +191,7 @@ class ChunkedAttention(Mixer):
         return ("chunked_attention.tiles", K.PREFILL_TILE) if self.ctx.act_dtype == torch.bfloat16 else None
 
     def prepare_step(self, shape):
-        """Tiles of up to PREFILL_TILE query rows as (sequence, first row among the sequence's new tokens), the
-        sequences with the most rows first.  Steps of single tokens need no list."""
-        if shape.all_decode:
-            return {}
-        lists = {"tile_seq": [], "tile_row0": []}
-        wide = []
-        for i in sorted(range(shape.n_seqs), key=lambda i: -shape.lens[i]):
-            for row0 in range(0, shape.lens[i], K.PREFILL_TILE):
-                lists["tile_seq"].append(i)
-                lists["tile_row0"].append(row0)
-            for row0 in range(0, shape.lens[i], 2 * K.PREFILL_TILE):
-                wide.append((shape.starts[i] + min(shape.lens[i], row0 + 2 * K.PREFILL_TILE), i, row0))
-        # the same rows in tiles of twice as many, for the tcgen05 kernel, which walks its list from the back
-        wide.sort()
-        lists["wide_seq"] = [i for _, i, _ in wide]
-        lists["wide_row0"] = [row0 for _, _, row0 in wide]
-        return lists
+        return prompt_tiles(shape)
 
     def forward(self, step, h, cache):
         T = h.shape[0]

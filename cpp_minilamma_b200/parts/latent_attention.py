@@ -27,6 +27,7 @@ import torch
 
 from ..csrc import kernels as K
 from .base import BuildContext, CacheNeed, KVNeed, Mixer, WeightSpec, register_part
+from .chunked_attention import prompt_tiles
 from .linear import Linear
 from .rope import shared_position_encoding
 
@@ -135,20 +136,7 @@ class LatentAttention(Mixer):
         return ("chunked_attention.tiles", K.PREFILL_TILE) if self.ctx.act_dtype == torch.bfloat16 else None
 
     def prepare_step(self, shape):
-        if shape.all_decode:
-            return {}
-        lists = {"tile_seq": [], "tile_row0": [], "wide_seq": [], "wide_row0": []}
-        wide = []
-        for i in sorted(range(shape.n_seqs), key=lambda i: -shape.lens[i]):
-            for row0 in range(0, shape.lens[i], K.PREFILL_TILE):
-                lists["tile_seq"].append(i)
-                lists["tile_row0"].append(row0)
-            for row0 in range(0, shape.lens[i], 2 * K.PREFILL_TILE):
-                wide.append((shape.starts[i] + min(shape.lens[i], row0 + 2 * K.PREFILL_TILE), i, row0))
-        wide.sort()
-        lists["wide_seq"] = [i for _, i, _ in wide]
-        lists["wide_row0"] = [row0 for _, _, row0 in wide]
-        return lists
+        return prompt_tiles(shape)
 
     def forward(self, step, h, cache):
         T, H = h.shape[0], self.n_heads

@@ -19,6 +19,7 @@ import torch
 
 from ..csrc import kernels as K
 from .base import BuildContext, CacheNeed, KVNeed, Mixer, WeightSpec, register_part
+from .chunked_attention import prompt_tiles
 from .linear import Linear
 from .rope import shared_position_encoding
 
@@ -112,7 +113,28 @@ class MixedHeadsAttention(Mixer):
         self._attend(step, q, cache, out)
         return self.o.forward(step, out, self.out_name)
 
+    def step_metadata_key(self):
+        # the tile list of prompt steps on tensor cores, shared with the other attention layers
+        return ("chunked_attention.tiles", K.PREFILL_TILE) if self.ctx.act_dtype == torch.bfloat16 else None
+
+    def prepare_step(self, shape):
+        return prompt_tiles(shape)
+
     def _attend(self, step, q, cache, out) -> None:
+        sizes = (self.n_heads, self.n_kv_heads, self.d, self.dv)
+        tiles = step.meta.get(self.step_metadata_key()) if not step.all_decode else None
+        if (step.all_decode or tiles) and K.mixed_attention_mma_supported(self.ctx.act_dtype, step.all_decode, *sizes):
+            seqs = (q, cache.k, cache.v, step.seq_slot, step.seq_ctx, step.seq_qstart, step.seq_qlen)
+            if tiles:
+                K.mixed_attention_tiles(*seqs, tiles["tile_seq"], tiles["tile_row0"], cache.block_table, self.mix, self.bias,
+                                        out, *sizes, self.window, self.scale)
+                return
+            splits = K.local_attention_heads_splits(step.n_seqs, 1, self.ctx.multiprocessors)
+            scratch = step.ws.buffer("attn.parts", (K.mixed_attention_single_scratch(step.n_seqs, self.n_heads, self.dv, splits),),
+                                     torch.float32) if splits > 1 else None
+            K.mixed_attention_single(*seqs, cache.block_table, self.mix, self.bias, out, step.n_seqs, *sizes, self.window,
+                                     self.scale, n_splits=splits, scratch=scratch)
+            return
         K.mixed_attention(q, cache.k, cache.v, step.tok_pos, step.tok_seq, step.seq_slot, cache.block_table, self.mix,
                           self.bias, out, self.n_heads, self.n_kv_heads, self.d, self.dv, self.window, self.scale)
 
