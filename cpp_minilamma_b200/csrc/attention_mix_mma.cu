@@ -4,16 +4,19 @@
 // A key's weight in head h needs the scores of all H heads at that key, so a block owns R query rows of one sequence with
 // all their heads and walks the window in runs of N keys.  Per run:
 //   1. S = q k^T by mma.sync: the 16 rows of a tile are R query rows of 16 / R heads of one key head's group; scores go to
-//      shared memory as float32.
-//   2. z = M S + b on the FMA pipe (two float32 FMAs an instruction), sigmoid, mask; weights go to shared memory as
-//      bfloat16.  A thread holds a few positions of a few output heads, so M is read as broadcasts.
-//   3. O += P V by mma.sync: a warp keeps up to TPW units of 16 rows x 64 value columns in registers for the whole walk.
+//      shared memory - for prompts as three bfloat16 planes that add up to all 24 bits of the float32 score.
+//   2. z = M S + b, sigmoid, mask; weights go to shared memory as bfloat16.  For prompts the mixing is three more mma.sync
+//      products (M is bfloat16, the planes are exact: a float32 product of float32 scores); for single tokens it is
+//      float32 FMAs, two an instruction.
+//   3. O += P V by mma.sync: a warp keeps TP x 16 rows x CP x 64 value columns in registers for the whole walk.
 // Nothing is normalised, so there is no running maximum and no rescaling, and context splits simply add up.
 // K and V of a run have one buffer each: the next run's keys load while 2 and 3 work, its values while 1 and 2 do.
 // Where the H x R rows' outputs exceed what one block's registers hold, grid y splits the output heads and every block
 // recomputes the scores.
 #include "attention_decode.cuh"
 #include "attention_mix.cuh"
+
+#include <type_traits>
 
 namespace mll {
 
@@ -25,10 +28,10 @@ struct MixMmaArgs {
   const int* seq_ctx;
   const int* seq_qstart;
   const int* seq_qlen;
-  const int* tile_seq;    // prompt tiles of 64 rows; null: single tokens, grid x runs over the sequences
+  const int* tile_seq;    // prompt tiles of 128 rows, walked from the back; null: single tokens, grid x runs over the sequences
   const int* tile_row0;
   const int* block_table;
-  const float* mix;       // [H, H] or null
+  const float* mix;       // [H, H] or null; prompts need entries that are bfloat16 values
   const float* bias;      // [H] or null
   __nv_bfloat16* out;
   float* part;            // [sequences, n_splits, H, dv] sums of the context's runs (n_splits > 1)
@@ -36,25 +39,28 @@ struct MixMmaArgs {
   float scale;
 };
 
-constexpr int MIX_WARPS = 8;
+constexpr int MIX_WARPS_PROMPT = 16, MIX_WARPS_SINGLE = 8;  // warps of a block
 
-// Shared memory of a block, in bytes from its start.  Rows of q and P are compact: row h * R + r.
+// Shared memory of a block, in bytes from its start.  Rows of q are compact: row h * R + r.  Scores and weights of head h
+// and row r begin at element h * ps + r * (N + 8): rows of 16-byte words of which neighbours - in a head, or of heads -
+// lie in different banks.
 struct MixMmaLayout {
-  int qs, vs, hp;                 // elements between rows of q / k and of v; heads rounded up to a multiple of 8
+  int qs, vs, ps, hp;             // elements between rows of q / k, of v, between heads of S / P; heads rounded up to 16
   int k, v, s, p, m, b, total;    // q starts at 0
 };
 __host__ __device__ inline MixMmaLayout mix_mma_layout(int H, int G, int d, int dv, int R, int N) {
   MixMmaLayout l;
   l.qs = ((d + 15) & ~15) + 8;
   l.vs = ((dv + 15) & ~15) + 8;
-  l.hp = (H + 7) & ~7;
+  l.ps = R * (N + 8) + (R > 1 ? 8 : 0);
+  l.hp = (H + 15) & ~15;
   int at = H * R * l.qs * 2;
   l.k = at; at += G * N * l.qs * 2;
   l.v = at; at += G * N * l.vs * 2;
-  l.s = at; at += H * R * (N + 8) * 4;
-  l.p = at; at += H * R * (N + 8) * 2;
+  l.s = at; at += R > 1 ? 3 * l.hp * l.ps * 2 : H * l.ps * 4;
+  l.p = at; at += l.hp * l.ps * 2;
   at = (at + 15) & ~15;
-  l.m = at; at += H * l.hp * 4;
+  l.m = at; at += R > 1 ? l.hp * (l.hp + 8) * 2 : H * l.hp * 4;
   l.b = at; at += l.hp * 4;
   l.total = at;
   return l;
@@ -74,32 +80,61 @@ __device__ __forceinline__ mix_f32x2 mix_fma2(mix_f32x2 a, mix_f32x2 b, mix_f32x
   asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
   return r;
 }
-// large |z|: e^-z overflows to infinity (weight 0) or falls to 0 (weight 1)
-__device__ __forceinline__ float mix_sigmoid(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+// sigmoid(z) from y = -z log2 e: 1 / (1 + 2^y); large |z|: 2^y overflows to infinity (weight 0) or falls to 0 (weight 1)
+__device__ __forceinline__ float mix_sigmoid(float y) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(y));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+  return r;
+}
+constexpr float MIX_LOG2E = 1.4426950408889634f;
 
-template <int R, int N, int TPW>
-__global__ void __launch_bounds__(MIX_WARPS * 32, TPW <= 2 ? 2 : 1) mixed_attention_mma_kernel(MixMmaArgs a) {
+// Shared memory by 32-bit address: the walk's inner loops add small offsets to a few bases.
+__device__ __forceinline__ void mix_ldsm(unsigned (&r)[4], unsigned at) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(at));
+}
+__device__ __forceinline__ void mix_ldsm_trans(unsigned (&r)[4], unsigned at) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(at));
+}
+__device__ __forceinline__ void mix_sts(unsigned at, unsigned v) {
+  asm volatile("st.shared.b32 [%0], %1;\n" ::"r"(at), "r"(v) : "memory");
+}
+__device__ __forceinline__ void mix_sts2(unsigned at, float x, float y) {
+  asm volatile("st.shared.v2.f32 [%0], {%1, %2};\n" ::"r"(at), "f"(x), "f"(y) : "memory");
+}
+__device__ __forceinline__ void mix_copy16(unsigned at, const void* src, bool valid) {
+  const int bytes = valid ? 16 : 0;  // fewer source bytes than 16: the rest is written as zero
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(at), "l"(src), "r"(bytes) : "memory");
+}
+
+template <int R, int N, int TP, int CP>
+__global__ void __launch_bounds__((R == 1 ? MIX_WARPS_SINGLE : MIX_WARPS_PROMPT) * 32, R == 1 ? 2 : 1)
+mixed_attention_mma_kernel(MixMmaArgs a) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
-  constexpr int THREADS = MIX_WARPS * 32;
+  constexpr int WARPS = R == 1 ? MIX_WARPS_SINGLE : MIX_WARPS_PROMPT, THREADS = WARPS * 32;
   constexpr int HPT = 16 / R;         // heads in the 16 rows of a tile
   constexpr int QP = R == 1 ? 1 : 2;  // tiles of one key head that share the key fragments in step 1
   constexpr int SS = N + 8;           // elements between rows of S and of P
   const int H = a.n_heads, G = a.n_kv_heads, group = H / G, d = a.d, dv = a.dv;
   const MixMmaLayout L = mix_mma_layout(H, G, d, dv, R, N);
   __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem_raw);
-  __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.k);
-  __nv_bfloat16* v_s = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.v);
   float* s_s = reinterpret_cast<float*>(smem_raw + L.s);
   __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.p);
-  float* m_s = reinterpret_cast<float*>(smem_raw + L.m);  // [H in][hp out], times scale
-  float* b_s = reinterpret_cast<float*>(smem_raw + L.b);
+  __nv_bfloat16* planes = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.s);  // R > 1: three of them, hp * ps elements each
+  float* m_s = reinterpret_cast<float*>(smem_raw + L.m);                     // R == 1: [H in][hp out], times -scale log2 e
+  __nv_bfloat16* mb_s = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.m);    // R > 1: [hp out][hp in + 8]
+  float* b_s = reinterpret_cast<float*>(smem_raw + L.b);                     // times -log2 e
 
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int tid = threadIdx.x, lane = tid & 31;
+  const int warp = __shfl_sync(0xffffffffu, tid >> 5, 0);  // the same register value in all lanes: branches on it are uniform
   const int g = lane >> 2, t = lane & 3;
   const bool single = a.tile_seq == nullptr;
-  constexpr int SUB = 64 / R;  // tiles of R rows in a listed tile of 64
-  const int seq = single ? blockIdx.x : a.tile_seq[blockIdx.x / SUB];
-  const int row0 = single ? 0 : a.tile_row0[blockIdx.x / SUB] + (int)(blockIdx.x % SUB) * R;
+  constexpr int SUB = 128 / R;  // tiles of R rows in a listed tile of 128
+  const int work = gridDim.x - 1 - blockIdx.x;  // from the back: the tiles with the most keys in front of them start first
+  const int seq = single ? blockIdx.x : a.tile_seq[work / SUB];
+  const int row0 = single ? 0 : a.tile_row0[work / SUB] + work % SUB * R;
   const int ctx = a.seq_ctx[seq], qlen = single ? 1 : a.seq_qlen[seq];
   const int rows = min(R, qlen - row0);
   if (rows <= 0) return;
@@ -114,177 +149,257 @@ __global__ void __launch_bounds__(MIX_WARPS * 32, TPW <= 2 ? 2 : 1) mixed_attent
     run_end = min(run_end, run + per);
   }
 
-  // the units (16 rows x 64 value columns) of this block and warp; neighbours share a key head where they can
-  const int tpg = (group + HPT - 1) / HPT;            // tiles of a key head
-  const int cps = (L.vs - 8 + 63) / 64;               // column parts of a value head
-  const int n_units = G * cps * tpg;
-  const int unit0 = (int)blockIdx.y * MIX_WARPS * TPW;
-  const int unit1 = min(n_units, unit0 + MIX_WARPS * TPW);
-  const int kv_lo = unit0 / (cps * tpg), kv_hi = (unit1 - 1) / (cps * tpg);
+  // the units of step 3 (TP tiles of 16 rows of one key head x CP x 64 value columns): one a warp
+  const int tpg = (group + HPT - 1) / HPT, tgs = (tpg + TP - 1) / TP;                  // tiles of a key head, groups of them
+  const int cgs = (L.vs - 8 + CP * 64 - 1) / (CP * 64);                                // column groups of a value head
+  const int unit0 = (int)blockIdx.y * WARPS, unit1 = min(G * cgs * tgs, unit0 + WARPS);
+  const int kv_lo = unit0 / (cgs * tgs), kv_hi = (unit1 - 1) / (cgs * tgs);
 
   const int kw = (L.qs - 8) >> 3, vw = (L.vs - 8) >> 3;  // 16-byte words of a padded row
-  auto load_run = [&](const __nv_bfloat16* cache, __nv_bfloat16* dst, int size, int stride, int words, int which) {
-    const int page = table[which * N / MLL_PAGE];
-    const int in_page = which * N % MLL_PAGE, valid = ctx - which * N;  // rows past the cached length hold no data
-    for (int i = tid; i < N * words; i += THREADS) {
-      const int r = i / words, c = (i - r * words) * 8;
-      const bool in = c < size && r < valid;
-      const __nv_bfloat16* src = cache + ((size_t)page * G * MLL_PAGE + in_page + r) * size + (in ? c : 0);
-      for (int h = 0; h < G; ++h)
-        cp_async16_zfill(dst + (size_t)(h * N + r) * stride + c, src + (size_t)h * MLL_PAGE * size, in);
-    }
+  // a thread's words of a run: the first (row, word) and the way to the next one
+  const int k_r = tid / kw, k_c = tid % kw * 8, v_r = tid / vw, v_c = tid % vw * 8;
+  const unsigned base = (unsigned)__cvta_generic_to_shared(smem_raw);
+  auto load_run = [&](const __nv_bfloat16* cache, unsigned dst, int size, int stride, int words, int r, int c, int which, int page) {
+    const int valid = ctx - which * N;  // rows past the cached length hold no data
+    const __nv_bfloat16* from = cache + (size_t)(page * G * MLL_PAGE + which * N % MLL_PAGE) * size;
+    const int head = MLL_PAGE * size, head_to = N * stride * 2;
+    auto column = [&](int row, int col) {  // the same word of every head
+      const bool in = col < size && row < valid;
+      const __nv_bfloat16* src = from + (in ? row * size + col : 0);
+      unsigned to = dst + (row * stride + col) * 2;
+      int h = 0;
+      for (; h + 4 <= G; h += 4) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) mix_copy16(to + i * head_to, src + (size_t)i * head, in);
+        src += (size_t)4 * head;
+        to += 4 * head_to;
+      }
+      for (; h < G; ++h, src += head, to += head_to) mix_copy16(to, src, in);
+    };
+    if (r < N) column(r, c);
+    if (N * words > THREADS)
+      for (int i = tid + THREADS; i < N * words; i += THREADS) column(i / words, i % words * 8);
   };
+  auto load_keys = [&](int which, int page) { load_run(a.k_cache, base + L.k, d, L.qs, kw, k_r, k_c, which, page); };
+  auto load_values = [&](int which, int page) { load_run(a.v_cache, base + L.v, dv, L.vs, vw, v_r, v_c, which, page); };
+  int page = run < run_end ? table[run * N / MLL_PAGE] : 0;  // of the run whose loads come next
   for (int i = tid; i < H * R * kw; i += THREADS) {
     const int row = i / kw, c = (i - row * kw) * 8, h = row / R, r = row % R;
     const bool in = c < d && r < rows;
     cp_async16_zfill(q_s + (size_t)row * L.qs + c, a.q + ((tok0 + (in ? r : 0)) * H + h) * d + (in ? c : 0), in);
   }
-  if (run < run_end) load_run(a.k_cache, k_s, d, L.qs, kw, run);
+  if (run < run_end) load_keys(run, page);
   cp_async_commit();
-  if (run < run_end) load_run(a.v_cache, v_s, dv, L.vs, vw, run);
+  if (run < run_end) load_values(run, page);
   cp_async_commit();
-  for (int i = tid; i < H * L.hp; i += THREADS) {
-    const int in = i / L.hp, to = i % L.hp;
-    m_s[i] = to < H ? (a.mix ? a.mix[(size_t)to * H + in] : (to == in ? 1.f : 0.f)) * a.scale : 0.f;
+  auto mix_at = [&](int to, int in) { return to >= H || in >= H ? 0.f : a.mix ? a.mix[(size_t)to * H + in] : (to == in ? 1.f : 0.f); };
+  if (R == 1) {
+    for (int i = tid; i < H * L.hp; i += THREADS) m_s[i] = mix_at(i % L.hp, i / L.hp) * (-MIX_LOG2E * a.scale);
+  } else {
+    for (int i = tid; i < L.hp * L.hp; i += THREADS) mb_s[i / L.hp * (L.hp + 8) + i % L.hp] = __float2bfloat16_rn(mix_at(i / L.hp, i % L.hp));
+    // heads that do not exist enter the products with a factor of 0: their scores must be numbers
+    for (int i = tid; i < 3 * (L.hp - H) * L.ps; i += THREADS)
+      planes[(size_t)(i / ((L.hp - H) * L.ps)) * L.hp * L.ps + (size_t)H * L.ps + i % ((L.hp - H) * L.ps)] = __float2bfloat16_rn(0.f);
   }
-  for (int i = tid; i < L.hp; i += THREADS) b_s[i] = (i < H && a.bias) ? a.bias[i] : 0.f;
+  for (int i = tid; i < L.hp; i += THREADS) b_s[i] = (i < H && a.bias) ? -MIX_LOG2E * a.bias[i] : 0.f;
 
-  float o[TPW][8][4];
+  float o[TP][CP][8][4];
 #pragma unroll
-  for (int j = 0; j < TPW; ++j)
-#pragma unroll
-    for (int n = 0; n < 8; ++n)
-#pragma unroll
-      for (int i = 0; i < 4; ++i) o[j][n][i] = 0.f;
+  for (int i = 0; i < TP * CP * 32; ++i) (&o[0][0][0][0])[i] = 0.f;
 
-  // step 1's units: QP tiles of one key head against N keys (or, where that leaves warps idle, half of them)
+  // the head that the tile's row rr stands for (rows past the group repeat its last head and are not stored)
+  auto head_of = [&](int kv, int tile, int rr) { return kv * group + min(tile * HPT + rr / R, group - 1); };
+  const int ld_row = (lane & 7) + (((lane >> 3) & 1) << 3), ld_col = (lane >> 4) << 3;  // ldmatrix: this lane's row and column
+
+  // step 3's unit of this warp: where the lane reads its rows of P and the values, how many of its columns exist (0: no unit)
+  const int unit = min(unit0 + warp, unit1 - 1), my_kv = unit / (cgs * tgs), my_col = unit / tgs % cgs * CP * 64, my_tile = unit % tgs * TP;
+  const int my_cols = unit0 + warp < unit1 ? min(CP * 64, L.vs - 8 - my_col) : 0;
+  unsigned p_at[TP];
+#pragma unroll
+  for (int i = 0; i < TP; ++i)
+    p_at[i] = base + L.p + (head_of(my_kv, min(my_tile + i, tpg - 1), ld_row) * L.ps + ld_row % R * SS + ld_col) * 2;
+  const unsigned v_at = base + L.v + ((my_kv * N + ld_row) * L.vs + my_col + ld_col) * 2;
+
+  // step 1's units: QP tiles of one key head against 16 keys.  Where the lane reads q and k and where its two rows of
+  // scores go (bytes from S's start; -1: nowhere)
   const int pairs = (tpg + QP - 1) / QP;
-  const int halves = (N == 32 && G * pairs * 2 <= MIX_WARPS) ? 2 : 1;
-  // row of q / P that the tile's row rr stands for (rows past the group repeat its last head and are not stored)
-  auto compact = [&](int kv, int tile, int rr) { return (kv * group + min(tile * HPT + rr / R, group - 1)) * R + rr % R; };
+  const int qk_units = G * pairs * (N / 16), plane = L.hp * L.ps * 2;
+  unsigned q_at[QP], k_at = 0;
+  int s_at[QP][2];
+  constexpr int SB = R == 1 ? 4 : 2;  // bytes of a score in S (R == 1), of one of its terms
+  auto set_qk = [&](int u) {
+    const int strip = u % (N / 16), pair = (u / (N / 16)) % pairs, kv = u / (N / 16 * pairs);
+    k_at = base + L.k + ((kv * N + strip * 16 + (lane & 7) + ((lane >> 4) << 3)) * L.qs + (((lane >> 3) & 1) << 3)) * 2;
+#pragma unroll
+    for (int m = 0; m < QP; ++m) {
+      const int tile = pair * QP + m;
+      q_at[m] = base + ((head_of(kv, min(tile, tpg - 1), ld_row) * R + ld_row % R) * L.qs + ld_col) * 2;
+#pragma unroll
+      for (int half8 = 0; half8 < 2; ++half8) {
+        const int rr = g + 8 * half8;
+        s_at[m][half8] = tile < tpg && tile * HPT + rr / R < group
+                             ? (head_of(kv, tile, rr) * L.ps + rr % R * SS + strip * 16 + 2 * t) * SB : -1;
+      }
+    }
+  };
+  set_qk(min(warp, qk_units - 1));
+  // step 3 of a run; `all`: every column of the unit exists
+  auto weigh_values = [&](auto all) {
+#pragma unroll
+    for (int ks = 0; ks < N / 16; ++ks) {
+      unsigned pf[TP][4];
+#pragma unroll
+      for (int i = 0; i < TP; ++i) mix_ldsm(pf[i], p_at[i] + ks * 32);
+      const unsigned v = v_at + ks * 32 * L.vs;
+#pragma unroll
+      for (int c = 0; c < CP; ++c)
+#pragma unroll
+        for (int np = 0; np < 4; ++np)
+          if (decltype(all)::value || c * 64 + np * 16 < my_cols) {
+            unsigned vf[4];
+            mix_ldsm_trans(vf, v + c * 128 + np * 32);
+#pragma unroll
+            for (int i = 0; i < TP; ++i) {
+              mma_16816(o[i][c][2 * np], pf[i], vf[0], vf[1]);
+              mma_16816(o[i][c][2 * np + 1], pf[i], vf[2], vf[3]);
+            }
+          }
+    }
+  };
+  const float neg_scale = -MIX_LOG2E * a.scale;
 
   cp_async_wait<1>();
   __syncthreads();
   for (; run < run_end; ++run) {
-    for (int u = warp; u < G * pairs * halves; u += MIX_WARPS) {
-      const int half = u % halves, pair = (u / halves) % pairs, kv = u / (halves * pairs);
-      const int np0 = half * (N / 16) / halves, np1 = (half + 1) * (N / 16) / halves;
-      float acc[QP][N / 8][4];
+    if (run + 1 < run_end) page = table[(run + 1) * N / MLL_PAGE];
+    for (int u = warp; u < qk_units; u += WARPS) {
+      if (qk_units > WARPS) set_qk(u);  // else the warp keeps the one it has
+      float acc[QP][2][4];
 #pragma unroll
       for (int m = 0; m < QP; ++m)
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int i = 0; i < 4; ++i) acc[m][n][i] = 0.f;
+#pragma unroll 4
+      for (int e = 0; e < (L.qs - 8) * 2; e += 32) {
+        unsigned qf[QP][4], kf[4];
+        mix_ldsm(kf, k_at + e);
+#pragma unroll
+        for (int m = 0; m < QP; ++m) mix_ldsm(qf[m], q_at[m] + e);
+#pragma unroll
+        for (int m = 0; m < QP; ++m) {
+          mma_16816(acc[m][0], qf[m], kf[0], kf[1]);
+          mma_16816(acc[m][1], qf[m], kf[2], kf[3]);
+        }
+      }
+#pragma unroll
+      for (int m = 0; m < QP; ++m)
+#pragma unroll
+        for (int half8 = 0; half8 < 2; ++half8) {
+          if (s_at[m][half8] < 0) continue;
+          const unsigned to = base + L.s + s_at[m][half8];
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            const float x = acc[m][n][2 * half8], y = acc[m][n][2 * half8 + 1];
+            if (R == 1) {
+              mix_sts2(to + n * 8 * SB, x, y);
+            } else {
+              const unsigned hi = pack_bf162(x, y);
+              const float2 h = unpack_bf162(hi);
+              const float rx = x - h.x, ry = y - h.y;  // exact
+              const unsigned mid = pack_bf162(rx, ry);
+              const float2 f = unpack_bf162(mid);
+              mix_sts(to + n * 8 * SB, hi);
+              mix_sts(to + n * 8 * SB + plane, mid);
+              mix_sts(to + n * 8 * SB + 2 * plane, pack_bf162(rx - f.x, ry - f.y));
+            }
+          }
+        }
+    }
+    __syncthreads();  // scores are there, this run's keys are done with
+    if (run + 1 < run_end) load_keys(run + 1, page);
+    cp_async_commit();
+
+    // step 2
+    if constexpr (R == 1) {
+      // one key x four output heads a thread
+      const int h_begin = kv_lo * group / 4, h_end = ((kv_hi + 1) * group + 3) / 4;
+      for (int item = tid; item < N * (h_end - h_begin); item += THREADS) {
+        const int key = item % N, hc = (h_begin + item / N) * 4;
+        mix_f32x2 z[2] = {mix_pack2(b_s[hc], b_s[hc + 1]), mix_pack2(b_s[hc + 2], b_s[hc + 3])};
+        const float* s = s_s + key;
+        const float* m = m_s + hc;
+#pragma unroll 8
+        for (int in = 0; in < H; ++in) {
+          const float sv = s[in * SS];
+          const ulonglong2 mv = *reinterpret_cast<const ulonglong2*>(m + in * L.hp);
+          const mix_f32x2 sd = mix_pack2(sv, sv);
+          z[0] = mix_fma2(sd, mv.x, z[0]);
+          z[1] = mix_fma2(sd, mv.y, z[1]);
+        }
+        const int kpos = run * N + key;
+        const bool ok = kpos <= pos0 && (a.window <= 0 || kpos > pos0 - a.window);
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          float lo, hi;
+          mix_unpack2(z[c], lo, hi);
+          p_s[(hc + 2 * c) * L.ps + key] = __float2bfloat16_rn(ok ? mix_sigmoid(lo) : 0.f);
+          p_s[(hc + 2 * c + 1) * L.ps + key] = __float2bfloat16_rn(ok ? mix_sigmoid(hi) : 0.f);
+        }
+      }
+    } else {
+      // a warp owns one row's keys x 16 output heads
+      const int mt0 = kv_lo * group / 16, mts = ((kv_hi + 1) * group + 15) / 16 - mt0;
+      const bool edge = rows < R || run * N + N - 1 > pos0 || (a.window > 0 && run * N <= last - a.window);
+      for (int item = warp; item < R * mts; item += WARPS) {
+        const int r = item % R, h = (mt0 + item / R) * 16;
+        float z[N / 8][4];
 #pragma unroll
         for (int n = 0; n < N / 8; ++n)
 #pragma unroll
-          for (int i = 0; i < 4; ++i) acc[m][n][i] = 0.f;
-      const __nv_bfloat16* qa[QP];
+          for (int i = 0; i < 4; ++i) z[n][i] = 0.f;
+        unsigned m = base + L.m + ((h + ld_row) * (L.hp + 8) + ld_col) * 2;
+        unsigned s = base + L.s + (ld_row * L.ps + r * SS + ld_col) * 2;
+        for (int kt = 0; kt < L.hp; kt += 16, m += 32, s += L.ps * 32) {
+          unsigned mf[4];
+          mix_ldsm(mf, m);
 #pragma unroll
-      for (int m = 0; m < QP; ++m)
-        qa[m] = q_s + (size_t)compact(kv, min(pair * QP + m, tpg - 1), (lane & 7) + (((lane >> 3) & 1) << 3)) * L.qs + ((lane >> 4) << 3);
-      const __nv_bfloat16* kb = k_s + (size_t)(kv * N + (lane & 7) + ((lane >> 4) << 3)) * L.qs + (((lane >> 3) & 1) << 3);
-#pragma unroll 4
-      for (int e = 0; e < L.qs - 8; e += 16) {
-        unsigned qf[QP][4];
+          for (int p = 2; p >= 0; --p) {
+            unsigned sf[N / 16][4];
 #pragma unroll
-        for (int m = 0; m < QP; ++m) ldmatrix_x4(qf[m], qa[m] + e);
+            for (int n = 0; n < N / 16; ++n) mix_ldsm_trans(sf[n], s + p * plane + n * 32);
 #pragma unroll
-        for (int np = 0; np < N / 16; ++np) {
-          if (np < np0 || np >= np1) continue;
-          unsigned kf[4];
-          ldmatrix_x4(kf, kb + (size_t)np * 16 * L.qs + e);
-#pragma unroll
-          for (int m = 0; m < QP; ++m) {
-            mma_16816(acc[m][2 * np], qf[m], kf[0], kf[1]);
-            mma_16816(acc[m][2 * np + 1], qf[m], kf[2], kf[3]);
+            for (int n = 0; n < N / 16; ++n) {
+              mma_16816(z[2 * n], mf, sf[n][0], sf[n][1]);
+              mma_16816(z[2 * n + 1], mf, sf[n][2], sf[n][3]);
+            }
           }
         }
-      }
+        const float b0 = b_s[h + g], b1 = b_s[h + g + 8];
+        const unsigned to = base + L.p + ((h + g) * L.ps + r * SS + 2 * t) * 2, to8 = to + 16 * L.ps;
 #pragma unroll
-      for (int m = 0; m < QP; ++m) {
-        const int tile = pair * QP + m;
-        if (tile >= tpg) continue;
-#pragma unroll
-        for (int half8 = 0; half8 < 2; ++half8) {
-          const int rr = g + 8 * half8;
-          if (tile * HPT + rr / R >= group) continue;
-          float* dst = s_s + (size_t)compact(kv, tile, rr) * SS + 2 * t;
+        for (int n = 0; n < N / 8; ++n) {
+          z[n][0] = mix_sigmoid(fmaf(z[n][0], neg_scale, b0));
+          z[n][1] = mix_sigmoid(fmaf(z[n][1], neg_scale, b0));
+          z[n][2] = mix_sigmoid(fmaf(z[n][2], neg_scale, b1));
+          z[n][3] = mix_sigmoid(fmaf(z[n][3], neg_scale, b1));
+        }
+        if (edge) {  // the run meets the diagonal, the window's far edge or a row that does not exist
+          const int qpos = pos0 + r, kpos = run * N + 2 * t;
+          const int lo = a.window > 0 ? qpos - a.window + 1 : 0, hi = r < rows ? qpos : -1;
 #pragma unroll
           for (int n = 0; n < N / 8; ++n)
-            if (n >= 2 * np0 && n < 2 * np1)
-              *reinterpret_cast<float2*>(dst + n * 8) = make_float2(acc[m][n][2 * half8], acc[m][n][2 * half8 + 1]);
-        }
-      }
-    }
-    __syncthreads();  // scores are there, this run's keys are done with
-    if (run + 1 < run_end) load_run(a.k_cache, k_s, d, L.qs, kw, run + 1);
-    cp_async_commit();
-
-    // step 2: PK positions (neighbouring keys of one row) x HC output heads a thread
-    constexpr int PK = R == 1 ? 1 : 4, HC = R == 1 ? 4 : 8;
-    const int h_begin = kv_lo * group / HC, h_end = ((kv_hi + 1) * group + HC - 1) / HC;
-    constexpr int POS = R * N / PK;
-    for (int item = tid; item < POS * (h_end - h_begin); item += THREADS) {
-      const int at = item % POS, hc = (h_begin + item / POS) * HC;
-      const int r = at / (N / PK), key = (at % (N / PK)) * PK;
-      mix_f32x2 z[PK][HC / 2];
 #pragma unroll
-      for (int c = 0; c < HC / 2; ++c) {
-        const mix_f32x2 b = mix_pack2(b_s[hc + 2 * c], b_s[hc + 2 * c + 1]);
-#pragma unroll
-        for (int k = 0; k < PK; ++k) z[k][c] = b;
-      }
-      const float* s = s_s + (size_t)r * SS + key;
-      const float* m = m_s + hc;
-#pragma unroll 4
-      for (int in = 0; in < H; ++in) {
-        float sv[PK];
-        if (PK == 4) {
-          const float4 v = *reinterpret_cast<const float4*>(s + (size_t)in * R * SS);
-          sv[0] = v.x; sv[1 % PK] = v.y; sv[2 % PK] = v.z; sv[3 % PK] = v.w;
-        } else {
-          sv[0] = s[(size_t)in * R * SS];
-        }
-        mix_f32x2 mv[HC / 2];
-#pragma unroll
-        for (int c = 0; c < HC / 4; ++c) {
-          const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(m + in * L.hp + 4 * c);
-          mv[2 * c] = v.x;
-          mv[2 * c + 1] = v.y;
+            for (int i = 0; i < 4; ++i) {
+              const int k = kpos + 8 * n + (i & 1);
+              if (k < lo || k > hi) z[n][i] = 0.f;
+            }
         }
 #pragma unroll
-        for (int k = 0; k < PK; ++k) {
-          const mix_f32x2 sd = mix_pack2(sv[k], sv[k]);
-#pragma unroll
-          for (int c = 0; c < HC / 2; ++c) z[k][c] = mix_fma2(sd, mv[c], z[k][c]);
-        }
-      }
-      const int qpos = pos0 + r, kpos = run * N + key;
-      bool ok[PK];
-#pragma unroll
-      for (int k = 0; k < PK; ++k)
-        ok[k] = r < rows && kpos + k <= qpos && (a.window <= 0 || kpos + k > qpos - a.window);
-#pragma unroll
-      for (int c = 0; c < HC / 2; ++c) {
-        float w[2][PK];
-#pragma unroll
-        for (int k = 0; k < PK; ++k) {
-          float lo, hi;
-          mix_unpack2(z[k][c], lo, hi);
-          w[0][k] = ok[k] ? mix_sigmoid(lo) : 0.f;
-          w[1][k] = ok[k] ? mix_sigmoid(hi) : 0.f;
-        }
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int h = hc + 2 * c + e;
-          if (h >= H) continue;
-          __nv_bfloat16* dst = p_s + (size_t)(h * R + r) * SS + key;
-          if (PK == 4) {
-            uint2 v;
-            v.x = pack_bf162(w[e][0], w[e][1 % PK]);
-            v.y = pack_bf162(w[e][2 % PK], w[e][3 % PK]);
-            *reinterpret_cast<uint2*>(dst) = v;
-          } else {
-            *dst = __float2bfloat16_rn(w[e][0]);
-          }
+        for (int n = 0; n < N / 8; ++n) {
+          mix_sts(to + 16 * n, pack_bf162(z[n][0], z[n][1]));
+          mix_sts(to8 + 16 * n, pack_bf162(z[n][2], z[n][3]));
         }
       }
     }
@@ -292,64 +407,37 @@ __global__ void __launch_bounds__(MIX_WARPS * 32, TPW <= 2 ? 2 : 1) mixed_attent
     __syncthreads();
 
     // step 3
-#pragma unroll
-    for (int ks = 0; ks < N / 16; ++ks) {
-      unsigned pf[TPW][4];
-#pragma unroll
-      for (int j = 0; j < TPW; ++j) {
-        const int u = min(unit0 + warp * TPW + j, n_units - 1);
-        const int kv = u / (cps * tpg), tile = u % tpg;
-        ldmatrix_x4(pf[j], p_s + (size_t)compact(kv, tile, (lane & 7) + (((lane >> 3) & 1) << 3)) * SS + ks * 16 + ((lane >> 4) << 3));
-      }
-#pragma unroll
-      for (int np = 0; np < 4; ++np) {
-        unsigned vf[4];
-        int held = -1;
-#pragma unroll
-        for (int j = 0; j < TPW; ++j) {
-          const int u = unit0 + warp * TPW + j;
-          if (u >= unit1) continue;
-          const int kc = u / tpg, kv = kc / cps, col = (kc % cps) * 64 + np * 16;
-          if (col >= L.vs - 8) continue;
-          if (kc != held) {
-            ldmatrix_x4_trans(vf, v_s + (size_t)(kv * N + ks * 16 + (lane & 7) + (((lane >> 3) & 1) << 3)) * L.vs + col + ((lane >> 4) << 3));
-            held = kc;
-          }
-          mma_16816(o[j][2 * np], pf[j], vf[0], vf[1]);
-          mma_16816(o[j][2 * np + 1], pf[j], vf[2], vf[3]);
-        }
-      }
-    }
+    if (my_cols == CP * 64)
+      weigh_values(std::true_type{});
+    else if (my_cols > 0)
+      weigh_values(std::false_type{});
     cp_async_wait<0>();  // the next run's keys
     __syncthreads();     // this run's values, weights and scores are done with
-    if (run + 1 < run_end) load_run(a.v_cache, v_s, dv, L.vs, vw, run + 1);
+    if (run + 1 < run_end) load_values(run + 1, page);
     cp_async_commit();
   }
   cp_async_wait<0>();
 
 #pragma unroll
-  for (int j = 0; j < TPW; ++j) {
-    const int u = unit0 + warp * TPW + j;
-    if (u >= unit1) continue;
-    const int kc = u / tpg, kv = kc / cps, tile = u % tpg;
+  for (int i = 0; i < TP; ++i)
 #pragma unroll
     for (int half8 = 0; half8 < 2; ++half8) {
-      const int rr = g + 8 * half8, r = rr % R;
+      const int rr = g + 8 * half8, r = rr % R, tile = my_tile + i;
       if (tile * HPT + rr / R >= group || r >= rows) continue;
-      const int h = kv * group + tile * HPT + rr / R;
+      const int h = my_kv * group + tile * HPT + rr / R;
 #pragma unroll
-      for (int n = 0; n < 8; ++n) {
-        const int col = (kc % cps) * 64 + n * 8 + 2 * t;
-        if (col >= dv) continue;  // dv is even: a pair is inside or outside as a whole
-        if (a.n_splits > 1)
-          *reinterpret_cast<float2*>(a.part + (((size_t)seq * a.n_splits + blockIdx.z) * H + h) * dv + col) =
-              make_float2(o[j][n][2 * half8], o[j][n][2 * half8 + 1]);
-        else
-          *reinterpret_cast<__nv_bfloat162*>(a.out + ((tok0 + r) * H + h) * dv + col) =
-              __floats2bfloat162_rn(o[j][n][2 * half8], o[j][n][2 * half8 + 1]);
-      }
+      for (int c = 0; c < CP; ++c)
+#pragma unroll
+        for (int n = 0; n < 8; ++n) {
+          const int col = c * 64 + n * 8 + 2 * t;
+          if (col >= my_cols || my_col + col >= dv) continue;  // dv is even: a pair is inside or outside as a whole
+          const float x = o[i][c][n][2 * half8], y = o[i][c][n][2 * half8 + 1];
+          if (a.n_splits > 1)
+            *reinterpret_cast<float2*>(a.part + (((size_t)seq * a.n_splits + blockIdx.z) * H + h) * dv + my_col + col) = make_float2(x, y);
+          else
+            *reinterpret_cast<__nv_bfloat162*>(a.out + ((tok0 + r) * H + h) * dv + my_col + col) = __floats2bfloat162_rn(x, y);
+        }
     }
-  }
 }
 
 // out[sequence's token] = the sum of its context splits, in split order; a thread owns a pair of columns
@@ -371,9 +459,9 @@ __global__ void __launch_bounds__(256) mixed_attention_sum_kernel(const float* _
 
 constexpr int MIX_SMEM_MAX = 227 * 1024;
 
-inline int mix_units(int H, int G, int dv, int R) {
+inline int mix_units(int H, int G, int dv, int R, int TP, int CP) {
   const int group = H / G, tpg = (group + 16 / R - 1) / (16 / R);
-  return G * tpg * ((((dv + 15) & ~15) + 63) / 64);
+  return G * ((tpg + TP - 1) / TP) * ((((dv + 15) & ~15) + CP * 64 - 1) / (CP * 64));
 }
 
 // Rows and keys per run of a launch: R * 256 + N, or 0 where shared memory holds no combination.
@@ -383,7 +471,7 @@ inline int mix_mma_shape(int single, int H, int G, int d, int dv) {
     if (fits(1, 32, MIX_SMEM_MAX / 2 - 1024)) return 256 + 32;  // two blocks a multiprocessor
     return fits(1, 16, MIX_SMEM_MAX) ? 256 + 16 : 0;
   }
-  if (mix_units(H, G, dv, 16) <= 4 * MIX_WARPS) {
+  if (mix_units(H, G, dv, 16, 2, 1) <= MIX_WARPS_PROMPT) {
     if (fits(16, 32, MIX_SMEM_MAX)) return 16 * 256 + 32;
     if (fits(16, 16, MIX_SMEM_MAX)) return 16 * 256 + 16;
   }
@@ -393,18 +481,19 @@ inline int mix_mma_shape(int single, int H, int G, int d, int dv) {
   return 0;
 }
 
-template <int R, int N, int TPW>
+template <int R, int N, int TP, int CP>
 int launch_mixed_mma(const MixMmaArgs& a, int n_blocks, cudaStream_t stream) {
   const int smem = mix_mma_layout(a.n_heads, a.n_kv_heads, a.d, a.dv, R, N).total;
-  auto kernel = mixed_attention_mma_kernel<R, N, TPW>;
+  auto kernel = mixed_attention_mma_kernel<R, N, TP, CP>;
   cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (err != cudaSuccess) {
     mll_set_error("mixed attention (mma): cannot reserve %d bytes of shared memory: %s", smem, cudaGetErrorString(err));
     return (int)err;
   }
-  const int units = mix_units(a.n_heads, a.n_kv_heads, a.dv, R);
-  const dim3 grid(n_blocks, (units + MIX_WARPS * TPW - 1) / (MIX_WARPS * TPW), a.n_splits);
-  MLL_LAUNCH((kernel), grid, MIX_WARPS * 32, smem, stream, a);
+  constexpr int WARPS = R == 1 ? MIX_WARPS_SINGLE : MIX_WARPS_PROMPT;
+  const int units = mix_units(a.n_heads, a.n_kv_heads, a.dv, R, TP, CP);
+  const dim3 grid(n_blocks, (units + WARPS - 1) / WARPS, a.n_splits);
+  MLL_LAUNCH((kernel), grid, WARPS * 32, smem, stream, a);
   MLL_LAUNCH_CHECK();
   return 0;
 }
@@ -416,7 +505,8 @@ MLL_API int mll_mixed_attention_mma_supported(int dtype, int single, int n_heads
          n_heads % n_kv_heads == 0 && mll::mix_mma_shape(single, n_heads, n_kv_heads, d, dv) != 0;
 }
 
-// tile_seq / tile_row0: tiles of up to 64 query rows as (sequence, first row among the sequence's new tokens), n_tiles of
+// mix: float32; for prompts its entries must be bfloat16 values (the kernel takes them as such).
+// tile_seq / tile_row0: tiles of up to 128 query rows as (sequence, first row among the sequence's new tokens), n_tiles of
 // them; null: every sequence brings one token and n_tiles is the number of sequences.  n_splits > 1 (single tokens only)
 // cuts every context into that many runs and needs scratch: n_tiles * n_splits * H * dv floats.
 MLL_API int mll_mixed_attention_mma(const void* q, const void* k_cache, const void* v_cache, const int* seq_slot,
@@ -435,19 +525,16 @@ MLL_API int mll_mixed_attention_mma(const void* q, const void* k_cache, const vo
                     seq_qstart, seq_qlen, tile_seq, tile_row0, block_table, mix, bias, (__nv_bfloat16*)out, scratch,
                     n_heads, n_kv_heads, d, dv, window, max_blocks, n_splits, scale};
   const int shape = mll::mix_mma_shape(single, n_heads, n_kv_heads, d, dv), R = shape / 256, N = shape % 256;
-  const int units = mll::mix_units(n_heads, n_kv_heads, dv, R);
   int code;
   if (R == 1) {
-    if (units <= mll::MIX_WARPS)
-      code = N == 32 ? mll::launch_mixed_mma<1, 32, 1>(a, n_tiles, stream) : mll::launch_mixed_mma<1, 16, 1>(a, n_tiles, stream);
+    if (mll::mix_units(n_heads, n_kv_heads, dv, 1, 1, 1) <= mll::MIX_WARPS_SINGLE)
+      code = N == 32 ? mll::launch_mixed_mma<1, 32, 1, 1>(a, n_tiles, stream) : mll::launch_mixed_mma<1, 16, 1, 1>(a, n_tiles, stream);
     else
-      code = N == 32 ? mll::launch_mixed_mma<1, 32, 2>(a, n_tiles, stream) : mll::launch_mixed_mma<1, 16, 2>(a, n_tiles, stream);
+      code = N == 32 ? mll::launch_mixed_mma<1, 32, 1, 2>(a, n_tiles, stream) : mll::launch_mixed_mma<1, 16, 1, 2>(a, n_tiles, stream);
   } else if (R == 8) {
-    code = N == 32 ? mll::launch_mixed_mma<8, 32, 4>(a, n_tiles * 8, stream) : mll::launch_mixed_mma<8, 16, 4>(a, n_tiles * 8, stream);
-  } else if (units <= 2 * mll::MIX_WARPS) {
-    code = N == 32 ? mll::launch_mixed_mma<16, 32, 2>(a, n_tiles * 4, stream) : mll::launch_mixed_mma<16, 16, 2>(a, n_tiles * 4, stream);
+    code = N == 32 ? mll::launch_mixed_mma<8, 32, 2, 1>(a, n_tiles * 16, stream) : mll::launch_mixed_mma<8, 16, 2, 1>(a, n_tiles * 16, stream);
   } else {
-    code = N == 32 ? mll::launch_mixed_mma<16, 32, 4>(a, n_tiles * 4, stream) : mll::launch_mixed_mma<16, 16, 4>(a, n_tiles * 4, stream);
+    code = N == 32 ? mll::launch_mixed_mma<16, 32, 2, 1>(a, n_tiles * 8, stream) : mll::launch_mixed_mma<16, 16, 2, 1>(a, n_tiles * 8, stream);
   }
   if (code != 0 || n_splits == 1) return code;
   const long long items = (long long)n_tiles * (n_heads * dv / 2);

@@ -1589,8 +1589,9 @@ def _mixed_mma(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_qlen, til
 
 def mixed_attention_tiles(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_qlen, tile_seq, tile_row0, block_table,
                           mix, bias, out, n_heads: int, n_kv_heads: int, d: int, dv: int, window: int, scale: float) -> None:
-    """`mixed_attention` for prompt steps in bfloat16 on tensor cores: the work is a list of tiles of up to PREFILL_TILE
-    query rows, (sequence, first row among the sequence's new tokens)."""
+    """`mixed_attention` for prompt steps in bfloat16 on tensor cores: the work is a list of tiles of up to twice
+    PREFILL_TILE query rows, (sequence, first row among the sequence's new tokens), walked from its end.  `mix` must hold
+    bfloat16 values (in float32): the scores pass it as exact sums of bfloat16 terms."""
     for name, t in (("tile_seq", tile_seq), ("tile_row0", tile_row0)):
         _need(t, f"mixed attention {name}", torch.int32, 1)
     if tile_seq.shape != tile_row0.shape:

@@ -10,7 +10,7 @@
 //
 // Kernels (each for prompts and single tokens alike; a step's tokens of one sequence are consecutive rows):
 //   * lru_gates       decay and write (sqrt(1 - decay^2) i u) of every token and channel.  A block owns a tile of tokens
-//                     and 64 channels of one diagonal block; it forms u for the tile's tokens and the whole diagonal
+//                     and channels of one diagonal block; it forms u for the tile's tokens and the whole diagonal
 //                     block in shared memory and multiplies.  Two versions: float32 FMAs (any block size, either dtype),
 //                     and mma.sync for bfloat16 matrices: u is cut into three bfloat16 terms that add up to all 24 bits
 //                     of its float32 value, so the products are those of the float32 u, accumulated in float32.
@@ -116,77 +116,148 @@ __global__ void __launch_bounds__(256) lru_gates_kernel(LruArgs a) {
     if (q0 + i < n) lru_finish<T>(a, t0 + q0 + i, block * bs + col, r[i], z[i], u_s[(q0 + i) * bs + col]);
 }
 
-// grid (ceil(tokens / (16 MT)), n * ceil(bs / 64)), 256 threads.  Warp w owns channels 8w .. 8w + 7 of the 64 and both
-// gates of them, so that a thread ends with r and i of the same four (token, channel) pairs per 16 tokens.
-// Shared memory: three bfloat16 planes [3][16 MT][row] of u (high, middle, low term).  The k-order inside a product is
-// free as long as both operands agree: a thread's 16 bytes (eight neighbouring inputs) serve two k-steps.
-template <int MT>
-__global__ void __launch_bounds__(256) lru_gates_mma_kernel(LruArgs a, int row) {
+// grid (ceil(tokens / M), n * column parts), 256 threads; M = 16 WM MT tokens.  A block forms u for its tokens and one
+// whole diagonal block in shared memory - three bfloat16 planes [3][M][row] (high, middle, low term) - and walks `passes`
+// runs of 64 channels of it.  Warps: WM along the tokens, 8 / WM along the channels; a warp owns MT x 16 tokens and NT x 8
+// channels of both gates, so that a thread ends with r and i of the same (token, channel) pairs.
+// The k-order inside a product is free as long as both operands agree: a thread's 16 bytes (eight neighbouring inputs)
+// serve two k-steps.
+template <int WM, int MT, int NT>
+__global__ void __launch_bounds__(256) lru_gates_mma_kernel(LruArgs a, int row, int passes) {
   extern __shared__ __align__(16) __nv_bfloat16 planes[];
-  constexpr int M = 16 * MT;
-  const int bs = a.width / a.blocks, tiles = (bs + 63) / 64;
-  const int block = blockIdx.y / tiles, c0 = (blockIdx.y % tiles) * 64;
+  constexpr int M = 16 * WM * MT;
+  static_assert(8 / WM * NT * 8 == 64, "a pass covers 64 channels");
+  __shared__ int pos_s[M], back_s[M];           // a token's position; how many of its inputs lie in this step
+  __shared__ const float* state_s[M];           // where its sequence's earlier inputs are
+  const int bs = a.width / a.blocks, tiles = (bs + 63) / 64, parts = (tiles + passes - 1) / passes;
+  const int block = blockIdx.y / parts, tile0 = (blockIdx.y % parts) * passes, tile1 = min(tiles, tile0 + passes);
   const int t0 = blockIdx.x * M, n = min(M, a.n_tokens - t0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3;
   const int k_pad = (bs + 31) & ~31;
-  for (int i = threadIdx.x; i < M * k_pad; i += 256) {
-    const int m = i / k_pad, k = i % k_pad;
-    float u = 0.f;
-    if (m < n && k < bs) {
-      const int t = t0 + m, seq = a.tok_seq[t];
-      u = lru_conv<__nv_bfloat16>(a, t, block * bs + k, a.tok_pos[t], t - a.seq_qstart[seq],
-                                  a.conv_state + (size_t)a.seq_slot[seq] * (a.taps - 1) * a.width);
-    }
-    const __nv_bfloat16 hi = __float2bfloat16_rn(u);
-    const float rest = u - __bfloat162float(hi);          // exact
-    const __nv_bfloat16 mid = __float2bfloat16_rn(rest);
-    planes[(size_t)m * row + k] = hi;
-    planes[(size_t)(M + m) * row + k] = mid;
-    planes[(size_t)(2 * M + m) * row + k] = __float2bfloat16_rn(rest - __bfloat162float(mid));
+  if (threadIdx.x < M && threadIdx.x < n) {
+    const int t = t0 + threadIdx.x, seq = a.tok_seq[t];
+    pos_s[threadIdx.x] = a.tok_pos[t];
+    back_s[threadIdx.x] = t - a.seq_qstart[seq];
+    state_s[threadIdx.x] = a.conv_state + (size_t)a.seq_slot[seq] * (a.taps - 1) * a.width;
   }
   __syncthreads();
-  float acc[2][MT][4];
+  // u: a thread owns a pair of channels and every (256 / pairs)-th token
+  const __nv_bfloat16* proj = (const __nv_bfloat16*)a.proj;
+  const int pairs = k_pad / 2;
+  for (int p = threadIdx.x % min(pairs, 256); p < pairs; p += 256) {
+    const int k = 2 * p, c = block * bs + k;
+    const bool real = k < bs;  // bs is even: both channels or none
+    const float2 xb = real ? make_float2(a.x_bias[c], a.x_bias[c + 1]) : make_float2(0.f, 0.f);
+    const float2 cb = real ? make_float2(a.conv_b[c], a.conv_b[c + 1]) : make_float2(0.f, 0.f);
+    const float* w = a.conv_w + (size_t)c * a.taps + a.taps - 1;
+    float2 w4[4];  // the taps of the last four inputs stay in registers
 #pragma unroll
-  for (int e = 0; e < 2; ++e)
+    for (int i = 0; i < 4; ++i) w4[i] = real && i < a.taps ? make_float2(w[-i], w[a.taps - i]) : make_float2(0.f, 0.f);
+    const int step = pairs >= 256 ? 1 : 256 / pairs;
+    if (pairs < 256 && threadIdx.x >= step * pairs) break;
+#pragma unroll 4
+    for (int m = pairs >= 256 ? 0 : threadIdx.x / pairs; m < M; m += step) {
+      float2 u = make_float2(0.f, 0.f);
+      if (real && m < n) {
+        u = cb;
+        const int local = back_s[m], reach = min(a.taps - 1, pos_s[m]);  // nothing before the sequence, not even the bias
+        const __nv_bfloat16* x0 = proj + (size_t)(t0 + m) * a.ld + a.x_col + c;
+        const float* s0 = state_s[m] + (size_t)(local + a.taps - 1) * a.width + c;
+        auto input = [&](int back) {
+          if (back <= local)
+            return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(x0 - (size_t)back * a.ld));
+          return make_float2(s0[-(ptrdiff_t)back * a.width], s0[1 - (ptrdiff_t)back * a.width]);
+        };
+        float2 x[4];
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
+        for (int back = 0; back < 4; ++back)
+          if (back <= reach) x[back] = input(back);
 #pragma unroll
-      for (int i = 0; i < 4; ++i) acc[e][m][i] = 0.f;
-  const int col = c0 + warp * 8 + g;  // this thread's row of the two matrices
-  const __nv_bfloat16* w = (const __nv_bfloat16*)a.gate_w + (size_t)block * 2 * bs * bs;
-  const uint4* wr = reinterpret_cast<const uint4*>(w + (size_t)min(col, bs - 1) * bs);
-  const uint4* wi = reinterpret_cast<const uint4*>(w + (size_t)(bs + min(col, bs - 1)) * bs);
-  const uint4 zero = make_uint4(0, 0, 0, 0);
-#pragma unroll 2
-  for (int k = 0; k < k_pad; k += 32) {
-    const bool in = k + 8 * q < bs && col < bs;  // bs is a multiple of 8: eight inputs are inside or outside together
-    const uint4 b[2] = {in ? wr[(k >> 3) + q] : zero, in ? wi[(k >> 3) + q] : zero};
-#pragma unroll
-    for (int p = 0; p < 3; ++p) {
-#pragma unroll
-      for (int m = 0; m < MT; ++m) {
-        const uint4 lo = *reinterpret_cast<const uint4*>(planes + (size_t)(p * M + m * 16 + g) * row + k + 8 * q);
-        const uint4 up = *reinterpret_cast<const uint4*>(planes + (size_t)(p * M + m * 16 + g + 8) * row + k + 8 * q);
-        const unsigned a0[4] = {lo.x, up.x, lo.y, up.y}, a1[4] = {lo.z, up.z, lo.w, up.w};
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          mma_16816(acc[e][m], a0, b[e].x, b[e].y);
-          mma_16816(acc[e][m], a1, b[e].z, b[e].w);
+        for (int back = 0; back < 4; ++back)
+          if (back <= reach) {
+            u.x = fmaf(w4[back].x, x[back].x + xb.x, u.x);
+            u.y = fmaf(w4[back].y, x[back].y + xb.y, u.y);
+          }
+        for (int back = 4; back <= reach; ++back) {
+          const float2 v = input(back);
+          u.x = fmaf(w[-back], v.x + xb.x, u.x);
+          u.y = fmaf(w[a.taps - back], v.y + xb.y, u.y);
         }
       }
+      const __nv_bfloat162 hi = __floats2bfloat162_rn(u.x, u.y);
+      const float2 h = __bfloat1622float2(hi);
+      const float2 rest = make_float2(u.x - h.x, u.y - h.y);  // exact
+      const __nv_bfloat162 mid = __floats2bfloat162_rn(rest.x, rest.y);
+      const float2 f = __bfloat1622float2(mid);
+      *reinterpret_cast<__nv_bfloat162*>(planes + (size_t)m * row + k) = hi;
+      *reinterpret_cast<__nv_bfloat162*>(planes + (size_t)(M + m) * row + k) = mid;
+      *reinterpret_cast<__nv_bfloat162*>(planes + (size_t)(2 * M + m) * row + k) = __floats2bfloat162_rn(rest.x - f.x, rest.y - f.y);
     }
   }
+  __syncthreads();
+  const int m0 = (warp % WM) * MT * 16, n0 = (warp / WM) * NT * 8;
+  const __nv_bfloat16* w = (const __nv_bfloat16*)a.gate_w + (size_t)block * 2 * bs * bs;
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  for (int tile = tile0; tile < tile1; ++tile) {
+    const int c0 = tile * 64 + n0;
+    if (c0 >= bs) break;
+    float acc[2][NT][MT][4];
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
+    for (int e = 0; e < 2; ++e)
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int tok = m * 16 + g + 8 * (i >> 1), c = c0 + warp * 8 + 2 * q + (i & 1);
-      if (tok < n && c < bs) {
-        const float u = __bfloat162float(planes[(size_t)tok * row + c]) + __bfloat162float(planes[(size_t)(M + tok) * row + c]) +
-                        __bfloat162float(planes[(size_t)(2 * M + tok) * row + c]);
-        lru_finish<__nv_bfloat16>(a, t0 + tok, block * bs + c, acc[0][m][i], acc[1][m][i], u);
-      }
+      for (int j = 0; j < NT; ++j)
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+          for (int i = 0; i < 4; ++i) acc[e][j][m][i] = 0.f;
+    const uint4* rows[2][NT];  // this lane's rows of the two matrices
+    bool have[NT];
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      const int col = min(c0 + 8 * j + g, bs - 1);
+      have[j] = c0 + 8 * j + g < bs;
+      rows[0][j] = reinterpret_cast<const uint4*>(w + (size_t)col * bs) + q;
+      rows[1][j] = reinterpret_cast<const uint4*>(w + (size_t)(bs + col) * bs) + q;
     }
+#pragma unroll 4
+    for (int k = 0; k < k_pad; k += 32) {
+      const bool in = k + 8 * q < bs;  // bs is a multiple of 8: eight inputs are inside or outside together
+      uint4 b[2][NT];
+#pragma unroll
+      for (int e = 0; e < 2; ++e)
+#pragma unroll
+        for (int j = 0; j < NT; ++j) b[e][j] = in && have[j] ? rows[e][j][k >> 3] : zero;
+#pragma unroll
+      for (int p = 0; p < 3; ++p)
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          const __nv_bfloat16* src = planes + (size_t)(p * M + m0 + m * 16 + g) * row + k + 8 * q;
+          const uint4 lo = *reinterpret_cast<const uint4*>(src);
+          const uint4 up = *reinterpret_cast<const uint4*>(src + 8 * row);
+          const unsigned a0[4] = {lo.x, up.x, lo.y, up.y}, a1[4] = {lo.z, up.z, lo.w, up.w};
+#pragma unroll
+          for (int e = 0; e < 2; ++e)
+#pragma unroll
+            for (int j = 0; j < NT; ++j) {
+              mma_16816(acc[e][j][m], a0, b[e][j].x, b[e][j].y);
+              mma_16816(acc[e][j][m], a1, b[e][j].z, b[e][j].w);
+            }
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int tok = m0 + m * 16 + g + 8 * (i >> 1), c = c0 + 8 * j + 2 * q + (i & 1);
+          if (tok < n && c < bs) {
+            const __nv_bfloat16* src = planes + (size_t)tok * row + c;
+            const float u = (__bfloat162float(src[0]) + __bfloat162float(src[(size_t)M * row])) + __bfloat162float(src[(size_t)2 * M * row]);
+            lru_finish<__nv_bfloat16>(a, t0 + tok, block * bs + c, acc[0][j][m][i], acc[1][j][m][i], u);
+          }
+        }
+  }
 }
 
 // grid (ceil(width / 32), sequences), (32, runs) threads: lane = channel, warp = run of tokens.
@@ -260,11 +331,12 @@ __global__ void __launch_bounds__(1024) lru_scan_kernel(LruArgs a) {
 // Bytes of shared memory and elements between rows of a plane: 16-byte words of neighbouring rows in different banks.
 inline int lru_plane_row(int bs) { return ((bs + 31) / 32) * 32 + (((bs + 31) / 32) % 2 ? 0 : 32); }
 
-template <int MT>
+template <int WM, int MT, int NT>
 int launch_lru_gates_mma(const LruArgs& a, cudaStream_t stream) {
-  const int bs = a.width / a.blocks, row = lru_plane_row(bs);
-  const size_t smem = (size_t)3 * 16 * MT * row * 2;
-  auto kernel = lru_gates_mma_kernel<MT>;
+  constexpr int M = 16 * WM * MT;
+  const int bs = a.width / a.blocks, row = lru_plane_row(bs), tiles = (bs + 63) / 64;
+  const size_t smem = (size_t)3 * M * row * 2;
+  auto kernel = lru_gates_mma_kernel<WM, MT, NT>;
   if (smem > 48 * 1024) {
     cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (err != cudaSuccess) {
@@ -272,8 +344,12 @@ int launch_lru_gates_mma(const LruArgs& a, cudaStream_t stream) {
       return (int)err;
     }
   }
-  const dim3 grid((a.n_tokens + 16 * MT - 1) / (16 * MT), a.blocks * ((bs + 63) / 64));
-  MLL_LAUNCH((kernel), grid, 256, smem, stream, a, row);
+  // a block that walks more channels forms u once for all of them; enough blocks for the device come first
+  const int n_tiles = (a.n_tokens + M - 1) / M;
+  int passes = tiles;
+  while (passes > 1 && (long long)n_tiles * a.blocks * ((tiles + passes - 1) / passes) < mll_sm_count()) passes = (passes + 1) / 2;
+  const dim3 grid(n_tiles, a.blocks * ((tiles + passes - 1) / passes));
+  MLL_LAUNCH((kernel), grid, 256, smem, stream, a, row, passes);
   MLL_LAUNCH_CHECK();
   return 0;
 }
@@ -322,12 +398,12 @@ MLL_API int mll_lru_gates(const void* proj, const float* x_bias, const float* y_
   mll::LruArgs a{proj, x_bias, y_bias, conv_w, conv_b, conv_state, gate_w, gate_b, lam, state, decay, write, out, tok_pos,
                  tok_seq, seq_slot, seq_qstart, nullptr, n_tokens, ld, x_col, y_col, width, blocks, taps, single, rate};
   if (mma) {
+    MLL_REQUIRE(ld % 2 == 0 && x_col % 2 == 0 && (uintptr_t)proj % 4 == 0, "linear recurrent unit: projection rows must be pairs");
     MLL_REQUIRE(mll_lru_mma_supported(dtype, bs), "linear recurrent unit: blocks of %d on tensor cores", bs);
     const size_t per16 = (size_t)3 * 16 * mll::lru_plane_row(bs) * 2;
     // a tall tile reads the matrices less often, a low one gives more blocks
-    if (n_tokens > 256 && 4 * per16 <= 110 * 1024) return mll::launch_lru_gates_mma<4>(a, stream);
-    if (n_tokens > 16 && 2 * per16 <= 110 * 1024) return mll::launch_lru_gates_mma<2>(a, stream);
-    return mll::launch_lru_gates_mma<1>(a, stream);
+    if (n_tokens > 256 && 4 * per16 <= 200 * 1024) return mll::launch_lru_gates_mma<2, 2, 2>(a, stream);
+    return mll::launch_lru_gates_mma<1, 1, 1>(a, stream);
   }
   if (dtype == MLL_F32) return mll::launch_lru_gates<float>(a, stream);
   if (dtype == MLL_BF16) return mll::launch_lru_gates<__nv_bfloat16>(a, stream);

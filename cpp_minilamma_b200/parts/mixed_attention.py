@@ -58,6 +58,7 @@ class MixedHeadsAttention(Mixer):
         self.qkv: Optional[Linear] = None
         self.o: Optional[Linear] = None
         self.q_weight = self.k_weight = self.mix = self.bias = None
+        self.mix_narrow = True  # the mixing matrix holds bfloat16 values: what the tensor-core prompt kernel takes
 
     def weight_specs(self) -> List[WeightSpec]:
         D, H, G = self.ctx.hidden_size, self.n_heads, self.n_kv_heads
@@ -85,6 +86,7 @@ class MixedHeadsAttention(Mixer):
         self.o = Linear(store.take(self.names["o"]), self.names["o"])
         if "mix" in self.names:
             self.mix = store.take(self.names["mix"])
+            self.mix_narrow = bool((self.mix.to(torch.bfloat16).float() == self.mix).all())
         if "bias" in self.names:
             self.bias = store.take(self.names["bias"])
         if self.qk_norm:
@@ -123,10 +125,10 @@ class MixedHeadsAttention(Mixer):
     def _attend(self, step, q, cache, out) -> None:
         sizes = (self.n_heads, self.n_kv_heads, self.d, self.dv)
         tiles = step.meta.get(self.step_metadata_key()) if not step.all_decode else None
-        if (step.all_decode or tiles) and K.mixed_attention_mma_supported(self.ctx.act_dtype, step.all_decode, *sizes):
+        if (step.all_decode or (tiles and self.mix_narrow)) and K.mixed_attention_mma_supported(self.ctx.act_dtype, step.all_decode, *sizes):
             seqs = (q, cache.k, cache.v, step.seq_slot, step.seq_ctx, step.seq_qstart, step.seq_qlen)
             if tiles:
-                K.mixed_attention_tiles(*seqs, tiles["tile_seq"], tiles["tile_row0"], cache.block_table, self.mix, self.bias,
+                K.mixed_attention_tiles(*seqs, tiles["wide_seq"], tiles["wide_row0"], cache.block_table, self.mix, self.bias,
                                         out, *sizes, self.window, self.scale)
                 return
             splits = K.local_attention_heads_splits(step.n_seqs, 1, self.ctx.multiprocessors)

@@ -346,7 +346,7 @@ def test_mixed_attention_kernels(dtype, H, G, d, dv, window):
     k_cache, v_cache, table = _paged(gen, ctxs, G, d, dv, dtype)
     T, group, scale = sum(lens), H // G, 1.2 / d ** 0.5
     q = torch.randn((T, H * d), generator=gen).to(dtype)
-    mix = (0.6 * torch.eye(H) + (torch.randn((H, H), generator=gen) / H ** 0.5 if H > 1 else 0.5)).contiguous()
+    mix = (0.6 * torch.eye(H) + (torch.randn((H, H), generator=gen) / H ** 0.5 if H > 1 else 0.5)).to(torch.bfloat16).float()
     bias = torch.linspace(-4.0, 1.0, H)
     for s in range(4):
         for edge in ((ctxs[s] - window, ctxs[s] - window - 1) if window else (0, 1)):
@@ -376,8 +376,8 @@ def test_mixed_attention_kernels(dtype, H, G, d, dv, window):
     K.mixed_attention(qd, kc, vc, state.tok_pos, state.tok_seq, state.seq_slot, table_dev, md, bd, out, H, G, d, dv, window, scale)
     assert (out.cpu().double() - want).abs().max().item() <= tol, "general kernel"
     if K.mixed_attention_mma_supported(dtype, False, H, G, d, dv):
-        tile_seq = [s for s, n in enumerate(lens) for _ in range(0, n, K.PREFILL_TILE)]
-        tile_row0 = [r for n in lens for r in range(0, n, K.PREFILL_TILE)]
+        tile_seq = [s for s, n in enumerate(lens) for _ in range(0, n, 2 * K.PREFILL_TILE)]
+        tile_row0 = [r for n in lens for r in range(0, n, 2 * K.PREFILL_TILE)]
         out = torch.zeros((T, H * dv), dtype=dtype, device=DEV)
         K.mixed_attention_tiles(qd, kc, vc, state.seq_slot, state.seq_ctx, state.seq_qstart, state.seq_qlen, _ints(tile_seq),
                                 _ints(tile_row0), table_dev, md, bd, out, H, G, d, dv, window, scale)
@@ -392,6 +392,34 @@ def test_mixed_attention_kernels(dtype, H, G, d, dv, window):
                                      table_dev, md, bd, out, 4, H, G, d, dv, window, scale, n_splits=splits, scratch=scratch)
             err = (out.cpu().double() - want[last]).abs().max().item()
             assert err <= tol, ("single tokens", splits, err, tol)
+
+
+def test_mixing_matrix_of_float32_values(models, tmp_path):
+    """A folder whose mixing matrix is stored in float32 with values bfloat16 does not have: bfloat16 prompts then go to
+    the general kernel instead of rounding the matrix."""
+    import struct
+    folder, cfg, W = tm.make_folder("talk", tmp_path / "m", seed=3)
+    blob = (tmp_path / "m" / "model.safetensors").read_bytes()
+    n, = struct.unpack("<Q", blob[:8])
+    header, data = json.loads(blob[8:8 + n]), blob[8 + n:]
+    values = (W["l0.mix.left.talk"] + 0.013 * np.arange(36).reshape(6, 6)).astype("<f4")
+    header["l0.mix.left.talk"] = {"dtype": "F32", "shape": [6, 6], "data_offsets": [len(data), len(data) + values.nbytes]}
+    # the old bytes stay behind as another tensor's: drop them by writing the file anew
+    order, parts, at = {}, [], 0
+    for name, info in header.items():
+        lo, hi = info["data_offsets"]
+        raw = values.tobytes() if info["dtype"] == "F32" else data[lo:hi]
+        order[name] = dict(info, data_offsets=[at, at + len(raw)])
+        parts.append(raw)
+        at += len(raw)
+    text = json.dumps(order).encode()
+    (tmp_path / "m" / "model.safetensors").write_bytes(struct.pack("<Q", len(text)) + text + b"".join(parts))
+    cfg, W = pm.read_folder(tmp_path / "m")
+    toks = tm.tokens(cfg, 80, 4)
+    for dtype in ("float32", "bfloat16"):
+        llm = ml.load(folder, dtype=dtype, max_tokens=256, max_positions=256)
+        assert not llm.model.layers[0].mixer.left.mix_narrow
+        close(run_alone(llm, toks, [70]), pm.forward(cfg, W, toks), dtype, f"float32 matrix, {dtype}")
 
 
 def test_mixed_attention_without_matrix_or_bias():
