@@ -10,7 +10,9 @@
 //      float32 FMAs, two an instruction.
 //   3. O += P V by mma.sync: a warp keeps TP x 16 rows x CP x 64 value columns in registers for the whole walk.
 // Nothing is normalised, so there is no running maximum and no rescaling, and context splits simply add up.
-// K and V of a run have one buffer each: the next run's keys load while 2 and 3 work, its values while 1 and 2 do.
+// K and V of a run have one buffer each.  Single tokens: the next run's keys load while 2 and 3 work, its values while 1
+// and 2 do.  Prompts: step 3 of a run shares an interval between barriers with step 1 of the next one (two streams of
+// independent products a warp), and the copies into both buffers pass while 2 works.
 // Where the H x R rows' outputs exceed what one block's registers hold, grid y splits the output heads and every block
 // recomputes the scores.
 #include "attention_decode.cuh"
@@ -109,7 +111,8 @@ __device__ __forceinline__ void mix_copy16(unsigned at, const void* src, bool va
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(at), "l"(src), "r"(bytes) : "memory");
 }
 
-template <int R, int N, int TP, int CP>
+// DIM: the head size of keys and values where it is known at compile time (strides and word counts are then constants), or 0.
+template <int R, int N, int TP, int CP, int DIM>
 __global__ void __launch_bounds__((R == 1 ? MIX_WARPS_SINGLE : MIX_WARPS_PROMPT) * 32, R == 1 ? 2 : 1)
 mixed_attention_mma_kernel(MixMmaArgs a) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -117,7 +120,8 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
   constexpr int HPT = 16 / R;         // heads in the 16 rows of a tile
   constexpr int QP = R == 1 ? 1 : 2;  // tiles of one key head that share the key fragments in step 1
   constexpr int SS = N + 8;           // elements between rows of S and of P
-  const int H = a.n_heads, G = a.n_kv_heads, group = H / G, d = a.d, dv = a.dv;
+  constexpr bool MERGED = R > 1;      // step 3 of a run beside step 1 of the next
+  const int H = a.n_heads, G = a.n_kv_heads, group = H / G, d = DIM ? DIM : a.d, dv = DIM ? DIM : a.dv;
   const MixMmaLayout L = mix_mma_layout(H, G, d, dv, R, N);
   __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem_raw);
   float* s_s = reinterpret_cast<float*>(smem_raw + L.s);
@@ -190,7 +194,7 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
   }
   if (run < run_end) load_keys(run, page);
   cp_async_commit();
-  if (run < run_end) load_values(run, page);
+  if (!MERGED && run < run_end) load_values(run, page);
   cp_async_commit();
   auto mix_at = [&](int to, int in) { return to >= H || in >= H ? 0.f : a.mix ? a.mix[(size_t)to * H + in] : (to == in ? 1.f : 0.f); };
   if (R == 1) {
@@ -214,33 +218,30 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
   // step 3's unit of this warp: where the lane reads its rows of P and the values, how many of its columns exist (0: no unit)
   const int unit = min(unit0 + warp, unit1 - 1), my_kv = unit / (cgs * tgs), my_col = unit / tgs % cgs * CP * 64, my_tile = unit % tgs * TP;
   const int my_cols = unit0 + warp < unit1 ? min(CP * 64, L.vs - 8 - my_col) : 0;
-  unsigned p_at[TP];
-#pragma unroll
-  for (int i = 0; i < TP; ++i)
-    p_at[i] = base + L.p + (head_of(my_kv, min(my_tile + i, tpg - 1), ld_row) * L.ps + ld_row % R * SS + ld_col) * 2;
+  const unsigned p_at = base + L.p + (head_of(my_kv, my_tile, ld_row) * L.ps + ld_row % R * SS + ld_col) * 2;
+  // the second tile's rows: HPT heads on, or the first tile's again where there is none (or where it is not whole)
+  const int p_step = my_tile + 1 < tpg ? HPT * L.ps * 2 : 0;
   const unsigned v_at = base + L.v + ((my_kv * N + ld_row) * L.vs + my_col + ld_col) * 2;
 
-  // step 1's units: QP tiles of one key head against 16 keys.  Where the lane reads q and k and where its two rows of
-  // scores go (bytes from S's start; -1: nowhere)
+  // step 1's units: QP tiles of one key head against 16 keys.  Where the lane reads q and k and where its scores
+  // go; the second tile and the rows 8 further down lie at fixed distances
   const int pairs = (tpg + QP - 1) / QP;
   const int qk_units = G * pairs * (N / 16), plane = L.hp * L.ps * 2;
-  unsigned q_at[QP], k_at = 0;
-  int s_at[QP][2];
+  unsigned q_at = 0, k_at = 0;
+  int q_step = 0, s_at = 0, rows_in = 0;  // rows_in: bit 2 m + i set where row i of tile m is a row of the group
   constexpr int SB = R == 1 ? 4 : 2;  // bytes of a score in S (R == 1), of one of its terms
   auto set_qk = [&](int u) {
     const int strip = u % (N / 16), pair = (u / (N / 16)) % pairs, kv = u / (N / 16 * pairs);
     k_at = base + L.k + ((kv * N + strip * 16 + (lane & 7) + ((lane >> 4) << 3)) * L.qs + (((lane >> 3) & 1) << 3)) * 2;
+    const int tile = pair * QP;
+    q_at = base + ((head_of(kv, tile, ld_row) * R + ld_row % R) * L.qs + ld_col) * 2;
+    q_step = tile + 1 < tpg ? HPT * R * L.qs * 2 : 0;
+    s_at = base + L.s + ((kv * group + tile * HPT + g / R) * L.ps + g % R * SS + strip * 16 + 2 * t) * SB;
+    rows_in = 0;
 #pragma unroll
-    for (int m = 0; m < QP; ++m) {
-      const int tile = pair * QP + m;
-      q_at[m] = base + ((head_of(kv, min(tile, tpg - 1), ld_row) * R + ld_row % R) * L.qs + ld_col) * 2;
+    for (int m = 0; m < QP; ++m)
 #pragma unroll
-      for (int half8 = 0; half8 < 2; ++half8) {
-        const int rr = g + 8 * half8;
-        s_at[m][half8] = tile < tpg && tile * HPT + rr / R < group
-                             ? (head_of(kv, tile, rr) * L.ps + rr % R * SS + strip * 16 + 2 * t) * SB : -1;
-      }
-    }
+      for (int i = 0; i < 2; ++i) rows_in |= (tile + m) * HPT + (g + 8 * i) / R < group ? 1 << (2 * m + i) : 0;
   };
   set_qk(min(warp, qk_units - 1));
   // step 3 of a run; `all`: every column of the unit exists
@@ -249,7 +250,7 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
     for (int ks = 0; ks < N / 16; ++ks) {
       unsigned pf[TP][4];
 #pragma unroll
-      for (int i = 0; i < TP; ++i) mix_ldsm(pf[i], p_at[i] + ks * 32);
+      for (int i = 0; i < TP; ++i) mix_ldsm(pf[i], p_at + i * p_step + ks * 32);
       const unsigned v = v_at + ks * 32 * L.vs;
 #pragma unroll
       for (int c = 0; c < CP; ++c)
@@ -268,9 +269,16 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
   };
   const float neg_scale = -MIX_LOG2E * a.scale;
 
+  auto step3 = [&] {
+    if (my_cols == CP * 64)
+      weigh_values(std::true_type{});
+    else if (my_cols > 0)
+      weigh_values(std::false_type{});
+  };
   cp_async_wait<1>();
   __syncthreads();
-  for (; run < run_end; ++run) {
+  for (const int run0 = run; run < run_end; ++run) {
+    const int page_now = page;
     if (run + 1 < run_end) page = table[(run + 1) * N / MLL_PAGE];
     for (int u = warp; u < qk_units; u += WARPS) {
       if (qk_units > WARPS) set_qk(u);  // else the warp keeps the one it has
@@ -286,7 +294,7 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
         unsigned qf[QP][4], kf[4];
         mix_ldsm(kf, k_at + e);
 #pragma unroll
-        for (int m = 0; m < QP; ++m) mix_ldsm(qf[m], q_at[m] + e);
+        for (int m = 0; m < QP; ++m) mix_ldsm(qf[m], q_at + m * q_step + e);
 #pragma unroll
         for (int m = 0; m < QP; ++m) {
           mma_16816(acc[m][0], qf[m], kf[0], kf[1]);
@@ -297,8 +305,8 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
       for (int m = 0; m < QP; ++m)
 #pragma unroll
         for (int half8 = 0; half8 < 2; ++half8) {
-          if (s_at[m][half8] < 0) continue;
-          const unsigned to = base + L.s + s_at[m][half8];
+          if (!(rows_in >> (2 * m + half8) & 1)) continue;
+          const unsigned to = s_at + (m * HPT * L.ps + half8 * (8 / R * L.ps + 8 % R * SS)) * SB;
 #pragma unroll
           for (int n = 0; n < 2; ++n) {
             const float x = acc[m][n][2 * half8], y = acc[m][n][2 * half8 + 1];
@@ -317,8 +325,10 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
           }
         }
     }
-    __syncthreads();  // scores are there, this run's keys are done with
+    if (MERGED && run > run0) step3();  // of the run before
+    __syncthreads();  // scores are there, this run's keys (and, merged, the values and weights of the run before) are done with
     if (run + 1 < run_end) load_keys(run + 1, page);
+    if (MERGED) load_values(run, page_now);
     cp_async_commit();
 
     // step 2
@@ -403,19 +413,20 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
         }
       }
     }
+    if (MERGED) {
+      cp_async_wait<0>();  // the next run's keys, this run's values
+      __syncthreads();
+      continue;
+    }
     cp_async_wait<1>();  // this run's values (the next run's keys may still be on their way)
     __syncthreads();
-
-    // step 3
-    if (my_cols == CP * 64)
-      weigh_values(std::true_type{});
-    else if (my_cols > 0)
-      weigh_values(std::false_type{});
+    step3();
     cp_async_wait<0>();  // the next run's keys
     __syncthreads();     // this run's values, weights and scores are done with
     if (run + 1 < run_end) load_values(run + 1, page);
     cp_async_commit();
   }
+  if (MERGED) step3();  // of the last run
   cp_async_wait<0>();
 
 #pragma unroll
@@ -481,10 +492,10 @@ inline int mix_mma_shape(int single, int H, int G, int d, int dv) {
   return 0;
 }
 
-template <int R, int N, int TP, int CP>
-int launch_mixed_mma(const MixMmaArgs& a, int n_blocks, cudaStream_t stream) {
+template <int R, int N, int TP, int CP, int DIM>
+int launch_mixed_mma_dim(const MixMmaArgs& a, int n_blocks, cudaStream_t stream) {
   const int smem = mix_mma_layout(a.n_heads, a.n_kv_heads, a.d, a.dv, R, N).total;
-  auto kernel = mixed_attention_mma_kernel<R, N, TP, CP>;
+  auto kernel = mixed_attention_mma_kernel<R, N, TP, CP, DIM>;
   cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (err != cudaSuccess) {
     mll_set_error("mixed attention (mma): cannot reserve %d bytes of shared memory: %s", smem, cudaGetErrorString(err));
@@ -496,6 +507,12 @@ int launch_mixed_mma(const MixMmaArgs& a, int n_blocks, cudaStream_t stream) {
   MLL_LAUNCH((kernel), grid, WARPS * 32, smem, stream, a);
   MLL_LAUNCH_CHECK();
   return 0;
+}
+
+template <int R, int N, int TP, int CP>
+int launch_mixed_mma(const MixMmaArgs& a, int n_blocks, cudaStream_t stream) {
+  return a.d == 128 && a.dv == 128 ? launch_mixed_mma_dim<R, N, TP, CP, 128>(a, n_blocks, stream)
+                                   : launch_mixed_mma_dim<R, N, TP, CP, 0>(a, n_blocks, stream);
 }
 
 }  // namespace mll
