@@ -1459,13 +1459,13 @@ def lru_mma_supported(dtype: torch.dtype, block: int) -> bool:
     return USE_TENSOR_CORE_LRU and dtype == torch.bfloat16 and bool(lib().mll_lru_mma_supported(dtype_code(dtype), block))
 
 
-def lru_gates(proj, x_col: int, y_col: int, x_bias, y_bias, conv_w, conv_b, conv_state, gate_w, gate_b, lam, state,
-              tok_pos, tok_seq, seq_slot, seq_qstart, blocks: int, rate: float, decay=None, write=None, out=None) -> None:
+def lru_gates(proj, x_col: int, y_col: int, x_bias, y_bias, conv_w, conv_b, conv_state, gate_w, gate_b, rates, state,
+              tok_pos, tok_seq, seq_slot, seq_qstart, blocks: int, decay=None, write=None, out=None) -> None:
     """The inputs of a gated linear recurrent unit from a step's projection rows (csrc/rglru.cu): u = short causal
     convolution of proj's columns x_col .. + width (+ x_bias) over conv_w float32 [width, taps] (+ conv_b), earlier
     inputs from conv_state [slots, taps - 1, width]; r, i = sigmoid of block-diagonal products of u (gate_w: bfloat16
     [n, 2, bs, bs] with rows as outputs, or float32 [n, bs, 2 bs] with columns as outputs; gate_b float32 [2, width]);
-    decay = exp(-rate r softplus(lam)) and write = sqrt(1 - decay^2) i u to float32 [T, width].  With `out` instead of
+    decay = exp(-rates r) (rates float32 [width], not negative) and write = sqrt(1 - decay^2) i u to float32 [T, width].  With `out` instead of
     `decay` and `write` every sequence brings one token: `state` float32 [slots, width] advances and out [T, width] =
     state * gelu(proj's columns y_col .. + y_bias)."""
     _need(proj, "lru proj", None, 2)
@@ -1473,7 +1473,7 @@ def lru_gates(proj, x_col: int, y_col: int, x_bias, y_bias, conv_w, conv_b, conv
     width, taps = conv_w.shape
     single = out is not None
     for name, t, shape in (("x bias", x_bias, (width,)), ("y bias", y_bias, (width,)), ("conv weights", conv_w, (width, taps)),
-                           ("conv bias", conv_b, (width,)), ("gate bias", gate_b, (2, width)), ("lam", lam, (width,))):
+                           ("conv bias", conv_b, (width,)), ("gate bias", gate_b, (2, width)), ("rates", rates, (width,))):
         _need(t, f"lru {name}", torch.float32)
         if tuple(t.shape) != shape:
             raise KernelError(f"lru: {name} {tuple(t.shape)}, expected {shape}")
@@ -1496,9 +1496,9 @@ def lru_gates(proj, x_col: int, y_col: int, x_bias, y_bias, conv_w, conv_b, conv
         _need(t, f"lru {name}", torch.int32, 1)
     _check(lib().mll_lru_gates(
         _ptr(proj), _ptr(x_bias), _ptr(y_bias), _ptr(conv_w), _ptr(conv_b), _ptr(conv_state), _ptr(gate_w), _ptr(gate_b),
-        _ptr(lam), _ptr(state), _ptr(decay), _ptr(write), _ptr(out), _ptr(tok_pos), _ptr(tok_seq), _ptr(seq_slot),
+        _ptr(rates), _ptr(state), _ptr(decay), _ptr(write), _ptr(out), _ptr(tok_pos), _ptr(tok_seq), _ptr(seq_slot),
         _ptr(seq_qstart), dtype_code(proj.dtype), ctypes.c_int(n), ctypes.c_int(ld), ctypes.c_int(x_col),
-        ctypes.c_int(y_col), ctypes.c_int(width), ctypes.c_int(blocks), ctypes.c_int(taps), ctypes.c_float(rate),
+        ctypes.c_int(y_col), ctypes.c_int(width), ctypes.c_int(blocks), ctypes.c_int(taps),
         ctypes.c_int(int(mma)), ctypes.c_int(int(single)), _stream()), "lru_gates (single tokens)" if single else "lru_gates")
 
 

@@ -2,7 +2,7 @@
 //
 //   u_t = conv(x_t + b_x) + b_c         causal, `taps` inputs per channel, nothing before a sequence's first token
 //   r_t = sigmoid(A u_t + a),  i_t = sigmoid(I u_t + c)       A, I block-diagonal: n square blocks of `bs` channels
-//   decay_t = exp(-rate * r_t * softplus(lam))
+//   decay_t = exp(-rate * r_t * softplus(lam))      rate * softplus(lam) is a number per channel, formed once
 //   S_t = decay_t S_(t-1) + sqrt(1 - decay_t^2) i_t u_t       one number per channel, float32, zero at the start
 //   out_t = S_t * gelu(y_t + b_y)       (the tanh form)
 //
@@ -23,8 +23,29 @@
 
 namespace mll {
 
-__device__ __forceinline__ float lru_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
-__device__ __forceinline__ float lru_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+// 1 / (1 + e^-z); FAST: the hardware's exponential and reciprocal (a few units in the last place of a float32)
+template <bool FAST>
+__device__ __forceinline__ float lru_sigmoid(float z) {
+  return FAST ? __fdividef(1.f, 1.f + __expf(-z)) : 1.f / (1.f + expf(-z));
+}
+template <bool FAST>
+__device__ __forceinline__ float lru_sqrt(float x) {
+  if (!FAST) return sqrtf(x);
+  float r;
+  asm("sqrt.approx.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
+}
+// 1 - e^-x for x >= 0, given e = e^-x: near 0 by the first terms of its Taylor series (the next one is below 1e-9 of the
+// result), else by the difference, which loses less than two bits there
+__device__ __forceinline__ float lru_one_minus(float x, float e) {
+  float p = fmaf(x, -1.f / 7.f, 1.f);
+  p = fmaf(x * p, -1.f / 6.f, 1.f);
+  p = fmaf(x * p, -1.f / 5.f, 1.f);
+  p = fmaf(x * p, -1.f / 4.f, 1.f);
+  p = fmaf(x * p, -1.f / 3.f, 1.f);
+  p = fmaf(x * p, -1.f / 2.f, 1.f);
+  return x < 0.25f ? x * p : 1.f - e;
+}
 __device__ __forceinline__ float lru_gelu(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
@@ -38,7 +59,7 @@ struct LruArgs {
   const float* conv_state;  // [slots, taps - 1, width]: the last inputs of every sequence, without x_bias
   const void* gate_w;       // mma: bfloat16 [n, 2, bs(out), bs(in)]; FMA: float32 [n, bs(in), 2 bs(out)]
   const float* gate_b;      // [2, width]: r's, then i's
-  const float* lam;         // [width]
+  const float* rates;       // [width]: rate * softplus(lam)
   float* state;             // [slots, width]
   float* decay;             // [T, width]
   float* write;             // [T, width]
@@ -49,7 +70,6 @@ struct LruArgs {
   const int* seq_qstart;
   const int* seq_qlen;
   int n_tokens, ld, x_col, y_col, width, blocks, taps, single;
-  float rate;
 };
 
 // u of token t, channel c (see above): inputs of this step come from the projection, earlier ones from the state.
@@ -66,23 +86,31 @@ __device__ __forceinline__ float lru_conv(const LruArgs& a, int t, int c, int po
   return u;
 }
 
-// From the two gates' pre-activations to the recurrence's inputs; with `single` also the step itself.
+// What one channel brings to every token: the gates' biases, its rate, y's bias.
+struct LruChannel {
+  float br, bi, rate, yb;
+};
+__device__ __forceinline__ LruChannel lru_channel(const LruArgs& a, int c) {
+  return {a.gate_b[c], a.gate_b[a.width + c], a.rates[c], a.y_bias[c]};
+}
+
+// From the two gates' pre-activations to the recurrence's inputs (decay, write).
+template <bool FAST>
+__device__ __forceinline__ float2 lru_inputs(const LruChannel& ch, float zr, float zi, float u) {
+  const float r = lru_sigmoid<FAST>(zr + ch.br), i = lru_sigmoid<FAST>(zi + ch.bi);
+  const float x = ch.rate * r;
+  const float decay = expf(-x);
+  return make_float2(decay, lru_sqrt<FAST>(lru_one_minus(2.f * x, decay * decay)) * i * u);
+}
+
+// A step of one token: the state advances, the output is written.
 template <typename T>
-__device__ __forceinline__ void lru_finish(const LruArgs& a, int t, int c, float zr, float zi, float u) {
-  const float r = lru_sigmoid(zr + a.gate_b[c]), i = lru_sigmoid(zi + a.gate_b[a.width + c]);
-  const float log_decay = -a.rate * r * lru_softplus(a.lam[c]);
-  const float decay = expf(log_decay);
-  const float write = sqrtf(-expm1f(2.f * log_decay)) * i * u;  // 1 - decay^2 without cancellation
-  if (a.single) {
-    float* S = a.state + (size_t)a.seq_slot[a.tok_seq[t]] * a.width + c;
-    const float s = fmaf(decay, *S, write);
-    *S = s;
-    const float y = to_float(((const T*)a.proj)[(size_t)t * a.ld + a.y_col + c]) + a.y_bias[c];
-    ((T*)a.out)[(size_t)t * a.width + c] = from_float<T>(s * lru_gelu(y));
-  } else {
-    a.decay[(size_t)t * a.width + c] = decay;
-    a.write[(size_t)t * a.width + c] = write;
-  }
+__device__ __forceinline__ void lru_advance(const LruArgs& a, const LruChannel& ch, int t, int slot, int c, float2 in) {
+  float* S = a.state + (size_t)slot * a.width + c;
+  const float y = to_float(((const T*)a.proj)[(size_t)t * a.ld + a.y_col + c]) + ch.yb;
+  const float s = fmaf(in.x, *S, in.y);
+  *S = s;
+  ((T*)a.out)[(size_t)t * a.width + c] = from_float<T>(s * lru_gelu(y));
 }
 
 // grid (ceil(tokens / 16), n * ceil(bs / 64)), 256 threads: a thread owns one channel and four tokens.
@@ -113,7 +141,17 @@ __global__ void __launch_bounds__(256) lru_gates_kernel(LruArgs a) {
   }
 #pragma unroll
   for (int i = 0; i < 4; ++i)
-    if (q0 + i < n) lru_finish<T>(a, t0 + q0 + i, block * bs + col, r[i], z[i], u_s[(q0 + i) * bs + col]);
+    if (q0 + i < n) {
+      const int t = t0 + q0 + i, c = block * bs + col;
+      const LruChannel ch = lru_channel(a, c);
+      const float2 in = lru_inputs<false>(ch, r[i], z[i], u_s[(q0 + i) * bs + col]);
+      if (a.single) {
+        lru_advance<T>(a, ch, t, a.seq_slot[a.tok_seq[t]], c, in);
+      } else {
+        a.decay[(size_t)t * a.width + c] = in.x;
+        a.write[(size_t)t * a.width + c] = in.y;
+      }
+    }
 }
 
 // grid (ceil(tokens / M), n * column parts), 256 threads; M = 16 WM MT tokens.  A block forms u for its tokens and one
@@ -128,7 +166,7 @@ __global__ void __launch_bounds__(256) lru_gates_mma_kernel(LruArgs a, int row, 
   constexpr int M = 16 * WM * MT;
   static_assert(8 / WM * NT * 8 == 64, "a pass covers 64 channels");
   __shared__ int pos_s[M], back_s[M];           // a token's position; how many of its inputs lie in this step
-  __shared__ const float* state_s[M];           // where its sequence's earlier inputs are
+  __shared__ int slot_s[M];                     // its sequence's slot
   const int bs = a.width / a.blocks, tiles = (bs + 63) / 64, parts = (tiles + passes - 1) / passes;
   const int block = blockIdx.y / parts, tile0 = (blockIdx.y % parts) * passes, tile1 = min(tiles, tile0 + passes);
   const int t0 = blockIdx.x * M, n = min(M, a.n_tokens - t0);
@@ -138,7 +176,7 @@ __global__ void __launch_bounds__(256) lru_gates_mma_kernel(LruArgs a, int row, 
     const int t = t0 + threadIdx.x, seq = a.tok_seq[t];
     pos_s[threadIdx.x] = a.tok_pos[t];
     back_s[threadIdx.x] = t - a.seq_qstart[seq];
-    state_s[threadIdx.x] = a.conv_state + (size_t)a.seq_slot[seq] * (a.taps - 1) * a.width;
+    slot_s[threadIdx.x] = a.seq_slot[seq];
   }
   __syncthreads();
   // u: a thread owns a pair of channels and every (256 / pairs)-th token
@@ -162,7 +200,7 @@ __global__ void __launch_bounds__(256) lru_gates_mma_kernel(LruArgs a, int row, 
         u = cb;
         const int local = back_s[m], reach = min(a.taps - 1, pos_s[m]);  // nothing before the sequence, not even the bias
         const __nv_bfloat16* x0 = proj + (size_t)(t0 + m) * a.ld + a.x_col + c;
-        const float* s0 = state_s[m] + (size_t)(local + a.taps - 1) * a.width + c;
+        const float* s0 = a.conv_state + ((size_t)slot_s[m] * (a.taps - 1) + local + a.taps - 1) * a.width + c;
         auto input = [&](int back) {
           if (back <= local)
             return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(x0 - (size_t)back * a.ld));
@@ -245,18 +283,30 @@ __global__ void __launch_bounds__(256) lru_gates_mma_kernel(LruArgs a, int row, 
         }
     }
 #pragma unroll
-    for (int j = 0; j < NT; ++j)
+    for (int j = 0; j < NT; ++j) {
+      const int c = c0 + 8 * j + 2 * q, full = block * bs + c;  // a pair of channels: bs is even, both or none
+      if (c >= bs) continue;
+      const LruChannel ch0 = lru_channel(a, full), ch1 = lru_channel(a, full + 1);
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const int tok = m0 + m * 16 + g + 8 * (i >> 1), c = c0 + 8 * j + 2 * q + (i & 1);
-          if (tok < n && c < bs) {
-            const __nv_bfloat16* src = planes + (size_t)tok * row + c;
-            const float u = (__bfloat162float(src[0]) + __bfloat162float(src[(size_t)M * row])) + __bfloat162float(src[(size_t)2 * M * row]);
-            lru_finish<__nv_bfloat16>(a, t0 + tok, block * bs + c, acc[0][j][m][i], acc[1][j][m][i], u);
+        for (int half = 0; half < 2; ++half) {
+          const int tok = m0 + m * 16 + g + 8 * half, t = t0 + tok;
+          if (tok >= n) continue;
+          const unsigned* src = reinterpret_cast<const unsigned*>(planes + (size_t)tok * row + c);
+          const float2 h = unpack_bf162(src[0]), mid = unpack_bf162(src[(size_t)M * row / 2]), lo = unpack_bf162(src[(size_t)M * row]);
+          const float2 in0 = lru_inputs<true>(ch0, acc[0][j][m][2 * half], acc[1][j][m][2 * half], (h.x + mid.x) + lo.x);
+          const float2 in1 = lru_inputs<true>(ch1, acc[0][j][m][2 * half + 1], acc[1][j][m][2 * half + 1], (h.y + mid.y) + lo.y);
+          if (a.single) {
+            lru_advance<__nv_bfloat16>(a, ch0, t, slot_s[tok], full, in0);
+            lru_advance<__nv_bfloat16>(a, ch1, t, slot_s[tok], full + 1, in1);
+          } else {
+            const size_t at = (size_t)t * a.width + full;
+            *reinterpret_cast<float2*>(a.decay + at) = make_float2(in0.x, in1.x);
+            *reinterpret_cast<float2*>(a.write + at) = make_float2(in0.y, in1.y);
           }
         }
+    }
   }
 }
 
@@ -383,9 +433,9 @@ MLL_API int mll_lru_mma_supported(int dtype, int bs) {
 // `single`: every sequence brings one token; the state advances and `out` is written here (decay, write may be null).
 MLL_API int mll_lru_gates(const void* proj, const float* x_bias, const float* y_bias, const float* conv_w,
                           const float* conv_b, const float* conv_state, const void* gate_w, const float* gate_b,
-                          const float* lam, float* state, float* decay, float* write, void* out, const int* tok_pos,
+                          const float* rates, float* state, float* decay, float* write, void* out, const int* tok_pos,
                           const int* tok_seq, const int* seq_slot, const int* seq_qstart, int dtype, int n_tokens, int ld,
-                          int x_col, int y_col, int width, int blocks, int taps, float rate, int mma, int single,
+                          int x_col, int y_col, int width, int blocks, int taps, int mma, int single,
                           cudaStream_t stream) {
   MLL_REQUIRE(n_tokens >= 0 && width > 0 && blocks > 0 && width % blocks == 0 && taps > 0, "linear recurrent unit: bad sizes");
   MLL_REQUIRE(x_col >= 0 && y_col >= 0 && x_col + width <= ld && y_col + width <= ld,
@@ -395,8 +445,8 @@ MLL_API int mll_lru_gates(const void* proj, const float* x_bias, const float* y_
   MLL_REQUIRE((size_t)16 * bs * 4 <= 200 * 1024, "linear recurrent unit: blocks of %d exceed the 3200 the kernel takes", bs);
   MLL_REQUIRE((long long)blocks * ((bs + 63) / 64) <= 65535, "linear recurrent unit: too many blocks for one launch");
   if (n_tokens == 0) return 0;
-  mll::LruArgs a{proj, x_bias, y_bias, conv_w, conv_b, conv_state, gate_w, gate_b, lam, state, decay, write, out, tok_pos,
-                 tok_seq, seq_slot, seq_qstart, nullptr, n_tokens, ld, x_col, y_col, width, blocks, taps, single, rate};
+  mll::LruArgs a{proj, x_bias, y_bias, conv_w, conv_b, conv_state, gate_w, gate_b, rates, state, decay, write, out, tok_pos,
+                 tok_seq, seq_slot, seq_qstart, nullptr, n_tokens, ld, x_col, y_col, width, blocks, taps, single};
   if (mma) {
     MLL_REQUIRE(ld % 2 == 0 && x_col % 2 == 0 && (uintptr_t)proj % 4 == 0, "linear recurrent unit: projection rows must be pairs");
     MLL_REQUIRE(mll_lru_mma_supported(dtype, bs), "linear recurrent unit: blocks of %d on tensor cores", bs);

@@ -63,7 +63,10 @@ class LinearRecurrentUnit(Mixer):
             fused = torch.cat([fused, torch.zeros((spare, fused.shape[1]), dtype=fused.dtype, device=fused.device)], dim=0)
         self.proj = Linear(fused, n["y"] + "+x")
         del mats, fused
-        self.y_bias, self.x_bias, self.conv_b, self.lam = (store.take(n[p]) for p in ("y_bias", "x_bias", "conv_bias", "lam"))
+        self.y_bias, self.x_bias, self.conv_b = (store.take(n[p]) for p in ("y_bias", "x_bias", "conv_bias"))
+        # the decay's exponent per channel, once: softplus(lam) = max(lam, 0) + log(1 + exp(-|lam|)) in double, then float32
+        lam = store.take(n["lam"]).double()
+        self.rates = (self.rate * (lam.clamp_min(0) + torch.log1p(torch.exp(-lam.abs())))).float().contiguous()
         self.conv_w = store.take(n["conv"]).contiguous()
         self.gate_b = torch.stack([store.take(n["ra_bias"]).reshape(W), store.take(n["ri_bias"]).reshape(W)]).contiguous()
         ra, ri = store.take(n["ra"]), store.take(n["ri"])
@@ -85,8 +88,8 @@ class LinearRecurrentUnit(Mixer):
         proj = self.proj.forward(step, h, "lru.proj")
         out = ws.buffer("lru.out", (T, W), self.ctx.act_dtype)
         gates = (proj, W, 0, self.x_bias, self.y_bias, self.conv_w, self.conv_b, cache.state["conv"], self.gate_w,
-                 self.gate_b, self.lam, cache.state["S"], step.tok_pos, step.tok_seq, step.seq_slot, step.seq_qstart,
-                 self.blocks, self.rate)
+                 self.gate_b, self.rates, cache.state["S"], step.tok_pos, step.tok_seq, step.seq_slot, step.seq_qstart,
+                 self.blocks)
         if step.all_decode:
             K.lru_gates(*gates, out=out)  # one token each: the state advances in the same kernel
         else:

@@ -456,6 +456,7 @@ def test_linear_recurrent_unit_kernels(dtype, W, n, taps):
     rnd = lambda *shape: torch.randn(shape, generator=gen)
     ra, ri = (rnd(n, bs, bs) * 1.5 / bs ** 0.5).to(dtype), (rnd(n, bs, bs) * 1.5 / bs ** 0.5).to(dtype)
     conv_w, conv_b, xb, yb, gb, lam = rnd(W, taps) * 0.6, rnd(W) * 0.3, rnd(W) * 0.3, rnd(W) * 0.3, rnd(2, W) * 0.4, rnd(W) * 3 - 3
+    rates = (8.0 * torch.nn.functional.softplus(lam.double(), threshold=40)).float()
     S0, C0 = rnd(7, W), rnd(7, taps - 1, W)
     S0[2], C0[2] = 0.0, 0.0
     mma = dtype == torch.bfloat16 and K.lru_mma_supported(dtype, bs)
@@ -473,8 +474,8 @@ def test_linear_recurrent_unit_kernels(dtype, W, n, taps):
                 proj = torch.cat([proj, torch.zeros(T, (-proj.shape[1]) % 8, dtype=dtype)], dim=1).contiguous()
             st = make_step_state(DEV, slots, starts, lens)
             pd = proj.to(DEV)
-            consts = (xb.to(DEV), yb.to(DEV), conv_w.to(DEV), conv_b.to(DEV), C_dev, gate_w.to(DEV), gb.to(DEV), lam.to(DEV), S_dev,
-                      st.tok_pos, st.tok_seq, st.seq_slot, st.seq_qstart, n, 8.0)
+            consts = (xb.to(DEV), yb.to(DEV), conv_w.to(DEV), conv_b.to(DEV), C_dev, gate_w.to(DEV), gb.to(DEV), rates.to(DEV), S_dev,
+                      st.tok_pos, st.tok_seq, st.seq_slot, st.seq_qstart, n)
             out = torch.zeros((T, W), dtype=dtype, device=DEV)
             single = max(lens) == 1
             decay, write = torch.zeros((T, W), device=DEV), torch.zeros((T, W), device=DEV)
