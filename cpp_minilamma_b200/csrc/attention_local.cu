@@ -24,6 +24,29 @@
 
 namespace mll {
 
+template <typename T>
+struct Vec16;  // 16 bytes of T as floats
+template <>
+struct Vec16<float> {
+  static __device__ __forceinline__ void load(const float* p, float* out) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    out[0] = v.x; out[1] = v.y; out[2] = v.z; out[3] = v.w;
+  }
+};
+template <>
+struct Vec16<__nv_bfloat16> {
+  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float* out) {
+    const uint4 v = *reinterpret_cast<const uint4*>(p);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&v);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 f = __bfloat1622float2(h[i]);
+      out[2 * i] = f.x;
+      out[2 * i + 1] = f.y;
+    }
+  }
+};
+
 struct LocalPrepArgs {
   const void* qkv;        // [T, ld]: q (Hq * d), k (Hk * d), v (Hk * dv)
   const float* q_weight;  // [Hq * d] or null: no norm of the projections
@@ -109,28 +132,84 @@ __global__ void __launch_bounds__(256) local_prepare_kernel(LocalPrepArgs a) {
   }
 }
 
-template <typename T>
-struct Vec16;  // 16 bytes of T as floats
-template <>
-struct Vec16<float> {
-  static __device__ __forceinline__ void load(const float* p, float* out) {
-    const float4 v = *reinterpret_cast<const float4*>(p);
-    out[0] = v.x; out[1] = v.y; out[2] = v.z; out[3] = v.w;
-  }
-};
-template <>
-struct Vec16<__nv_bfloat16> {
-  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float* out) {
-    const uint4 v = *reinterpret_cast<const uint4*>(p);
-    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&v);
+// The same for bfloat16 rows that are whole 16-byte words and rotated halves of whole words: a thread owns eight
+// neighbouring dimensions.  The row waits in shared memory between the norm's sums and the rotation, which needs the
+// partner half.
+__global__ void __launch_bounds__(256) local_prepare_vec_kernel(LocalPrepArgs a) {
+  extern __shared__ __align__(16) uint4 row_s[];
+  __shared__ float scratch[32];
+  const int t = blockIdx.x;
+  const int dw = a.d >> 3, vw = a.dv >> 3, nq = a.n_heads * dw, nk = a.write_kv ? a.n_kv_heads * dw : 0;
+  const int nv = a.write_kv ? a.n_kv_heads * vw : 0;
+  const __nv_bfloat16* row = (const __nv_bfloat16*)a.qkv + (size_t)t * a.ld;
+  const int pos = a.tok_pos[t];
+  const int page = a.write_kv ? a.block_table[(size_t)a.seq_slot[a.tok_seq[t]] * a.max_blocks + pos / MLL_PAGE] : 0;
+  const int in_page = pos % MLL_PAGE;
+  float sq = 0.f, sk = 0.f;
+  for (int i = threadIdx.x; i < nq + nk; i += 256) {
+    const uint4 v = reinterpret_cast<const uint4*>(row)[i];
+    row_s[i] = v;
+    if (a.q_weight) {
+      float x[8];
+      Vec16<__nv_bfloat16>::load(reinterpret_cast<const __nv_bfloat16*>(&v), x);
+      float s = 0.f;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const float2 f = __bfloat1622float2(h[i]);
-      out[2 * i] = f.x;
-      out[2 * i + 1] = f.y;
+      for (int k = 0; k < 8; ++k) s += x[k] * x[k];
+      if (i < nq) sq += s;
+      else sk += s;
     }
   }
-};
+  for (int i = threadIdx.x; i < nv; i += 256) {
+    const int head = i / vw, e = i - head * vw;
+    reinterpret_cast<uint4*>((__nv_bfloat16*)a.v_cache + (((size_t)page * a.n_kv_heads + head) * MLL_PAGE + in_page) * a.dv)[e] =
+        reinterpret_cast<const uint4*>(row + a.v_col)[i];
+  }
+  float fq = 1.f, fk = 1.f;
+  if (a.q_weight) {
+    sq = block_sum(sq, scratch);
+    sk = block_sum(sk, scratch);
+    fq = 1.f / sqrtf(sq / (float)(nq * 8) + a.eps);
+    fk = 1.f / sqrtf(sk / (float)(nk * 8) + a.eps);
+  }
+  if (a.q_temp_every > 0) fq *= 1.f + a.q_temp_coef * logf((float)((pos + 1) / a.q_temp_every) + 1.f);
+  __syncthreads();
+  const int hw = a.rot >> 4;  // words of a rotated half
+  const float* cs = a.cos_table ? a.cos_table + (size_t)pos * (a.rot >> 1) : nullptr;
+  const float* sn = a.cos_table ? a.sin_table + (size_t)pos * (a.rot >> 1) : nullptr;
+  auto scaled = [&](int word, bool is_q, float* x) {  // eight normalised dimensions of the row
+    Vec16<__nv_bfloat16>::load(reinterpret_cast<const __nv_bfloat16*>(row_s + word), x);
+    const float f = is_q ? fq : fk;
+    const float* w = a.q_weight ? (is_q ? a.q_weight + word * 8 : a.k_weight + (word - nq) * 8) : nullptr;
+#pragma unroll
+    for (int k = 0; k < 8; k += 4) {
+      const float4 m = w ? *reinterpret_cast<const float4*>(w + k) : make_float4(1.f, 1.f, 1.f, 1.f);
+      x[k] = x[k] * f * m.x; x[k + 1] = x[k + 1] * f * m.y; x[k + 2] = x[k + 2] * f * m.z; x[k + 3] = x[k + 3] * f * m.w;
+    }
+  };
+  for (int i = threadIdx.x; i < nq + nk; i += 256) {
+    const bool is_q = i < nq;
+    const int c = is_q ? i : i - nq, head = c / dw, e = c - head * dw;
+    float x[8];
+    scaled(i, is_q, x);
+    if (cs && e < 2 * hw) {
+      const bool first = e < hw;
+      float y[8];
+      scaled(first ? i + hw : i - hw, is_q, y);
+      const float* co = cs + (first ? e : e - hw) * 8;
+      const float* si = sn + (first ? e : e - hw) * 8;
+#pragma unroll
+      for (int k = 0; k < 8; ++k) x[k] = first ? x[k] * co[k] - y[k] * si[k] : x[k] * co[k] + y[k] * si[k];
+    }
+    uint4 v;
+    __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) p[k] = __floats2bfloat162_rn(x[2 * k], x[2 * k + 1]);
+    if (is_q)
+      reinterpret_cast<uint4*>((__nv_bfloat16*)a.q_out + (size_t)t * nq * 8)[c] = v;
+    else
+      reinterpret_cast<uint4*>((__nv_bfloat16*)a.k_cache + (((size_t)page * a.n_kv_heads + head) * MLL_PAGE + in_page) * a.d)[e] = v;
+  }
+}
 
 struct LocalAttnArgs {
   const void* q;         // [T, Hq * d]
@@ -379,6 +458,14 @@ MLL_API int mll_local_attention_prepare(const void* qkv, const float* q_weight, 
                        block_table, q_out, k_cache, v_cache, ld, n_heads, n_kv_heads, d, dv, rot, interleaved,
                        max_blocks, eps, q_temp_coef, q_temp_every,
                        v_from_k ? n_heads * d : n_heads * d + n_kv_heads * d, write_kv ? 1 : 0};
+  const auto whole = [](const void* p) { return (uintptr_t)p % 16 == 0; };
+  const size_t row_bytes = (size_t)(n_heads + (write_kv ? n_kv_heads : 0)) * d * 2;
+  if (dtype == MLL_BF16 && d % 8 == 0 && dv % 8 == 0 && ld % 8 == 0 && (rot == 0 || (!interleaved && rot % 16 == 0)) &&
+      row_bytes <= 48 * 1024 && whole(qkv) && whole(q_out) && whole(k_cache) && whole(v_cache) && whole(q_weight) && whole(k_weight)) {
+    MLL_LAUNCH((mll::local_prepare_vec_kernel), n_tokens, 256, row_bytes, stream, a);
+    MLL_LAUNCH_CHECK();
+    return 0;
+  }
   if (dtype == MLL_F32)
     MLL_LAUNCH((mll::local_prepare_kernel<float>), n_tokens, 256, 0, stream, a);
   else if (dtype == MLL_BF16)

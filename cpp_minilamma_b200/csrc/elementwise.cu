@@ -329,6 +329,26 @@ __global__ void heads_gate_kernel(const T* __restrict__ in, const T* __restrict_
   }
 }
 
+// The same in bfloat16 with one gate per head, eight neighbouring values a thread (dv and the strides multiples of 8).
+__global__ void __launch_bounds__(256) heads_gate_vec_kernel(const __nv_bfloat16* in, const __nv_bfloat16* gate, __nv_bfloat16* out,
+                                                             size_t words, int n_heads, int dv, long long in_t, long long in_h,
+                                                             int gate_ld) {
+  const int per_head = dv / 8, per_token = n_heads * per_head;
+  for (size_t i = (size_t)blockIdx.x * 256 + threadIdx.x; i < words; i += (size_t)gridDim.x * 256) {
+    const size_t t = i / per_token;
+    const int w = (int)(i - t * per_token), h = w / per_head;
+    uint4 v = *reinterpret_cast<const uint4*>(in + t * in_t + (size_t)h * in_h + (w - h * per_head) * 8);
+    const float f = 1.f / (1.f + expf(-__bfloat162float(gate[t * gate_ld + h])));
+    __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const float2 x = __bfloat1622float2(p[k]);
+      p[k] = __floats2bfloat162_rn(x.x * f, x.y * f);
+    }
+    *reinterpret_cast<uint4*>(out + i * 8) = v;
+  }
+}
+
 // out = act(in), elementwise, evaluated in float32.  kind 0: gelu in its erf form, 0.5 z (1 + erf(z / sqrt 2));
 // 1: gelu in its tanh form, 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))).
 template <typename T>
@@ -540,6 +560,13 @@ MLL_API int mll_heads_gate(const void* in, const void* gate, void* out, int dtyp
   MLL_REQUIRE(n_tokens >= 0 && n_heads > 0 && dv > 0 && gate_ld > 0, "heads_gate: bad sizes");
   if (n_tokens == 0) return 0;
   const size_t total = (size_t)n_tokens * n_heads * dv;
+  if (dtype == MLL_BF16 && per_head && dv % 8 == 0 && in_t % 8 == 0 && in_h % 8 == 0 && (uintptr_t)in % 16 == 0 && (uintptr_t)out % 16 == 0) {
+    const long long want = (long long)((total / 8 + 255) / 256), most = (long long)mll_sm_count() * 8;
+    MLL_LAUNCH((mll::heads_gate_vec_kernel), (int)(want < most ? want : most), 256, 0, stream, (const __nv_bfloat16*)in,
+               (const __nv_bfloat16*)gate, (__nv_bfloat16*)out, total / 8, n_heads, dv, in_t, in_h, gate_ld);
+    MLL_LAUNCH_CHECK();
+    return 0;
+  }
   long long blocks = (long long)((total + 255) / 256);
   if (blocks > mll_sm_count() * 16) blocks = mll_sm_count() * 16;
   if (dtype == MLL_F32)
