@@ -13,14 +13,20 @@
 // K and V of a run have one buffer each.  Single tokens: the next run's keys load while 2 and 3 work, its values while 1
 // and 2 do.  Prompts: step 3 of a run shares an interval between barriers with step 1 of the next one (two streams of
 // independent products a warp), and the copies into both buffers pass while 2 works.
+// A prompt's tile may be cut along its keys too: the blocks of a thread-block cluster walk a share of the runs each and add
+// their sums up through distributed shared memory, every block the columns it writes.
 // Where the H x R rows' outputs exceed what one block's registers hold, grid y splits the output heads and every block
 // recomputes the scores.
 #include "attention_decode.cuh"
 #include "attention_mix.cuh"
 
+#include <cooperative_groups.h>
+
 #include <type_traits>
 
 namespace mll {
+
+namespace cg = cooperative_groups;
 
 struct MixMmaArgs {
   const __nv_bfloat16* q;
@@ -36,12 +42,12 @@ struct MixMmaArgs {
   const float* mix;       // [H, H] or null; prompts need entries that are bfloat16 values
   const float* bias;      // [H] or null
   __nv_bfloat16* out;
-  float* part;            // [sequences, n_splits, H, dv] sums of the context's runs (n_splits > 1)
-  int n_heads, n_kv_heads, d, dv, window, max_blocks, n_splits;
+  float* part;            // single tokens: [sequences, n_splits, H, dv] sums of the context's runs (n_splits > 1)
+  int n_heads, n_kv_heads, d, dv, window, max_blocks;
+  int n_splits;           // blocks (grid z) that share a tile's runs; for prompts they are one cluster
   float scale;
 };
 
-constexpr int MIX_WARPS_PROMPT = 16, MIX_WARPS_SINGLE = 8;  // warps of a block
 
 // Shared memory of a block, in bytes from its start.  Rows of q are compact: row h * R + r.  Scores and weights of head h
 // and row r begin at element h * ps + r * (N + 8): rows of 16-byte words of which neighbours - in a head, or of heads -
@@ -112,13 +118,14 @@ __device__ __forceinline__ void mix_copy16(unsigned at, const void* src, bool va
 }
 
 // DIM: the head size of keys and values where it is known at compile time (strides and word counts are then constants), or 0.
-template <int R, int N, int TP, int CP, int DIM>
-__global__ void __launch_bounds__((R == 1 ? MIX_WARPS_SINGLE : MIX_WARPS_PROMPT) * 32, R == 1 ? 2 : 1)
+// W warps a block; with 8 of them two blocks share a multiprocessor.
+template <int R, int N, int W, int TP, int CP, int DIM>
+__global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1)
 mixed_attention_mma_kernel(MixMmaArgs a) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
-  constexpr int WARPS = R == 1 ? MIX_WARPS_SINGLE : MIX_WARPS_PROMPT, THREADS = WARPS * 32;
+  constexpr int WARPS = W, THREADS = W * 32;
   constexpr int HPT = 16 / R;         // heads in the 16 rows of a tile
-  constexpr int QP = R == 1 ? 1 : 2;  // tiles of one key head that share the key fragments in step 1
+  constexpr int QP = W == 8 ? 1 : 2;  // tiles of one key head that share the key fragments in step 1
   constexpr int SS = N + 8;           // elements between rows of S and of P
   constexpr bool MERGED = R > 1;      // step 3 of a run beside step 1 of the next
   const int H = a.n_heads, G = a.n_kv_heads, group = H / G, d = DIM ? DIM : a.d, dv = DIM ? DIM : a.dv;
@@ -277,6 +284,7 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
   };
   cp_async_wait<1>();
   __syncthreads();
+  const bool any_runs = run < run_end;
   for (const int run0 = run; run < run_end; ++run) {
     const int page_now = page;
     if (run + 1 < run_end) page = table[(run + 1) * N / MLL_PAGE];
@@ -426,9 +434,48 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
     if (run + 1 < run_end) load_values(run + 1, page);
     cp_async_commit();
   }
-  if (MERGED) step3();  // of the last run
+  if (MERGED && any_runs) step3();  // of the last run
   cp_async_wait<0>();
 
+  if constexpr (R > 1) {
+    if (a.n_splits > 1) {  // the same in all blocks of the cluster: each gets here, with or without runs of its own
+      cg::cluster_group cluster = cg::this_cluster();
+      float2* mine = reinterpret_cast<float2*>(smem_raw);  // [TP * CP * 16][THREADS], over what the walk no longer needs
+      __syncthreads();
+#pragma unroll
+      for (int i = 0; i < TP * CP * 8; ++i)
+#pragma unroll
+        for (int half8 = 0; half8 < 2; ++half8) {
+          const float* f = &o[0][0][0][0] + i * 4 + 2 * half8;
+          mine[(i * 2 + half8) * THREADS + tid] = make_float2(f[0], f[1]);
+        }
+      cluster.sync();
+      const int rank = (int)cluster.block_rank(), share = 8 / a.n_splits;  // n_splits divides 8
+#pragma unroll
+      for (int i = 0; i < TP; ++i)
+#pragma unroll
+        for (int half8 = 0; half8 < 2; ++half8) {
+          const int rr = g + 8 * half8, r = rr % R, tile = my_tile + i;
+          if (tile * HPT + rr / R >= group || r >= rows) continue;
+          const int h = my_kv * group + tile * HPT + rr / R;
+          for (int c = 0; c < CP; ++c)
+            for (int n = rank * share; n < (rank + 1) * share; ++n) {
+              const int col = c * 64 + n * 8 + 2 * t;
+              if (col >= my_cols || my_col + col >= dv) continue;
+              const float2* at = mine + (((i * CP + c) * 8 + n) * 2 + half8) * THREADS + tid;
+              float2 sum = make_float2(0.f, 0.f);
+              for (int sp = 0; sp < a.n_splits; ++sp) {  // in the order of the runs
+                const float2 v = *cluster.map_shared_rank(at, sp);
+                sum.x += v.x;
+                sum.y += v.y;
+              }
+              *reinterpret_cast<__nv_bfloat162*>(a.out + ((tok0 + r) * H + h) * dv + my_col + col) = __floats2bfloat162_rn(sum.x, sum.y);
+            }
+        }
+      cluster.sync();  // nobody leaves while another block may still read its shared memory
+      return;
+    }
+  }
 #pragma unroll
   for (int i = 0; i < TP; ++i)
 #pragma unroll
@@ -475,57 +522,75 @@ inline int mix_units(int H, int G, int dv, int R, int TP, int CP) {
   return G * ((tpg + TP - 1) / TP) * ((((dv + 15) & ~15) + CP * 64 - 1) / (CP * 64));
 }
 
-// Rows and keys per run of a launch: R * 256 + N, or 0 where shared memory holds no combination.
-inline int mix_mma_shape(int single, int H, int G, int d, int dv) {
+// How a launch cuts its work: rows, keys per run and warps of a block (rows 0: shared memory holds no cut).
+struct MixShape {
+  int R, N, W;
+};
+inline MixShape mix_mma_shape(int single, int H, int G, int d, int dv) {
   auto fits = [&](int R, int N, int limit) { return mix_mma_layout(H, G, d, dv, R, N).total <= limit; };
+  const int half = MIX_SMEM_MAX / 2 - 1024;  // two blocks a multiprocessor
   if (single) {
-    if (fits(1, 32, MIX_SMEM_MAX / 2 - 1024)) return 256 + 32;  // two blocks a multiprocessor
-    return fits(1, 16, MIX_SMEM_MAX) ? 256 + 16 : 0;
+    if (fits(1, 32, half)) return {1, 32, 8};
+    return {fits(1, 16, MIX_SMEM_MAX) ? 1 : 0, 16, 8};
   }
-  if (mix_units(H, G, dv, 16, 2, 1) <= MIX_WARPS_PROMPT) {
-    if (fits(16, 32, MIX_SMEM_MAX)) return 16 * 256 + 32;
-    if (fits(16, 16, MIX_SMEM_MAX)) return 16 * 256 + 16;
+  if (mix_units(H, G, dv, 16, 2, 1) <= 16) {
+    if (fits(16, 32, MIX_SMEM_MAX)) return {16, 32, 16};
+    if (fits(16, 16, MIX_SMEM_MAX)) return {16, 16, 16};
   }
   for (int R = 8; R <= 16; R += 8)
     for (int N = 32; N >= 16; N -= 16)
-      if (fits(R, N, MIX_SMEM_MAX)) return R * 256 + N;
-  return 0;
+      if (fits(R, N, MIX_SMEM_MAX)) return {R, N, 16};
+  return {0, 0, 0};
 }
 
-template <int R, int N, int TP, int CP, int DIM>
+template <int R, int N, int W, int TP, int CP, int DIM>
 int launch_mixed_mma_dim(const MixMmaArgs& a, int n_blocks, cudaStream_t stream) {
-  const int smem = mix_mma_layout(a.n_heads, a.n_kv_heads, a.d, a.dv, R, N).total;
-  auto kernel = mixed_attention_mma_kernel<R, N, TP, CP, DIM>;
+  const int exchange = R > 1 && a.n_splits > 1 ? TP * CP * 16 * W * 32 * (int)sizeof(float2) : 0;
+  const int smem = max(mix_mma_layout(a.n_heads, a.n_kv_heads, a.d, a.dv, R, N).total, exchange);
+  auto kernel = mixed_attention_mma_kernel<R, N, W, TP, CP, DIM>;
   cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (err != cudaSuccess) {
     mll_set_error("mixed attention (mma): cannot reserve %d bytes of shared memory: %s", smem, cudaGetErrorString(err));
     return (int)err;
   }
-  constexpr int WARPS = R == 1 ? MIX_WARPS_SINGLE : MIX_WARPS_PROMPT;
   const int units = mix_units(a.n_heads, a.n_kv_heads, a.dv, R, TP, CP);
-  const dim3 grid(n_blocks, (units + WARPS - 1) / WARPS, a.n_splits);
-  MLL_LAUNCH((kernel), grid, WARPS * 32, smem, stream, a);
+  cudaLaunchConfig_t config = {};
+  config.gridDim = dim3(n_blocks, (units + W - 1) / W, a.n_splits);
+  config.blockDim = dim3(W * 32);
+  config.dynamicSmemBytes = smem;
+  config.stream = stream;
+  cudaLaunchAttribute attr[1];
+  if (R > 1 && a.n_splits > 1) {
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = 1;
+    attr[0].val.clusterDim.y = 1;
+    attr[0].val.clusterDim.z = a.n_splits;
+    config.attrs = attr;
+    config.numAttrs = 1;
+  }
+  mll_launch_status = cudaLaunchKernelEx(&config, kernel, a);
   MLL_LAUNCH_CHECK();
   return 0;
 }
 
-template <int R, int N, int TP, int CP>
+template <int R, int N, int W, int TP, int CP>
 int launch_mixed_mma(const MixMmaArgs& a, int n_blocks, cudaStream_t stream) {
-  return a.d == 128 && a.dv == 128 ? launch_mixed_mma_dim<R, N, TP, CP, 128>(a, n_blocks, stream)
-                                   : launch_mixed_mma_dim<R, N, TP, CP, 0>(a, n_blocks, stream);
+  return a.d == 128 && a.dv == 128 ? launch_mixed_mma_dim<R, N, W, TP, CP, 128>(a, n_blocks, stream)
+                                   : launch_mixed_mma_dim<R, N, W, TP, CP, 0>(a, n_blocks, stream);
 }
 
 }  // namespace mll
 
 MLL_API int mll_mixed_attention_mma_supported(int dtype, int single, int n_heads, int n_kv_heads, int d, int dv) {
   return dtype == MLL_BF16 && d % 8 == 0 && d >= 8 && d <= 256 && dv % 8 == 0 && dv >= 8 && dv <= 256 && n_kv_heads > 0 &&
-         n_heads % n_kv_heads == 0 && mll::mix_mma_shape(single, n_heads, n_kv_heads, d, dv) != 0;
+         n_heads % n_kv_heads == 0 && mll::mix_mma_shape(single, n_heads, n_kv_heads, d, dv).R != 0;
 }
 
 // mix: float32; for prompts its entries must be bfloat16 values (the kernel takes them as such).
 // tile_seq / tile_row0: tiles of up to 128 query rows as (sequence, first row among the sequence's new tokens), n_tiles of
-// them; null: every sequence brings one token and n_tiles is the number of sequences.  n_splits > 1 (single tokens only)
-// cuts every context into that many runs and needs scratch: n_tiles * n_splits * H * dv floats.
+// them; null: every sequence brings one token and n_tiles is the number of sequences.  n_splits > 1 blocks share every
+// tile's keys: the blocks of a cluster for prompts (2, 4 or 8), else blocks that need scratch, n_tiles * n_splits * H * dv
+// floats.
 MLL_API int mll_mixed_attention_mma(const void* q, const void* k_cache, const void* v_cache, const int* seq_slot,
                                     const int* seq_ctx, const int* seq_qstart, const int* seq_qlen, const int* tile_seq,
                                     const int* tile_row0, const int* block_table, const float* mix, const float* bias,
@@ -535,28 +600,36 @@ MLL_API int mll_mixed_attention_mma(const void* q, const void* k_cache, const vo
   MLL_REQUIRE(mll_mixed_attention_mma_supported(MLL_BF16, single, n_heads, n_kv_heads, d, dv),
               "mixed attention (mma): %d heads of %d / %d over %d", n_heads, d, dv, n_kv_heads);
   MLL_REQUIRE(n_tiles >= 0 && window >= 0 && (single || tile_row0), "mixed attention (mma): bad tile list or window");
-  MLL_REQUIRE(n_splits >= 1 && n_splits <= 64 && (n_splits == 1 || (single && scratch)),
-              "mixed attention (mma): %d context splits need single tokens and scratch memory", n_splits);
+  MLL_REQUIRE(n_splits >= 1 && n_splits <= 64 && (n_splits == 1 || (single ? scratch != nullptr : 8 % n_splits == 0)),
+              "mixed attention (mma): %d context splits (single tokens: scratch memory; prompts: 1, 2, 4 or 8)", n_splits);
   if (n_tiles == 0) return 0;
   mll::MixMmaArgs a{(const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, seq_slot, seq_ctx,
                     seq_qstart, seq_qlen, tile_seq, tile_row0, block_table, mix, bias, (__nv_bfloat16*)out, scratch,
                     n_heads, n_kv_heads, d, dv, window, max_blocks, n_splits, scale};
-  const int shape = mll::mix_mma_shape(single, n_heads, n_kv_heads, d, dv), R = shape / 256, N = shape % 256;
+  const mll::MixShape shape = mll::mix_mma_shape(single, n_heads, n_kv_heads, d, dv);
+  const bool wide = shape.N == 32;
   int code;
-  if (R == 1) {
-    if (mll::mix_units(n_heads, n_kv_heads, dv, 1, 1, 1) <= mll::MIX_WARPS_SINGLE)
-      code = N == 32 ? mll::launch_mixed_mma<1, 32, 1, 1>(a, n_tiles, stream) : mll::launch_mixed_mma<1, 16, 1, 1>(a, n_tiles, stream);
+  if (shape.R == 1) {
+    if (mll::mix_units(n_heads, n_kv_heads, dv, 1, 1, 1) <= 8)
+      code = wide ? mll::launch_mixed_mma<1, 32, 8, 1, 1>(a, n_tiles, stream) : mll::launch_mixed_mma<1, 16, 8, 1, 1>(a, n_tiles, stream);
     else
-      code = N == 32 ? mll::launch_mixed_mma<1, 32, 1, 2>(a, n_tiles, stream) : mll::launch_mixed_mma<1, 16, 1, 2>(a, n_tiles, stream);
-  } else if (R == 8) {
-    code = N == 32 ? mll::launch_mixed_mma<8, 32, 2, 1>(a, n_tiles * 16, stream) : mll::launch_mixed_mma<8, 16, 2, 1>(a, n_tiles * 16, stream);
+      code = wide ? mll::launch_mixed_mma<1, 32, 8, 1, 2>(a, n_tiles, stream) : mll::launch_mixed_mma<1, 16, 8, 1, 2>(a, n_tiles, stream);
+  } else if (shape.R == 8) {
+    code = wide ? mll::launch_mixed_mma<8, 32, 16, 2, 1>(a, n_tiles * 16, stream) : mll::launch_mixed_mma<8, 16, 16, 2, 1>(a, n_tiles * 16, stream);
   } else {
-    code = N == 32 ? mll::launch_mixed_mma<16, 32, 2, 1>(a, n_tiles * 8, stream) : mll::launch_mixed_mma<16, 16, 2, 1>(a, n_tiles * 8, stream);
+    code = wide ? mll::launch_mixed_mma<16, 32, 16, 2, 1>(a, n_tiles * 8, stream) : mll::launch_mixed_mma<16, 16, 16, 2, 1>(a, n_tiles * 8, stream);
   }
-  if (code != 0 || n_splits == 1) return code;
+  if (code != 0 || n_splits == 1 || !single) return code;
   const long long items = (long long)n_tiles * (n_heads * dv / 2);
   MLL_LAUNCH((mll::mixed_attention_sum_kernel), (unsigned)((items + 255) / 256), 256, 0, stream, scratch, seq_qstart,
              (__nv_bfloat16*)out, n_tiles, n_splits, n_heads * dv);
   MLL_LAUNCH_CHECK();
   return 0;
+}
+
+// Blocks along the rows that a prompt tile of 128 rows becomes (what a choice of n_splits goes by), or 0.
+MLL_API int mll_mixed_attention_mma_blocks(int n_heads, int n_kv_heads, int d, int dv) {
+  const mll::MixShape shape = mll::mix_mma_shape(0, n_heads, n_kv_heads, d, dv);
+  if (shape.R == 0) return 0;
+  return 128 / shape.R * ((mll::mix_units(n_heads, n_kv_heads, dv, shape.R, 2, 1) + shape.W - 1) / shape.W);
 }

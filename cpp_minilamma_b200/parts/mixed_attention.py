@@ -128,8 +128,9 @@ class MixedHeadsAttention(Mixer):
         if (step.all_decode or (tiles and self.mix_narrow)) and K.mixed_attention_mma_supported(self.ctx.act_dtype, step.all_decode, *sizes):
             seqs = (q, cache.k, cache.v, step.seq_slot, step.seq_ctx, step.seq_qstart, step.seq_qlen)
             if tiles:
+                splits = K.mixed_attention_tile_splits(tiles["wide_seq"].shape[0], *sizes, self.ctx.multiprocessors)
                 K.mixed_attention_tiles(*seqs, tiles["wide_seq"], tiles["wide_row0"], cache.block_table, self.mix, self.bias,
-                                        out, *sizes, self.window, self.scale)
+                                        out, *sizes, self.window, self.scale, n_splits=splits)
                 return
             splits = K.local_attention_heads_splits(step.n_seqs, 1, self.ctx.multiprocessors)
             scratch = step.ws.buffer("attn.parts", (K.mixed_attention_single_scratch(step.n_seqs, self.n_heads, self.dv, splits),),

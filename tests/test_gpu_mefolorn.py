@@ -378,11 +378,12 @@ def test_mixed_attention_kernels(dtype, H, G, d, dv, window):
     if K.mixed_attention_mma_supported(dtype, False, H, G, d, dv):
         tile_seq = [s for s, n in enumerate(lens) for _ in range(0, n, 2 * K.PREFILL_TILE)]
         tile_row0 = [r for n in lens for r in range(0, n, 2 * K.PREFILL_TILE)]
-        out = torch.zeros((T, H * dv), dtype=dtype, device=DEV)
-        K.mixed_attention_tiles(qd, kc, vc, state.seq_slot, state.seq_ctx, state.seq_qstart, state.seq_qlen, _ints(tile_seq),
-                                _ints(tile_row0), table_dev, md, bd, out, H, G, d, dv, window, scale)
-        err = (out.cpu().double() - want).abs()
-        assert err.max().item() <= tol, ("prompt kernel", err.max().item(), tol, int(err.max(dim=1).values.argmax()))
+        for splits in (1, 2, 4, 8):  # blocks that share a tile's keys, many of them with none
+            out = torch.zeros((T, H * dv), dtype=dtype, device=DEV)
+            K.mixed_attention_tiles(qd, kc, vc, state.seq_slot, state.seq_ctx, state.seq_qstart, state.seq_qlen, _ints(tile_seq),
+                                    _ints(tile_row0), table_dev, md, bd, out, H, G, d, dv, window, scale, n_splits=splits)
+            err = (out.cpu().double() - want).abs()
+            assert err.max().item() <= tol, ("prompt kernel", splits, err.max().item(), tol, int(err.max(dim=1).values.argmax()))
     if K.mixed_attention_mma_supported(dtype, True, H, G, d, dv):
         one = make_step_state(DEV, [0, 1, 2, 3], [c - 1 for c in ctxs], [1] * 4)
         for splits in (1, 2, 7):
