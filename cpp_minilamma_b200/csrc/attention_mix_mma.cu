@@ -6,8 +6,8 @@
 //   1. S = q k^T by mma.sync: the 16 rows of a tile are R query rows of 16 / R heads of one key head's group; scores go to
 //      shared memory - for prompts as three bfloat16 planes that add up to all 24 bits of the float32 score.
 //   2. z = M S + b, sigmoid, mask; weights go to shared memory as bfloat16.  For prompts the mixing is three more mma.sync
-//      products (M is bfloat16, the planes are exact: a float32 product of float32 scores); for single tokens it is
-//      float32 FMAs, two an instruction.
+//      products (the planes are exact: a float32 product of float32 scores), or six where M has values that are no
+//      bfloat16 numbers and is cut into planes as well; for single tokens it is float32 FMAs, two an instruction.
 //   3. O += P V by mma.sync: a warp keeps TP x 16 rows x CP x 64 value columns in registers for the whole walk.
 // Nothing is normalised, so there is no running maximum and no rescaling, and context splits simply add up.
 // K and V of a run have one buffer each.  Single tokens: the next run's keys load while 2 and 3 work, its values while 1
@@ -39,11 +39,12 @@ struct MixMmaArgs {
   const int* tile_seq;    // prompt tiles of 128 rows, walked from the back; null: single tokens, grid x runs over the sequences
   const int* tile_row0;
   const int* block_table;
-  const float* mix;       // [H, H] or null; prompts need entries that are bfloat16 values
+  const float* mix;       // [H, H] or null
   const float* bias;      // [H] or null
   __nv_bfloat16* out;
   float* part;            // single tokens: [sequences, n_splits, H, dv] sums of the context's runs (n_splits > 1)
   int n_heads, n_kv_heads, d, dv, window, max_blocks;
+  int mix_planes;         // prompts: 1 where every entry of mix is a bfloat16 number, else 3
   int n_splits;           // blocks (grid z) that share a tile's runs; for prompts they are one cluster
   float scale;
 };
@@ -68,7 +69,7 @@ __host__ __device__ inline MixMmaLayout mix_mma_layout(int H, int G, int d, int 
   l.s = at; at += R > 1 ? 3 * l.hp * l.ps * 2 : H * l.ps * 4;
   l.p = at; at += l.hp * l.ps * 2;
   at = (at + 15) & ~15;
-  l.m = at; at += R > 1 ? l.hp * (l.hp + 8) * 2 : H * l.hp * 4;
+  l.m = at; at += R > 1 ? 3 * l.hp * (l.hp + 8) * 2 : H * l.hp * 4;
   l.b = at; at += l.hp * 4;
   l.total = at;
   return l;
@@ -106,6 +107,12 @@ __device__ __forceinline__ void mix_ldsm_trans(unsigned (&r)[4], unsigned at) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(at));
 }
+// as mma_16816, free to move between the fragment loads around it
+__device__ __forceinline__ void mix_mma(float (&c)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
 __device__ __forceinline__ void mix_sts(unsigned at, unsigned v) {
   asm volatile("st.shared.b32 [%0], %1;\n" ::"r"(at), "r"(v) : "memory");
 }
@@ -135,7 +142,7 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
   __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.p);
   __nv_bfloat16* planes = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.s);  // R > 1: three of them, hp * ps elements each
   float* m_s = reinterpret_cast<float*>(smem_raw + L.m);                     // R == 1: [H in][hp out], times -scale log2 e
-  __nv_bfloat16* mb_s = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.m);    // R > 1: [hp out][hp in + 8]
+  __nv_bfloat16* mb_s = reinterpret_cast<__nv_bfloat16*>(smem_raw + L.m);    // R > 1: planes of [hp out][hp in + 8]
   float* b_s = reinterpret_cast<float*>(smem_raw + L.b);                     // times -log2 e
 
   const int tid = threadIdx.x, lane = tid & 31;
@@ -207,7 +214,14 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
   if (R == 1) {
     for (int i = tid; i < H * L.hp; i += THREADS) m_s[i] = mix_at(i % L.hp, i / L.hp) * (-MIX_LOG2E * a.scale);
   } else {
-    for (int i = tid; i < L.hp * L.hp; i += THREADS) mb_s[i / L.hp * (L.hp + 8) + i % L.hp] = __float2bfloat16_rn(mix_at(i / L.hp, i % L.hp));
+    for (int i = tid; i < L.hp * L.hp; i += THREADS) {
+      float rest = mix_at(i / L.hp, i % L.hp);
+      for (int p = 0; p < a.mix_planes; ++p) {
+        const __nv_bfloat16 term = __float2bfloat16_rn(rest);
+        mb_s[(p * L.hp + i / L.hp) * (L.hp + 8) + i % L.hp] = term;
+        rest -= __bfloat162float(term);  // exact
+      }
+    }
     // heads that do not exist enter the products with a factor of 0: their scores must be numbers
     for (int i = tid; i < 3 * (L.hp - H) * L.ps; i += THREADS)
       planes[(size_t)(i / ((L.hp - H) * L.ps)) * L.hp * L.ps + (size_t)H * L.ps + i % ((L.hp - H) * L.ps)] = __float2bfloat16_rn(0.f);
@@ -255,23 +269,21 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
   auto weigh_values = [&](auto all) {
 #pragma unroll
     for (int ks = 0; ks < N / 16; ++ks) {
-      unsigned pf[TP][4];
+      unsigned pf[TP][4], vf[2][4];
 #pragma unroll
       for (int i = 0; i < TP; ++i) mix_ldsm(pf[i], p_at + i * p_step + ks * 32);
       const unsigned v = v_at + ks * 32 * L.vs;
+      mix_ldsm_trans(vf[0], v);
 #pragma unroll
-      for (int c = 0; c < CP; ++c)
+      for (int np = 0; np < CP * 4; ++np)
+        if (decltype(all)::value || np * 16 < my_cols) {
+          if (np + 1 < CP * 4 && (decltype(all)::value || np * 16 + 16 < my_cols)) mix_ldsm_trans(vf[(np + 1) & 1], v + np * 32 + 32);
 #pragma unroll
-        for (int np = 0; np < 4; ++np)
-          if (decltype(all)::value || c * 64 + np * 16 < my_cols) {
-            unsigned vf[4];
-            mix_ldsm_trans(vf, v + c * 128 + np * 32);
-#pragma unroll
-            for (int i = 0; i < TP; ++i) {
-              mma_16816(o[i][c][2 * np], pf[i], vf[0], vf[1]);
-              mma_16816(o[i][c][2 * np + 1], pf[i], vf[2], vf[3]);
-            }
+          for (int i = 0; i < TP; ++i) {
+            mix_mma(o[i][np / 4][np % 4 * 2], pf[i], vf[np & 1][0], vf[np & 1][1]);
+            mix_mma(o[i][np / 4][np % 4 * 2 + 1], pf[i], vf[np & 1][2], vf[np & 1][3]);
           }
+        }
     }
   };
   const float neg_scale = -MIX_LOG2E * a.scale;
@@ -297,16 +309,28 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
         for (int n = 0; n < 2; ++n)
 #pragma unroll
           for (int i = 0; i < 4; ++i) acc[m][n][i] = 0.f;
-#pragma unroll 4
-      for (int e = 0; e < (L.qs - 8) * 2; e += 32) {
-        unsigned qf[QP][4], kf[4];
-        mix_ldsm(kf, k_at + e);
+      unsigned qf[2][QP][4], kf[2][4];  // this step's fragments and the next one's
+      auto fetch = [&](int to, int e) {
+        mix_ldsm(kf[to], k_at + e);
 #pragma unroll
-        for (int m = 0; m < QP; ++m) mix_ldsm(qf[m], q_at + m * q_step + e);
+        for (int m = 0; m < QP; ++m) mix_ldsm(qf[to][m], q_at + m * q_step + e);
+      };
+      auto multiply = [&](int from) {
 #pragma unroll
         for (int m = 0; m < QP; ++m) {
-          mma_16816(acc[m][0], qf[m], kf[0], kf[1]);
-          mma_16816(acc[m][1], qf[m], kf[2], kf[3]);
+          mix_mma(acc[m][0], qf[from][m], kf[from][0], kf[from][1]);
+          mix_mma(acc[m][1], qf[from][m], kf[from][2], kf[from][3]);
+        }
+      };
+      const int e_end = (L.qs - 8) * 2;
+      fetch(0, 0);
+#pragma unroll 4
+      for (int e = 0; e < e_end; e += 64) {
+        if (e + 32 < e_end) fetch(1, e + 32);
+        multiply(0);
+        if (e + 32 < e_end) {
+          if (e + 64 < e_end) fetch(0, e + 64);
+          multiply(1);
         }
       }
 #pragma unroll
@@ -380,19 +404,33 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
         unsigned m = base + L.m + ((h + ld_row) * (L.hp + 8) + ld_col) * 2;
         unsigned s = base + L.s + (ld_row * L.ps + r * SS + ld_col) * 2;
         for (int kt = 0; kt < L.hp; kt += 16, m += 32, s += L.ps * 32) {
-          unsigned mf[4];
+          unsigned mf[4], sf[3][N / 16][4];
           mix_ldsm(mf, m);
 #pragma unroll
-          for (int p = 2; p >= 0; --p) {
-            unsigned sf[N / 16][4];
+          for (int p = 0; p < 3; ++p)
 #pragma unroll
-            for (int n = 0; n < N / 16; ++n) mix_ldsm_trans(sf[n], s + p * plane + n * 32);
+            for (int n = 0; n < N / 16; ++n) mix_ldsm_trans(sf[p][n], s + p * plane + n * 32);
+          if (a.mix_planes > 1) {  // the smaller terms of M with the terms of S that still count, smallest first
 #pragma unroll
-            for (int n = 0; n < N / 16; ++n) {
-              mma_16816(z[2 * n], mf, sf[n][0], sf[n][1]);
-              mma_16816(z[2 * n + 1], mf, sf[n][2], sf[n][3]);
+            for (int k = 2; k >= 1; --k) {
+              unsigned mk[4];
+              mix_ldsm(mk, m + k * L.hp * (L.hp + 8) * 2);
+#pragma unroll
+              for (int p = 2 - k; p >= 0; --p)
+#pragma unroll
+                for (int n = 0; n < N / 16; ++n) {
+                  mix_mma(z[2 * n], mk, sf[p][n][0], sf[p][n][1]);
+                  mix_mma(z[2 * n + 1], mk, sf[p][n][2], sf[p][n][3]);
+                }
             }
           }
+#pragma unroll
+          for (int p = 2; p >= 0; --p)
+#pragma unroll
+            for (int n = 0; n < N / 16; ++n) {
+              mix_mma(z[2 * n], mf, sf[p][n][0], sf[p][n][1]);
+              mix_mma(z[2 * n + 1], mf, sf[p][n][2], sf[p][n][3]);
+            }
         }
         const float b0 = b_s[h + g], b1 = b_s[h + g + 8];
         const unsigned to = base + L.p + ((h + g) * L.ps + r * SS + 2 * t) * 2, to8 = to + 16 * L.ps;
@@ -586,7 +624,7 @@ MLL_API int mll_mixed_attention_mma_supported(int dtype, int single, int n_heads
          n_heads % n_kv_heads == 0 && mll::mix_mma_shape(single, n_heads, n_kv_heads, d, dv).R != 0;
 }
 
-// mix: float32; for prompts its entries must be bfloat16 values (the kernel takes them as such).
+// mix: float32; mix_planes: for prompts, 1 says that every entry is a bfloat16 number, 3 that it may be any float32.
 // tile_seq / tile_row0: tiles of up to 128 query rows as (sequence, first row among the sequence's new tokens), n_tiles of
 // them; null: every sequence brings one token and n_tiles is the number of sequences.  n_splits > 1 blocks share every
 // tile's keys: the blocks of a cluster for prompts (2, 4 or 8), else blocks that need scratch, n_tiles * n_splits * H * dv
@@ -595,17 +633,18 @@ MLL_API int mll_mixed_attention_mma(const void* q, const void* k_cache, const vo
                                     const int* seq_ctx, const int* seq_qstart, const int* seq_qlen, const int* tile_seq,
                                     const int* tile_row0, const int* block_table, const float* mix, const float* bias,
                                     void* out, float* scratch, int n_tiles, int n_heads, int n_kv_heads, int d, int dv,
-                                    int window, int max_blocks, int n_splits, float scale, cudaStream_t stream) {
+                                    int window, int max_blocks, int mix_planes, int n_splits, float scale, cudaStream_t stream) {
   const int single = tile_seq == nullptr;
   MLL_REQUIRE(mll_mixed_attention_mma_supported(MLL_BF16, single, n_heads, n_kv_heads, d, dv),
               "mixed attention (mma): %d heads of %d / %d over %d", n_heads, d, dv, n_kv_heads);
   MLL_REQUIRE(n_tiles >= 0 && window >= 0 && (single || tile_row0), "mixed attention (mma): bad tile list or window");
   MLL_REQUIRE(n_splits >= 1 && n_splits <= 64 && (n_splits == 1 || (single ? scratch != nullptr : 8 % n_splits == 0)),
               "mixed attention (mma): %d context splits (single tokens: scratch memory; prompts: 1, 2, 4 or 8)", n_splits);
+  MLL_REQUIRE(mix_planes == 1 || mix_planes == 3, "mixed attention (mma): a matrix of 1 or 3 planes, not %d", mix_planes);
   if (n_tiles == 0) return 0;
   mll::MixMmaArgs a{(const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, seq_slot, seq_ctx,
                     seq_qstart, seq_qlen, tile_seq, tile_row0, block_table, mix, bias, (__nv_bfloat16*)out, scratch,
-                    n_heads, n_kv_heads, d, dv, window, max_blocks, n_splits, scale};
+                    n_heads, n_kv_heads, d, dv, window, max_blocks, mix_planes, n_splits, scale};
   const mll::MixShape shape = mll::mix_mma_shape(single, n_heads, n_kv_heads, d, dv);
   const bool wide = shape.N == 32;
   int code;

@@ -1573,7 +1573,7 @@ def mixed_attention_mma_supported(dtype: torch.dtype, single: bool, n_heads: int
 
 
 def _mixed_mma(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_qlen, tile_seq, tile_row0, block_table, mix, bias,
-               out, scratch, n_tiles, n_heads, n_kv_heads, d, dv, window, n_splits, scale, what) -> None:
+               out, scratch, n_tiles, n_heads, n_kv_heads, d, dv, window, n_splits, scale, what, mix_planes: int = 3) -> None:
     _need(q, "mixed attention q", torch.bfloat16)
     _check_mixed(q, k_cache, v_cache, out, mix, bias, n_heads, n_kv_heads, d, dv)
     for name, t in (("seq_slot", seq_slot), ("seq_ctx", seq_ctx), ("seq_qstart", seq_qstart), ("seq_qlen", seq_qlen)):
@@ -1583,37 +1583,36 @@ def _mixed_mma(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_qlen, til
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(seq_slot), _ptr(seq_ctx), _ptr(seq_qstart), _ptr(seq_qlen),
         _ptr(tile_seq), _ptr(tile_row0), _ptr(block_table), _ptr(mix), _ptr(bias), _ptr(out), _ptr(scratch),
         ctypes.c_int(n_tiles), ctypes.c_int(n_heads), ctypes.c_int(n_kv_heads), ctypes.c_int(d), ctypes.c_int(dv),
-        ctypes.c_int(window), ctypes.c_int(block_table.shape[1]), ctypes.c_int(n_splits), ctypes.c_float(scale),
-        _stream()), what, kernels=2 if n_splits > 1 and tile_seq is None else 1)
+        ctypes.c_int(window), ctypes.c_int(block_table.shape[1]), ctypes.c_int(mix_planes), ctypes.c_int(n_splits),
+        ctypes.c_float(scale), _stream()), what, kernels=2 if n_splits > 1 and tile_seq is None else 1)
 
 
 def mixed_attention_tiles(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_qlen, tile_seq, tile_row0, block_table,
                           mix, bias, out, n_heads: int, n_kv_heads: int, d: int, dv: int, window: int, scale: float,
-                          n_splits: int = 1) -> None:
+                          n_splits: int = 1, narrow_mix: bool = False) -> None:
     """`mixed_attention` for prompt steps in bfloat16 on tensor cores: the work is a list of tiles of up to twice
-    PREFILL_TILE query rows, (sequence, first row among the sequence's new tokens), walked from its end.  `mix` must hold
-    bfloat16 values (in float32): the scores pass it as exact sums of bfloat16 terms.  `n_splits` (1, 2, 4 or 8): blocks
-    of a cluster that share every tile's keys."""
+    PREFILL_TILE query rows, (sequence, first row among the sequence's new tokens), walked from its end.  The scores pass
+    `mix` as exact sums of bfloat16 terms; `narrow_mix` says that every entry of `mix` is a bfloat16 number itself, which
+    halves those products.  `n_splits` (1, 2, 4 or 8): blocks of a cluster that share every tile's keys."""
     for name, t in (("tile_seq", tile_seq), ("tile_row0", tile_row0)):
         _need(t, f"mixed attention {name}", torch.int32, 1)
     if tile_seq.shape != tile_row0.shape:
         raise KernelError("mixed attention: the tile lists differ in length")
     _mixed_mma(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_qlen, tile_seq, tile_row0, block_table, mix, bias, out,
                None, tile_seq.shape[0], n_heads, n_kv_heads, d, dv, window, n_splits, scale,
-               "mixed_attention_mma")
+               "mixed_attention_mma", 1 if narrow_mix or mix is None else 3)
 
 
 def mixed_attention_tile_splits(n_tiles: int, n_heads: int, n_kv_heads: int, d: int, dv: int, multiprocessors: int) -> int:
-    """Blocks that should share a prompt tile's keys: as many as the device has multiprocessors for, and once more where a
-    second wave of smaller pieces evens out the tiles' unequal numbers of keys."""
+    """Blocks that should share a prompt tile's keys: as many as give the device two waves of blocks, and two at least up
+    to four waves (smaller pieces even out the tiles' unequal numbers of keys).  Measured at 2,048 tokens under a window of
+    1,024, 1 / 2 / 4 blocks a tile: 16 heads over 4 of 128 (128 tiles) 147 / 139 / 151 us, 32 over 8 (256 tiles)
+    299 / 266 / 336 us."""
     blocks = n_tiles * int(lib().mll_mixed_attention_mma_blocks(n_heads, n_kv_heads, d, dv))
     splits = 1
-    while splits < 8 and 2 * splits * blocks <= MIXED_TILE_WAVES * max(multiprocessors, 1):
+    while splits < 8 and 2 * splits * blocks <= (4 if splits == 1 else 2) * max(multiprocessors, 1):
         splits *= 2
     return splits
-
-
-MIXED_TILE_WAVES = 2
 
 
 def mixed_attention_single_scratch(n_seqs: int, n_heads: int, dv: int, n_splits: int) -> int:

@@ -58,7 +58,7 @@ class MixedHeadsAttention(Mixer):
         self.qkv: Optional[Linear] = None
         self.o: Optional[Linear] = None
         self.q_weight = self.k_weight = self.mix = self.bias = None
-        self.mix_narrow = True  # the mixing matrix holds bfloat16 values: what the tensor-core prompt kernel takes
+        self.mix_narrow = True  # the mixing matrix holds bfloat16 numbers: fewer products in the prompt kernel
 
     def weight_specs(self) -> List[WeightSpec]:
         D, H, G = self.ctx.hidden_size, self.n_heads, self.n_kv_heads
@@ -125,12 +125,12 @@ class MixedHeadsAttention(Mixer):
     def _attend(self, step, q, cache, out) -> None:
         sizes = (self.n_heads, self.n_kv_heads, self.d, self.dv)
         tiles = step.meta.get(self.step_metadata_key()) if not step.all_decode else None
-        if (step.all_decode or (tiles and self.mix_narrow)) and K.mixed_attention_mma_supported(self.ctx.act_dtype, step.all_decode, *sizes):
+        if (step.all_decode or tiles) and K.mixed_attention_mma_supported(self.ctx.act_dtype, step.all_decode, *sizes):
             seqs = (q, cache.k, cache.v, step.seq_slot, step.seq_ctx, step.seq_qstart, step.seq_qlen)
             if tiles:
                 splits = K.mixed_attention_tile_splits(tiles["wide_seq"].shape[0], *sizes, self.ctx.multiprocessors)
                 K.mixed_attention_tiles(*seqs, tiles["wide_seq"], tiles["wide_row0"], cache.block_table, self.mix, self.bias,
-                                        out, *sizes, self.window, self.scale, n_splits=splits)
+                                        out, *sizes, self.window, self.scale, n_splits=splits, narrow_mix=self.mix_narrow)
                 return
             splits = K.local_attention_heads_splits(step.n_seqs, 1, self.ctx.multiprocessors)
             scratch = step.ws.buffer("attn.parts", (K.mixed_attention_single_scratch(step.n_seqs, self.n_heads, self.dv, splits),),
