@@ -665,11 +665,20 @@ def llama_like_config(size):
         "tie_word_embeddings": False})
 
 
-def kernel_times_of_a_step(llm, entries_of, launches=3):
-    """Device time of every kernel of this library in one eager step (CUDA events around each launch), after two
-    warm-up steps of the same kind: {kernel: (calls, ms)}."""
+def kernel_times_of_a_step(llm, entries_of):
+    """Device time of every kernel of this library in one eager step on one stream (CUDA events around each launch),
+    after two warm-up steps of the same kind: {kernel: (calls, ms)}."""
     from cpp_minilamma_b200.csrc import kernels as K
+    from cpp_minilamma_b200.parts import branches
     import torch
+    beside, branches.USE_SIDE_STREAMS = branches.USE_SIDE_STREAMS, False
+    try:
+        return _kernel_times_of_a_step(llm, entries_of, K, torch)
+    finally:
+        branches.USE_SIDE_STREAMS = beside
+
+
+def _kernel_times_of_a_step(llm, entries_of, K, torch):
     for _ in range(2):
         slots, entries = entries_of()
         llm.engine.step_borrowed(entries)

@@ -341,6 +341,7 @@ EMBEDDING_ENTRY = -1  # the key of the embedding's per-sequence state among the 
 
 class Mixer(Part):
     role = "mixer"
+    workspace: Optional[str] = None  # family of its workspace buffers' names: mixers of two families share none of them
     takes_prenormed = False  # True: `h` may be a PreNormed
     adds_residual = False    # True: forward has a keyword `into` (a ResidualTarget or None) and may return a PreNormed
 

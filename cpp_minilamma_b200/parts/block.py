@@ -20,6 +20,7 @@ from __future__ import annotations
 from dataclasses import replace
 from typing import List
 
+from .branches import run_both
 from .mlp import NoFeedForward
 from .base import Block, NormedDelta, PendingSum, ResidualTarget, ScaledDelta, register_part
 
@@ -84,7 +85,8 @@ class ParallelBlock(Block):
 class ParallelTwoNormsBlock(Block):
     """Two norms of one stream:   x' = x + mixer(norm_m(x)) + feed_forward(norm_f(x)), norms "mixer" and "feed_forward".
     The norms run together where their kind has a kernel for the pair (`Norm.forward_pair`); all outputs - the mixer's
-    may be a `PendingSum` itself - stay pending until the next norm."""
+    may be a `PendingSum` itself - stay pending until the next norm.  In steps of single tokens the two sub-layers run on
+    two streams."""
 
     capturable = True
 
@@ -96,8 +98,8 @@ class ParallelTwoNormsBlock(Block):
         if isinstance(layer.feed_forward, NoFeedForward):
             return layer.mixer.forward(step, norm.forward(step, x, pending), cache)
         h, h_ff = norm.forward_pair(step, x, pending, layer.norms["feed_forward"])
-        mixed = layer.mixer.forward(step, h, cache)
-        fed = layer.feed_forward.forward(step, h_ff)
+        mixed, fed = run_both(step, self.ctx, "feed_forward", lambda: layer.mixer.forward(step, h, cache),
+                              lambda: layer.feed_forward.forward(step, h_ff))
         return replace(mixed, third=fed) if isinstance(mixed, PendingSum) else PendingSum(mixed, fed)
 
 

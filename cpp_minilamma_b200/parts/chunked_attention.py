@@ -81,6 +81,7 @@ class ChunkedAttention(Mixer):
     """
 
     capturable = True
+    workspace = "attention"
 
     def __init__(self, params, ctx: BuildContext):
         super().__init__(params, ctx)

@@ -48,6 +48,7 @@ class LatentAttention(Mixer):
     """
 
     capturable = True
+    workspace = "attention"
 
     def __init__(self, params, ctx: BuildContext):
         super().__init__(params, ctx)

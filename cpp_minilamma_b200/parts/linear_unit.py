@@ -27,6 +27,7 @@ class LinearRecurrentUnit(Mixer):
     "conv_bias", "ra", "ra_bias", "ri", "ri_bias", "lam", "o"."""
 
     capturable = True
+    workspace = "lru"
 
     def __init__(self, params, ctx: BuildContext):
         super().__init__(params, ctx)

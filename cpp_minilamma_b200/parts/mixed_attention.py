@@ -37,6 +37,7 @@ class MixedHeadsAttention(Mixer):
     """
 
     capturable = True
+    workspace = "attention"
 
     def __init__(self, params, ctx: BuildContext):
         super().__init__(params, ctx)

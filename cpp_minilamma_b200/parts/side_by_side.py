@@ -5,12 +5,14 @@
 `left` and `right` are any two registered mixers (attention beside a recurrent layer, say); each keeps what it
 needs in the cache - one of them keys and values, the other a fixed-size state, or either both - and the pair asks the
 cache for the union.  Nothing is added here: the pair hands both results on as a `PendingSum` with the two
-weights, and the norm kernel that reads the residual stream next forms the weighted sum in float32 on its way in.
+weights, and the norm kernel that reads the residual stream next forms the weighted sum in float32 on its way in.  In
+steps of single tokens two mixers whose workspace buffers are of different families run on two streams.
 """
 from __future__ import annotations
 
 from typing import List
 
+from .branches import run_both
 from .base import BuildContext, CacheNeed, Mixer, PartSpec, PendingSum, StateNeed, WeightSpec, build_part, register_part
 
 
@@ -24,6 +26,9 @@ class SideBySideMixer(Mixer):
         self.right: Mixer = build_part("mixer", _as_spec(params["right"]), ctx)
         self.scale_left = float(params.get("scale_left", 1.0))
         self.scale_right = float(params.get("scale_right", 1.0))
+        # two streams only where no scratch buffer is shared
+        self.apart = (self.left.workspace is not None and self.right.workspace is not None
+                      and self.left.workspace != self.right.workspace)
         self.capturable = self.left.capturable and self.right.capturable
         left, right = self.left.cache_need(), self.right.cache_need()
         if left.kv is not None and right.kv is not None:
@@ -52,8 +57,8 @@ class SideBySideMixer(Mixer):
         return CacheNeed(kv=left.kv if left.kv is not None else right.kv, state=StateNeed(tensors) if tensors else None)
 
     def forward(self, step, h, cache):
-        first = self.left.forward(step, h, cache)
-        second = self.right.forward(step, h, cache)
+        first, second = run_both(step, self.ctx, "side_by_side", lambda: self.left.forward(step, h, cache),
+                                 lambda: self.right.forward(step, h, cache), self.apart)
         if first.data_ptr() == second.data_ptr():
             raise RuntimeError("side-by-side mixers: both results live in the same workspace buffer (give one an out_name)")
         return PendingSum(first, second, self.scale_left, self.scale_right)

@@ -55,6 +55,7 @@ class Retention(Mixer):
     names {"q","k","v","g","o"}: tensor names."""
 
     capturable = True
+    workspace = "mix"
 
     def __init__(self, params, ctx: BuildContext):
         super().__init__(params, ctx)
@@ -118,6 +119,7 @@ class GatedDeltaRule(Mixer):
     "A_log", "g1", "g2", "norm", "o"; decay_rank, gate_rank: inner sizes of the two low-rank pairs (-1: as stored)."""
 
     capturable = True
+    workspace = "mix"
 
     def __init__(self, params, ctx: BuildContext):
         super().__init__(params, ctx)
@@ -212,6 +214,7 @@ class GatedLinearAttention(Mixer):
     names: tensor names for "q", "k", "v", "g", "a1", "a2", "a2_bias", "norm", "o"."""
 
     capturable = True
+    workspace = "gla"
 
     def __init__(self, params, ctx: BuildContext):
         super().__init__(params, ctx)
@@ -288,6 +291,7 @@ class StateSpace(Mixer):
     names: tensor names for "in", "conv", "conv_bias", "dt_bias", "A_log", "D", "norm", "o"."""
 
     capturable = True
+    workspace = "ssd"
 
     def __init__(self, params, ctx: BuildContext):
         super().__init__(params, ctx)
