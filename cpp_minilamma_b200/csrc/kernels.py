@@ -1615,6 +1615,13 @@ def mixed_attention_tile_splits(n_tiles: int, n_heads: int, n_kv_heads: int, d: 
     return splits
 
 
+def mixed_attention_single_splits(n_seqs: int, multiprocessors: int) -> int:
+    """Context splits of a single-token step: as many blocks as two a multiprocessor hold at once (a second wave costs more
+    than the shorter runs save: 64 sequences at 32 heads over 8 of 128, 4 / 5 splits 71 / 94 us), at most 16 a sequence; a
+    function of the batch size alone, so that a captured step keeps its launch."""
+    return max(1, min(16, 2 * max(multiprocessors, 1) // max(n_seqs, 1)))
+
+
 def mixed_attention_single_scratch(n_seqs: int, n_heads: int, dv: int, n_splits: int) -> int:
     return n_seqs * n_splits * n_heads * dv
 

@@ -65,8 +65,8 @@ class MixedHeadsAttention(Mixer):
         D, H, G = self.ctx.hidden_size, self.n_heads, self.n_kv_heads
         specs = [WeightSpec(self.names["q"], (H * self.d, D)), WeightSpec(self.names["k"], (G * self.d, D)),
                  WeightSpec(self.names["v"], (G * self.dv, D)), WeightSpec(self.names["o"], (D, H * self.dv))]
-        if "mix" in self.names:  # a score is float32: so is what mixes it
-            specs.append(WeightSpec(self.names["mix"], (H, H), kind="vector"))
+        if "mix" in self.names:
+            specs.append(WeightSpec(self.names["mix"], (H, H)))
         if "bias" in self.names:
             specs.append(WeightSpec(self.names["bias"], (H,), kind="vector"))
         if self.qk_norm:
@@ -86,7 +86,7 @@ class MixedHeadsAttention(Mixer):
         del mats, fused
         self.o = Linear(store.take(self.names["o"]), self.names["o"])
         if "mix" in self.names:
-            self.mix = store.take(self.names["mix"])
+            self.mix = store.take(self.names["mix"]).float()  # a score is float32: so is what mixes it
             self.mix_narrow = bool((self.mix.to(torch.bfloat16).float() == self.mix).all())
         if "bias" in self.names:
             self.bias = store.take(self.names["bias"])
@@ -133,7 +133,7 @@ class MixedHeadsAttention(Mixer):
                 K.mixed_attention_tiles(*seqs, tiles["wide_seq"], tiles["wide_row0"], cache.block_table, self.mix, self.bias,
                                         out, *sizes, self.window, self.scale, n_splits=splits, narrow_mix=self.mix_narrow)
                 return
-            splits = K.local_attention_heads_splits(step.n_seqs, 1, self.ctx.multiprocessors)
+            splits = K.mixed_attention_single_splits(step.n_seqs, self.ctx.multiprocessors)
             scratch = step.ws.buffer("attn.parts", (K.mixed_attention_single_scratch(step.n_seqs, self.n_heads, self.dv, splits),),
                                      torch.float32) if splits > 1 else None
             K.mixed_attention_single(*seqs, cache.block_table, self.mix, self.bias, out, step.n_seqs, *sizes, self.window,
