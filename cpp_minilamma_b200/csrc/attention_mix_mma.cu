@@ -125,8 +125,8 @@ __device__ __forceinline__ void mix_copy16(unsigned at, const void* src, bool va
 }
 
 // DIM: the head size of keys and values where it is known at compile time (strides and word counts are then constants), or 0.
-// W warps a block; with 8 of them two blocks share a multiprocessor.
-template <int R, int N, int W, int TP, int CP, int DIM>
+// W warps a block; with 8 of them two blocks share a multiprocessor.  CUT: the mixing matrix comes in three terms.
+template <int R, int N, int W, int TP, int CP, int DIM, bool CUT>
 __global__ void __launch_bounds__(W * 32, W == 8 ? 2 : 1)
 mixed_attention_mma_kernel(MixMmaArgs a) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -216,7 +216,7 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
   } else {
     for (int i = tid; i < L.hp * L.hp; i += THREADS) {
       float rest = mix_at(i / L.hp, i % L.hp);
-      for (int p = 0; p < a.mix_planes; ++p) {
+      for (int p = 0; p < (CUT ? 3 : 1); ++p) {
         const __nv_bfloat16 term = __float2bfloat16_rn(rest);
         mb_s[(p * L.hp + i / L.hp) * (L.hp + 8) + i % L.hp] = term;
         rest -= __bfloat162float(term);  // exact
@@ -410,7 +410,7 @@ mixed_attention_mma_kernel(MixMmaArgs a) {
           for (int p = 0; p < 3; ++p)
 #pragma unroll
             for (int n = 0; n < N / 16; ++n) mix_ldsm_trans(sf[p][n], s + p * plane + n * 32);
-          if (a.mix_planes > 1) {  // the smaller terms of M with the terms of S that still count, smallest first
+          if (CUT) {  // the smaller terms of M with the terms of S that still count, smallest first
 #pragma unroll
             for (int k = 2; k >= 1; --k) {
               unsigned mk[4];
@@ -581,11 +581,11 @@ inline MixShape mix_mma_shape(int single, int H, int G, int d, int dv) {
   return {0, 0, 0};
 }
 
-template <int R, int N, int W, int TP, int CP, int DIM>
-int launch_mixed_mma_dim(const MixMmaArgs& a, int n_blocks, cudaStream_t stream) {
+template <int R, int N, int W, int TP, int CP, int DIM, bool CUT>
+int launch_mixed_mma_cut(const MixMmaArgs& a, int n_blocks, cudaStream_t stream) {
   const int exchange = R > 1 && a.n_splits > 1 ? TP * CP * 16 * W * 32 * (int)sizeof(float2) : 0;
   const int smem = max(mix_mma_layout(a.n_heads, a.n_kv_heads, a.d, a.dv, R, N).total, exchange);
-  auto kernel = mixed_attention_mma_kernel<R, N, W, TP, CP, DIM>;
+  auto kernel = mixed_attention_mma_kernel<R, N, W, TP, CP, DIM, CUT>;
   cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (err != cudaSuccess) {
     mll_set_error("mixed attention (mma): cannot reserve %d bytes of shared memory: %s", smem, cudaGetErrorString(err));
@@ -609,6 +609,14 @@ int launch_mixed_mma_dim(const MixMmaArgs& a, int n_blocks, cudaStream_t stream)
   mll_launch_status = cudaLaunchKernelEx(&config, kernel, a);
   MLL_LAUNCH_CHECK();
   return 0;
+}
+
+template <int R, int N, int W, int TP, int CP, int DIM>
+int launch_mixed_mma_dim(const MixMmaArgs& a, int n_blocks, cudaStream_t stream) {
+  if constexpr (R > 1) {
+    if (a.mix_planes > 1) return launch_mixed_mma_cut<R, N, W, TP, CP, DIM, true>(a, n_blocks, stream);
+  }
+  return launch_mixed_mma_cut<R, N, W, TP, CP, DIM, false>(a, n_blocks, stream);
 }
 
 template <int R, int N, int W, int TP, int CP>

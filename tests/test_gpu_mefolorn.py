@@ -4,8 +4,8 @@ alone.
 Every test makes its own small configuration and weights (`tiny_mefolorn`).  float32 runs must agree with the oracle to
 2e-4 of the largest logit (at least 2e-4 absolute): with the test weights a sink left out, a window one token off, a lost
 state, scores mixed by the transposed matrix or a bias forgotten moves logits by percents.  bfloat16 runs are compared
-with the same unrounded oracle, so their bound is that of rounding noise: largest error at most 10 %, mean error at most
-2.5 % of the largest logit (the bound of the other designs' tests).  The sharp test is float32."""
+with the same unrounded oracle, so their bound is that of rounding noise: largest error at most 3 %, mean error at most
+0.5 % of the largest logit.  The sharp test is float32."""
 import json
 import os
 import subprocess
@@ -58,7 +58,7 @@ def close(got, ref, dtype, what):
     if dtype == "float32":
         assert err.max() <= 2e-4 * scale, f"{what}: err {err.max():.3e} of {scale:.2f}, first at row {row}"
         return
-    assert err.max() <= 1e-1 * scale and err.mean() <= 2.5e-2 * scale, \
+    assert err.max() <= 3e-2 * scale and err.mean() <= 5e-3 * scale, \
         f"{what}: max {err.max():.3e} mean {err.mean():.3e} of {scale:.2f}, worst row {row}"
 
 
