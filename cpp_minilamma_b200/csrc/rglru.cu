@@ -87,7 +87,7 @@ __device__ __forceinline__ float lru_conv(const LruArgs& a, int t, int c, int po
 }
 
 // What one channel brings to every token: the gates' biases, its rate, y's bias.
-struct LruChannel {
+struct __align__(16) LruChannel {
   float br, bi, rate, yb;
 };
 __device__ __forceinline__ LruChannel lru_channel(const LruArgs& a, int c) {
@@ -172,6 +172,8 @@ __global__ void __launch_bounds__(256) lru_gates_mma_kernel(LruArgs a, int row, 
   const int t0 = blockIdx.x * M, n = min(M, a.n_tokens - t0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, q = lane & 3;
   const int k_pad = (bs + 31) & ~31;
+  LruChannel* channel_s = reinterpret_cast<LruChannel*>(planes + (size_t)3 * M * row);  // of the block's channels
+  for (int i = threadIdx.x; i < min(bs, tile1 * 64) - tile0 * 64; i += 256) channel_s[i] = lru_channel(a, block * bs + tile0 * 64 + i);
   if (threadIdx.x < M && threadIdx.x < n) {
     const int t = t0 + threadIdx.x, seq = a.tok_seq[t];
     pos_s[threadIdx.x] = a.tok_pos[t];
@@ -257,14 +259,23 @@ __global__ void __launch_bounds__(256) lru_gates_mma_kernel(LruArgs a, int row, 
       rows[0][j] = reinterpret_cast<const uint4*>(w + (size_t)col * bs) + q;
       rows[1][j] = reinterpret_cast<const uint4*>(w + (size_t)(bs + col) * bs) + q;
     }
-#pragma unroll 4
-    for (int k = 0; k < k_pad; k += 32) {
+    uint4 next[2][NT];  // the matrices' words of the step ahead
+    auto fetch = [&](int k) {
       const bool in = k + 8 * q < bs;  // bs is a multiple of 8: eight inputs are inside or outside together
+#pragma unroll
+      for (int e = 0; e < 2; ++e)
+#pragma unroll
+        for (int j = 0; j < NT; ++j) next[e][j] = in && have[j] ? rows[e][j][k >> 3] : zero;
+    };
+    fetch(0);
+#pragma unroll 2
+    for (int k = 0; k < k_pad; k += 32) {
       uint4 b[2][NT];
 #pragma unroll
       for (int e = 0; e < 2; ++e)
 #pragma unroll
-        for (int j = 0; j < NT; ++j) b[e][j] = in && have[j] ? rows[e][j][k >> 3] : zero;
+        for (int j = 0; j < NT; ++j) b[e][j] = next[e][j];
+      if (k + 32 < k_pad) fetch(k + 32);
 #pragma unroll
       for (int p = 0; p < 3; ++p)
 #pragma unroll
@@ -286,7 +297,7 @@ __global__ void __launch_bounds__(256) lru_gates_mma_kernel(LruArgs a, int row, 
     for (int j = 0; j < NT; ++j) {
       const int c = c0 + 8 * j + 2 * q, full = block * bs + c;  // a pair of channels: bs is even, both or none
       if (c >= bs) continue;
-      const LruChannel ch0 = lru_channel(a, full), ch1 = lru_channel(a, full + 1);
+      const LruChannel ch0 = channel_s[c - tile0 * 64], ch1 = channel_s[c - tile0 * 64 + 1];
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -385,7 +396,11 @@ template <int WM, int MT, int NT>
 int launch_lru_gates_mma(const LruArgs& a, cudaStream_t stream) {
   constexpr int M = 16 * WM * MT;
   const int bs = a.width / a.blocks, row = lru_plane_row(bs), tiles = (bs + 63) / 64;
-  const size_t smem = (size_t)3 * M * row * 2;
+  // a block that walks more channels forms u once for all of them; enough blocks for the device come first
+  const int n_tiles = (a.n_tokens + M - 1) / M;
+  int passes = tiles;
+  while (passes > 1 && (long long)n_tiles * a.blocks * ((tiles + passes - 1) / passes) < mll_sm_count()) passes = (passes + 1) / 2;
+  const size_t smem = (size_t)3 * M * row * 2 + (size_t)passes * 64 * sizeof(LruChannel);
   auto kernel = lru_gates_mma_kernel<WM, MT, NT>;
   if (smem > 48 * 1024) {
     cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -394,10 +409,6 @@ int launch_lru_gates_mma(const LruArgs& a, cudaStream_t stream) {
       return (int)err;
     }
   }
-  // a block that walks more channels forms u once for all of them; enough blocks for the device come first
-  const int n_tiles = (a.n_tokens + M - 1) / M;
-  int passes = tiles;
-  while (passes > 1 && (long long)n_tiles * a.blocks * ((tiles + passes - 1) / passes) < mll_sm_count()) passes = (passes + 1) / 2;
   const dim3 grid(n_tiles, a.blocks * ((tiles + passes - 1) / passes));
   MLL_LAUNCH((kernel), grid, 256, smem, stream, a, row, passes);
   MLL_LAUNCH_CHECK();
@@ -426,7 +437,7 @@ int launch_lru_gates(const LruArgs& a, cudaStream_t stream) {
 
 // Whether the tensor-core version takes diagonal blocks of this size (bfloat16 matrices).
 MLL_API int mll_lru_mma_supported(int dtype, int bs) {
-  return dtype == MLL_BF16 && bs % 8 == 0 && bs >= 8 && (size_t)3 * 16 * mll::lru_plane_row(bs) * 2 <= 200 * 1024;
+  return dtype == MLL_BF16 && bs % 8 == 0 && bs >= 8 && (size_t)3 * 16 * mll::lru_plane_row(bs) * 2 <= 160 * 1024;  // and the channels' numbers beside them
 }
 
 // `mma`: gate_w is bfloat16 [n, 2, bs, bs] (rows are outputs), else float32 [n, bs(in), 2 bs(out)].
@@ -452,7 +463,7 @@ MLL_API int mll_lru_gates(const void* proj, const float* x_bias, const float* y_
     MLL_REQUIRE(mll_lru_mma_supported(dtype, bs), "linear recurrent unit: blocks of %d on tensor cores", bs);
     const size_t per16 = (size_t)3 * 16 * mll::lru_plane_row(bs) * 2;
     // a tall tile reads the matrices less often, a low one gives more blocks
-    if (n_tokens > 256 && 4 * per16 <= 200 * 1024) return mll::launch_lru_gates_mma<2, 2, 2>(a, stream);
+    if (n_tokens > 256 && 4 * per16 <= 190 * 1024) return mll::launch_lru_gates_mma<2, 2, 2>(a, stream);
     return mll::launch_lru_gates_mma<1, 1, 1>(a, stream);
   }
   if (dtype == MLL_F32) return mll::launch_lru_gates<float>(a, stream);
