@@ -331,7 +331,7 @@ def _mixed_reference(q, keys, values, pos0, scale, window, mix, bias, group):
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("H,G,d,dv,window", [
-    (4, 2, 16, 16, 40), (8, 2, 64, 64, 70), (8, 2, 96, 96, 1), (6, 3, 24, 40, 63), (16, 4, 128, 128, 100), (3, 3, 32, 8, 65),
+    (4, 2, 16, 16, 40), (8, 2, 64, 64, 70), (12, 4, 96, 80, 1), (6, 3, 24, 40, 63), (16, 4, 128, 128, 100), (3, 3, 32, 8, 65),
     (32, 8, 128, 128, 90), (24, 3, 16, 72, 0), (40, 5, 8, 16, 128), (5, 1, 6, 10, 33), (12, 1, 256, 256, 50), (1, 1, 8, 8, 17),
     (64, 8, 64, 64, 45)])
 def test_mixed_attention_kernels(dtype, H, G, d, dv, window):
@@ -467,7 +467,7 @@ def test_mixed_attention_without_matrix_or_bias():
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("W,n,taps", [(40, 2, 4), (160, 2, 4), (24, 24, 3), (30, 3, 1), (256, 1, 2), (200, 5, 5), (1024, 4, 4), (1, 1, 4)])
+@pytest.mark.parametrize("W,n,taps", [(40, 2, 4), (144, 2, 3), (24, 24, 3), (30, 3, 1), (256, 1, 2), (200, 5, 5), (1024, 4, 4), (1, 1, 4)])
 def test_linear_recurrent_unit_kernels(dtype, W, n, taps):
     """Gates, convolution state and scan against the recurrence walked token by token in float64: sequences of 150, 2, 1
     and 37 tokens, three of which go on from a state and convolution inputs that are not zero; portions shorter than
