@@ -4,3 +4,5 @@ from .llama import LlamaConfig, RopeScaling
 from .kupirax import KupiraxConfig
 from .sopanex import SopanexConfig
 from .badolix import BadolixConfig
+from .mefolorn import MefolornConfig
+from .gopitar import GopitarConfig

@@ -12,11 +12,17 @@
 // its own position), and a score may be capped smoothly (s <- cap * tanh(s / cap) after the scale).  A layer that reads
 // another layer's keys and values prepares its queries only (`write_kv` 0).
 //
-// Two kernels, for prompts and single tokens alike:
+// The projections may have biases and pass a short causal convolution over time, per channel of q, k and v, before the
+// rotation (the last taps - 1 inputs of every sequence, biases included, are state; nothing comes before the first token).
+//
+// Kernels, for prompts and single tokens alike:
 //   * prepare: one block per token.  q and k are each divided by the root mean square of their whole
 //     projection (all heads at once) and multiplied by a weight, the pairs of the first `rot`
 //     dimensions of every head are rotated by position * frequency (cos / sin from a table), q goes to
 //     a buffer and k, v into the pages of the cache.  All arithmetic in float32.
+//   * prepare behind a convolution: the same without norms; a thread owns four neighbouring channels (with their
+//     partners where the rotation pairs them) and walks a run of rows, with taps and last inputs in registers; a
+//     version of a channel a thread takes every other size.
 //   * attend: one block per (token, kv head) and the query heads of its group.  Pages of keys and values pass
 //     through shared memory; scores are float32 dot products over the head, the softmax runs online in
 //     float32.  Any d and dv (16-byte copies where rows are whole 16-byte words).
@@ -209,6 +215,217 @@ __global__ void __launch_bounds__(256) local_prepare_vec_kernel(LocalPrepArgs a)
     else
       reinterpret_cast<uint4*>((__nv_bfloat16*)a.k_cache + (((size_t)page * a.n_kv_heads + head) * MLL_PAGE + in_page) * a.d)[e] = v;
   }
+}
+
+struct ConvPrepArgs {
+  const void* qkv;        // [T, ld]: q (Hq * d), k (Hk * d), v (Hk * dv): C channels
+  const float* bias;      // [C] or null
+  const float* conv_w;    // [C, taps], the last tap meets the current token
+  const float* conv_state; // [slots, taps - 1, C]: the last inputs, biases included
+  float* advance;         // conv_state to be moved on by the same kernel (every sequence brings one token), or null
+  const float* cos_table; // [max_pos, rot / 2] or null
+  const float* sin_table;
+  const int* tok_pos;
+  const int* tok_seq;
+  const int* seq_slot;
+  const int* seq_qstart;
+  const int* block_table;
+  void* q_out;            // [T, Hq * d]
+  void* k_cache;          // [pages, Hk, PAGE, d]
+  void* v_cache;          // [pages, Hk, PAGE, dv]
+  int ld, n_heads, n_kv_heads, d, dv, rot, interleaved, max_blocks, taps;
+};
+
+// grid (tokens), 256 threads: a channel a thread; the partner of a rotated dimension is convolved again
+template <typename T>
+__global__ void __launch_bounds__(256) conv_prepare_kernel(ConvPrepArgs a) {
+  const int t = blockIdx.x;
+  const int d = a.d, nq = a.n_heads * d, nk = a.n_kv_heads * d, nv = a.n_kv_heads * a.dv, C = nq + nk + nv;
+  const int seq = a.tok_seq[t], local = t - a.seq_qstart[seq], slot = a.seq_slot[seq], pos = a.tok_pos[t];
+  const float* state = a.conv_state + (size_t)slot * (a.taps - 1) * C;
+  const int page = a.block_table[(size_t)slot * a.max_blocks + pos / MLL_PAGE], in_page = pos % MLL_PAGE;
+  const int half = a.rot >> 1;
+  auto convolved = [&](int c) {
+    const float b = a.bias ? a.bias[c] : 0.f;
+    float y = 0.f;
+    for (int back = 0; back < a.taps; ++back) {
+      const float u = back <= local ? to_float(((const T*)a.qkv)[(size_t)(t - back) * a.ld + c]) + b
+                                    : state[(size_t)(local - back + a.taps - 1) * C + c];
+      y = fmaf(a.conv_w[(size_t)c * a.taps + (a.taps - 1 - back)], u, y);
+    }
+    return y;
+  };
+  for (int c = threadIdx.x; c < C; c += 256) {
+    float x = convolved(c);
+    if (c >= nq + nk) {
+      const int i = c - nq - nk, head = i / a.dv, e = i % a.dv;
+      ((T*)a.v_cache)[(((size_t)page * a.n_kv_heads + head) * MLL_PAGE + in_page) * a.dv + e] = from_float<T>(x);
+      continue;
+    }
+    const int head = c / d, e = c % d;  // k heads follow the q heads
+    if (e < a.rot) {
+      int pair, partner;
+      bool first;
+      if (a.interleaved) {
+        pair = e >> 1; first = !(e & 1); partner = e ^ 1;
+      } else {
+        first = e < half; pair = first ? e : e - half; partner = first ? e + half : e - half;
+      }
+      const float y = convolved(head * d + partner);
+      const float co = a.cos_table[(size_t)pos * half + pair], si = a.sin_table[(size_t)pos * half + pair];
+      x = first ? x * co - y * si : x * co + y * si;
+    }
+    if (c < nq)
+      ((T*)a.q_out)[(size_t)t * nq + c] = from_float<T>(x);
+    else
+      ((T*)a.k_cache)[(((size_t)page * a.n_kv_heads + (head - a.n_heads)) * MLL_PAGE + in_page) * d + e] = from_float<T>(x);
+  }
+}
+
+// V channels on their way through the convolution: taps and last inputs of this thread's channels in registers
+template <typename T, int V, int TAPS>
+struct ConvWalk {
+  float w[V * TAPS], b[V], past[TAPS > 1 ? TAPS - 1 : 1][V];  // past[i]: the input i + 1 tokens ago
+
+  __device__ __forceinline__ void begin(const ConvPrepArgs& a, int c) {
+    load_floats<float, V * TAPS>(a.conv_w + (size_t)c * TAPS, w);
+#pragma unroll
+    for (int j = 0; j < V; ++j) b[j] = a.bias ? a.bias[c + j] : 0.f;
+  }
+  __device__ __forceinline__ void fetch(const ConvPrepArgs& a, int t, int c, float* x) const {
+    load_floats<T, V>((const T*)a.qkv + (size_t)t * a.ld + c, x);
+#pragma unroll
+    for (int j = 0; j < V; ++j) x[j] += b[j];
+  }
+  // the inputs before row t, the local-th of its sequence in this step
+  __device__ __forceinline__ void look_back(const ConvPrepArgs& a, int t, int local, const float* state, int C, int c) {
+#pragma unroll
+    for (int i = 0; i < TAPS - 1; ++i) {
+      if (i < local) fetch(a, t - i - 1, c, past[i]);
+      else load_floats<float, V>(state + (size_t)(local - i - 1 + TAPS - 1) * C + c, past[i]);
+    }
+  }
+  // y = the convolution's value at row t; the row becomes the newest of the last inputs
+  __device__ __forceinline__ void next(const ConvPrepArgs& a, int t, int c, float* y, float* advance, int C) {
+    float x[V];
+    fetch(a, t, c, x);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      y[j] = w[j * TAPS + TAPS - 1] * x[j];
+#pragma unroll
+      for (int i = 0; i < TAPS - 1; ++i) y[j] = fmaf(w[j * TAPS + TAPS - 2 - i], past[i][j], y[j]);
+    }
+    if constexpr (TAPS > 1) {
+      if (advance) {
+#pragma unroll
+        for (int i = 0; i < TAPS - 1; ++i)
+          store_floats<float, V>(advance + (size_t)(TAPS - 2 - i) * C + c, i == 0 ? x : past[i - 1]);
+      }
+#pragma unroll
+      for (int i = TAPS - 2; i > 0; --i)
+#pragma unroll
+        for (int j = 0; j < V; ++j) past[i][j] = past[i - 1][j];
+#pragma unroll
+      for (int j = 0; j < V; ++j) past[0][j] = x[j];
+    }
+  }
+};
+
+// grid (ceil(tokens / TB), ceil(units / 256)), 256 threads; a unit is a word of V channels, or the two words that the
+// rotation (pairs half a rotated part apart) turns together
+template <typename T, int TAPS, int TB>
+__global__ void __launch_bounds__(256) conv_prepare_walk_kernel(ConvPrepArgs a, int n_tokens) {
+  constexpr int V = 4;
+  const int u = blockIdx.y * 256 + threadIdx.x;
+  const int H = a.n_heads, G = a.n_kv_heads, d = a.d, dv = a.dv;
+  const int hw = a.rot / (2 * V), nu = d / V - hw, vw = dv / V;
+  const int nqk = (H + G) * nu;
+  if (u >= nqk + G * vw) return;
+  const int C = (H + G) * d + G * dv;
+  const bool is_v = u >= nqk;
+  int head, e, c;       // head among the q and k heads (or among the v heads), first dimension in it, column
+  bool pair = false;
+  if (is_v) {
+    head = (u - nqk) / vw;
+    e = (u - nqk - head * vw) * V;
+    c = (H + G) * d + head * dv + e;
+  } else {
+    head = u / nu;
+    const int i = u - head * nu;
+    pair = i < hw;
+    e = (pair ? i : i + hw) * V;
+    c = head * d + e;
+  }
+  const int far = hw * V;  // distance to the partner
+  ConvWalk<T, V, TAPS> one, two;
+  one.begin(a, c);
+  if (pair) two.begin(a, c + far);
+  const int t0 = blockIdx.x * TB, t1 = min(n_tokens, t0 + TB);
+  for (int t = t0; t < t1; ++t) {
+    const int seq = a.tok_seq[t], local = t - a.seq_qstart[seq], slot = a.seq_slot[seq], pos = a.tok_pos[t];
+    if (TAPS > 1 && (t == t0 || local == 0)) {
+      const float* state = a.conv_state + (size_t)slot * (TAPS - 1) * C;
+      one.look_back(a, t, local, state, C, c);
+      if (pair) two.look_back(a, t, local, state, C, c + far);
+    }
+    float* advance = a.advance ? a.advance + (size_t)slot * (TAPS - 1) * C : nullptr;
+    float x[V], y[V];
+    one.next(a, t, c, x, advance, C);
+    if (pair) {
+      two.next(a, t, c + far, y, advance, C);
+      float co[V], si[V];
+      load_floats<float, V>(a.cos_table + (size_t)pos * (a.rot >> 1) + e, co);
+      load_floats<float, V>(a.sin_table + (size_t)pos * (a.rot >> 1) + e, si);
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        const float p = x[j], q = y[j];
+        x[j] = p * co[j] - q * si[j];
+        y[j] = q * co[j] + p * si[j];
+      }
+    }
+    T* dst;
+    if (!is_v && head < H) {
+      dst = (T*)a.q_out + (size_t)t * H * d + c;
+    } else {
+      const int page = a.block_table[(size_t)slot * a.max_blocks + pos / MLL_PAGE], in_page = pos % MLL_PAGE;
+      dst = is_v ? (T*)a.v_cache + (((size_t)page * G + head) * MLL_PAGE + in_page) * dv + e
+                 : (T*)a.k_cache + (((size_t)page * G + (head - H)) * MLL_PAGE + in_page) * d + e;
+    }
+    store_floats<T, V>(dst, x);
+    if (pair) store_floats<T, V>(dst + far, y);
+  }
+}
+
+static bool conv_walk_takes(int d, int dv, int rot, int interleaved, int taps, int ld) {
+  return taps >= 2 && taps <= 4 && d % 4 == 0 && dv % 4 == 0 && rot % 8 == 0 && ld % 4 == 0 && (!interleaved || rot == 0);
+}
+
+template <typename T, int TAPS>
+static int launch_conv_walk(const ConvPrepArgs& a, int n_tokens, cudaStream_t stream) {
+  const int units = (a.n_heads + a.n_kv_heads) * (a.d / 4 - a.rot / 8) + a.n_kv_heads * (a.dv / 4);
+  const int columns = (units + 255) / 256;
+  // rows a thread walks: eight, as long as that leaves every multiprocessor four blocks
+  if ((long long)((n_tokens + 7) / 8) * columns >= (long long)mll_sm_count() * 4)
+    MLL_LAUNCH((conv_prepare_walk_kernel<T, TAPS, 8>), dim3((n_tokens + 7) / 8, columns), 256, 0, stream, a, n_tokens);
+  else
+    MLL_LAUNCH((conv_prepare_walk_kernel<T, TAPS, 1>), dim3(n_tokens, columns), 256, 0, stream, a, n_tokens);
+  MLL_LAUNCH_CHECK();
+  return 0;
+}
+
+template <typename T>
+static int launch_conv_prepare(const ConvPrepArgs& a, int n_tokens, cudaStream_t stream) {
+  const uintptr_t all = (uintptr_t)a.qkv | (uintptr_t)a.conv_w | (uintptr_t)a.conv_state | (uintptr_t)a.cos_table |
+                        (uintptr_t)a.sin_table | (uintptr_t)a.q_out | (uintptr_t)a.k_cache | (uintptr_t)a.v_cache;
+  if (conv_walk_takes(a.d, a.dv, a.rot, a.interleaved, a.taps, a.ld) && all % 16 == 0) {
+    if (a.taps == 2) return launch_conv_walk<T, 2>(a, n_tokens, stream);
+    if (a.taps == 3) return launch_conv_walk<T, 3>(a, n_tokens, stream);
+    return launch_conv_walk<T, 4>(a, n_tokens, stream);
+  }
+  MLL_REQUIRE(!a.advance, "conv prepare: this size moves its state on in a kernel of its own");
+  MLL_LAUNCH((conv_prepare_kernel<T>), n_tokens, 256, 0, stream, a);
+  MLL_LAUNCH_CHECK();
+  return 0;
 }
 
 struct LocalAttnArgs {
@@ -439,6 +656,32 @@ int launch_local_attention(const LocalAttnArgs& a, cudaStream_t stream) {
 }
 
 }  // namespace mll
+// Whether mll_conv_attention_prepare can also move the convolution's state on (`advance`).
+MLL_API int mll_conv_attention_advances(int d, int dv, int rot, int interleaved, int taps, int ld) {
+  return mll::conv_walk_takes(d, dv, rot, interleaved, taps, ld) ? 1 : 0;
+}
+
+// qkv [n_tokens, ld] of `dtype`; see ConvPrepArgs.  advance: conv_state itself, or null.
+MLL_API int mll_conv_attention_prepare(const void* qkv, const float* bias, const float* conv_w, float* conv_state, int advance,
+                                       const float* cos_table, const float* sin_table, const int* tok_pos,
+                                       const int* tok_seq, const int* seq_slot, const int* seq_qstart,
+                                       const int* block_table, void* q_out, void* k_cache, void* v_cache, int dtype,
+                                       int n_tokens, int ld, int n_heads, int n_kv_heads, int d, int dv, int rot,
+                                       int interleaved, int max_blocks, int taps, cudaStream_t stream) {
+  MLL_REQUIRE(n_tokens >= 0 && n_heads > 0 && n_kv_heads > 0 && d > 0 && dv > 0 && taps >= 1 && max_blocks > 0,
+              "conv prepare: bad sizes");
+  MLL_REQUIRE(rot >= 0 && rot <= d && rot % 2 == 0 && (rot == 0 || (cos_table && sin_table)),
+              "conv prepare: %d rotated dimensions of %d, or no table", rot, d);
+  MLL_REQUIRE(ld >= (n_heads + n_kv_heads) * d + n_kv_heads * dv, "conv prepare: row stride %d too short", ld);
+  if (n_tokens == 0) return 0;
+  mll::ConvPrepArgs a{qkv, bias, conv_w, conv_state, advance ? conv_state : nullptr, rot ? cos_table : nullptr,
+                      rot ? sin_table : nullptr, tok_pos, tok_seq, seq_slot, seq_qstart, block_table, q_out, k_cache, v_cache,
+                      ld, n_heads, n_kv_heads, d, dv, rot, interleaved, max_blocks, taps};
+  if (dtype == MLL_F32) return mll::launch_conv_prepare<float>(a, n_tokens, stream);
+  if (dtype == MLL_BF16) return mll::launch_conv_prepare<__nv_bfloat16>(a, n_tokens, stream);
+  MLL_REQUIRE(false, "conv prepare: unknown dtype %d", dtype);
+  return -1;
+}
 
 MLL_API int mll_local_attention_prepare(const void* qkv, const float* q_weight, const float* k_weight,
                                         const float* cos_table, const float* sin_table, const int* tok_pos,

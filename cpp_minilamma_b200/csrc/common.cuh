@@ -121,6 +121,66 @@ __device__ __forceinline__ int decode_first_key(int ctx, int window) {
   return 0;
 }
 
+// V neighbouring values (V * sizeof(T) a power of two; p aligned to as many bytes, 16 at most) as floats
+template <typename T, int V>
+__device__ __forceinline__ void load_floats(const T* p, float* out) {
+  if constexpr (sizeof(T) == 4) {
+    if constexpr (V % 4 == 0) {
+#pragma unroll
+      for (int i = 0; i < V; i += 4) {
+        const float4 v = *reinterpret_cast<const float4*>((const float*)p + i);
+        out[i] = v.x; out[i + 1] = v.y; out[i + 2] = v.z; out[i + 3] = v.w;
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < V; ++i) out[i] = to_float(p[i]);
+    }
+  } else if constexpr (V == 1) {
+    out[0] = to_float(p[0]);
+  } else {
+    unsigned raw[(V + 1) / 2];
+    if constexpr (V == 8) {
+      const uint4 v = *reinterpret_cast<const uint4*>(p);
+      raw[0] = v.x; raw[1] = v.y; raw[2] = v.z; raw[3] = v.w;
+    } else if constexpr (V == 4) {
+      const uint2 v = *reinterpret_cast<const uint2*>(p);
+      raw[0] = v.x; raw[1] = v.y;
+    } else {
+      raw[0] = *reinterpret_cast<const unsigned*>(p);
+    }
+#pragma unroll
+    for (int i = 0; i < V / 2; ++i) {
+      const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw[i]));
+      out[2 * i] = f.x;
+      out[2 * i + 1] = f.y;
+    }
+  }
+}
+template <typename T, int V>
+__device__ __forceinline__ void store_floats(T* p, const float* v) {
+  if constexpr (sizeof(T) == 4) {
+    if constexpr (V % 4 == 0) {
+#pragma unroll
+      for (int i = 0; i < V; i += 4) *reinterpret_cast<float4*>((float*)p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < V; ++i) p[i] = from_float<T>(v[i]);
+    }
+  } else if constexpr (V == 1) {
+    p[0] = from_float<T>(v[0]);
+  } else {
+    unsigned raw[(V + 1) / 2];
+#pragma unroll
+    for (int i = 0; i < V / 2; ++i) {
+      const __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+      raw[i] = *reinterpret_cast<const unsigned*>(&h);
+    }
+    if constexpr (V == 8) *reinterpret_cast<uint4*>(p) = make_uint4(raw[0], raw[1], raw[2], raw[3]);
+    else if constexpr (V == 4) *reinterpret_cast<uint2*>(p) = make_uint2(raw[0], raw[1]);
+    else *reinterpret_cast<unsigned*>(p) = raw[0];
+  }
+}
+
 // 16-byte asynchronous copy global -> shared (both 16-byte aligned)
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
   unsigned s = (unsigned)__cvta_generic_to_shared(smem);
@@ -130,6 +190,18 @@ __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commi
 template <int N>
 __device__ __forceinline__ void cp_async_wait() {
   asm volatile("cp.async.wait_group %0;\n" ::"n"(N));
+}
+
+// Activations of a gated feed-forward's gate (GATE_ACT_*), exact and as one multiplication and one division:
+// silu(z) = z / (1 + e^-z); gelu in its tanh form, 0.5 z (1 + tanh y) with y = sqrt(2 / pi) (z + 0.044715 z^3), is
+// z / (1 + e^-2y), since (1 + tanh y) / 2 is the logistic function of 2y.  FAST: hardware exponential and division, for
+// results that are rounded to bfloat16.
+enum : int { GATE_ACT_SILU = 0, GATE_ACT_GELU_TANH = 1 };
+
+template <bool FAST>
+__device__ __forceinline__ float gate_act_mul(int kind, float g, float u) {
+  const float y = kind == GATE_ACT_GELU_TANH ? 1.5957691216057308f * fmaf(0.044715f * g * g, g, g) : g;
+  return FAST ? __fdividef(g, 1.f + __expf(-y)) * u : g / (1.f + expf(-y)) * u;
 }
 
 // Rows whose RMS norm is still to be applied.  The kernel that added to the residual stream wrote, for

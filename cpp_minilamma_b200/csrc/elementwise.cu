@@ -1,4 +1,4 @@
-// Embedding gather, dtype casts and the SwiGLU activation.
+// Embedding gather, dtype casts and the gated activations (SwiGLU and its relatives).
 //
 // Replaces the reference's EmbeddingKernel, SiluKernel and ElementWiseMulKernel
 // (src/cuda_ops.cu:165-192) with batched kernels; SiLU and the product are one pass.
@@ -21,7 +21,7 @@ MLL_API const char* mll_last_error() { return g_error; }
 thread_local cudaError_t mll_launch_status = cudaSuccess;
 
 // Identifies the build; the Python side checks it after loading the library.
-MLL_API int mll_abi_version() { return 34; }
+MLL_API int mll_abi_version() { return 35; }
 
 // Cache positions per page, for the Python side to check against its own constant.
 MLL_API int mll_page() { return MLL_PAGE; }
@@ -128,13 +128,13 @@ __global__ void cast_kernel(const In* __restrict__ in, Out* __restrict__ out, si
   for (; i < n; i += stride) out[i] = from_float<Out>(to_float(in[i]));
 }
 
-// out[t, i] = silu(gate) * up.  `gu` rows hold gate and up either as two halves
+// out[t, i] = act(gate) * up, act silu or gelu in its tanh form (GATE_ACT_*).  `gu` rows hold gate and up either as two halves
 // ([gate(0..I) | up(0..I)], block == 0) or interleaved in blocks of `block` columns
 // ([gate(0..b) | up(0..b) | gate(b..2b) | ...]); I is a multiple of `block` then.
 // `bias` (float32 [2 I], in the order of a row of gu, or null) is added to gate and up first.
 template <typename T>
 __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int tokens,
-                              int inter, int block, const float* __restrict__ bias) {
+                              int inter, int block, const float* __restrict__ bias, int act) {
   const size_t total = (size_t)tokens * inter;
   size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   const size_t stride = (size_t)gridDim.x * blockDim.x;
@@ -150,8 +150,7 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int
       g += bias[gc];
       u += bias[uc];
     }
-    const float act = g / (1.f + expf(-g));
-    out[idx] = from_float<T>(act * u);
+    out[idx] = from_float<T>(gate_act_mul<false>(act, g, u));
   }
 }
 
@@ -191,19 +190,12 @@ struct Pack8<float> {
   }
 };
 
-// silu(g) * u.  The float32 path keeps the accurate exponential and division; a bfloat16 result
+// The float32 path keeps the accurate exponential and division; a bfloat16 result
 // is rounded to 8 bits anyway, so it takes the fast ones (a prefill step spends a tenth of its
 // non-GEMM time here, and the accurate forms make the kernel compute-bound).
 template <typename T>
-__device__ __forceinline__ float silu_mul(float g, float u);
-template <>
-__device__ __forceinline__ float silu_mul<float>(float g, float u) { return g / (1.f + expf(-g)) * u; }
-template <>
-__device__ __forceinline__ float silu_mul<__nv_bfloat16>(float g, float u) { return __fdividef(g, 1.f + __expf(-g)) * u; }
-
-template <typename T>
 __global__ void swiglu_vec8_kernel(const T* __restrict__ gu, T* __restrict__ out, int tokens, int inter, int block,
-                                   const float* __restrict__ bias) {
+                                   const float* __restrict__ bias, int act) {
   const int groups = inter >> 3;
   const size_t total = (size_t)tokens * groups;
   size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -227,7 +219,7 @@ __global__ void swiglu_vec8_kernel(const T* __restrict__ gu, T* __restrict__ out
       }
     }
 #pragma unroll
-    for (int i = 0; i < 8; ++i) r[i] = silu_mul<T>(g[i], u[i]);
+    for (int i = 0; i < 8; ++i) r[i] = gate_act_mul<sizeof(T) == 2>(act, g[i], u[i]);
     Pack8<T>::store(out + (size_t)t * inter + (size_t)b * 8, r);
   }
 }
@@ -238,6 +230,22 @@ __global__ void scale_kernel(float* __restrict__ x, size_t n, float factor) {
   for (; idx < n; idx += stride) x[idx] *= factor;
 }
 
+// x = cap * tanh(factor * x / cap)
+__global__ void softcap_kernel(float* __restrict__ x, size_t n, float factor, float cap) {
+  const size_t at = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 4, stride = (size_t)gridDim.x * blockDim.x * 4;
+  const float inv = 1.f / cap;
+  for (size_t i = at; i < n; i += stride) {
+    if (i + 4 <= n) {  // the launch checks that x starts on a 16-byte boundary
+      float4 v = *reinterpret_cast<float4*>(x + i);
+      v.x = cap * tanhf(factor * v.x * inv); v.y = cap * tanhf(factor * v.y * inv);
+      v.z = cap * tanhf(factor * v.z * inv); v.w = cap * tanhf(factor * v.w * inv);
+      *reinterpret_cast<float4*>(x + i) = v;
+    } else {
+      for (size_t j = i; j < n; ++j) x[j] = cap * tanhf(factor * x[j] * inv);
+    }
+  }
+}
+
 // x[t, i] += bias[i] (bias float32, sum in float32)
 template <typename T>
 __global__ void add_bias_kernel(T* __restrict__ x, const float* __restrict__ bias, size_t total, int width) {
@@ -246,11 +254,24 @@ __global__ void add_bias_kernel(T* __restrict__ x, const float* __restrict__ bia
   for (; idx < total; idx += stride) x[idx] = from_float<T>(to_float(x[idx]) + bias[idx % width]);
 }
 
+// The same in bfloat16, eight neighbouring columns a thread (width a multiple of 8).
+__global__ void __launch_bounds__(256) add_bias_vec8_kernel(__nv_bfloat16* __restrict__ x, const float* __restrict__ bias,
+                                                            size_t words, int row_words) {
+  for (size_t i = (size_t)blockIdx.x * 256 + threadIdx.x; i < words; i += (size_t)gridDim.x * 256) {
+    float v[8], b[8];
+    Pack8<__nv_bfloat16>::load(x + i * 8, v);
+    Pack8<float>::load(bias + (i % row_words) * 8, b);
+#pragma unroll
+    for (int k = 0; k < 8; ++k) v[k] += b[k];
+    Pack8<__nv_bfloat16>::store(x + i * 8, v);
+  }
+}
+
 // As swiglu_vec8_kernel (bfloat16, gate and up interleaved in blocks of 8), for rows of gate/up that still lack their
 // RMS norm's factor (the product ran on x * w_norm): both are multiplied by the row's factor first.  One row per
 // blockIdx.y; warp 0 computes the factor from the row's partial sums of squares.
 __global__ void swiglu_rows_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ out, int inter,
-                                   int block, RowNormIn in, int width) {
+                                   int block, RowNormIn in, int width, int act) {
   __shared__ float factor;
   const int m = blockIdx.y;
   if (threadIdx.x < 32) {
@@ -270,7 +291,7 @@ __global__ void swiglu_rows_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bf
   Pack8<__nv_bfloat16>::load(gp, g);
   Pack8<__nv_bfloat16>::load(up, u);
 #pragma unroll
-  for (int i = 0; i < 8; ++i) r[i] = silu_mul<__nv_bfloat16>(g[i] * f, u[i] * f);
+  for (int i = 0; i < 8; ++i) r[i] = gate_act_mul<true>(act, g[i] * f, u[i] * f);
   Pack8<__nv_bfloat16>::store(out + (size_t)m * inter + (size_t)b * 8, r);
 }
 
@@ -409,10 +430,29 @@ MLL_API int mll_scale(float* x, long long n, float factor, cudaStream_t stream) 
   return 0;
 }
 
+// x[i] = cap * tanh(factor * x[i] / cap) (float32, in place)
+MLL_API int mll_softcap(float* x, long long n, float factor, float cap, cudaStream_t stream) {
+  MLL_REQUIRE(n >= 0 && cap > 0.f, "softcap: bad size %lld or cap", n);
+  MLL_REQUIRE((uintptr_t)x % 16 == 0, "softcap: the tensor must be 16-byte aligned");
+  if (n == 0) return 0;
+  long long blocks = (n + 1023) / 1024;
+  if (blocks > mll_sm_count() * 16) blocks = mll_sm_count() * 16;
+  MLL_LAUNCH((mll::softcap_kernel), (int)blocks, 256, 0, stream, x, (size_t)n, factor, cap);
+  MLL_LAUNCH_CHECK();
+  return 0;
+}
+
 MLL_API int mll_add_bias(void* x, const float* bias, int dtype, int n_rows, int width, cudaStream_t stream) {
   MLL_REQUIRE(n_rows >= 0 && width > 0, "add_bias: bad sizes rows=%d width=%d", n_rows, width);
   if (n_rows == 0) return 0;
   const size_t total = (size_t)n_rows * width;
+  if (dtype == MLL_BF16 && width % 8 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)bias % 16 == 0) {
+    const long long want = (long long)((total / 8 + 255) / 256), most = (long long)mll_sm_count() * 16;
+    MLL_LAUNCH((mll::add_bias_vec8_kernel), (int)(want < most ? want : most), 256, 0, stream, (__nv_bfloat16*)x, bias,
+               total / 8, width / 8);
+    MLL_LAUNCH_CHECK();
+    return 0;
+  }
   long long blocks = (long long)((total + 255) / 256);
   if (blocks > mll_sm_count() * 16) blocks = mll_sm_count() * 16;
   if (dtype == MLL_F32)
@@ -483,9 +523,10 @@ MLL_API int mll_cast(const void* in, int in_dtype, void* out, int out_dtype, lon
 }
 
 // bfloat16 gu [n_tokens, 2 inter] (halves: block 0; blocks of 8: block 8) computed from rows that lack their RMS
-// norm's factor 1 / sqrt(sum_p sumsq[m][p] / width + eps): out = silu(gate f) * (up f).
+// norm's factor 1 / sqrt(sum_p sumsq[m][p] / width + eps): out = act(gate f) * (up f).
 MLL_API int mll_swiglu_rows(const void* gu, void* out, int n_tokens, int inter, int block, const float* sumsq, int partials,
-                            int stride, float eps, int width, cudaStream_t stream) {
+                            int stride, float eps, int width, int act, cudaStream_t stream) {
+  MLL_REQUIRE(act == mll::GATE_ACT_SILU || act == mll::GATE_ACT_GELU_TANH, "swiglu_rows: unknown activation %d", act);
   MLL_REQUIRE(n_tokens >= 0 && n_tokens <= 65535 && inter > 0 && inter % 8 == 0 && (block == 0 || block == 8),
               "swiglu_rows: bad sizes tokens=%d inter=%d block=%d", n_tokens, inter, block);
   MLL_REQUIRE(sumsq && partials >= 1 && stride >= partials && eps >= 0.f && width > 0,
@@ -494,13 +535,14 @@ MLL_API int mll_swiglu_rows(const void* gu, void* out, int n_tokens, int inter, 
   if (n_tokens == 0) return 0;
   const int groups = inter / 8;
   MLL_LAUNCH((mll::swiglu_rows_kernel), dim3((groups + 255) / 256, n_tokens), 256, 0, stream, (const __nv_bfloat16*)gu,
-             (__nv_bfloat16*)out, inter, block, mll::RowNormIn{sumsq, partials, stride, eps}, width);
+             (__nv_bfloat16*)out, inter, block, mll::RowNormIn{sumsq, partials, stride, eps}, width, act);
   MLL_LAUNCH_CHECK();
   return 0;
 }
 
 MLL_API int mll_swiglu(const void* gu, void* out, int dtype, int n_tokens, int inter, int block, const float* bias,
-                       cudaStream_t stream) {
+                       int act, cudaStream_t stream) {
+  MLL_REQUIRE(act == mll::GATE_ACT_SILU || act == mll::GATE_ACT_GELU_TANH, "swiglu: unknown activation %d", act);
   MLL_REQUIRE(n_tokens >= 0 && inter > 0, "swiglu: bad sizes tokens=%d inter=%d", n_tokens, inter);
   MLL_REQUIRE(block >= 0 && (block == 0 || inter % block == 0),
               "swiglu: intermediate size %d is not a multiple of the interleave block %d", inter, block);
@@ -513,9 +555,9 @@ MLL_API int mll_swiglu(const void* gu, void* out, int dtype, int n_tokens, int i
     if (groups > mll_sm_count() * 32) groups = mll_sm_count() * 32;
     if (dtype == MLL_F32)
       MLL_LAUNCH((mll::swiglu_vec8_kernel<float>), (int)groups, threads, 0, stream, (const float*)gu, (float*)out, n_tokens,
-                                                                       inter, block, bias);
+                                                                       inter, block, bias, act);
     else if (dtype == MLL_BF16)
-      MLL_LAUNCH((mll::swiglu_vec8_kernel<__nv_bfloat16>), (int)groups, threads, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, n_tokens, inter, block, bias);
+      MLL_LAUNCH((mll::swiglu_vec8_kernel<__nv_bfloat16>), (int)groups, threads, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, n_tokens, inter, block, bias, act);
     else
       MLL_REQUIRE(false, "swiglu: unknown dtype %d", dtype);
     MLL_LAUNCH_CHECK();
@@ -524,9 +566,9 @@ MLL_API int mll_swiglu(const void* gu, void* out, int dtype, int n_tokens, int i
   long long blocks = ((long long)n_tokens * inter + threads - 1) / threads;
   if (blocks > mll_sm_count() * 32) blocks = mll_sm_count() * 32;
   if (dtype == MLL_F32)
-    MLL_LAUNCH((mll::swiglu_kernel<float>), (int)blocks, threads, 0, stream, (const float*)gu, (float*)out, n_tokens, inter, block, bias);
+    MLL_LAUNCH((mll::swiglu_kernel<float>), (int)blocks, threads, 0, stream, (const float*)gu, (float*)out, n_tokens, inter, block, bias, act);
   else if (dtype == MLL_BF16)
-    MLL_LAUNCH((mll::swiglu_kernel<__nv_bfloat16>), (int)blocks, threads, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, n_tokens, inter, block, bias);
+    MLL_LAUNCH((mll::swiglu_kernel<__nv_bfloat16>), (int)blocks, threads, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, n_tokens, inter, block, bias, act);
   else
     MLL_REQUIRE(false, "swiglu: unknown dtype %d", dtype);
   MLL_LAUNCH_CHECK();

@@ -14,7 +14,7 @@ import torch
 from ..cache.paged import PAGE  # cache positions per page; the library's MLL_PAGE is checked against it on load
 from .build import KernelBuildError, load_library
 
-ABI_VERSION = 34
+ABI_VERSION = 35
 MAX_TOP_K = 1024
 
 
@@ -156,6 +156,13 @@ def scale_(x: torch.Tensor, factor: float) -> None:
     _check(lib().mll_scale(_ptr(x), ctypes.c_longlong(x.numel()), ctypes.c_float(factor), _stream()), "scale")
 
 
+def softcap_(x: torch.Tensor, cap: float, factor: float = 1.0) -> None:
+    """x = cap * tanh(factor * x / cap) (float32, in place)."""
+    _need(x, "softcap x", torch.float32)
+    _check(lib().mll_softcap(_ptr(x), ctypes.c_longlong(x.numel()), ctypes.c_float(factor), ctypes.c_float(cap), _stream()),
+           "softcap")
+
+
 def embedding_pair(tokens, tok_pos, tok_seq, seq_slot, seq_qstart, seq_qlen, prev_token, table, pairs, out,
                    buckets: int, mul_prev: int, mul_cur: int, scale: float) -> None:
     """out[t, :] = scale * table[tokens[t], :] + pairs[row(t), :] (float32 [T, D]), row(t) = (mul_prev * the token
@@ -237,7 +244,7 @@ def gather_int32(dst: torch.Tensor, src: torch.Tensor, index: torch.Tensor, n: i
                                   _stream()), "gather_int32")
 
 
-EPI_BF16, EPI_F32, EPI_SWIGLU, EPI_RESID = 0, 1, 2, 3
+EPI_BF16, EPI_F32, EPI_SWIGLU, EPI_RESID, EPI_GEGLU = 0, 1, 2, 3, 4
 NORM_TILE = 16  # columns per partial sum of squares that the residual epilogue writes
 
 
@@ -277,7 +284,8 @@ def linear_small(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor],
     """out = x . w^T for at most 64 rows of bfloat16 x [M, K] and bfloat16 w [N, K], read once.
 
     epilogue EPI_BF16 / EPI_F32: out [M, N] in that dtype (+ float32 bias [N]);
-    EPI_SWIGLU: w holds gate and up rows interleaved in blocks of 8, out [M, N / 2] = silu(gate) * up;
+    EPI_SWIGLU: w holds gate and up rows interleaved in blocks of 8, out [M, N / 2] = silu(gate) * up (EPI_GEGLU: gelu
+    in its tanh form);
     EPI_RESID (at most 16 rows, with `residual`): the result is added to the residual stream, out [M, N]
     is the new stream times the next norm's weight (not yet its factor), with partial sums of squares.
     `row_norm`: x is such an output; the result is multiplied by the rows' factors."""
@@ -287,7 +295,7 @@ def linear_small(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor],
     n = w.shape[0]
     if w.shape[1] != k:
         raise KernelError(f"linear_small: x width {k} differs from w width {w.shape[1]}")
-    want = (rows, n // 2) if epilogue == EPI_SWIGLU else (rows, n)
+    want = (rows, n // 2) if epilogue in (EPI_SWIGLU, EPI_GEGLU) else (rows, n)
     _need(out, "linear_small out", torch.float32 if epilogue == EPI_F32 else torch.bfloat16, 2)
     if tuple(out.shape) != want:
         raise KernelError(f"linear_small: out {tuple(out.shape)}, expected {want}")
@@ -328,7 +336,7 @@ def linear_tma(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], o
     n = w.shape[0]
     if w.shape[1] != k:
         raise KernelError(f"linear_tma: x width {k} differs from w width {w.shape[1]}")
-    want = (rows, n // 2) if epilogue == EPI_SWIGLU else (rows, n)
+    want = (rows, n // 2) if epilogue in (EPI_SWIGLU, EPI_GEGLU) else (rows, n)
     _need(out, "linear_tma out", torch.float32 if epilogue == EPI_F32 else torch.bfloat16, 2)
     if tuple(out.shape) != want:
         raise KernelError(f"linear_tma: out {tuple(out.shape)}, expected {want}")
@@ -357,7 +365,7 @@ def linear_tc5(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], o
     n = w.shape[0]
     if w.shape[1] != k:
         raise KernelError(f"linear_tc5: x width {k} differs from w width {w.shape[1]}")
-    want = (rows, n // 2) if epilogue == EPI_SWIGLU else (rows, n)
+    want = (rows, n // 2) if epilogue in (EPI_SWIGLU, EPI_GEGLU) else (rows, n)
     _need(out, "linear_tc5 out", torch.float32 if epilogue == EPI_F32 else torch.bfloat16, 2)
     if tuple(out.shape) != want:
         raise KernelError(f"linear_tc5: out {tuple(out.shape)}, expected {want}")
@@ -476,9 +484,12 @@ FUSE_NORM = True  # off: every norm is a kernel of its own
 SMALL_LINEAR = "auto"  # "auto", a forced kind ("tc5", "tma", "direct"), or "none" (library GEMM only)
 
 
+GATE_ACT_SILU, GATE_ACT_GELU_TANH = 0, 1
+
+
 def swiglu(gate_up: torch.Tensor, out: torch.Tensor, block: int, row_norm: Optional[RowNorm] = None,
-           width: int = 0, bias: Optional[torch.Tensor] = None) -> None:
-    """out[t, i] = silu(gate) * up; gate_up [T, 2I] holds halves (block 0) or blocks of `block`.
+           width: int = 0, bias: Optional[torch.Tensor] = None, act: int = GATE_ACT_SILU) -> None:
+    """out[t, i] = act(gate) * up (silu, or gelu in its tanh form); gate_up [T, 2I] holds halves (block 0) or blocks of `block`.
     `bias` (float32 [2I], in the order of gate_up's columns) is added to gate and up first, in float32.
     `row_norm` (bfloat16, I a multiple of 8): gate_up was computed from rows of `width` columns that lacked their
     norm's factor; gate and up are multiplied by it first."""
@@ -496,11 +507,11 @@ def swiglu(gate_up: torch.Tensor, out: torch.Tensor, block: int, row_norm: Optio
             raise KernelError("swiglu: rows without their norm's factor need bfloat16, I % 8 == 0 and the rows' width")
         sumsq, partials, stride, eps = _row_norm_args(row_norm, tokens, "swiglu")
         _check(lib().mll_swiglu_rows(_ptr(gate_up), _ptr(out), ctypes.c_int(tokens), ctypes.c_int(inter),
-                                     ctypes.c_int(block), sumsq, partials, stride, eps, ctypes.c_int(width), _stream()),
-               "swiglu_rows")
+                                     ctypes.c_int(block), sumsq, partials, stride, eps, ctypes.c_int(width), ctypes.c_int(act),
+                                     _stream()), "swiglu_rows")
         return
     _check(lib().mll_swiglu(_ptr(gate_up), _ptr(out), dtype_code(out.dtype), ctypes.c_int(tokens),
-                            ctypes.c_int(inter), ctypes.c_int(block), _ptr(bias), _stream()), "swiglu")
+                            ctypes.c_int(inter), ctypes.c_int(block), _ptr(bias), ctypes.c_int(act), _stream()), "swiglu")
 
 
 class DeltaNorm(NamedTuple):
@@ -510,6 +521,7 @@ class DeltaNorm(NamedTuple):
     eps: float = 0.0
     scale1: float = 1.0
     scale2: float = 1.0
+    again: Optional[torch.Tensor] = None  # float32, shaped like the stream: joins it behind the delta
 
 
 def add_rmsnorm(x: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, out: torch.Tensor,
@@ -549,15 +561,19 @@ def add_rmsnorm(x: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Te
     if out.shape[0] != n_rows:
         raise KernelError(f"rmsnorm: out has {out.shape[0]} rows, expected {n_rows}")
     if delta_norm is not None:
-        if delta is None:
+        if delta is None and (delta_norm.weight is not None or delta_norm.again is None):
             raise KernelError("rmsnorm: a norm of the delta without a delta")
+        if delta_norm.again is not None:
+            _need(delta_norm.again, "rmsnorm earlier stream", torch.float32, 2)
+            if delta_norm.again.shape != x.shape:
+                raise KernelError("rmsnorm: the earlier stream differs from x in shape")
         if delta_norm.weight is not None:
             _need(delta_norm.weight, "rmsnorm delta weight", torch.float32, 1)
             if delta_norm.weight.shape[0] != width:
                 raise KernelError("rmsnorm: the delta's norm weight differs in width")
         _check(lib().mll_add_normed_rmsnorm(
             _ptr(x), _ptr(delta), _ptr(delta2), ctypes.c_float(delta_norm.scale1), ctypes.c_float(delta_norm.scale2),
-            _ptr(delta_norm.weight), ctypes.c_float(delta_norm.eps), _ptr(weight), _ptr(out), _ptr(rows),
+            _ptr(delta_norm.weight), ctypes.c_float(delta_norm.eps), _ptr(delta_norm.again), _ptr(weight), _ptr(out), _ptr(rows),
             dtype_code(delta_dtype), dtype_code(out.dtype), ctypes.c_int(n_rows), ctypes.c_int(width),
             ctypes.c_float(eps), _stream()), "rmsnorm (normed delta)")
         return
@@ -637,6 +653,23 @@ def add_dynamic_tanh(x: torch.Tensor, deltas, norms, rows: Optional[torch.Tensor
     _check(lib().mll_add_tanh_norm(_ptr(x), *(p for p, _ in d), *(f for _, f in d), *n[0], *n[1], _ptr(rows),
                                    dtype_code(delta_dtype), dtype_code(out_dtype), ctypes.c_int(n_rows),
                                    ctypes.c_int(width), _stream()), "tanh_norm")
+
+
+def stream_add(x: torch.Tensor, delta=None, delta2=None, scale1: float = 1.0, scale2: float = 1.0,
+               again: Optional[torch.Tensor] = None) -> None:
+    """x += scale1 * delta (+ scale2 * delta2) (+ again), the float32 stream in place."""
+    _need(x, "stream_add x", torch.float32, 2)
+    for name, t, dtype in (("delta", delta, None), ("delta2", delta2, delta.dtype if delta is not None else None),
+                           ("earlier stream", again, torch.float32)):
+        if t is not None:
+            _need(t, f"stream_add {name}", dtype, 2)
+            if t.shape != x.shape:
+                raise KernelError(f"stream_add: {name} differs from x in shape")
+    if delta2 is not None and delta is None:
+        raise KernelError("stream_add: a second delta without a first")
+    _check(lib().mll_stream_add(_ptr(x), _ptr(delta), _ptr(delta2), ctypes.c_float(scale1), ctypes.c_float(scale2), _ptr(again),
+                                dtype_code(delta.dtype if delta is not None else torch.float32),
+                                ctypes.c_longlong(x.numel()), _stream()), "stream_add")
 
 
 def stream_concat(x: torch.Tensor, delta: Optional[torch.Tensor], x0: torch.Tensor, out: torch.Tensor) -> None:
@@ -1115,6 +1148,55 @@ def local_attention_prepare(qkv, q_weight, k_weight, cos, sin, tok_pos, tok_seq,
         "local_attention_prepare")
 
 
+def conv_attention_advances(d: int, dv: int, rot: int, interleaved: bool, taps: int, row: int) -> bool:
+    """Whether `conv_attention_prepare` on rows of `row` columns can move the convolution's state on itself (`advance`)."""
+    return bool(lib().mll_conv_attention_advances(d, dv, rot, int(interleaved), taps, row))
+
+
+def conv_attention_prepare(qkv, bias, conv_w, conv_state, cos, sin, tok_pos, tok_seq, seq_slot, seq_qstart, block_table,
+                           q_out, k_cache, v_cache, n_heads: int, n_kv_heads: int, d: int, dv: int, rot: int,
+                           interleaved: bool, taps: int, advance: bool = False) -> None:
+    """As `local_attention_prepare` (without norms) for projections that pass a short causal convolution over time, per
+    channel of q, k and v, before the rotation: qkv [T, ld] holds the projections, `bias` (float32 [C] or None) is added to
+    them first, conv_w float32 [C, taps] (the last tap meets the current token), conv_state float32 [slots, taps - 1, C] the
+    last inputs of every sequence, biases included.  `advance` (every sequence brings one token, sizes as
+    `conv_attention_advances` says): conv_state moves on in the same kernel."""
+    _need(qkv, "conv attention qkv", None, 2)
+    _need(q_out, "conv attention q", qkv.dtype, 2)
+    _need(k_cache, "conv attention k cache", qkv.dtype, 4)
+    _need(v_cache, "conv attention v cache", qkv.dtype, 4)
+    _need(conv_w, "conv attention taps", torch.float32, 2)
+    _need(conv_state, "conv attention state", torch.float32, 3)
+    n, C = qkv.shape[0], (n_heads + n_kv_heads) * d + n_kv_heads * dv
+    if tuple(k_cache.shape[1:]) != (n_kv_heads, PAGE, d) or tuple(v_cache.shape[1:]) != (n_kv_heads, PAGE, dv):
+        raise KernelError(f"conv attention: caches {tuple(k_cache.shape)} / {tuple(v_cache.shape)} do not fit "
+                          f"{n_kv_heads} heads of {d} / {dv}")
+    if tuple(q_out.shape) != (n, n_heads * d):
+        raise KernelError(f"conv attention: q out {tuple(q_out.shape)}, expected {(n, n_heads * d)}")
+    if tuple(conv_w.shape) != (C, taps) or tuple(conv_state.shape[1:]) != (taps - 1, C):
+        raise KernelError(f"conv attention: taps {tuple(conv_w.shape)} / state {tuple(conv_state.shape)} for {C} channels of "
+                          f"{taps} taps")
+    if bias is not None:
+        _need(bias, "conv attention bias", torch.float32, 1)
+        if bias.shape[0] != C:
+            raise KernelError(f"conv attention: bias of {bias.shape[0]}, expected {C}")
+    if rot:
+        _need(cos, "conv attention cos", torch.float32, 2)
+        _need(sin, "conv attention sin", torch.float32, 2)
+        if cos.shape[1] != rot // 2 or sin.shape != cos.shape:
+            raise KernelError(f"conv attention: rotary table {tuple(cos.shape)} for {rot} rotated dimensions")
+    for name, t in (("tok_pos", tok_pos), ("tok_seq", tok_seq), ("seq_slot", seq_slot), ("seq_qstart", seq_qstart)):
+        _need(t, f"conv attention {name}", torch.int32, 1)
+    _need(block_table, "conv attention block table", torch.int32, 2)
+    _check(lib().mll_conv_attention_prepare(
+        _ptr(qkv), _ptr(bias), _ptr(conv_w), _ptr(conv_state), ctypes.c_int(int(advance)), _ptr(cos if rot else None),
+        _ptr(sin if rot else None), _ptr(tok_pos), _ptr(tok_seq), _ptr(seq_slot), _ptr(seq_qstart), _ptr(block_table),
+        _ptr(q_out), _ptr(k_cache), _ptr(v_cache), dtype_code(qkv.dtype), ctypes.c_int(n), ctypes.c_int(qkv.shape[1]),
+        ctypes.c_int(n_heads), ctypes.c_int(n_kv_heads), ctypes.c_int(d), ctypes.c_int(dv), ctypes.c_int(rot),
+        ctypes.c_int(int(interleaved)), ctypes.c_int(block_table.shape[1]), ctypes.c_int(taps), _stream()),
+        "conv_attention_prepare")
+
+
 def _check_local_caches(k_cache, v_cache, n_kv_heads: int, d: int, dv: int, v_in_k: bool) -> None:
     if tuple(k_cache.shape[1:]) != (n_kv_heads, PAGE, d):
         raise KernelError(f"local attention: key cache {tuple(k_cache.shape)} does not fit {n_kv_heads} heads of {d}")
@@ -1232,9 +1314,10 @@ def local_attention_heads_splits(n_seqs: int, blocks_per_seq: int, multiprocesso
 # mixers with a matrix-valued state per sequence and head
 # --------------------------------------------------------------------------- #
 def retention_prepare(proj, cos, sin, tok_pos, q, k, v, n_heads: int, d: int, dv: int, rot: int, interleaved: bool,
-                      k_scale: float) -> None:
+                      k_scale: float, silu: bool = False) -> None:
     """proj [T, ld] (q heads of d, k heads of d, v heads of dv, ...) -> float32 q, k [T, H, d] with the first `rot`
-    dimensions of every head rotated and k * k_scale, v [T, H, dv]."""
+    dimensions of every head rotated and k * k_scale, v [T, H, dv].  `silu` (without a rotation): q, k and v pass silu
+    first."""
     _need(proj, "retention proj", None, 2)
     n = proj.shape[0]
     for name, t, width in (("q", q, n_heads * d), ("k", k, n_heads * d), ("v", v, n_heads * dv)):
@@ -1250,17 +1333,27 @@ def retention_prepare(proj, cos, sin, tok_pos, q, k, v, n_heads: int, d: int, dv
     _check(lib().mll_retention_prepare(
         _ptr(proj), _ptr(cos if rot else None), _ptr(sin if rot else None), _ptr(tok_pos), _ptr(q), _ptr(k), _ptr(v),
         dtype_code(proj.dtype), ctypes.c_int(n), ctypes.c_int(proj.shape[1]), ctypes.c_int(n_heads), ctypes.c_int(d),
-        ctypes.c_int(dv), ctypes.c_int(rot), ctypes.c_int(int(interleaved)), ctypes.c_float(k_scale), _stream()),
-        "retention_prepare")
+        ctypes.c_int(dv), ctypes.c_int(rot), ctypes.c_int(int(interleaved)), ctypes.c_float(k_scale),
+        ctypes.c_int(int(silu)), _stream()), "lightning_prepare" if silu else "retention_prepare")
+
+
+def delta_prepare_advances(n_heads: int, n_kv_heads: int, d: int, dv: int, taps: int, row: int) -> bool:
+    """Whether `delta_prepare` on rows of `row` columns can move the convolution's state on itself (`advance`)."""
+    return bool(lib().mll_delta_prepare_advances(n_heads, n_kv_heads, d, dv, taps, row))
 
 
 def delta_prepare(proj, rate, conv_w, conv_state, a_log, dt_bias, tok_seq, seq_slot, seq_qstart, q, k, v, g, beta,
-                  n_heads: int, n_kv_heads: int, d: int, dv: int, taps: int, unit_eps: float) -> None:
+                  n_heads: int, n_kv_heads: int, d: int, dv: int, taps: int, unit_eps: float,
+                  advance: bool = False) -> None:
     """The inputs of the gated delta rule from the projections of a step (see csrc/recurrent.cu): proj [T, ld]
     holds q, k (G heads of d), v (H heads of dv) and beta's pre-activation (H); rate float32 [T, >= H * d] the
-    decay's; conv_w float32 [C, taps]; conv_state float32 [slots, taps - 1, C]."""
+    decay's; conv_w float32 [C, taps]; conv_state float32 [slots, taps - 1, C].  rate None: one decay per head (g [T, H],
+    dt_bias [H]), whose pre-activations (H) follow beta's in proj.  `advance` (every sequence brings one token, sizes as
+    `delta_prepare_advances` says): conv_state moves on in the same kernel."""
     _need(proj, "delta proj", None, 2)
-    _need(rate, "delta rate", torch.float32, 2)
+    per_head = rate is None
+    if not per_head:
+        _need(rate, "delta rate", torch.float32, 2)
     _need(conv_w, "delta conv weights", torch.float32, 2)
     _need(conv_state, "delta conv state", torch.float32, 3)
     _need(a_log, "delta A_log", torch.float32, 1)
@@ -1270,31 +1363,36 @@ def delta_prepare(proj, rate, conv_w, conv_state, a_log, dt_bias, tok_seq, seq_s
     if tuple(conv_w.shape) != (C, taps) or tuple(conv_state.shape[1:]) != (max(taps - 1, 0), C):
         raise KernelError(f"delta prepare: conv weights {tuple(conv_w.shape)} / state {tuple(conv_state.shape)} "
                           f"for {C} channels of {taps} taps")
-    if a_log.shape[0] != n_heads or dt_bias.shape[0] != n_heads * d or rate.shape[0] != n:
+    decays = n_heads if per_head else n_heads * d
+    if a_log.shape[0] != n_heads or dt_bias.shape[0] != decays or (not per_head and rate.shape[0] != n):
         raise KernelError("delta prepare: A_log, dt_bias or rate of the wrong size")
     for name, t, width in (("q", q, n_kv_heads * d), ("k", k, n_kv_heads * d), ("v", v, n_heads * dv),
-                           ("g", g, n_heads * d), ("beta", beta, n_heads)):
+                           ("g", g, decays), ("beta", beta, n_heads)):
         _need(t, f"delta {name}", torch.float32, 2)
         if tuple(t.shape) != (n, width):
             raise KernelError(f"delta prepare: {name} {tuple(t.shape)}, expected {(n, width)}")
     _check(lib().mll_delta_prepare(
         _ptr(proj), _ptr(rate), _ptr(conv_w), _ptr(conv_state), _ptr(a_log), _ptr(dt_bias), _ptr(tok_seq),
         _ptr(seq_slot), _ptr(seq_qstart), _ptr(q), _ptr(k), _ptr(v), _ptr(g), _ptr(beta), dtype_code(proj.dtype),
-        ctypes.c_int(n), ctypes.c_int(proj.shape[1]), ctypes.c_int(rate.shape[1]), ctypes.c_int(n_heads),
+        ctypes.c_int(n), ctypes.c_int(proj.shape[1]), ctypes.c_int(0 if per_head else rate.shape[1]), ctypes.c_int(n_heads),
         ctypes.c_int(n_kv_heads), ctypes.c_int(d), ctypes.c_int(dv), ctypes.c_int(taps), ctypes.c_float(unit_eps),
-        _stream()), "delta_prepare")
+        _ptr(conv_state if advance else None), _stream()), "delta_prepare")
 
 
 def conv_state_update(proj, conv_state, seq_slot, seq_qstart, seq_qlen, n_seqs: int, channels: int, taps: int,
-                      first_column: int = 0) -> None:
+                      first_column: int = 0, bias: Optional[torch.Tensor] = None) -> None:
     """conv_state[slot] <- the last taps - 1 rows of (conv_state[slot], this step's rows of
-    proj[:, first_column:first_column + channels])."""
+    proj[:, first_column:first_column + channels] + bias)."""
+    if bias is not None:
+        _need(bias, "conv state bias", torch.float32, 1)
+        if bias.shape[0] < channels:
+            raise KernelError("conv state update: the bias has one value per channel")
     _need(proj, "conv state proj", None, 2)
     _need(conv_state, "conv state", torch.float32, 3)
     if tuple(conv_state.shape[1:]) != (max(taps - 1, 0), channels):
         raise KernelError(f"conv state update: state {tuple(conv_state.shape)} for {channels} channels of {taps} taps")
     _check(lib().mll_conv_state_update(
-        _ptr(proj), dtype_code(proj.dtype), ctypes.c_int(first_column), ctypes.c_int(proj.shape[1]), _ptr(conv_state),
+        _ptr(proj), dtype_code(proj.dtype), ctypes.c_int(first_column), ctypes.c_int(proj.shape[1]), _ptr(bias), _ptr(conv_state),
         _ptr(seq_slot),
         _ptr(seq_qstart), _ptr(seq_qlen), ctypes.c_int(n_seqs), ctypes.c_int(channels), ctypes.c_int(taps), _stream()),
         "conv_state_update")
@@ -1304,14 +1402,16 @@ def state_scan(q, k, v, g, beta, head_decay, state, out, seq_slot, seq_qstart, s
                n_kv_heads: int, d: int, dv: int, token_decay: Optional[torch.Tensor] = None) -> None:
     """The recurrence S <- decay S + k u^T, o = S^T q over each sequence's tokens of the step, from and to
     state [slots, H, d, dv] (float32).  With g [T, H * d] and beta [T, H]: the gated delta rule
-    (u = beta (v - S^T k) after the decay); with g alone: a decay per key channel and u = v; with `token_decay`
+    (u = beta (v - S^T k) after the decay); with `token_decay` float32 [T, H] and beta: the same with one decay per token
+    and head; with g alone: a decay per key channel and u = v; with `token_decay`
     float32 [T, H]: one decay per token and head and u = v; else head_decay float32 [H] and u = v."""
     n = q.shape[0]
+    scalar_delta = token_decay is not None and beta is not None
     delta = g is not None and beta is not None
     channel = g is not None and beta is None
-    per_token = token_decay is not None
-    if per_token and (g is not None or beta is not None or head_decay is not None):
-        raise KernelError("state scan: a decay per token and head stands alone")
+    per_token = token_decay is not None and beta is None
+    if token_decay is not None and (g is not None or head_decay is not None):
+        raise KernelError("state scan: a decay per token and head goes with no other decay")
     for name, t, width in (("q", q, n_kv_heads * d), ("k", k, n_kv_heads * d), ("v", v, n_heads * dv),
                            ("out", out, n_heads * dv)):
         _need(t, f"state scan {name}", torch.float32, 2)
@@ -1320,7 +1420,13 @@ def state_scan(q, k, v, g, beta, head_decay, state, out, seq_slot, seq_qstart, s
     _need(state, "state scan state", torch.float32, 4)
     if tuple(state.shape[1:]) != (n_heads, d, dv):
         raise KernelError(f"state scan: state {tuple(state.shape)} for {n_heads} heads of {d} x {dv}")
-    if delta:
+    if scalar_delta:
+        for name, t in (("token decay", token_decay), ("beta", beta)):
+            _need(t, f"state scan {name}", torch.float32, 2)
+            if tuple(t.shape) != (n, n_heads):
+                raise KernelError(f"state scan: one {name} per token and head is needed")
+        g = token_decay
+    elif delta:
         _need(g, "state scan g", torch.float32, 2)
         _need(beta, "state scan beta", torch.float32, 2)
         if tuple(g.shape) != (n, n_heads * d) or tuple(beta.shape) != (n, n_heads):
@@ -1341,9 +1447,9 @@ def state_scan(q, k, v, g, beta, head_decay, state, out, seq_slot, seq_qstart, s
     _check(lib().mll_state_scan(
         _ptr(q), _ptr(k), _ptr(v), _ptr(g), _ptr(beta), _ptr(head_decay), _ptr(state), _ptr(out), _ptr(seq_slot),
         _ptr(seq_qstart), _ptr(seq_qlen), ctypes.c_int(n_seqs), ctypes.c_int(n_heads), ctypes.c_int(n_kv_heads),
-        ctypes.c_int(d), ctypes.c_int(dv), ctypes.c_int(1 if delta else (2 if channel else (3 if per_token else 0))),
+        ctypes.c_int(d), ctypes.c_int(dv), ctypes.c_int(4 if scalar_delta else (1 if delta else (2 if channel else (3 if per_token else 0)))),
         _stream()),
-        "state_scan (delta rule)" if delta else ("state_scan (channel decay)" if channel else
+        "state_scan (delta rule, head decay)" if scalar_delta else "state_scan (delta rule)" if delta else ("state_scan (channel decay)" if channel else
                                                  ("state_scan (token decay)" if per_token else "state_scan (retention)")))
 
 
@@ -1446,6 +1552,22 @@ def head_norm_gate(o, weight, gate, out, n_heads: int, dv: int, eps: float, act:
         dtype_code(gate.dtype), ctypes.c_int(gate.shape[1]), _ptr(out),
         dtype_code(out.dtype), ctypes.c_int(n), ctypes.c_int(n_heads), ctypes.c_int(dv), ctypes.c_float(eps),
         ctypes.c_int(act), _stream()), "head_norm_gate")
+
+
+def row_norm_gate(o, weight, gate, out, eps: float, act: int, gate_col: int = 0) -> None:
+    """out[t, :] = o[t, :] / sqrt(mean(o[t, :]^2) + eps) * weight * act(gate[t, :]), the whole row at once; o float32
+    [T, W], weight float32 [W], gate [T, ld] in out's dtype, of which columns gate_col .. gate_col + W are read."""
+    _need(o, "row norm o", torch.float32, 2)
+    _need(weight, "row norm weight", torch.float32, 1)
+    _need(out, "row norm out", None, 2)
+    _need(gate, "row norm gate", out.dtype, 2)
+    n, width = o.shape
+    if out.shape != o.shape or weight.shape[0] != width or gate.shape[0] != n or not 0 <= gate_col <= gate.shape[1] - width:
+        raise KernelError(f"row norm gate: o {tuple(o.shape)}, out {tuple(out.shape)}, gate {tuple(gate.shape)}")
+    _check(lib().mll_row_norm_gate(
+        _ptr(o), _ptr(weight), ctypes.c_void_p(gate.data_ptr() + gate_col * gate.element_size()), dtype_code(gate.dtype),
+        ctypes.c_int(gate.shape[1]), _ptr(out), dtype_code(out.dtype), ctypes.c_int(n), ctypes.c_int(width),
+        ctypes.c_float(eps), ctypes.c_int(act), _stream()), "row_norm_gate")
 
 
 # --------------------------------------------------------------------------- #

@@ -26,7 +26,7 @@ namespace cg = cooperative_groups;
 
 namespace mll {
 
-enum : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_RESID = 3 };
+enum : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_RESID = 3, EPI_GEGLU = 4 };
 
 struct LinearArgs {
   const __nv_bfloat16* x;  // [M, K]
@@ -239,7 +239,8 @@ linear_small_kernel(LinearArgs a) {
   __syncthreads();
 
   // epilogue on the full sums: element (row, m) of the tile is y[m][n0 + row]
-  if (a.epilogue == EPI_SWIGLU) {
+  if (a.epilogue == EPI_SWIGLU || a.epilogue == EPI_GEGLU) {
+    const int act = a.epilogue == EPI_GEGLU ? GATE_ACT_GELU_TANH : GATE_ACT_SILU;
     __nv_bfloat16* out = (__nv_bfloat16*)a.out;
     const int half = a.N >> 1;
     for (int i = threadIdx.x; i < 8 * 8 * NT; i += LS_WARPS * 32) {
@@ -247,7 +248,7 @@ linear_small_kernel(LinearArgs a) {
       if (m < a.M && n0 + r + 8 < a.N) {
         const float f = a.in.sumsq ? row_factor[m] : 1.f;
         const float gate = red[0][r][m] * f, up = red[0][r + 8][m] * f;
-        out[(size_t)m * half + (n0 >> 1) + r] = __float2bfloat16_rn(gate / (1.f + expf(-gate)) * up);
+        out[(size_t)m * half + (n0 >> 1) + r] = __float2bfloat16_rn(gate_act_mul<false>(act, gate, up));
       }
     }
   } else if (a.epilogue == EPI_RESID) {
@@ -319,13 +320,13 @@ int launch_linear_small(const LinearArgs& a, int tiles, int ranks, cudaStream_t 
 // Whether mll_linear_small takes this problem (the caller uses the library GEMM otherwise).
 MLL_API int mll_linear_small_supported(int M, int N, int K, int epilogue) {
   if (M < 1 || M > 64 || N < 16 || K < 32 || K % 32 != 0) return 0;
-  if (epilogue == mll::EPI_SWIGLU && N % 16 != 0) return 0;
+  if ((epilogue == mll::EPI_SWIGLU || epilogue == mll::EPI_GEGLU) && N % 16 != 0) return 0;
   return 1;
 }
 
 // x: bfloat16 [M, K]; w: bfloat16 [N, K]; bias: optional float32 [N];
 // out: bfloat16 [M, N] (epilogue 0), float32 [M, N] (1), or bfloat16 [M, N / 2] = silu(gate) * up
-// with gate and up rows of w interleaved in blocks of 8 (2).  ranks: cluster size along K
+// with gate and up rows of w interleaved in blocks of 8 (2; 4: gelu in its tanh form in silu's place).  ranks: cluster size along K
 // (1, 2, 4 or 8), 0 = choose.
 // in_sumsq (optional, float32 [M, in_stride], in_partials of each row used): x lacks its RMS norm's
 // factor 1 / sqrt(sum / K + in_eps), which the result is multiplied by.
@@ -336,11 +337,11 @@ MLL_API int mll_linear_small_fused(const void* x, const void* w, const float* bi
                                    int epilogue, int ranks, const float* in_sumsq, int in_partials, int in_stride,
                                    float in_eps, float* resid, const float* next_w, float* out_sumsq, int out_stride,
                                    cudaStream_t stream) {
-  MLL_REQUIRE(epilogue >= 0 && epilogue <= 3, "linear_small: unknown epilogue %d", epilogue);
+  MLL_REQUIRE(epilogue >= 0 && epilogue <= 4, "linear_small: unknown epilogue %d", epilogue);
   MLL_REQUIRE(mll_linear_small_supported(M, N, K, epilogue == mll::EPI_RESID ? 0 : epilogue),
               "linear_small: unsupported sizes M=%d N=%d K=%d", M, N, K);
   MLL_REQUIRE(((uintptr_t)x % 16 == 0) && ((uintptr_t)w % 16 == 0), "linear_small: operands must be 16-byte aligned");
-  MLL_REQUIRE(epilogue != mll::EPI_SWIGLU || bias == nullptr, "linear_small: the SwiGLU epilogue takes no bias");
+  MLL_REQUIRE((epilogue != mll::EPI_SWIGLU && epilogue != mll::EPI_GEGLU) || bias == nullptr, "linear_small: the gated epilogues take no bias");
   if (in_sumsq) {
     MLL_REQUIRE(in_partials >= 1 && in_stride >= in_partials, "linear_small: partial sums: %d of stride %d",
                 in_partials, in_stride);

@@ -46,7 +46,7 @@ __device__ int mll_tc5_error_flag = 0;
 
 namespace mll {
 
-enum : int { CEPI_BF16 = 0, CEPI_F32 = 1, CEPI_SWIGLU = 2, CEPI_RESID = 3 };
+enum : int { CEPI_BF16 = 0, CEPI_F32 = 1, CEPI_SWIGLU = 2, CEPI_RESID = 3, CEPI_GEGLU = 4 };
 constexpr int C_ROWS = 128;     // weight rows per block (the MMA's M)
 constexpr int C_KB = 64;        // k elements per stage: one 128-byte swizzle span
 constexpr int C_THREADS = 256;  // 4 epilogue warps, then producer A, MMA A, producer B, MMA B (even / odd k-blocks)
@@ -292,7 +292,8 @@ linear_tc5_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constan
 
   // red[m][row] is y[m][n0 + row]; neighbouring threads take neighbouring weight rows
   const int span = max(0, m_end - m_begin);
-  if (a.epilogue == CEPI_SWIGLU) {
+  if (a.epilogue == CEPI_SWIGLU || a.epilogue == CEPI_GEGLU) {
+    const int act = a.epilogue == CEPI_GEGLU ? GATE_ACT_GELU_TANH : GATE_ACT_SILU;
     __nv_bfloat16* out = (__nv_bfloat16*)a.out;
     const int half = a.N >> 1;
     for (int i = tid; i < span * (C_ROWS / 2); i += C_THREADS) {
@@ -301,7 +302,7 @@ linear_tc5_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constan
       if (n0 + row + 8 < a.N) {
         const float f = a.in.sumsq ? row_factor[m] : 1.f;
         const float gate = red[m * C_ROWS + row] * f, up = red[m * C_ROWS + row + 8] * f;
-        out[(size_t)m * half + (n0 >> 1) + j] = __float2bfloat16_rn(gate / (1.f + expf(-gate)) * up);
+        out[(size_t)m * half + (n0 >> 1) + j] = __float2bfloat16_rn(gate_act_mul<false>(act, gate, up));
       }
     }
   } else if (a.epilogue == CEPI_RESID) {
@@ -398,7 +399,7 @@ extern "C" int* mll_linear_tc5_error_address() {
 // Up to 64 rows: 16, 32 or 64 batch columns per MMA, chosen by the row count.
 MLL_API int mll_linear_tc5_supported(int M, int N, int K, int epilogue) {
   if (M < 1 || M > 64 || N < 1 || K < 8 || K % 8 != 0) return 0;
-  if (epilogue == mll::CEPI_SWIGLU && N % 16 != 0) return 0;
+  if ((epilogue == mll::CEPI_SWIGLU || epilogue == mll::CEPI_GEGLU) && N % 16 != 0) return 0;
   return 1;
 }
 
@@ -410,11 +411,11 @@ MLL_API int mll_linear_tc5_fused(const void* x, const void* w, const float* bias
                                  cudaStream_t stream) {
   MLL_REQUIRE(!in_sumsq || (in_partials >= 1 && in_stride >= in_partials && in_eps >= 0.f),
               "linear_tc5: partial sums: %d of stride %d", in_partials, in_stride);
-  MLL_REQUIRE(epilogue >= 0 && epilogue <= 3, "linear_tc5: unknown epilogue %d", epilogue);
+  MLL_REQUIRE(epilogue >= 0 && epilogue <= 4, "linear_tc5: unknown epilogue %d", epilogue);
   MLL_REQUIRE(mll_linear_tc5_supported(M, N, K, epilogue == mll::CEPI_RESID ? 0 : epilogue),
               "linear_tc5: unsupported sizes M=%d N=%d K=%d", M, N, K);
   MLL_REQUIRE(((uintptr_t)x % 16 == 0) && ((uintptr_t)w % 16 == 0), "linear_tc5: operands must be 16-byte aligned");
-  MLL_REQUIRE(epilogue != mll::CEPI_SWIGLU || bias == nullptr, "linear_tc5: the SwiGLU epilogue takes no bias");
+  MLL_REQUIRE((epilogue != mll::CEPI_SWIGLU && epilogue != mll::CEPI_GEGLU) || bias == nullptr, "linear_tc5: the gated epilogues take no bias");
   if (epilogue == mll::CEPI_RESID)
     MLL_REQUIRE(resid && next_w && out_sumsq && out_stride >= (N + 15) / 16,
                 "linear_tc5: the residual epilogue needs resid, next_w and out_sumsq with stride >= %d", (N + 15) / 16);

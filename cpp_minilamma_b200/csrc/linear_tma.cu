@@ -35,7 +35,7 @@ __device__ int mll_device_error_flag = 0;
 
 namespace mll {
 
-enum : int { TEPI_BF16 = 0, TEPI_F32 = 1, TEPI_SWIGLU = 2 };
+enum : int { TEPI_BF16 = 0, TEPI_F32 = 1, TEPI_SWIGLU = 2, TEPI_GEGLU = 4 };  // codes shared with the other small products
 constexpr int T_ROWS = 64;     // weight rows per block
 constexpr int T_KB = 64;       // k elements per stage (128 bytes: one swizzle span)
 constexpr int T_STAGES = 3;
@@ -240,7 +240,8 @@ linear_tma_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constan
 
   // epilogue on the full sums: red[row][m] is y[m][n0 + row]
   constexpr int COLS = 8 * NT;
-  if (a.epilogue == TEPI_SWIGLU) {
+  if (a.epilogue == TEPI_SWIGLU || a.epilogue == TEPI_GEGLU) {
+    const int act = a.epilogue == TEPI_GEGLU ? GATE_ACT_GELU_TANH : GATE_ACT_SILU;
     __nv_bfloat16* out = (__nv_bfloat16*)a.out;
     const int half = a.N >> 1;
     for (int i = tid; i < (T_ROWS / 2) * COLS; i += T_THREADS) {
@@ -249,7 +250,7 @@ linear_tma_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constan
       if (m < a.M && n0 + row + 8 < a.N) {
         const float f = a.in.sumsq ? row_factor[m] : 1.f;
         const float gate = red[row * COLS + m] * f, up = red[(row + 8) * COLS + m] * f;
-        out[(size_t)m * half + (n0 >> 1) + j] = __float2bfloat16_rn(gate / (1.f + expf(-gate)) * up);
+        out[(size_t)m * half + (n0 >> 1) + j] = __float2bfloat16_rn(gate_act_mul<false>(act, gate, up));
       }
     }
   } else {
@@ -390,7 +391,7 @@ extern "C" int* mll_linear_tma_error_address() {
 
 MLL_API int mll_linear_tma_supported(int M, int N, int K, int epilogue) {
   if (M < 1 || M > 64 || N < 1 || K < 8 || K % 8 != 0) return 0;
-  if (epilogue == mll::TEPI_SWIGLU && N % 16 != 0) return 0;
+  if ((epilogue == mll::TEPI_SWIGLU || epilogue == mll::TEPI_GEGLU) && N % 16 != 0) return 0;
   return 1;
 }
 
@@ -403,9 +404,9 @@ MLL_API int mll_linear_tma_fused(const void* x, const void* w, const float* bias
   MLL_REQUIRE(!in_sumsq || (in_partials >= 1 && in_stride >= in_partials && in_eps >= 0.f),
               "linear_tma: partial sums: %d of stride %d", in_partials, in_stride);
   MLL_REQUIRE(mll_linear_tma_supported(M, N, K, epilogue), "linear_tma: unsupported sizes M=%d N=%d K=%d", M, N, K);
-  MLL_REQUIRE(epilogue >= 0 && epilogue <= 2, "linear_tma: unknown epilogue %d", epilogue);
+  MLL_REQUIRE((epilogue >= 0 && epilogue <= 2) || epilogue == mll::TEPI_GEGLU, "linear_tma: unknown epilogue %d", epilogue);
   MLL_REQUIRE(((uintptr_t)x % 16 == 0) && ((uintptr_t)w % 16 == 0), "linear_tma: operands must be 16-byte aligned");
-  MLL_REQUIRE(epilogue != mll::TEPI_SWIGLU || bias == nullptr, "linear_tma: the SwiGLU epilogue takes no bias");
+  MLL_REQUIRE((epilogue != mll::TEPI_SWIGLU && epilogue != mll::TEPI_GEGLU) || bias == nullptr, "linear_tma: the gated epilogues take no bias");
   const int tiles = (N + mll::T_ROWS - 1) / mll::T_ROWS;
   const int k_blocks = (K + mll::T_KB - 1) / mll::T_KB;
   if (ranks <= 0) {

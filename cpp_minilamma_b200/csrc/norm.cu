@@ -12,10 +12,12 @@ namespace mll {
 
 // What happens to the delta on its way into the stream: delta = scale1 * delta (+ scale2 * delta2), and with a
 // weight the delta is normalised by its own root mean square first: x += delta / sqrt(mean(delta^2) + eps) * weight
-// (a block whose sub-layers end in a norm of their own).
+// (a block whose sub-layers end in a norm of their own).  `again` joins the stream as well (a stretch of layers that gets
+// the embedding's output anew before each of its runs).
 struct DeltaNorm {
   const float* weight;  // [width] or null: the delta is added as it is
   float eps, scale1, scale2;
+  const float* again;   // [*, width] or null: an earlier state of the stream, added behind the delta
 };
 
 // One block per output row.  The row (after the add) is kept in shared memory between
@@ -48,8 +50,9 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ x, const DeltaT* __restri
     if (dr) {
       const float d = dr2 ? dn.scale1 * to_float(dr[i]) + dn.scale2 * to_float(dr2[i]) : dn.scale1 * to_float(dr[i]);
       v += dn.weight ? d * fd * dn.weight[i] : d;
-      if (!rows) xr[i] = v;
     }
+    if (dn.again) v += dn.again[(size_t)src * width + i];
+    if ((dr || dn.again) && !rows) xr[i] = v;
     row_buf[i] = v;
     ss += v * v;
   }
@@ -144,6 +147,17 @@ add_rmsnorm_vec_kernel(float* __restrict__ x, const DeltaT* __restrict__ delta,
       const int g = threadIdx.x + k * 256;
       if (g < groups) {
         v[k].x += dl[k].x; v[k].y += dl[k].y; v[k].z += dl[k].z; v[k].w += dl[k].w;
+        if (!rows && !dn.again) store4(xr + 4 * g, v[k]);
+      }
+    }
+  }
+  if (dn.again) {
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int g = threadIdx.x + k * 256;
+      if (g < groups) {
+        const float4 e = load4<float>(dn.again + (size_t)src * width + 4 * g);
+        v[k].x += e.x; v[k].y += e.y; v[k].z += e.z; v[k].w += e.w;
         if (!rows) store4(xr + 4 * g, v[k]);
       }
     }
@@ -171,7 +185,8 @@ int launch_add_rmsnorm(float* x, const void* delta, const void* delta2, const fl
                        const int* rows, int n_rows, int width, float eps, DeltaNorm dn, cudaStream_t stream) {
   const bool aligned = width % 4 == 0 && ((uintptr_t)x % 16 == 0) && ((uintptr_t)weight % 16 == 0) &&
                        ((uintptr_t)out % 16 == 0) && (!delta || (uintptr_t)delta % 8 == 0) &&
-                       (!delta2 || (uintptr_t)delta2 % 8 == 0) && (!dn.weight || (uintptr_t)dn.weight % 16 == 0);
+                       (!delta2 || (uintptr_t)delta2 % 8 == 0) && (!dn.weight || (uintptr_t)dn.weight % 16 == 0) &&
+                       (uintptr_t)dn.again % 16 == 0;
   if (aligned && width <= 4 * 256 * 8) {
     const int groups = width / 4;
     if (groups <= 256 * 2)
@@ -421,6 +436,23 @@ int launch_add_tanh_norm(const TanhNormArgs& a, cudaStream_t stream) {
   return 0;
 }
 
+// x += scale1 * delta (+ scale2 * delta2) (+ again): the stream alone, for a norm that cannot add all of it itself.
+template <typename DeltaT>
+__global__ void __launch_bounds__(256) stream_add_kernel(float* __restrict__ x, const DeltaT* __restrict__ delta,
+                                                         const DeltaT* __restrict__ delta2, float scale1, float scale2,
+                                                         const float* __restrict__ again, size_t total) {
+  for (size_t i = (size_t)blockIdx.x * 256 + threadIdx.x; i < total; i += (size_t)gridDim.x * 256) {
+    float v = x[i];
+    if (delta) {
+      float d = scale1 * to_float(delta[i]);
+      if (delta2) d = fmaf(scale2, to_float(delta2[i]), d);
+      v += d;
+    }
+    if (again) v += again[i];
+    x[i] = v;
+  }
+}
+
 // Finishes a norm whose rows were left without their factor (RowNormIn), for a product that cannot do
 // it itself: out[m, i] = values[m, i] * factor(m).  One block per row.
 __global__ void apply_row_norm_kernel(const __nv_bfloat16* __restrict__ values, RowNormIn in,
@@ -454,9 +486,9 @@ MLL_API int mll_apply_row_norm(const void* values, const float* sumsq, int parti
 }
 
 MLL_API int mll_add_normed_rmsnorm(float* x, const void* delta, const void* delta2, float scale1, float scale2,
-                                   const float* delta_weight, float delta_eps, const float* weight, void* out,
-                                   const int* rows, int delta_dtype, int out_dtype, int n_rows, int width, float eps,
-                                   cudaStream_t stream);
+                                   const float* delta_weight, float delta_eps, const float* again, const float* weight,
+                                   void* out, const int* rows, int delta_dtype, int out_dtype, int n_rows, int width,
+                                   float eps, cudaStream_t stream);
 
 // x: float32 [*, width] residual stream; delta, delta2: optional [*, width] of `delta_dtype` (delta2 only with
 // delta: the outputs of two parts that read the same norm); weight: float32 [width]; out: [n_rows, width] of
@@ -465,21 +497,21 @@ MLL_API int mll_add_normed_rmsnorm(float* x, const void* delta, const void* delt
 MLL_API int mll_add2_rmsnorm(float* x, const void* delta, const void* delta2, const float* weight, void* out,
                              const int* rows, int delta_dtype, int out_dtype, int n_rows, int width, float eps,
                              cudaStream_t stream) {
-  return mll_add_normed_rmsnorm(x, delta, delta2, 1.f, 1.f, nullptr, 0.f, weight, out, rows, delta_dtype, out_dtype,
+  return mll_add_normed_rmsnorm(x, delta, delta2, 1.f, 1.f, nullptr, 0.f, nullptr, weight, out, rows, delta_dtype, out_dtype,
                                 n_rows, width, eps, stream);
 }
 
 // As mll_add2_rmsnorm with the delta scaled and normalised on its way into the stream:
 //   d = scale1 * delta (+ scale2 * delta2);  with delta_weight: d <- d / sqrt(mean(d^2) + delta_eps) * delta_weight;
-//   x += d;  out = x / sqrt(mean(x^2) + eps) * weight.   All of it float32.
+//   x += d (+ again, float32 [*, width]);  out = x / sqrt(mean(x^2) + eps) * weight.   All of it float32.
 MLL_API int mll_add_normed_rmsnorm(float* x, const void* delta, const void* delta2, float scale1, float scale2,
-                                   const float* delta_weight, float delta_eps, const float* weight, void* out,
-                                   const int* rows, int delta_dtype, int out_dtype, int n_rows, int width, float eps,
-                                   cudaStream_t stream) {
+                                   const float* delta_weight, float delta_eps, const float* again, const float* weight,
+                                   void* out, const int* rows, int delta_dtype, int out_dtype, int n_rows, int width,
+                                   float eps, cudaStream_t stream) {
   MLL_REQUIRE(n_rows >= 0 && width > 0, "rmsnorm: bad sizes rows=%d width=%d", n_rows, width);
   MLL_REQUIRE(delta || !delta_weight, "rmsnorm: a norm of the delta without a delta");
   MLL_REQUIRE(delta_eps >= 0.f, "rmsnorm: the delta's eps must be non-negative");
-  const mll::DeltaNorm dn{delta_weight, delta_eps, scale1, scale2};
+  const mll::DeltaNorm dn{delta_weight, delta_eps, scale1, scale2, again};
   MLL_REQUIRE(width <= 50 * 1024, "rmsnorm: width %d exceeds the 51200 floats one block can hold", width);
   MLL_REQUIRE(eps >= 0.f, "rmsnorm: eps must be non-negative");
   MLL_REQUIRE(delta || !delta2, "rmsnorm: a second delta without a first");
@@ -500,6 +532,25 @@ MLL_API int mll_add_rmsnorm(float* x, const void* delta, const float* weight, vo
                             const int* rows, int act_dtype, int n_rows, int width, float eps,
                             cudaStream_t stream) {
   return mll_add2_rmsnorm(x, delta, nullptr, weight, out, rows, act_dtype, act_dtype, n_rows, width, eps, stream);
+}
+
+// x: float32 [n]; delta, delta2: optional [n] of `dtype`; again: optional float32 [n].
+MLL_API int mll_stream_add(float* x, const void* delta, const void* delta2, float scale1, float scale2, const float* again,
+                           int dtype, long long n, cudaStream_t stream) {
+  MLL_REQUIRE(n >= 0 && (delta || !delta2), "stream add: bad size or a second delta without a first");
+  if (n == 0) return 0;
+  long long blocks = (n + 255) / 256;
+  if (blocks > mll_sm_count() * 16) blocks = mll_sm_count() * 16;
+  if (dtype == MLL_F32)
+    MLL_LAUNCH((mll::stream_add_kernel<float>), (int)blocks, 256, 0, stream, x, (const float*)delta, (const float*)delta2,
+               scale1, scale2, again, (size_t)n);
+  else if (dtype == MLL_BF16)
+    MLL_LAUNCH((mll::stream_add_kernel<__nv_bfloat16>), (int)blocks, 256, 0, stream, x, (const __nv_bfloat16*)delta,
+               (const __nv_bfloat16*)delta2, scale1, scale2, again, (size_t)n);
+  else
+    MLL_REQUIRE(false, "stream add: unknown dtype %d", dtype);
+  MLL_LAUNCH_CHECK();
+  return 0;
 }
 
 // Layer norm with weight and (optional) bias after the residual add; arguments as for mll_add2_rmsnorm.

@@ -152,8 +152,7 @@ class Model:
         for i, entry in enumerate(schedule):
             layer = self.layers[entry.layer]
             if entry.enter is not None:
-                self.stream_ops[entry.enter[0]].forward(step, x, pending, x0, entry.enter[1])
-                pending = None
+                pending = self.stream_ops[entry.enter[0]].forward(step, x, pending, x0, entry.enter[1])
             if layer.block.first_reader(layer) is None:
                 pending = layer.block.forward(step, x, pending, layer, cache.view(i))
                 continue

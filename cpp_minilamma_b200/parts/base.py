@@ -143,6 +143,11 @@ class PreNormed:
     norm: "Norm"
 
 
+def row_count(h) -> int:
+    """Rows of a part's input, which may be a `PreNormed`."""
+    return (h.values if isinstance(h, PreNormed) else h).shape[0]
+
+
 @dataclass
 class ResidualTarget:
     """Offered to a part with `adds_residual`: it may add its output to the float32 residual stream `x`
@@ -185,6 +190,16 @@ class NormedDelta:
 
     delta: Any
     norm: "Norm"
+
+
+@dataclass
+class PendingStream:
+    """What is still to be added to the residual stream - a part's output in any of the forms above, or None - and an
+    earlier state of the stream, float32 [T, D], that joins it as well (`x += delta + again`).  The next RMS norm does both
+    in its one kernel; other norms add to the stream first."""
+
+    delta: Any
+    again: torch.Tensor
 
 
 # --------------------------------------------------------------------------- #
@@ -330,9 +345,10 @@ class StreamOp(Part):
 
     role = "stream_op"
 
-    def forward(self, step, x: torch.Tensor, pending, x0: torch.Tensor, pass_number: int) -> None:
-        """Rewrite the float32 stream `x` [T, D] in place.  `pending` is the output of the part before, still
-        to be added to x first (a tensor or None); `x0` is the stream as the embedding left it."""
+    def forward(self, step, x: torch.Tensor, pending, x0: torch.Tensor, pass_number: int):
+        """Rewrite the float32 stream `x` [T, D] in place and return None, or leave the work to the norm that reads the
+        stream next by returning what it has to add.  `pending` is the output of the part before, still to be added to x
+        first; `x0` is the stream as the embedding left it."""
         raise NotImplementedError
 
 

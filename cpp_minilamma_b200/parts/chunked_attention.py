@@ -13,7 +13,9 @@ no value), or a learned one (exp(c_h) in place of the 1, c_h a number per query 
 that are the keys themselves as projected, before norm and rotation (no W_v; dv == d); an output gate read from the mixer's own input, one number per head (head h's output times
 sigmoid(W_g h)_h) or one per element, applied before W_o; a smooth cap on the scores, s <- cap * tanh(s / cap) after the
 scale; a window that keeps the sequence's first tokens (key j < keep_first stays visible whatever its distance, at its own
-position); keys and values that are another layer's (`kv_shared`: the layer has queries and an output projection only and
+position); biases on the four projections, and a short causal convolution over time on every channel of q, k and v behind
+its bias and before the rotation, u_t <- sum_j w[:, j] u_(t - taps + 1 + j) with nothing before the sequence's first token
+(the last taps - 1 inputs of a sequence are state beside its keys and values); keys and values that are another layer's (`kv_shared`: the layer has queries and an output projection only and
 reads the cache of the schedule entry named by its own entry's `cache_of`, with its own mask, scale and cap).
 
 Chunks count from position 0 of the sequence, not from where a step's tokens begin.  Keys and values live in
@@ -29,7 +31,7 @@ from typing import List, Optional
 import torch
 
 from ..csrc import kernels as K
-from .base import BuildContext, CacheNeed, KVNeed, Mixer, WeightSpec, register_part
+from .base import BuildContext, CacheNeed, KVNeed, Mixer, StateNeed, WeightSpec, register_part, row_count
 from .linear import Linear
 from .rope import shared_position_encoding
 
@@ -75,6 +77,10 @@ class ChunkedAttention(Mixer):
       keep_first                                    with a window: keys at positions below this stay visible
       kv_shared                                     True: no names["k"] / ["v"]; keys and values are read from the cache
                                                     of another schedule entry (the entry's `cache_of`)
+      conv                                          0 / None, or the taps of a short convolution on q, k and v; its weights
+                                                    are loaded as names["q"] + ".conv" and so on, [channels, taps]
+      bias                                          True: biases names["q"] + ".b" and so on, of q, k, v (with `conv` only)
+                                                    and of the output projection
       cache_window, cache_keep_first                what the cache must keep when other layers read this layer's keys
                                                     with masks of their own (default: this layer's window / keep_first)
       names                                         {"q","k","v","o"} (and "g"): tensor names
@@ -82,6 +88,7 @@ class ChunkedAttention(Mixer):
 
     capturable = True
     workspace = "attention"
+    takes_prenormed = True  # the fused product finishes the norm in front of it
 
     def __init__(self, params, ctx: BuildContext):
         super().__init__(params, ctx)
@@ -130,9 +137,21 @@ class ChunkedAttention(Mixer):
         if self.dv > 256:
             raise ValueError(f"attention: value heads of {self.dv} exceed the 256 the kernel takes")
         self.position = shared_position_encoding(params["position"], ctx) if self.rot else None
+        self.taps = int(params.get("conv") or 0)
+        self.bias = bool(params.get("bias", False))
+        self.channels = self.n_heads * self.d + self.n_kv_heads * (self.d + self.dv)  # that pass the convolution
+        if self.taps < 0:
+            raise ValueError(f"attention: a convolution of {self.taps} taps")
+        if self.taps and (self.kv_shared or self.qk_norm or self.q_temp or self.v_from_k):
+            raise ValueError("attention: a convolution goes with plain projections of the layer's own")
+        if self.bias and not self.taps:
+            raise ValueError("attention: biases go with a convolution")
         self.qkv: Optional[Linear] = None
         self.o: Optional[Linear] = None
         self.q_weight = self.k_weight = None
+        self.conv_w: Optional[torch.Tensor] = None
+        self.qkv_bias: Optional[torch.Tensor] = None
+        self.advances: Optional[bool] = None  # the preparation kernel moves the convolution's state on itself
 
     def weight_specs(self) -> List[WeightSpec]:
         D = self.ctx.hidden_size
@@ -142,6 +161,13 @@ class ChunkedAttention(Mixer):
             if not self.v_from_k:
                 specs.append(WeightSpec(self.names["v"], (self.n_kv_heads * self.dv, D)))
         specs.append(WeightSpec(self.names["o"], (D, self.n_heads * self.dv)))
+        for p, channels in (("q", self.n_heads * self.d), ("k", self.n_kv_heads * self.d), ("v", self.n_kv_heads * self.dv)):
+            if self.bias:
+                specs.append(WeightSpec(self.names[p] + ".b", (channels,), kind="vector"))
+            if self.taps:
+                specs.append(WeightSpec(self.names[p] + ".conv", (channels, self.taps), kind="vector"))
+        if self.bias:
+            specs.append(WeightSpec(self.names["o"] + ".b", (D,), kind="vector"))
         if self.sink_name:
             specs.append(WeightSpec(self.sink_name, (self.n_heads,), kind="vector", init="normal"))
         if self.gate:
@@ -169,7 +195,12 @@ class ChunkedAttention(Mixer):
         del mats, fused
         if self.sink_name:
             self.sink_values = store.take(self.sink_name)
-        self.o = Linear(store.take(self.names["o"]), self.names["o"])
+        if self.taps:
+            self.conv_w = torch.cat([store.take(self.names[p] + ".conv") for p in ("q", "k", "v")], dim=0).contiguous()
+        if self.bias:
+            self.qkv_bias = torch.cat([store.take(self.names[p] + ".b") for p in ("q", "k", "v")], dim=0).contiguous()
+        self.o = Linear(store.take(self.names["o"]), self.names["o"],
+                        store.take(self.names["o"] + ".b").contiguous() if self.bias else None)
         if self.qk_norm:
             self.q_weight = store.take(self.qk_norm["q"])
             self.k_weight = store.take(self.qk_norm["k"])
@@ -181,8 +212,9 @@ class ChunkedAttention(Mixer):
         # a query reads nothing before its chunk's first key, which lies less than `chunk` positions back
         window = self.cache_window
         reach = self.chunk if window <= 0 else (min(self.chunk, window) if self.chunk else window)
+        state = StateNeed((("conv", (self.taps - 1, self.channels)),)) if self.taps else None
         return CacheNeed(kv=KVNeed(self.n_kv_heads, self.d, reach, self.dv if self.dv != self.d else 0,
-                                   keep_first=self.cache_keep_first if reach > 0 and not self.chunk else 0))
+                                   keep_first=self.cache_keep_first if reach > 0 and not self.chunk else 0), state=state)
 
     def _tensor_cores(self) -> bool:
         return K.local_attention_mma_supported(self.ctx.act_dtype, self.d, self.dv)
@@ -195,7 +227,7 @@ class ChunkedAttention(Mixer):
         return prompt_tiles(shape)
 
     def forward(self, step, h, cache):
-        T = h.shape[0]
+        T = row_count(h)
         act = self.ctx.act_dtype
         if cache.k is None:
             raise RuntimeError("attention: the cache view has no key/value storage")
@@ -204,12 +236,15 @@ class ChunkedAttention(Mixer):
         qkv = self.qkv.forward(step, h, "qkv")
         cos, sin = self.position.tables() if self.position is not None else (None, None)
         q = step.ws.buffer("q", (T, self.n_heads * self.d), act)
-        K.local_attention_prepare(qkv, self.q_weight, self.k_weight, cos, sin, step.tok_pos, step.tok_seq,
-                                  step.seq_slot, cache.block_table, q, cache.k, cache.v, self.n_heads,
-                                  self.n_kv_heads, self.d, self.dv, self.rot,
-                                  bool(self.position.interleaved) if self.position is not None else False,
-                                  float(self.qk_norm["eps"]) if self.qk_norm else 0.0, q_temp=self.q_temp,
-                                  v_from_k=self.v_from_k, write_kv=not self.kv_shared)
+        if self.taps:
+            self._prepare_behind_convolution(step, qkv, cos, sin, q, cache)
+        else:
+            K.local_attention_prepare(qkv, self.q_weight, self.k_weight, cos, sin, step.tok_pos, step.tok_seq,
+                                      step.seq_slot, cache.block_table, q, cache.k, cache.v, self.n_heads,
+                                      self.n_kv_heads, self.d, self.dv, self.rot,
+                                      bool(self.position.interleaved) if self.position is not None else False,
+                                      float(self.qk_norm["eps"]) if self.qk_norm else 0.0, q_temp=self.q_temp,
+                                      v_from_k=self.v_from_k, write_kv=not self.kv_shared)
         out = step.ws.buffer("attn", (T, self.n_heads * self.dv), act)
         self._attend(step, q, cache, out)
         if self.gate:
@@ -217,6 +252,18 @@ class ChunkedAttention(Mixer):
                                                 self.n_kv_heads * (self.d if self.v_from_k else self.d + self.dv))
             K.heads_gate(out, qkv, gate_col, out, self.n_heads, self.dv, per_head=self.gate == "head")
         return self.o.forward(step, out, self.out_name)
+
+    def _prepare_behind_convolution(self, step, qkv, cos, sin, q, cache) -> None:
+        interleaved = bool(self.position.interleaved) if self.position is not None else False
+        if self.advances is None:
+            self.advances = K.conv_attention_advances(self.d, self.dv, self.rot, interleaved, self.taps, qkv.shape[1])
+        advance = self.advances and step.all_decode
+        K.conv_attention_prepare(qkv, self.qkv_bias, self.conv_w, cache.state["conv"], cos, sin, step.tok_pos, step.tok_seq,
+                                 step.seq_slot, step.seq_qstart, cache.block_table, q, cache.k, cache.v, self.n_heads,
+                                 self.n_kv_heads, self.d, self.dv, self.rot, interleaved, self.taps, advance=advance)
+        if self.taps > 1 and not advance:
+            K.conv_state_update(qkv, cache.state["conv"], step.seq_slot, step.seq_qstart, step.seq_qlen, step.n_seqs,
+                                self.channels, self.taps, bias=self.qkv_bias)
 
     def _attend(self, step, q, cache, out) -> None:
         act = self.ctx.act_dtype

@@ -103,7 +103,7 @@ class PairHashEmbedding(TokenEmbedding):
 
 class LMHead(Part):
     """params: vocab, name, tied_to (name of the embedding tensor, or None), scale (a factor on the float32 logits,
-    default 1)."""
+    default 1), softcap (0 / None, or the cap c: logits <- c * tanh(logits / c) behind the scale)."""
 
     capturable = True
 
@@ -115,6 +115,9 @@ class LMHead(Part):
         self.name = params["name"]
         self.tied_to = params.get("tied_to")
         self.scale = float(params.get("scale", 1.0))
+        self.softcap = float(params.get("softcap") or 0.0)
+        if self.softcap < 0:
+            raise ValueError(f"lm head: a cap of {self.softcap}")
         self.linear: Optional[Linear] = None
 
     def weight_specs(self) -> List[WeightSpec]:
@@ -131,7 +134,9 @@ class LMHead(Part):
 
     def forward(self, step, h: torch.Tensor, out_name: str = "logits") -> torch.Tensor:
         logits = self.linear.forward(step, h, out_name, out_dtype=torch.float32)
-        if self.scale != 1.0:
+        if self.softcap:
+            K.softcap_(logits, self.softcap, self.scale)
+        elif self.scale != 1.0:
             K.scale_(logits, self.scale)
         return logits
 

@@ -5,6 +5,8 @@ W is row-major [out, in] as in the reference (src/cuda_matmul.cc:181-186, one
   * bfloat16 weight, bfloat16 x: tensor-core product with float32 accumulation;
   * float32 weight: a true float32 product (TF32 must be off; it is refused otherwise);
     bfloat16 activations are widened first and the result narrowed afterwards.
+A bias (float32 [N], not in the reference) is added in float32 by the weight-streaming kernels' epilogues, or by a
+kernel behind the library product.
 Large products go to the library GEMM (as the reference's do); small batches of rows go
 to this package's own weight-streaming kernel when it is available for the shape.  That kernel can
 also finish the norm in front of the product (input `PreNormed`) and start the one behind it
@@ -21,7 +23,7 @@ from .base import PreNormed, ResidualTarget
 
 
 class Linear:
-    def __init__(self, weight: torch.Tensor, name: str = "linear"):
+    def __init__(self, weight: torch.Tensor, name: str = "linear", bias: Optional[torch.Tensor] = None):
         if weight.dim() != 2:
             raise ValueError(f"{name}: weight must be [out, in], got {tuple(weight.shape)}")
         if weight.dtype not in (torch.float32, torch.bfloat16):
@@ -29,9 +31,12 @@ class Linear:
         self.weight = weight.contiguous()
         self.name = name
         self.out_features, self.in_features = weight.shape
+        if bias is not None and (bias.dtype != torch.float32 or tuple(bias.shape) != (self.out_features,)):
+            raise ValueError(f"{name}: the bias must be float32 [{self.out_features}], got {bias.dtype} {tuple(bias.shape)}")
+        self.bias = bias
 
     def parameter_bytes(self) -> int:
-        return self.weight.numel() * self.weight.element_size()
+        return self.weight.numel() * self.weight.element_size() + (4 * self.out_features if self.bias is not None else 0)
 
     def forward(self, step, x, out_name: str, out_dtype: Optional[torch.dtype] = None,
                 into: Optional[ResidualTarget] = None, out: Optional[torch.Tensor] = None):
@@ -70,9 +75,10 @@ class Linear:
             if out_dtype == torch.float32:
                 out = given if given is not None else ws.buffer(out_name, (rows, self.out_features), torch.float32)
                 torch.mm(x, w.t(), out=out)
-                return out
+                return self._biased(out)
             wide_out = ws.buffer(out_name + ".y32", (rows, self.out_features), torch.float32)
             torch.mm(x, w.t(), out=wide_out)
+            self._biased(wide_out)
             out = given if given is not None else ws.buffer(out_name, (rows, self.out_features), out_dtype)
             K.cast(wide_out, out)
             return out
@@ -85,7 +91,7 @@ class Linear:
             if made is not None:
                 return made
         out = given if given is not None else ws.buffer(out_name, (rows, self.out_features), out_dtype)
-        if rows <= step.small_rows and K.small_linear(x, w, None, out,
+        if rows <= step.small_rows and K.small_linear(x, w, self.bias, out,
                                                        K.EPI_F32 if out_dtype == torch.float32 else K.EPI_BF16,
                                                        row_norm):
             return out
@@ -97,8 +103,12 @@ class Linear:
             torch.mm(x, w.t(), out=out)
         else:  # bfloat16 operands, float32 result (the logits)
             _mm_bf16_to_f32(x, w, out)
-        return out
+        return self._biased(out)
 
+    def _biased(self, out: torch.Tensor) -> torch.Tensor:
+        if self.bias is not None:
+            K.add_bias(out, self.bias)
+        return out
 
     def _into_residual(self, ws, x, row_norm, out_name: str, into: ResidualTarget) -> Optional[PreNormed]:
         prenorm = into.norm.prenorm_weight()
@@ -109,7 +119,7 @@ class Linear:
         partials = -(-width // K.NORM_TILE)
         values = ws.buffer(out_name + ".pre", (rows, width), torch.bfloat16)
         sumsq = ws.buffer(out_name + ".sumsq", (rows, partials), torch.float32)
-        if not K.small_linear(x, self.weight, None, values, K.EPI_RESID, row_norm, K.ResidualOut(into.x, weight, sumsq)):
+        if not K.small_linear(x, self.weight, self.bias, values, K.EPI_RESID, row_norm, K.ResidualOut(into.x, weight, sumsq)):
             return None
         return PreNormed(values, sumsq, partials, eps, into.norm)
 

@@ -7,7 +7,8 @@ The reference's FfnForward (src/forward.cc:313-322) with SiLU as x / (1 + exp(-x
 8-15, ...), which puts a gate value and its up value into the same thread of a
 tensor-core accumulator tile.  With biases (not in the reference) the form is
 down( silu(gate(h) + b_g) * (up(h) + b_u) ) + b_d: the gate and up biases are added in float32 inside the activation
-kernel, in the fused matrix's row order.
+kernel, in the fused matrix's row order.  `activation` "gelu_tanh" (not in the reference) puts gelu in its tanh form in
+silu's place, everywhere the same kernels.
 """
 from __future__ import annotations
 
@@ -37,7 +38,8 @@ def fuse_gate_up(gate: torch.Tensor, up: torch.Tensor):
 class SwiGLUFeedForward(FeedForward):
     """params: intermediate, names {"gate","up","down"} (tensor name stems, ".weight" is appended; with
     `bare_names` they are the tensor names themselves); bias_names {"gate","up","down"}: tensor names of the three
-    biases, or None for a feed-forward without biases; out_name: workspace name of the result (default "down")."""
+    biases, or None for a feed-forward without biases; activation: "silu" (default) or "gelu_tanh"; out_name: workspace
+    name of the result (default "down")."""
 
     capturable = True
     takes_prenormed = True  # the gate/up product may read rows whose norm it finishes itself
@@ -50,6 +52,11 @@ class SwiGLUFeedForward(FeedForward):
         self.names = {k: v + suffix for k, v in dict(params["names"]).items()}
         self.bias_names = dict(params["bias_names"]) if params.get("bias_names") else None
         self.out_name = params.get("out_name") or "down"
+        forms = {"silu": (K.GATE_ACT_SILU, K.EPI_SWIGLU), "gelu_tanh": (K.GATE_ACT_GELU_TANH, K.EPI_GEGLU)}
+        name = params.get("activation") or "silu"
+        if name not in forms:
+            raise ValueError(f"feed-forward: activation {name!r} is not one of {sorted(forms)}")
+        self.act, self.epilogue = forms[name]
         if self.bias_names:  # the products that fold norms away know no bias: this instance takes plain rows
             self.takes_prenormed = self.adds_residual = False
         self.gate_up_bias = self.down_bias = None
@@ -86,7 +93,7 @@ class SwiGLUFeedForward(FeedForward):
         if self.gate_up_bias is not None:
             gu = self.gate_up.forward(step, h, "gu")
             act = step.ws.buffer("act", (h.shape[0], self.inter), gu.dtype)
-            K.swiglu(gu, act, self.block, bias=self.gate_up_bias)
+            K.swiglu(gu, act, self.block, bias=self.gate_up_bias, act=self.act)
             out = self.down.forward(step, act, self.out_name)
             K.add_bias(out, self.down_bias)
             return out
@@ -95,22 +102,22 @@ class SwiGLUFeedForward(FeedForward):
         w = self.gate_up.weight
         fused = (rows <= step.small_rows and self.block == INTERLEAVE and w.dtype == torch.bfloat16
                  and values.dtype == torch.bfloat16
-                 and bool(K.small_linear_kind(rows, 2 * self.inter, w.shape[1], K.EPI_SWIGLU)))
+                 and bool(K.small_linear_kind(rows, 2 * self.inter, w.shape[1], self.epilogue)))
         if fused:
             # few rows: one weight-streaming kernel whose epilogue applies the activation
             act = step.ws.buffer("act", (rows, self.inter), torch.bfloat16)
-            K.small_linear(values, w, None, act, K.EPI_SWIGLU, row_norm)
+            K.small_linear(values, w, None, act, self.epilogue, row_norm)
         elif (row_norm is not None and w.dtype == torch.bfloat16 and self.inter % 8 == 0
               and not K.small_linear_kind(rows, 2 * self.inter, w.shape[1], K.EPI_BF16)):
             # the library product cannot finish the norm in front of it: it runs on the rows as they are and
             # the activation kernel multiplies gate and up by the rows' factors
             gu = self.gate_up.forward(step, values, "gu")
             act = step.ws.buffer("act", (rows, self.inter), torch.bfloat16)
-            K.swiglu(gu, act, self.block, row_norm, w.shape[1])
+            K.swiglu(gu, act, self.block, row_norm, w.shape[1], act=self.act)
         else:
             gu = self.gate_up.forward(step, h, "gu")
             act = step.ws.buffer("act", (rows, self.inter), gu.dtype)
-            K.swiglu(gu, act, self.block)
+            K.swiglu(gu, act, self.block, act=self.act)
         return self.down.forward(step, act, self.out_name, into=into)
 
 

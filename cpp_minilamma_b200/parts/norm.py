@@ -24,11 +24,14 @@ from typing import List, Optional
 import torch
 
 from ..csrc import kernels as K
-from .base import BuildContext, Norm, NormedDelta, PendingSum, PreNormed, ScaledDelta, WeightSpec, register_part
+from .base import BuildContext, Norm, NormedDelta, PendingStream, PendingSum, PreNormed, ScaledDelta, WeightSpec, register_part
 
 
 def _delta_parts(delta):
     """(first, second, DeltaNorm or None) of whatever a block left pending."""
+    if isinstance(delta, PendingStream):
+        first, second, form = _delta_parts(delta.delta)
+        return first, second, (form or K.DeltaNorm(None))._replace(again=delta.again)
     norm = None
     if isinstance(delta, NormedDelta):
         norm = delta.norm
@@ -47,8 +50,19 @@ def _delta_parts(delta):
     return first, second, K.DeltaNorm(norm.weight if norm is not None else None, norm.eps if norm is not None else 0.0, s1, s2)
 
 
+def _add_earlier_stream(x, delta):
+    """For a norm that adds outputs only: an earlier state of the stream joins it in a kernel of its own first.  (For
+    gathered rows, whose norm leaves the stream alone, too: nothing reads the stream after them.)"""
+    if isinstance(delta, PendingStream):
+        K.stream_add(x, again=delta.again)
+        return delta.delta
+    return delta
+
+
 def _add_third(x, delta):
     """The norms below take two outputs: a third one joins the stream in a kernel of its own first."""
+    if isinstance(delta, PendingStream):
+        return replace(delta, delta=_add_third(x, delta.delta))
     if isinstance(delta, PendingSum) and delta.third is not None:
         K.add_dynamic_tanh(x, [(delta.third, 1.0)], [])
         return replace(delta, third=None)
@@ -137,7 +151,7 @@ class LayerNorm(Norm):
             raise RuntimeError(f"{self.name}: a layer norm cannot finish rows that were prepared for another norm")
         n = x.shape[0] if rows is None else rows.shape[0]
         out = step.ws.buffer(out_name, (n, self.width), self.ctx.act_dtype)
-        delta = _add_third(x, delta)
+        delta = _add_third(x, _add_earlier_stream(x, delta))
         if isinstance(delta, (NormedDelta, ScaledDelta)) or (isinstance(delta, PendingSum) and (delta.scale_first != 1.0 or delta.scale_second != 1.0)):
             raise RuntimeError(f"{self.name}: a layer norm adds its delta as it is (no norm or factor on the way in)")
         if isinstance(delta, PendingSum):
@@ -199,14 +213,14 @@ class DynamicTanh(Norm):
     def forward(self, step, x, delta, rows=None, out_name: str = "h"):
         n = x.shape[0] if rows is None else rows.shape[0]
         out = step.ws.buffer(out_name, (n, self.width), self.ctx.act_dtype)
-        K.add_dynamic_tanh(x, self._deltas(delta), [self._form(out)], rows)
+        K.add_dynamic_tanh(x, self._deltas(_add_earlier_stream(x, delta)), [self._form(out)], rows)
         return out
 
     def forward_pair(self, step, x, delta, other, out_names=("h", "h2")):
         if not isinstance(other, DynamicTanh):
             return super().forward_pair(step, x, delta, other, out_names)
         first, second = (step.ws.buffer(name, (x.shape[0], self.width), self.ctx.act_dtype) for name in out_names)
-        K.add_dynamic_tanh(x, self._deltas(delta), [self._form(first), other._form(second)])
+        K.add_dynamic_tanh(x, self._deltas(_add_earlier_stream(x, delta)), [self._form(first), other._form(second)])
         return first, second
 
 

@@ -6,6 +6,9 @@ A model that runs a stretch of its layers several times gives every pass the ori
 of its own so that the passes can tell each other apart.  W_in is [D, 2 D] with x's columns first; `step` is
 [passes, D].  The sum x + (pending output of the layer before) is formed in float32 and the result is written to
 the float32 stream; the product itself runs in the activation dtype like every other projection.
+
+`embedding_again` is the form without weights, x <- x + x0: no kernel of its own - the norm that reads the stream next
+adds x0 together with the output that is still pending.
 """
 from __future__ import annotations
 
@@ -14,7 +17,7 @@ from typing import List, Optional
 import torch
 
 from ..csrc import kernels as K
-from .base import BuildContext, PendingSum, PreNormed, StreamOp, WeightSpec, register_part
+from .base import BuildContext, PendingStream, PendingSum, PreNormed, StreamOp, WeightSpec, register_part
 from .linear import Linear
 
 
@@ -58,4 +61,16 @@ class Reentry(StreamOp):
         K.add_bias(x, self.step_vectors[pass_number])
 
 
+class EmbeddingAgain(StreamOp):
+    """x <- x + x0.  No params."""
+
+    capturable = True
+
+    def forward(self, step, x, pending, x0, pass_number: int):
+        if isinstance(pending, PreNormed):
+            pending = None  # the part before has added its output to the stream already
+        return PendingStream(pending, x0)
+
+
 register_part("stream_op", "reentry", Reentry)
+register_part("stream_op", "embedding_again", EmbeddingAgain)

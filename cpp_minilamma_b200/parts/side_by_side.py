@@ -30,6 +30,7 @@ class SideBySideMixer(Mixer):
         self.apart = (self.left.workspace is not None and self.right.workspace is not None
                       and self.left.workspace != self.right.workspace)
         self.capturable = self.left.capturable and self.right.capturable
+        self.takes_prenormed = self.left.takes_prenormed and self.right.takes_prenormed
         left, right = self.left.cache_need(), self.right.cache_need()
         if left.kv is not None and right.kv is not None:
             raise ValueError("side-by-side mixers: only one of the two may keep keys and values")

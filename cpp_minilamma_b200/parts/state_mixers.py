@@ -1,8 +1,8 @@
 """Mixers that keep a matrix per sequence and head instead of keys and values.
 
-Both run   S_t = diag(g_t) S_(t-1) + k_t u_t^T,   o_t = S_t^T q_t   (S is [d, dv], float32, zero at the start of a
+All run   S_t = diag(g_t) S_(t-1) + k_t u_t^T,   o_t = S_t^T q_t   (S is [d, dv], float32, zero at the start of a
 sequence, carried from step to step in the cache's per-slot state), so the read-out sees the current token's
-write, and both normalise every head's o by its root mean square before a gate and the output projection.
+write, and normalise o by its root mean square (per head, or a row at once) before a gate and the output projection.
 
 `retention`          one fixed decay per head, u = v; q and k carry rotary positions, k / sqrt(d);
                      out = W_o (o / rms(o) * silu(W_g h))
@@ -11,6 +11,12 @@ write, and both normalise every head's o by its root mean square before a gate a
                      convolution over time and silu, q and k are scaled to unit length per head, q / sqrt(d);
                      the last taps - 1 convolution inputs of a sequence are state too;
                      out = W_o (o / rms(o) * w * sigmoid(W_g2 W_g1 h))
+
+`delta_rule_head_decay`  the delta rule with one decay per head, g = exp(-exp(A) softplus(W_a h + b)), and an output
+                     gate of full rank: out = W_o (o / rms(o) * w * silu(W_g h)); everything else as above
+
+`lightning_attention`  one fixed decay per head, u = v, silu on q, k and v; the row of all heads' o is normalised at once:
+                     out = W_o (o / rms(o) * w * sigmoid(W_g h))
 
 `gated_linear_attention`  a decay per head and key channel, g = sigmoid(W_a2 W_a1 h + b)^(1 / tau), u = v, q / sqrt(d);
                      out = W_o (o / rms(o) * w * silu(W_g h))
@@ -32,7 +38,7 @@ from typing import List, Optional
 import torch
 
 from ..csrc import kernels as K
-from .base import BuildContext, CacheNeed, Mixer, StateNeed, WeightSpec, register_part
+from .base import BuildContext, CacheNeed, Mixer, StateNeed, WeightSpec, register_part, row_count
 from .linear import Linear
 from .rope import shared_position_encoding
 
@@ -208,6 +214,153 @@ class GatedDeltaRule(Mixer):
         return self.o.forward(step, gated, "o")
 
 
+class HeadDecayDeltaRule(Mixer):
+    """params: n_heads, n_kv_heads (q and k heads; value head h reads q/k head h // (n_heads / n_kv_heads)), head_dim,
+    v_head_dim, conv (taps), eps (of the head norm), unit_eps (inside the root of the unit length), out_name (workspace name
+    of the result, default "o"), names: tensor names for "q", "k", "v" (their convolution taps are "<name>.conv"), "b", "a",
+    "dt_bias", "A_log", "g", "norm", "o"."""
+
+    capturable = True
+    workspace = "mix"
+    takes_prenormed = True
+    adds_residual = True
+
+    def __init__(self, params, ctx: BuildContext):
+        super().__init__(params, ctx)
+        self.n_heads = int(params["n_heads"])
+        self.n_kv_heads = int(params["n_kv_heads"])
+        self.d = int(params["head_dim"])
+        self.dv = int(params["v_head_dim"])
+        self.taps = int(params["conv"])
+        self.eps = float(params["eps"])
+        self.unit_eps = float(params.get("unit_eps", 1e-6))
+        self.names = dict(params["names"])
+        self.out_name = params.get("out_name") or "o"
+        if self.n_heads % self.n_kv_heads:
+            raise ValueError(f"delta rule: {self.n_heads} heads are not a multiple of {self.n_kv_heads} q/k heads")
+        if self.taps < 1:
+            raise ValueError("delta rule: the convolution needs at least one tap")
+        self.channels = 2 * self.n_kv_heads * self.d + self.n_heads * self.dv
+        # a row of the one product: q, k, v | beta, decay | the gate, from a multiple of eight columns on
+        self.gate_col = self.channels + 2 * self.n_heads
+        self.gate_col += -self.gate_col % 8
+        self.proj: Optional[Linear] = None
+        self.o: Optional[Linear] = None
+        self.advances: Optional[bool] = None  # the preparation kernel moves the convolution's state on itself
+
+    def weight_specs(self) -> List[WeightSpec]:
+        D, H, G, d, dv, n = self.ctx.hidden_size, self.n_heads, self.n_kv_heads, self.d, self.dv, self.names
+        return [WeightSpec(n["q"], (G * d, D)), WeightSpec(n["q"] + ".conv", (G * d, self.taps), kind="vector"),
+                WeightSpec(n["k"], (G * d, D)), WeightSpec(n["k"] + ".conv", (G * d, self.taps), kind="vector"),
+                WeightSpec(n["v"], (H * dv, D)), WeightSpec(n["v"] + ".conv", (H * dv, self.taps), kind="vector"),
+                WeightSpec(n["b"], (H, D)), WeightSpec(n["A_log"], (H,), kind="vector"),
+                WeightSpec(n["norm"], (dv,), kind="vector", init="norm"), WeightSpec(n["a"], (H, D)),
+                WeightSpec(n["dt_bias"], (H,), kind="vector"), WeightSpec(n["g"], (H * dv, D)),
+                WeightSpec(n["o"], (D, H * dv))]
+
+    def bind(self, store) -> None:
+        n = self.names
+        mats = _same_dtype([store.take(n[p]) for p in ("q", "k", "v", "b", "a", "g")])
+        front = _pad_rows(torch.cat(mats[:5], dim=0))
+        self.proj = Linear(_pad_rows(torch.cat([front, mats[5]], dim=0)), n["q"] + "+k+v+b+a+g")
+        del mats, front
+        self.conv_w = torch.cat([store.take(n[p] + ".conv") for p in ("q", "k", "v")], dim=0).contiguous()
+        self.a_log = store.take(n["A_log"])
+        self.dt_bias = store.take(n["dt_bias"])
+        self.norm_w = store.take(n["norm"])
+        self.o = Linear(store.take(n["o"]), n["o"])
+
+    def parameter_bytes(self) -> int:
+        return self.proj.parameter_bytes() + self.o.parameter_bytes()
+
+    def cache_need(self) -> CacheNeed:
+        return CacheNeed(state=StateNeed((("S", (self.n_heads, self.d, self.dv)),
+                                          ("conv", (self.taps - 1, self.channels)))))
+
+    def forward(self, step, h, cache, into=None):
+        T, H, G, d, dv = row_count(h), self.n_heads, self.n_kv_heads, self.d, self.dv
+        ws = step.ws
+        proj = self.proj.forward(step, h, "mix.proj")
+        q = ws.buffer("mix.q", (T, G * d), torch.float32)
+        k = ws.buffer("mix.k", (T, G * d), torch.float32)
+        v = ws.buffer("mix.v", (T, H * dv), torch.float32)
+        decay = ws.buffer("mix.decay", (T, H), torch.float32)
+        beta = ws.buffer("mix.beta", (T, H), torch.float32)
+        if self.advances is None:
+            self.advances = K.delta_prepare_advances(H, G, d, dv, self.taps, proj.shape[1])
+        advance = self.advances and step.all_decode
+        K.delta_prepare(proj, None, self.conv_w, cache.state["conv"], self.a_log, self.dt_bias, step.tok_seq,
+                        step.seq_slot, step.seq_qstart, q, k, v, decay, beta, H, G, d, dv, self.taps, self.unit_eps,
+                        advance=advance)
+        if self.taps > 1 and not advance:
+            K.conv_state_update(proj, cache.state["conv"], step.seq_slot, step.seq_qstart, step.seq_qlen, step.n_seqs,
+                                self.channels, self.taps)
+        o = ws.buffer("mix.o", (T, H * dv), torch.float32)
+        K.state_scan(q, k, v, None, beta, None, cache.state["S"], o, step.seq_slot, step.seq_qstart, step.seq_qlen,
+                     step.n_seqs, H, G, d, dv, token_decay=decay)
+        gated = ws.buffer("mix.gated", (T, H * dv), self.ctx.act_dtype)
+        K.head_norm_gate(o, self.norm_w, proj, gated, H, dv, self.eps, K.GATE_SILU, gate_col=self.gate_col)
+        return self.o.forward(step, gated, self.out_name, into=into)
+
+
+class LightningAttention(Mixer):
+    """params: n_heads, head_dim, v_head_dim, decay (one per head), eps (of the norm over the row of all heads), out_name
+    (workspace name of the result, default "o"), names: tensor names for "q", "k", "v", "g", "norm", "o"."""
+
+    capturable = True
+    workspace = "lightning"
+    takes_prenormed = True
+
+    def __init__(self, params, ctx: BuildContext):
+        super().__init__(params, ctx)
+        self.n_heads = int(params["n_heads"])
+        self.d = int(params["head_dim"])
+        self.dv = int(params["v_head_dim"])
+        self.decay = [float(x) for x in params["decay"]]
+        self.eps = float(params["eps"])
+        self.names = dict(params["names"])
+        self.out_name = params.get("out_name") or "o"
+        if len(self.decay) != self.n_heads:
+            raise ValueError(f"lightning attention: {len(self.decay)} decays for {self.n_heads} heads")
+        self.decay_t = torch.tensor(self.decay, dtype=torch.float32, device=ctx.device)
+        self.proj: Optional[Linear] = None
+        self.o: Optional[Linear] = None
+
+    def weight_specs(self) -> List[WeightSpec]:
+        D, H, d, dv, n = self.ctx.hidden_size, self.n_heads, self.d, self.dv, self.names
+        return [WeightSpec(n["q"], (H * d, D)), WeightSpec(n["k"], (H * d, D)), WeightSpec(n["v"], (H * dv, D)),
+                WeightSpec(n["g"], (H * dv, D)), WeightSpec(n["norm"], (H * dv,), kind="vector", init="norm"),
+                WeightSpec(n["o"], (D, H * dv))]
+
+    def bind(self, store) -> None:
+        mats = _same_dtype([store.take(self.names[p]) for p in ("q", "k", "v", "g")])
+        self.proj = Linear(_pad_rows(torch.cat(mats, dim=0)), self.names["q"] + "+k+v+g")
+        del mats
+        self.norm_w = store.take(self.names["norm"])
+        self.o = Linear(store.take(self.names["o"]), self.names["o"])
+
+    def parameter_bytes(self) -> int:
+        return self.proj.parameter_bytes() + self.o.parameter_bytes()
+
+    def cache_need(self) -> CacheNeed:
+        return CacheNeed(state=StateNeed((("S", (self.n_heads, self.d, self.dv)),)))
+
+    def forward(self, step, h, cache):
+        T, H, d, dv = row_count(h), self.n_heads, self.d, self.dv
+        ws = step.ws
+        proj = self.proj.forward(step, h, "lightning.proj")
+        q = ws.buffer("lightning.q", (T, H * d), torch.float32)
+        k = ws.buffer("lightning.k", (T, H * d), torch.float32)
+        v = ws.buffer("lightning.v", (T, H * dv), torch.float32)
+        K.retention_prepare(proj, None, None, step.tok_pos, q, k, v, H, d, dv, 0, False, 1.0, silu=True)
+        o = ws.buffer("lightning.o", (T, H * dv), torch.float32)
+        K.state_scan(q, k, v, None, None, self.decay_t, cache.state["S"], o, step.seq_slot, step.seq_qstart,
+                     step.seq_qlen, step.n_seqs, H, H, d, dv)
+        gated = ws.buffer("lightning.gated", (T, H * dv), self.ctx.act_dtype)
+        K.row_norm_gate(o, self.norm_w, proj, gated, self.eps, K.GATE_SIGMOID, gate_col=H * (2 * d + dv))
+        return self.o.forward(step, gated, self.out_name)
+
+
 class GatedLinearAttention(Mixer):
     """params: n_heads, head_dim, v_head_dim, tau (the decay is sigmoid(z)^(1 / tau)), eps (of the head norm),
     decay_rank (inner size of the low-rank pair, -1: as stored), out_name (workspace name of the result, default "o"),
@@ -366,6 +519,8 @@ class StateSpace(Mixer):
 
 
 register_part("mixer", "state_space", StateSpace)
+register_part("mixer", "delta_rule_head_decay", HeadDecayDeltaRule)
+register_part("mixer", "lightning_attention", LightningAttention)
 register_part("mixer", "gated_linear_attention", GatedLinearAttention)
 register_part("mixer", "retention", Retention)
 register_part("mixer", "gated_delta_rule", GatedDeltaRule)
