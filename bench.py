@@ -654,6 +654,58 @@ def mefolorn_rooflines(size, tokens, batch, context, peaks):
     return out
 
 
+def gopitar_config(size):
+    """Six layers: the pair twice and the delta rule, twice over.  The pair: attention with query and key heads of 64 and
+    value heads of 128 under a window of 1,024 behind a convolution of 3 taps, beside lightning attention with heads of
+    128 x 128; the delta rule with heads of 128 x 128 and 4 taps; a dense feed-forward behind every mixer."""
+    import cpp_minilamma_b200 as ml
+    s = DESIGN_SIZES[size]
+    mlp = {"kind": "dense", "ff": s["ff"]}
+    R = s["ret_heads"]
+    pair = {"type": "parallel", "mlp": mlp,
+            "mixer": {"left": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": 64, "vdim": 128, "conv": 3, "scale": 0.125,
+                               "mask": {"size": 1024}, "rot": {"base": 10000.0, "dims": 32}},
+                      "right": {"heads": R, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-5 - 4 * i / R) for i in range(R)]},
+                      "left_scale": 0.8, "right_scale": 1.1}}
+    delta = {"type": "delta", "mlp": mlp, "mixer": {"heads": s["heads"], "kv_heads": s["heads"], "dim": 128, "vdim": 128, "conv": 4}}
+    return ml.config_from_dict({"architecture": "Gopitar", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5},
+                                "embedding": {"scale": 12.0}, "logit_softcap": 30.0, "layers": [pair, pair, delta] * s["groups"],
+                                "torch_dtype": "bfloat16"})
+
+
+def gopitar_rooflines(size, tokens, batch, context, peaks):
+    """As `design_rooflines`, for the kernels of the Gopitar decoder and their like in the Kupirax decoder."""
+    s = DESIGN_SIZES[size]
+    H, G, d, dv, R, D, ff = s["heads"], s["kv_heads"], 64, 128, s["ret_heads"], s["width"], s["ff"]
+    e = 128  # rows and columns of every state
+    out = {k: v for k, v in design_rooflines(size, tokens, batch, context, peaks).items() if k[0] == "kupirax"}
+    seen = sum(min(i + 1, 1024) for i in range(tokens))
+    visible = min(context, 1024)
+    for name in ("attention_prefill", "local_attention_mma"):
+        out["gopitar", "prefill", name] = ("tensor", 2.0 * H * seen * (d + dv))
+    for name in ("attention_decode", "local_attention_heads"):
+        out["gopitar", "decode", name] = ("hbm", batch * visible * G * (d + dv) * 2)
+    qkv = (H * d + G * (d + dv)) * 2
+    for kind, n, seqs in (("prefill", tokens, 1), ("decode", batch, batch)):
+        out["gopitar", kind, "conv_attention_prepare"] = ("hbm", n * 2 * qkv + (n * 4 * qkv if kind == "decode" else 0))
+        out["gopitar", kind, "lightning_prepare"] = ("hbm", n * R * 3 * e * (2 + 4))
+        out["gopitar", kind, "state_scan (retention)"] = ("hbm", n * R * 4 * e * 4 + seqs * R * e * e * 8)
+        out["gopitar", kind, "row_norm_gate"] = ("hbm", n * R * e * (4 + 2 + 2))
+        conv = n * H * 3 * e * 2 * 3 * 4 if kind == "decode" else 0  # the convolution's state, in and out
+        out["gopitar", kind, "delta_prepare"] = ("hbm", n * H * 3 * e * (2 + 4) + conv)
+        out["gopitar", kind, "state_scan (delta rule, head decay)"] = ("hbm", n * H * 4 * e * 4 + seqs * H * e * e * 8)
+        out["gopitar", kind, "head_norm_gate"] = ("hbm", n * H * e * (4 + 2 + 2))
+        out["gopitar", kind, "heads_gate"] = ("hbm", n * H * dv * 4)
+        for model in ("gopitar", "kupirax"):
+            out[model, kind, "swiglu"] = ("hbm", n * ff * (4 + 2))
+        for name in ("rmsnorm", "rmsnorm (normed delta)"):  # the stream in and out, the outputs that join it, the result
+            out["gopitar", kind, name] = ("hbm", n * D * (8 + 2 + (4 if "delta" in name else 2)))
+            out["kupirax", kind, name] = ("hbm", n * D * (8 + 2 + 4))
+        out["gopitar", kind, "add_bias"] = ("hbm", n * D * 4)
+        out["gopitar", kind, "softcap"] = ("hbm", seqs * s["vocab"] * 8)
+    return out
+
+
 def llama_like_config(size):
     import cpp_minilamma_b200 as ml
     s = DESIGN_SIZES[size]
@@ -730,8 +782,8 @@ def design_rooflines(size, tokens, batch, context, peaks):
 
 def bench_design(args):
     """Prompt and decode throughput of the Kupirax or Malulorn decoder and of the Llama decoder (of the Sopanex or Badolix
-    decoder and of the Malulorn decoder, the closest to them; of the Mefolorn decoder and of the Badolix decoder) at equal width,
-    feed-forward, heads and layer count (random bfloat16 weights), and the device time of each of this library's kernels in one
+    decoder and of the Malulorn decoder, the closest to them; of the Mefolorn decoder and of the Badolix decoder; of the
+    Gopitar decoder and of the Kupirax decoder) at equal width, feed-forward, heads and layer count (random bfloat16 weights), and the device time of each of this library's kernels in one
     prompt step and one decode step of either, with the fraction of the measured peak it reaches."""
     import numpy as np
     import torch
@@ -742,11 +794,12 @@ def bench_design(args):
     tokens, batch, context = PREFILL_TOKENS, 64, 1024
     design = args.design
     make_config = {"kupirax": kupirax_config, "malulorn": malulorn_config, "sopanex": sopanex_config,
-                   "badolix": badolix_config, "mefolorn": mefolorn_config}[design]
+                   "badolix": badolix_config, "mefolorn": mefolorn_config, "gopitar": gopitar_config}[design]
     rooflines = {"kupirax": design_rooflines, "malulorn": malulorn_rooflines, "sopanex": sopanex_rooflines,
-                 "badolix": badolix_rooflines, "mefolorn": mefolorn_rooflines}[design]
+                 "badolix": badolix_rooflines, "mefolorn": mefolorn_rooflines, "gopitar": gopitar_rooflines}[design]
     beside, beside_config = {"sopanex": ("malulorn", malulorn_config), "badolix": ("malulorn", malulorn_config),
-                             "mefolorn": ("badolix", badolix_config)}.get(design, ("llama", llama_like_config))
+                             "mefolorn": ("badolix", badolix_config),
+                             "gopitar": ("kupirax", kupirax_config)}.get(design, ("llama", llama_like_config))
     result = {"design": design, "beside": beside, "dtype": "bf16", "data": "synthetic token ids, random-init weights",
               "prefill_tokens": tokens, "decode_prompts": "uniform[128,1024)", "steps": steps, "warmup": warmup,
               "peaks": {"hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"], "source": peaks["source"]},
@@ -818,7 +871,7 @@ def main():
     parser.add_argument("--shape", choices=sorted(SHAPES), default="llama31_8b", help="model shape of the --profile step")
     parser.add_argument("--batch", type=int, default=BATCH, help="batch of the --profile decode step")
     parser.add_argument("--context", type=int, default=1024, help="prompt length of the --profile decode step")
-    parser.add_argument("--design", choices=["kupirax", "malulorn", "sopanex", "badolix", "mefolorn"], default=None,
+    parser.add_argument("--design", choices=["kupirax", "malulorn", "sopanex", "badolix", "mefolorn", "gopitar"], default=None,
                         help="instead of the default workload: prompt and decode throughput and kernel times of that "
                              "decoder beside the Llama decoder (sopanex, badolix: beside the Malulorn decoder; mefolorn: beside the Badolix decoder) at equal sizes")
     parser.add_argument("--size", choices=sorted(DESIGN_SIZES), default=None, help="one size of --design (default: all)")

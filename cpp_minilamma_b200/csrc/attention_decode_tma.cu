@@ -1,5 +1,5 @@
-// Decode attention (one query token per sequence) over the paged cache, bfloat16, head_dim 64 or
-// 128: pages arrive by TMA, and the four compute warps of a block never meet inside the page loop.
+// Decode attention (one query token per sequence) over the paged cache, bfloat16, head sizes 64 and
+// 128 (the values' may differ from the queries' and keys'): pages arrive by TMA, and the four compute warps of a block never meet inside the page loop.
 //
 // One block per (sequence, kv head [, chunk of 16 query heads], split of the context):
 //   * warp 4, one thread: producer.  Per page it loads the keys and the values of the block's kv
@@ -46,15 +46,15 @@ constexpr int DT_STAGES = 3;
 constexpr int DT_THREADS = 160;  // four compute warps and the producer warp
 constexpr long long DT_WAIT_CLOCKS = 2ll << 30;
 
-template <int D>
+template <int D, int DV>
 struct DecodeTmaSmem {
-  static constexpr int BOXES = D / 64;
+  static constexpr int BOXES = D / 64, V_BOXES = DV / 64;
   static constexpr int BOX_BYTES = MLL_PAGE * 128;      // [64 rows x 128 bytes]
-  static constexpr int HALF = BOXES * BOX_BYTES;        // one page's keys (or values)
-  static constexpr int STAGE = 2 * HALF;
+  static constexpr int HALF = BOXES * BOX_BYTES;        // one page's keys; its values follow
+  static constexpr int STAGE = (BOXES + V_BOXES) * BOX_BYTES;
   static constexpr int RING = DT_STAGES * STAGE;        // 96 KB for head_dim 128: two blocks per multiprocessor
-  static constexpr int MERGE_FLOATS = 4 * (16 * D + 32);  // the warps' partial results, over the ring once it is drained
-  static_assert(MERGE_FLOATS * 4 + (16 * D + 32) * 4 <= RING, "the merge buffers must fit into the ring");
+  static constexpr int MERGE_FLOATS = 4 * (16 * DV + 32);  // the warps' partial results, over the ring once it is drained
+  static_assert(MERGE_FLOATS * 4 + (16 * DV + 32) * 4 <= RING, "the merge buffers must fit into the ring");
   static constexpr int BAR_OFF = RING;                  // full[S], empty[S]
   static constexpr size_t BYTES = (size_t)RING + 64;
 };
@@ -87,7 +87,7 @@ __device__ __forceinline__ void dt_tma_load_2d(unsigned dst, const CUtensorMap* 
       ::"r"(dst), "l"(map), "r"(c0), "r"(c1), "r"(bar) : "memory");
 }
 // Byte offset of 16-byte chunk `chunk` (8 bfloat16) of row `row` in a K or V half: the half is
-// D / 64 boxes of [64 rows x 128 bytes], and the 128-byte swizzle xors the chunk index within
+// boxes of [64 rows x 128 bytes], and the 128-byte swizzle xors the chunk index within
 // the box with the row's low three bits.
 __device__ __forceinline__ unsigned dt_chunk_offset(int row, int chunk) {
   return (unsigned)((chunk >> 3) * (MLL_PAGE * 128) + row * 128 + (((chunk & 7) ^ (row & 7)) << 4));
@@ -182,15 +182,17 @@ __device__ __forceinline__ void dt_load_query(const DecodeMmaArgs& a, int b, int
 // the sequence.  On the sequence's last page the fused variant first puts the step's new key and value into the
 // stage and into the cache (the block that owns that page; the four compute warps meet once for it), and rows
 // beyond the context are masked (keys) and zeroed (values).
-template <int D, bool FUSED>
+template <int D, int DV, bool FUSED>
 __device__ __forceinline__ void dt_page_step(const DecodeMmaArgs& a, unsigned char* stage, int p, int ctx, int first_key,
                                              int kept, int pages_total, bool owns_new_row, const int* table, int kvh,
                                              __nv_bfloat16 new_k0, __nv_bfloat16 new_k1, unsigned new_v,
-                                             const unsigned (&qf)[D / 16][4], float (&o)[D / 8][4], float (&m_run)[2],
+                                             const unsigned (&qf)[D / 16][4], float (&o)[DV / 8][4], float (&m_run)[2],
                                              float (&l_run)[2]) {
-  constexpr int KSTEPS = D / 16, NT = D / 8;
+  using L = DecodeTmaSmem<D, DV>;
+  static_assert(!FUSED || D == DV, "the fused variant writes rows of one size");
+  constexpr int KSTEPS = D / 16, NT = DV / 8;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, t = lane & 3;
-  const unsigned kt = dt_smem(stage), vt = kt + DecodeTmaSmem<D>::HALF;
+  const unsigned kt = dt_smem(stage), vt = kt + L::HALF;
   if (p == pages_total - 1) {
     if (FUSED && owns_new_row) {
       // the step's token lies in this page: its key (rotated) and value replace whatever the cache held
@@ -199,7 +201,7 @@ __device__ __forceinline__ void dt_page_step(const DecodeMmaArgs& a, unsigned ch
         const size_t cache_row = (((size_t)table[p] * a.n_kv_heads + kvh) * MLL_PAGE + row) * D;
         const int e0 = a.interleaved ? 2 * tid : tid, e1 = a.interleaved ? 2 * tid + 1 : tid + D / 2;
         unsigned char* k_half = stage;
-        unsigned char* v_half = k_half + DecodeTmaSmem<D>::HALF;
+        unsigned char* v_half = k_half + L::HALF;
         *reinterpret_cast<__nv_bfloat16*>(k_half + dt_chunk_offset(row, e0 >> 3) + (e0 & 7) * 2) = new_k0;
         *reinterpret_cast<__nv_bfloat16*>(k_half + dt_chunk_offset(row, e1 >> 3) + (e1 & 7) * 2) = new_k1;
         a.k_write[cache_row + e0] = new_k0;
@@ -211,9 +213,9 @@ __device__ __forceinline__ void dt_page_step(const DecodeMmaArgs& a, unsigned ch
     }
     const int valid = ctx - p * MLL_PAGE;  // positions of this page that the sequence has
     if (valid < MLL_PAGE) {                // the rest of the page may hold anything: zero this warp's value rows
-      unsigned char* v_half = stage + DecodeTmaSmem<D>::HALF;
-      for (int idx = lane; idx < 16 * (D / 8); idx += 32) {
-        const int row = warp * 16 + idx / (D / 8), ch = idx % (D / 8);
+      unsigned char* v_half = stage + L::HALF;
+      for (int idx = lane; idx < 16 * (DV / 8); idx += 32) {
+        const int row = warp * 16 + idx / (DV / 8), ch = idx % (DV / 8);
         if (row >= valid) *reinterpret_cast<uint4*>(v_half + dt_chunk_offset(row, ch)) = make_uint4(0, 0, 0, 0);
       }
       __syncwarp();
@@ -239,7 +241,7 @@ __device__ __forceinline__ void dt_page_step(const DecodeMmaArgs& a, unsigned ch
   for (int ks = 0; ks < KSTEPS; ++ks) {
     // matrices: (keys 0-7, dims 0-7), (keys 0-7, dims 8-15), (keys 8-15, dims 0-7), (keys 8-15, dims 8-15)
     unsigned kb[4];
-    dt_ldmatrix_x4(kb, (k_lane ^ (unsigned)(((ks * 2) & 7) << 4)) + (ks >> 2) * DecodeTmaSmem<D>::BOX_BYTES);
+    dt_ldmatrix_x4(kb, (k_lane ^ (unsigned)(((ks * 2) & 7) << 4)) + (ks >> 2) * L::BOX_BYTES);
     if (D == 64 && (ks & 1)) {
       mma_16816(s_odd[0], qf[ks], kb[0], kb[1]);
       mma_16816(s_odd[1], qf[ks], kb[2], kb[3]);
@@ -310,20 +312,20 @@ __device__ __forceinline__ void dt_page_step(const DecodeMmaArgs& a, unsigned ch
   for (int n = 0; n < NT; n += 2) {
     // transposed 8x8 tiles of V: (keys 0-7, cols n), (keys 8-15, cols n), (keys 0-7, cols n+1), (keys 8-15, cols n+1)
     unsigned vb[4];
-    dt_ldmatrix_x4_trans(vb, (v_lane ^ (unsigned)((n & 7) << 4)) + (n >> 3) * DecodeTmaSmem<D>::BOX_BYTES);
+    dt_ldmatrix_x4_trans(vb, (v_lane ^ (unsigned)((n & 7) << 4)) + (n >> 3) * L::BOX_BYTES);
     mma_16816(o[n], pa, vb[0], vb[1]);
     mma_16816(o[n + 1], pa, vb[2], vb[3]);
   }
 }
 
 // grid (Hk * head_chunks, B, n_splits); 160 threads.
-template <int D, bool FUSED, bool CLUSTER>
+template <int D, int DV, bool FUSED, bool CLUSTER>
 __global__ void __launch_bounds__(DT_THREADS, 2)
 attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant__ CUtensorMap vmap,
                        DecodeMmaArgs a) {
-  using L = DecodeTmaSmem<D>;
+  using L = DecodeTmaSmem<D, DV>;
   constexpr int KSTEPS = D / 16;  // k-steps of the score product
-  constexpr int NT = D / 8;       // output n-tiles (8 columns) per warp: every warp holds all columns
+  constexpr int NT = DV / 8;      // output n-tiles (8 columns) per warp: every warp holds all columns
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   unsigned long long* bars = reinterpret_cast<unsigned long long*>(smem_raw + L::BAR_OFF);
   // no static shared memory in this kernel: it would sit before the ring and could move it off its boundary
@@ -365,11 +367,11 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
   const bool active = split < n_eff && !misplaced;
   if (!CLUSTER && !active) return;
   // where the block's result lies once its four warps are merged (over the drained ring)
-  float* part = reinterpret_cast<float*>(smem_raw);       // [4 warps][16 rows][D], then [4][16] maxima, [4][16] sums
-  float* part_m = part + 4 * 16 * D;
+  float* part = reinterpret_cast<float*>(smem_raw);       // [4 warps][16 rows][DV], then [4][16] maxima, [4][16] sums
+  float* part_m = part + 4 * 16 * DV;
   float* part_l = part_m + 4 * 16;
-  float* merged = part_l + 4 * 16;                        // [16][D], then [16] maxima, [16] sums
-  float* merged_m = merged + 16 * D;
+  float* merged = part_l + 4 * 16;                        // [16][DV], then [16] maxima, [16] sums
+  float* merged_m = merged + 16 * DV;
   float* merged_l = merged_m + 16;
   bool failed = true;
   if (active) {
@@ -413,10 +415,10 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
                        : "memory");
           const unsigned dst = ring + st * L::STAGE;
 #pragma unroll
-          for (int bx = 0; bx < L::BOXES; ++bx) {
-            dt_tma_load_2d(dst + bx * L::BOX_BYTES, &kmap, bx * 64, row, full + 8 * st);
+          for (int bx = 0; bx < L::BOXES; ++bx) dt_tma_load_2d(dst + bx * L::BOX_BYTES, &kmap, bx * 64, row, full + 8 * st);
+#pragma unroll
+          for (int bx = 0; bx < L::V_BOXES; ++bx)
             dt_tma_load_2d(dst + L::HALF + bx * L::BOX_BYTES, &vmap, bx * 64, row, full + 8 * st);
-          }
         }
       }
     } else {
@@ -441,7 +443,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
         const int p = page_at(w_begin + it);
         const int st = it % DT_STAGES;
         dt_mbar_wait(full + 8 * st, (it / DT_STAGES) & 1, abort_flag);
-        dt_page_step<D, FUSED>(a, smem_raw + st * L::STAGE, p, ctx, first_key, kept, pages_total, owns_new_row, table, kvh,
+        dt_page_step<D, DV, FUSED>(a, smem_raw + st * L::STAGE, p, ctx, first_key, kept, pages_total, owns_new_row, table, kvh,
                                new_k0, new_k1, new_v, qf, o, m_run, l_run);
         __syncwarp();
         if (lane == 0) asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(empty + 8 * st) : "memory");
@@ -459,8 +461,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
 #pragma unroll
       for (int n = 0; n < NT; ++n) {
         const int col = n * 8 + 2 * t;
-        *reinterpret_cast<float2*>(part + ((size_t)warp * 16 + g) * D + col) = make_float2(o[n][0], o[n][1]);
-        *reinterpret_cast<float2*>(part + ((size_t)warp * 16 + g + 8) * D + col) = make_float2(o[n][2], o[n][3]);
+        *reinterpret_cast<float2*>(part + ((size_t)warp * 16 + g) * DV + col) = make_float2(o[n][0], o[n][1]);
+        *reinterpret_cast<float2*>(part + ((size_t)warp * 16 + g + 8) * DV + col) = make_float2(o[n][2], o[n][3]);
       }
       if (t == 0) {
         part_m[warp * 16 + g] = m_run[0];
@@ -471,16 +473,16 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
     }
     __syncthreads();
     failed = *abort_flag != 0;
-    for (int idx = tid; idx < ng * D; idx += DT_THREADS) {
-      const int row = idx / D, col = idx % D;
+    for (int idx = tid; idx < ng * DV; idx += DT_THREADS) {
+      const int row = idx / DV, col = idx % DV;
       const float m0 = part_m[row], m1 = part_m[16 + row], m2 = part_m[32 + row], m3 = part_m[48 + row];
       const float m = fmaxf(fmaxf(m0, m1), fmaxf(m2, m3));
       const float w0 = m0 > -INFINITY ? __expf(m0 - m) : 0.f, w1 = m1 > -INFINITY ? __expf(m1 - m) : 0.f;
       const float w2 = m2 > -INFINITY ? __expf(m2 - m) : 0.f, w3 = m3 > -INFINITY ? __expf(m3 - m) : 0.f;
       const float l = (part_l[row] * w0 + part_l[16 + row] * w1) + (part_l[32 + row] * w2 + part_l[48 + row] * w3);
-      const float v = (part[(size_t)row * D + col] * w0 + part[((size_t)16 + row) * D + col] * w1) +
-                      (part[((size_t)32 + row) * D + col] * w2 + part[((size_t)48 + row) * D + col] * w3);
-      merged[(size_t)row * D + col] = v;
+      const float v = (part[(size_t)row * DV + col] * w0 + part[((size_t)16 + row) * DV + col] * w1) +
+                      (part[((size_t)32 + row) * DV + col] * w2 + part[((size_t)48 + row) * DV + col] * w3);
+      merged[(size_t)row * DV + col] = v;
       if (col == 0) {
         merged_m[row] = m;
         merged_l[row] = l;
@@ -495,9 +497,9 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
     cg::cluster_group cluster = cg::this_cluster();
     cluster.sync();  // every block's merged result is in its shared memory
     if (active && !failed) {
-      const int share = (ng * D + n_eff - 1) / n_eff;  // split number `split` writes outputs [split * share, + share)
-      for (int idx = split * share + tid; idx < min(ng * D, (split + 1) * share); idx += DT_THREADS) {
-        const int row = idx / D, col = idx % D;
+      const int share = (ng * DV + n_eff - 1) / n_eff;  // split number `split` writes outputs [split * share, + share)
+      for (int idx = split * share + tid; idx < min(ng * DV, (split + 1) * share); idx += DT_THREADS) {
+        const int row = idx / DV, col = idx % DV;
         float m = -INFINITY;
         for (int sp = 0; sp < n_eff; ++sp) m = fmaxf(m, *cluster.map_shared_rank(merged_m + row, sp));
         float l = 0.f, v = 0.f;
@@ -505,23 +507,23 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
           const float ms = *cluster.map_shared_rank(merged_m + row, sp);
           const float w = ms > -INFINITY ? __expf(ms - m) : 0.f;
           l = fmaf(*cluster.map_shared_rank(merged_l + row, sp), w, l);
-          v = fmaf(*cluster.map_shared_rank(merged + (size_t)row * D + col, sp), w, v);
+          v = fmaf(*cluster.map_shared_rank(merged + (size_t)row * DV + col, sp), w, v);
         }
-        a.out[((size_t)b * a.n_heads + h0 + row) * D + col] = __float2bfloat16_rn(l > 0.f ? v / l : 0.f);
+        a.out[((size_t)b * a.n_heads + h0 + row) * DV + col] = __float2bfloat16_rn(l > 0.f ? v / l : 0.f);
       }
     }
     cluster.sync();  // nobody leaves while another block may still read its shared memory
     return;
   }
   if (failed) return;
-  for (int idx = tid; idx < ng * D; idx += DT_THREADS) {
-    const int row = idx / D, col = idx % D;
+  for (int idx = tid; idx < ng * DV; idx += DT_THREADS) {
+    const int row = idx / DV, col = idx % DV;
     const size_t head = (size_t)b * a.n_heads + h0 + row;
     if (n_eff == 1) {
       const float l = merged_l[row];
-      a.out[head * D + col] = __float2bfloat16_rn(l > 0.f ? merged[(size_t)row * D + col] / l : 0.f);
+      a.out[head * DV + col] = __float2bfloat16_rn(l > 0.f ? merged[(size_t)row * DV + col] / l : 0.f);
     } else {
-      a.part_o[(head * a.n_splits + split) * D + col] = merged[(size_t)row * D + col];
+      a.part_o[(head * a.n_splits + split) * DV + col] = merged[(size_t)row * DV + col];
       if (col == 0) {
         float* ml = a.part_ml + (head * a.n_splits + split) * 2;
         ml[0] = merged_m[row];
@@ -530,16 +532,16 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
     }
   }
   if (n_eff == 1) return;
-  merge_decode_splits<D, DT_THREADS>(a, b, item, gridDim.x, h0, ng, n_eff, merged_l + 16);
+  merge_decode_splits<DV, DT_THREADS>(a, b, item, gridDim.x, h0, ng, n_eff, merged_l + 16);
 }
 
 // cluster: the splits of a group are the blocks of one thread-block cluster and merge through distributed
 // shared memory (n_splits 2 .. 16); otherwise through global memory and arrival counters.
-template <int D, bool FUSED, bool CLUSTER>
+template <int D, int DV, bool FUSED, bool CLUSTER>
 int launch_decode_tma_as(const CUtensorMap& kmap, const CUtensorMap& vmap, const DecodeMmaArgs& a, int n_seqs,
                          cudaStream_t stream) {
-  const size_t smem = DecodeTmaSmem<D>::BYTES;
-  auto kernel = attn_decode_tma_kernel<D, FUSED, CLUSTER>;
+  const size_t smem = DecodeTmaSmem<D, DV>::BYTES;
+  auto kernel = attn_decode_tma_kernel<D, DV, FUSED, CLUSTER>;
   cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (err == cudaSuccess && CLUSTER && a.n_splits > 8)
     err = cudaFuncSetAttribute(kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
@@ -573,13 +575,13 @@ int launch_decode_tma_as(const CUtensorMap& kmap, const CUtensorMap& vmap, const
 
 // How many clusters of `n_splits` of these blocks the device holds at once (0: such a cluster cannot be
 // launched); asked once per kernel and size.
-template <int D, bool FUSED>
+template <int D, int DV, bool FUSED>
 int decode_clusters_resident(int n_splits) {
   static int known[17] = {0};  // 0 unknown, -1 none, else the count
   if (n_splits < 2 || n_splits > 16) return 0;
   if (known[n_splits] == 0) {
-    auto kernel = attn_decode_tma_kernel<D, FUSED, true>;
-    const size_t smem = DecodeTmaSmem<D>::BYTES;
+    auto kernel = attn_decode_tma_kernel<D, DV, FUSED, true>;
+    const size_t smem = DecodeTmaSmem<D, DV>::BYTES;
     int clusters = 0;
     cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (err == cudaSuccess && n_splits > 8)
@@ -604,12 +606,12 @@ int decode_clusters_resident(int n_splits) {
   return max(known[n_splits], 0);
 }
 
-template <int D, bool FUSED>
+template <int D, int DV, bool FUSED>
 int launch_decode_tma(const CUtensorMap& kmap, const CUtensorMap& vmap, const DecodeMmaArgs& a, int n_seqs,
                       int cluster_merge, cudaStream_t stream) {
-  if (cluster_merge && a.work == nullptr && decode_clusters_resident<D, FUSED>(a.n_splits) >= 1)
-    return launch_decode_tma_as<D, FUSED, true>(kmap, vmap, a, n_seqs, stream);
-  return launch_decode_tma_as<D, FUSED, false>(kmap, vmap, a, n_seqs, stream);
+  if (cluster_merge && a.work == nullptr && decode_clusters_resident<D, DV, FUSED>(a.n_splits) >= 1)
+    return launch_decode_tma_as<D, DV, FUSED, true>(kmap, vmap, a, n_seqs, stream);
+  return launch_decode_tma_as<D, DV, FUSED, false>(kmap, vmap, a, n_seqs, stream);
 }
 
 }  // namespace mll
@@ -631,15 +633,18 @@ MLL_API int mll_attn_decode_tma_supported(int dtype, int head_dim) {
 
 // Clusters of `n_splits` blocks of the (fused) kernel for this head size that the device holds at once; 0 if
 // such a cluster cannot be launched or the head size is not taken.
-MLL_API int mll_attn_decode_tma_resident_clusters(int head_dim, int fused, int n_splits) {
-  if (head_dim == 64)
-    return fused ? mll::decode_clusters_resident<64, true>(n_splits) : mll::decode_clusters_resident<64, false>(n_splits);
-  if (head_dim == 128)
-    return fused ? mll::decode_clusters_resident<128, true>(n_splits) : mll::decode_clusters_resident<128, false>(n_splits);
+MLL_API int mll_attn_decode_tma_resident_clusters(int head_dim, int v_head_dim, int fused, int n_splits) {
+  if (head_dim == 64 && v_head_dim == 64)
+    return fused ? mll::decode_clusters_resident<64, 64, true>(n_splits) : mll::decode_clusters_resident<64, 64, false>(n_splits);
+  if (head_dim == 128 && v_head_dim == 128)
+    return fused ? mll::decode_clusters_resident<128, 128, true>(n_splits) : mll::decode_clusters_resident<128, 128, false>(n_splits);
+  if (head_dim == 64 && v_head_dim == 128 && !fused) return mll::decode_clusters_resident<64, 128, false>(n_splits);
+  if (head_dim == 128 && v_head_dim == 64 && !fused) return mll::decode_clusters_resident<128, 64, false>(n_splits);
   return 0;
 }
 
-// One query token per sequence over the paged cache (bfloat16, head_dim 64 or 128).  Either q [B, Hq d]
+// One query token per sequence over the paged cache (bfloat16, head_dim and v_head_dim 64 or 128; the fused variant only
+// where they are equal).  Either q [B, Hq d]
 // (already rotated) or, for the fused variant, qkv [B, qkv_ld] with the rotary tables as in
 // mll_attn_decode_mma_fused (then q is ignored).  n_pages: pages of k_cache and v_cache.  With
 // n_splits > 1, scratch and counters (int32, one per (sequence, kv head x head chunk), zero
@@ -654,10 +659,12 @@ MLL_API int mll_attn_decode_tma(const void* q, const void* qkv, int qkv_ld, cons
                                 const float* sin_table, int interleaved, int write_kv, void* k_cache, void* v_cache,
                                 long long n_pages, const int* seq_slot, const int* seq_ctx, const int* block_table,
                                 float* scratch, void* out, int n_seqs, int n_heads, int n_kv_heads, int head_dim,
-                                int max_blocks, int n_splits, int window, float scale, int* counters,
+                                int v_head_dim, int max_blocks, int n_splits, int window, float scale, int* counters,
                                 int cluster_merge, const int* seq_order, const int* work, int work_pairs, int sink,
                                 const float* sink_values, int keep_first, float softcap, cudaStream_t stream) {
-  MLL_REQUIRE(mll_attn_decode_tma_supported(MLL_BF16, head_dim), "attention decode (tma): head_dim %d", head_dim);
+  MLL_REQUIRE(mll_attn_decode_tma_supported(MLL_BF16, head_dim) && mll_attn_decode_tma_supported(MLL_BF16, v_head_dim) &&
+                  (qkv == nullptr || head_dim == v_head_dim),
+              "attention decode (tma): head sizes %d / %d", head_dim, v_head_dim);
   MLL_REQUIRE(n_heads > 0 && n_kv_heads > 0 && n_heads % n_kv_heads == 0, "attention decode (tma): bad head counts");
   MLL_REQUIRE(n_seqs >= 0 && n_splits >= 1 && n_splits <= 65535, "attention decode (tma): bad batch or split count");
   MLL_REQUIRE(work == nullptr || (work_pairs >= n_seqs && work_pairs <= 65535 && n_seqs <= 65535 && n_splits <= 127),
@@ -674,11 +681,11 @@ MLL_API int mll_attn_decode_tma(const void* q, const void* qkv, int qkv_ld, cons
   if (n_seqs == 0) return 0;
   CUtensorMap kmap, vmap;
   if (mll::tensor_map_bf16(k_cache, n_pages * n_kv_heads * MLL_PAGE, head_dim, MLL_PAGE, &kmap) != 0) return -1;
-  if (mll::tensor_map_bf16(v_cache, n_pages * n_kv_heads * MLL_PAGE, head_dim, MLL_PAGE, &vmap) != 0) return -1;
+  if (mll::tensor_map_bf16(v_cache, n_pages * n_kv_heads * MLL_PAGE, v_head_dim, MLL_PAGE, &vmap) != 0) return -1;
   const bool fused = qkv != nullptr;
   mll::DecodeMmaArgs a{(const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache,
                        seq_slot, seq_ctx, block_table, scratch,
-                       scratch ? scratch + (size_t)n_seqs * n_heads * n_splits * head_dim : nullptr,
+                       scratch ? scratch + (size_t)n_seqs * n_heads * n_splits * v_head_dim : nullptr,
                        (__nv_bfloat16*)out, n_heads, n_kv_heads, max_blocks, n_splits, window, scale, counters,
                        (const __nv_bfloat16*)qkv, fused ? cos_table : nullptr, fused ? sin_table : nullptr,
                        fused && write_kv ? (__nv_bfloat16*)k_cache : nullptr,
@@ -690,9 +697,12 @@ MLL_API int mll_attn_decode_tma(const void* q, const void* qkv, int qkv_ld, cons
   a.keep_first = keep_first;
   a.softcap = softcap;
   const int rows = work != nullptr ? work_pairs : n_seqs;  // the grid's second index
+  if (head_dim != v_head_dim)
+    return head_dim == 64 ? mll::launch_decode_tma<64, 128, false>(kmap, vmap, a, rows, cluster_merge, stream)
+                          : mll::launch_decode_tma<128, 64, false>(kmap, vmap, a, rows, cluster_merge, stream);
   if (head_dim == 64)
-    return fused ? mll::launch_decode_tma<64, true>(kmap, vmap, a, rows, cluster_merge, stream)
-                 : mll::launch_decode_tma<64, false>(kmap, vmap, a, rows, cluster_merge, stream);
-  return fused ? mll::launch_decode_tma<128, true>(kmap, vmap, a, rows, cluster_merge, stream)
-               : mll::launch_decode_tma<128, false>(kmap, vmap, a, rows, cluster_merge, stream);
+    return fused ? mll::launch_decode_tma<64, 64, true>(kmap, vmap, a, rows, cluster_merge, stream)
+                 : mll::launch_decode_tma<64, 64, false>(kmap, vmap, a, rows, cluster_merge, stream);
+  return fused ? mll::launch_decode_tma<128, 128, true>(kmap, vmap, a, rows, cluster_merge, stream)
+               : mll::launch_decode_tma<128, 128, false>(kmap, vmap, a, rows, cluster_merge, stream);
 }

@@ -1,5 +1,6 @@
 // Causal attention of many query tokens over the paged cache on the fifth-generation tensor
-// cores: TMA -> shared memory -> tcgen05.mma -> tensor memory (bfloat16, head_dim 64 or 128).
+// cores: TMA -> shared memory -> tcgen05.mma -> tensor memory (bfloat16, head sizes 64 and 128, the
+// values' of their own: d for queries and keys, dv for values).
 //
 // One block owns 128 query rows of one head.  Its warps:
 //   * warps 0-3, the softmax: thread i owns query row i, which is lane i of tensor memory, so the
@@ -8,10 +9,10 @@
 //     tile, keeps the running maximum and sum in float32 (base 2), and writes P back over the first
 //     half of the S columns as packed bfloat16 (tcgen05.st);
 //   * warp 4, one thread: TMA loads with the 128-byte swizzle - the query tile once, then the key and
-//     the value pages (64 positions each) into a ring of two stages (three at head size 64) guarded by
+//     the value pages (64 positions each) into a ring of two stages (three where both sizes are 64) guarded by
 //     full / empty mbarriers;
 //   * warp 5, one thread: S = Q K^T (M = 128 rows, N = 64 keys, both operands K-major) into one of two
-//     64-column buffers of tensor memory (three at head size 64, where O takes half the columns); S_i is issued
+//     64-column buffers of tensor memory (three at value size 64, where O takes half the columns); S_i is issued
 //     as soon as page i's keys are there and the buffer's last user, the P V of two (three) pages before, is
 //     done, so it runs under the softmax of the pages between.  The warp also
 //     allocates and frees the block's 256 columns;
@@ -66,7 +67,7 @@ struct PrefillTc5Args {
   const int* tile_seq;   // tiles of 128 rows (entries that do not start a multiple of 128 are skipped)
   const int* tile_row0;
   const int* block_table;
-  __nv_bfloat16* out;    // [T, Hq * d]
+  __nv_bfloat16* out;    // [T, Hq * dv]
   int n_heads, n_kv_heads, max_blocks, window;
   int chunk;  // > 0: key j is visible from query i only if j / chunk == i / chunk (chunks count from position 0)
   float scale_log2;
@@ -280,26 +281,27 @@ __device__ __forceinline__ void a_mbar_arrive(unsigned bar) {
 constexpr int A_SOFTMAX_REGS = 168, A_OTHER_REGS = 40;
 constexpr float A_RESCALE_STEP = 8.f;  // the output is rescaled only when a row's maximum grows by more than 2^8
 
-template <int D>
+template <int D, int DV>
 struct PrefillTc5Smem {
   static constexpr int THREADS = 256;
-  static constexpr int KV_STAGES = D == 64 ? 3 : 2;   // as many key/value stages as S buffers (80 KB a block either way)
+  static constexpr int KV_STAGES = D == 64 && DV == 64 ? 3 : 2;  // at most 80 KB a block
   static constexpr int Q_BYTES = A_ROWS * D * 2;       // D / 64 boxes of [128 rows x 128 bytes]
-  static constexpr int KV_BYTES = MLL_PAGE * D * 2;    // D / 64 boxes of [64 rows x 128 bytes]
-  static constexpr int Q_OFF = 0, K_OFF = Q_BYTES, V_OFF = K_OFF + KV_STAGES * KV_BYTES;
-  static constexpr int BAR_OFF = V_OFF + KV_STAGES * KV_BYTES;
+  static constexpr int K_BYTES = MLL_PAGE * D * 2;     // D / 64 boxes of [64 rows x 128 bytes]
+  static constexpr int V_BYTES = MLL_PAGE * DV * 2;    // DV / 64 boxes
+  static constexpr int Q_OFF = 0, K_OFF = Q_BYTES, V_OFF = K_OFF + KV_STAGES * K_BYTES;
+  static constexpr int BAR_OFF = V_OFF + KV_STAGES * V_BYTES;
   // Two blocks per multiprocessor (their tensor memory: 2 x 256 columns); never three: the request
   // is padded above a third of the shared memory.  The kernel checks that its dynamic shared
   // memory starts on a 1024-byte boundary (the swizzle's period) and refuses otherwise.
   static constexpr size_t USED = (size_t)BAR_OFF + 512;
   static constexpr size_t BYTES = USED < 80 * 1024 ? 80 * 1024 : USED;
-  // Tensor memory, 256 columns a block: S / P buffers of 64 columns, then O (D columns).  Head size 128 leaves room
-  // for two S buffers, head size 64 for three: the chain softmax -> P V -> S -> softmax that bounds a block's pace
+  // Tensor memory, 256 columns a block: S / P buffers of 64 columns, then O (DV columns).  Value size 128 leaves room
+  // for two S buffers, value size 64 for three: the chain softmax -> P V -> S -> softmax that bounds a block's pace
   // then runs over three pages instead of two.
-  static constexpr int S_BUFS = D == 64 ? 3 : 2;
+  static constexpr int S_BUFS = DV == 64 ? 3 : 2;
   static constexpr int TMEM_COLS = 256;
   static constexpr int O_COL = S_BUFS * MLL_PAGE;
-  static_assert(O_COL + D <= TMEM_COLS, "S buffers and O must fit the block's columns");
+  static_assert(O_COL + DV <= TMEM_COLS, "S buffers and O must fit the block's columns");
   // barrier slots: the queries; keys and values full / empty per ring stage; per S buffer: S full, P ready,
   // P V done
   static constexpr int AB_Q = 0, AB_K_FULL = 1, AB_V_FULL = AB_K_FULL + KV_STAGES, AB_K_EMPTY = AB_V_FULL + KV_STAGES,
@@ -309,12 +311,12 @@ struct PrefillTc5Smem {
   static_assert(AB_COUNT * 8 + 16 <= 512, "the barriers must fit behind the tiles");
 };
 
-template <int D>
-__global__ void __launch_bounds__(PrefillTc5Smem<D>::THREADS, 2)
+template <int D, int DV>
+__global__ void __launch_bounds__(PrefillTc5Smem<D, DV>::THREADS, 2)
 attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant__ CUtensorMap kmap,
                         const __grid_constant__ CUtensorMap vmap, PrefillTc5Args a) {
-  using L = PrefillTc5Smem<D>;
-  constexpr int DB = D / 64;  // 64-column boxes per row of Q, K or V
+  using L = PrefillTc5Smem<D, DV>;
+  constexpr int DB = D / 64, VB = DV / 64;  // 64-column boxes per row of Q and K, and of V
   constexpr int KS = L::KV_STAGES, SB = L::S_BUFS;
   constexpr int LOAD_WARP = 4, MMA_WARP = 5, PV_WARP = 6;
   // later tiles of a sequence see more keys: they go first, so that the short ones fill the tail
@@ -389,15 +391,15 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_c
         const int row = (page * a.n_kv_heads + kvh) * MLL_PAGE;
         if (i + 1 < n_pages) page = table[page_at(i + 1)];  // looked up while this page's loads fly
         wait(bar(L::AB_K_EMPTY, st), parity);
-        a_mbar_expect_tx(bar(L::AB_K_FULL, st), L::KV_BYTES);
+        a_mbar_expect_tx(bar(L::AB_K_FULL, st), L::K_BYTES);
 #pragma unroll
         for (int b = 0; b < DB; ++b)
-          a_tma_load_2d(k_s + st * L::KV_BYTES + b * (MLL_PAGE * 128), &kmap, b * 64, row, bar(L::AB_K_FULL, st));
+          a_tma_load_2d(k_s + st * L::K_BYTES + b * (MLL_PAGE * 128), &kmap, b * 64, row, bar(L::AB_K_FULL, st));
         wait(bar(L::AB_V_EMPTY, st), parity);
-        a_mbar_expect_tx(bar(L::AB_V_FULL, st), L::KV_BYTES);
+        a_mbar_expect_tx(bar(L::AB_V_FULL, st), L::V_BYTES);
 #pragma unroll
-        for (int b = 0; b < DB; ++b)
-          a_tma_load_2d(v_s + st * L::KV_BYTES + b * (MLL_PAGE * 128), &vmap, b * 64, row, bar(L::AB_V_FULL, st));
+        for (int b = 0; b < VB; ++b)
+          a_tma_load_2d(v_s + st * L::V_BYTES + b * (MLL_PAGE * 128), &vmap, b * 64, row, bar(L::AB_V_FULL, st));
       }
     }
   } else if (warp == MMA_WARP) {
@@ -410,7 +412,7 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_c
       const unsigned long long q_desc = a_desc(q_s, 16);
       unsigned long long k_desc[KS];
 #pragma unroll
-      for (int s = 0; s < KS; ++s) k_desc[s] = a_desc(k_s + s * L::KV_BYTES, 16);
+      for (int s = 0; s < KS; ++s) k_desc[s] = a_desc(k_s + s * L::K_BYTES, 16);
       wait(bar(L::AB_Q, 0), 0);
       for (int i = 0; i < n_pages && !*abort_flag; ++i) {
         const int sb = i % SB, st = i % KS;
@@ -438,10 +440,10 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_c
     // the other (75 clocks apiece for S, 135 for P V, and a hundred for every wait, even one that is over),
     // 2,400 to 3,000 clocks a page of which the tensor cores worked 640, and the softmax warps waited
     if (lane == 0) {
-      constexpr unsigned idesc_o = a_idesc(A_ROWS, D, true);
+      constexpr unsigned idesc_o = a_idesc(A_ROWS, DV, true);
       unsigned long long v_desc[KS];
 #pragma unroll
-      for (int s = 0; s < KS; ++s) v_desc[s] = a_desc(v_s + s * L::KV_BYTES, MLL_PAGE * 128);
+      for (int s = 0; s < KS; ++s) v_desc[s] = a_desc(v_s + s * L::V_BYTES, MLL_PAGE * 128);
       for (int i = 0; i < n_pages && !*abort_flag; ++i) {
         const int sb = i % SB, st = i % KS;
         unsigned long long vd = v_desc[0];
@@ -514,7 +516,7 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_c
         wait(bar(L::AB_PV_DONE, (i - 1) % SB), ((i - 1) / SB) & 1);  // O holds every page before this one
         a_fence_after();
 #pragma unroll
-        for (int c = 0; c < D; c += 32) {
+        for (int c = 0; c < DV; c += 32) {
           float o[32];
           a_tmem_ld32(tmem_row + L::O_COL + c, o);
 #pragma unroll
@@ -557,9 +559,9 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_c
       const int valid = ctx - k0;  // positions of this page that the sequence has
       if (valid < MLL_PAGE) {      // only the sequence's last page: the rest of it may hold anything
         wait(bar(L::AB_V_FULL, st), (i / KS) & 1);
-        unsigned char* vt = base + L::V_OFF + st * L::KV_BYTES;
+        unsigned char* vt = base + L::V_OFF + st * L::V_BYTES;
         const int n_chunks = (MLL_PAGE - valid) * 8;  // 16-byte chunks per box
-        for (int b = 0; b < DB; ++b)
+        for (int b = 0; b < VB; ++b)
           for (int c = r; c < n_chunks; c += A_ROWS)
             *reinterpret_cast<uint4*>(vt + b * (MLL_PAGE * 128) + valid * 128 + c * 16) = make_uint4(0, 0, 0, 0);
         a_fence_async_smem();
@@ -577,9 +579,9 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_c
       // threads that own a row of the sequence store
       const bool store = !*abort_flag && r < rows;
       const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-      __nv_bfloat16* dst = a.out + ((size_t)qstart + row0 + (store ? r : 0)) * a.n_heads * D + (size_t)h * D;
+      __nv_bfloat16* dst = a.out + ((size_t)qstart + row0 + (store ? r : 0)) * a.n_heads * DV + (size_t)h * DV;
 #pragma unroll
-      for (int c = 0; c < D; c += 32) {
+      for (int c = 0; c < DV; c += 32) {
         float o[32];
         a_tmem_ld32(tmem_row + L::O_COL + c, o);
         if (store) {
@@ -608,12 +610,12 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_c
   }
 }
 
-template <int D>
+template <int D, int DV>
 int launch_prefill_tc5(const CUtensorMap& qmap, const CUtensorMap& kmap, const CUtensorMap& vmap,
                        const PrefillTc5Args& a, int n_tiles, cudaStream_t stream) {
-  using L = PrefillTc5Smem<D>;
+  using L = PrefillTc5Smem<D, DV>;
   const size_t smem = L::BYTES;
-  auto kernel = attn_prefill_tc5_kernel<D>;
+  auto kernel = attn_prefill_tc5_kernel<D, DV>;
   cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (err != cudaSuccess) {
     mll_set_error("attention prefill (tcgen05): cannot reserve %zu bytes of shared memory: %s", smem,
@@ -642,15 +644,17 @@ MLL_API int mll_attn_prefill_tc5_supported(int dtype, int head_dim) {
   return dtype == MLL_BF16 && (head_dim == 64 || head_dim == 128);
 }
 
-// Same contract as mll_attn_prefill (bfloat16, head_dim 64 or 128); n_tokens is the number of
+// Same contract as mll_attn_prefill (bfloat16, head_dim and v_head_dim 64 or 128; value pages and out rows have
+// v_head_dim columns a head); n_tokens is the number of
 // rows of q and out, n_pages the number of pages of k_cache and v_cache.
 MLL_API int mll_attn_prefill_tc5(const void* q, const void* k_cache, const void* v_cache, const int* seq_slot,
                                  const int* seq_ctx, const int* seq_qstart, const int* seq_qlen, const int* tile_seq,
                                  const int* tile_row0, const int* block_table, void* out, int n_tokens,
                                  long long n_pages, int n_tiles, int n_heads, int n_kv_heads, int head_dim,
-                                 int max_blocks, int window, int chunk, float scale, int sink,
+                                 int v_head_dim, int max_blocks, int window, int chunk, float scale, int sink,
                                  const float* sink_values, int keep_first, float softcap, cudaStream_t stream) {
-  MLL_REQUIRE(mll_attn_prefill_tc5_supported(MLL_BF16, head_dim), "attention prefill (tcgen05): head_dim %d", head_dim);
+  MLL_REQUIRE(mll_attn_prefill_tc5_supported(MLL_BF16, head_dim) && mll_attn_prefill_tc5_supported(MLL_BF16, v_head_dim),
+              "attention prefill (tcgen05): head sizes %d / %d", head_dim, v_head_dim);
   MLL_REQUIRE(n_heads > 0 && n_kv_heads > 0 && n_heads % n_kv_heads == 0, "attention prefill (tcgen05): bad head counts");
   MLL_REQUIRE(n_tiles >= 0 && n_tokens >= 0 && (long long)n_tiles * n_heads < (1ll << 31),
               "attention prefill (tcgen05): bad tile or head count");
@@ -665,11 +669,13 @@ MLL_API int mll_attn_prefill_tc5(const void* q, const void* k_cache, const void*
   CUtensorMap qmap, kmap, vmap;
   if (mll::tensor_map_bf16(q, n_tokens, (long long)n_heads * head_dim, mll::A_ROWS, &qmap) != 0) return -1;
   if (mll::tensor_map_bf16(k_cache, n_pages * n_kv_heads * MLL_PAGE, head_dim, MLL_PAGE, &kmap) != 0) return -1;
-  if (mll::tensor_map_bf16(v_cache, n_pages * n_kv_heads * MLL_PAGE, head_dim, MLL_PAGE, &vmap) != 0) return -1;
+  if (mll::tensor_map_bf16(v_cache, n_pages * n_kv_heads * MLL_PAGE, v_head_dim, MLL_PAGE, &vmap) != 0) return -1;
   mll::PrefillTc5Args a{seq_slot, seq_ctx, seq_qstart, seq_qlen, tile_seq, tile_row0, block_table,
                         (__nv_bfloat16*)out, n_heads, n_kv_heads, max_blocks, window, chunk, scale * 1.4426950408889634f,
                         (sink || sink_values) ? 1 : 0, sink_values, keep_first, softcap > 0.f ? scale / softcap : 0.f,
                         softcap > 0.f ? softcap / scale : 0.f};
-  if (head_dim == 64) return mll::launch_prefill_tc5<64>(qmap, kmap, vmap, a, n_tiles, stream);
-  return mll::launch_prefill_tc5<128>(qmap, kmap, vmap, a, n_tiles, stream);
+  if (head_dim == 64 && v_head_dim == 64) return mll::launch_prefill_tc5<64, 64>(qmap, kmap, vmap, a, n_tiles, stream);
+  if (head_dim == 64) return mll::launch_prefill_tc5<64, 128>(qmap, kmap, vmap, a, n_tiles, stream);
+  if (v_head_dim == 64) return mll::launch_prefill_tc5<128, 64>(qmap, kmap, vmap, a, n_tiles, stream);
+  return mll::launch_prefill_tc5<128, 128>(qmap, kmap, vmap, a, n_tiles, stream);
 }

@@ -761,7 +761,8 @@ def rope_cache_write(qkv, bias, cos, sin, tok_pos, tok_seq, seq_slot, block_tabl
                                 ctypes.c_int(int(write_kv)), _stream()), "rope_cache_write")
 
 
-def _check_attention(q, k_cache, v_cache, out, n_heads, n_kv_heads, head_dim):
+def _check_attention(q, k_cache, v_cache, out, n_heads, n_kv_heads, head_dim, v_head_dim=0):
+    v_head_dim = v_head_dim or head_dim
     _need(q, "attention q", None, 2)
     _need(out, "attention out", q.dtype, 2)
     _need(k_cache, "attention k_cache", q.dtype, 4)
@@ -770,9 +771,10 @@ def _check_attention(q, k_cache, v_cache, out, n_heads, n_kv_heads, head_dim):
         raise KernelError(f"attention: head_dim {head_dim} is not a multiple of 16 in [16, 256]")
     if n_heads % n_kv_heads != 0:
         raise KernelError(f"attention: {n_heads} heads are not a multiple of {n_kv_heads} kv heads")
-    if q.shape[1] != n_heads * head_dim or out.shape[1] != n_heads * head_dim:
+    if q.shape[1] != n_heads * head_dim or out.shape[1] != n_heads * v_head_dim:
         raise KernelError("attention: q/out width differs from heads * head_dim")
-    if tuple(k_cache.shape[1:]) != (n_kv_heads, PAGE, head_dim) or k_cache.shape != v_cache.shape:
+    if (tuple(k_cache.shape[1:]) != (n_kv_heads, PAGE, head_dim)
+            or tuple(v_cache.shape) != (k_cache.shape[0], n_kv_heads, PAGE, v_head_dim)):
         raise KernelError(f"attention: cache shape {tuple(k_cache.shape)} is not "
                           f"[pages, {n_kv_heads}, {PAGE}, {head_dim}]")
 
@@ -789,6 +791,11 @@ def _check_sink_values(sink_values, n_heads: int) -> None:
             raise KernelError(f"attention: {sink_values.shape[0]} sink values for {n_heads} heads")
 
 
+def attention_decode_takes_value_size(dtype: torch.dtype, head_dim: int, v_head_dim: int) -> bool:
+    """Whether `attention_decode` would run a kernel that knows value heads of another size than the keys'."""
+    return attention_decode_takes_window_extras(dtype, head_dim) and attention_decode_takes_window_extras(dtype, v_head_dim)
+
+
 def attention_decode_takes_window_extras(dtype: torch.dtype, head_dim: int) -> bool:
     """Whether `attention_decode` would run the kernel that knows kept first tokens and capped scores."""
     return bool(USE_TMA_DECODE and USE_TENSOR_CORE_DECODE and dtype == torch.bfloat16
@@ -803,8 +810,11 @@ def attention_decode(q, k_cache, v_cache, seq_slot, seq_ctx, block_table, scratc
                      n_heads: int, n_kv_heads: int, head_dim: int, n_splits: int, window: int,
                      scale: float, counters: Optional[torch.Tensor] = None, order: Optional[torch.Tensor] = None,
                      work: Optional[torch.Tensor] = None, chunk: int = 0, sink: bool = False,
-                     sink_values: Optional[torch.Tensor] = None, keep_first: int = 0, softcap: float = 0.0) -> None:
+                     sink_values: Optional[torch.Tensor] = None, keep_first: int = 0, softcap: float = 0.0,
+                     v_head_dim: int = 0) -> None:
     """One query token per sequence (q row i belongs to sequence i) over the paged cache.
+    `v_head_dim` (0: head_dim): the values' head size, where it differs from the keys' (the TMA-fed kernel only; ask
+    `attention_decode_takes_value_size` first).
     `keep_first` (with a window) and `softcap`: the TMA-fed kernel only (ask `attention_decode_takes_window_extras`
     first) - keys below `keep_first` stay visible; a score s becomes softcap * tanh(s / softcap) after the scale.
     `sink` (bfloat16 tensor-core kernels only): one more term exp(0) in the softmax's denominator, or
@@ -814,7 +824,8 @@ def attention_decode(q, k_cache, v_cache, seq_slot, seq_ctx, block_table, scratc
     bfloat16 runs on tensor cores (head sizes 16 .. 256 in steps of 16), float32 on the general kernel.
     `order`: optional int32 permutation of the sequences, longest context first; the TMA-fed kernel starts its
     blocks in that order so that short sequences fill the end of the launch (the others ignore it)."""
-    _check_attention(q, k_cache, v_cache, out, n_heads, n_kv_heads, head_dim)
+    v_head_dim = v_head_dim or head_dim
+    _check_attention(q, k_cache, v_cache, out, n_heads, n_kv_heads, head_dim, v_head_dim)
     _check_sink_values(sink_values, n_heads)
     sink = bool(sink or sink_values is not None)
     if chunk:
@@ -828,7 +839,7 @@ def attention_decode(q, k_cache, v_cache, seq_slot, seq_ctx, block_table, scratc
         raise KernelError("attention decode: an input has fewer rows than sequences")
     if n_splits > 1:
         _need(scratch, "attention scratch", torch.float32)
-        if scratch.numel() < attention_decode_scratch_floats(n_seqs, n_heads, head_dim, n_splits):
+        if scratch.numel() < attention_decode_scratch_floats(n_seqs, n_heads, v_head_dim, n_splits):
             raise KernelError("attention decode: scratch too small for the split count")
     code = dtype_code(q.dtype)
     if counters is not None:
@@ -839,10 +850,11 @@ def attention_decode(q, k_cache, v_cache, seq_slot, seq_ctx, block_table, scratc
     if q.dtype == torch.bfloat16 and _tma_decode(q, None, None, None, False, False, k_cache, v_cache, seq_slot, seq_ctx,
                                                 block_table, scratch, out, n_seqs, n_heads, n_kv_heads, head_dim,
                                                 n_splits, window, scale, counters, _order(order, n_seqs), work,
-                                                sink=sink, sink_values=sink_values, keep_first=keep_first, softcap=softcap):
+                                                sink=sink, sink_values=sink_values, keep_first=keep_first, softcap=softcap,
+                                                v_head_dim=v_head_dim):
         return
-    if keep_first or softcap:
-        raise KernelError("attention decode: only the TMA-fed kernel keeps first tokens or caps scores")
+    if keep_first or softcap or v_head_dim != head_dim:
+        raise KernelError("attention decode: only the TMA-fed kernel keeps first tokens, caps scores or has values of another size")
     if work is not None:
         raise KernelError("attention decode: a work list was given, but the kernel that takes one does not run here")
     if USE_TENSOR_CORE_DECODE and lib().mll_attn_decode_mma_supported(code, head_dim):
@@ -903,19 +915,20 @@ def _work(work, n_seqs: int, n_splits: int):
 def _tma_decode(q, qkv, cos, sin, interleaved, write_kv, k_cache, v_cache, seq_slot, seq_ctx, block_table, scratch, out,
                 n_seqs, n_heads, n_kv_heads, head_dim, n_splits, window, scale, counters, order=None, work=None,
                 sink: bool = False, sink_values: Optional[torch.Tensor] = None, keep_first: int = 0,
-                softcap: float = 0.0) -> bool:
+                softcap: float = 0.0, v_head_dim: int = 0) -> bool:
     """Runs the TMA-fed decode kernel when it takes the problem (bfloat16, head_dim 64/128, arrival
     counters whenever the context is split); returns whether it did."""
     if not (USE_TMA_DECODE and USE_TENSOR_CORE_DECODE and lib().mll_attn_decode_tma_supported(dtype_code(out.dtype), head_dim)):
         return False
-    if n_splits > 1 and counters is None:
+    v_head_dim = v_head_dim or head_dim
+    if (n_splits > 1 and counters is None) or not lib().mll_attn_decode_tma_supported(dtype_code(out.dtype), v_head_dim):
         return False
     work = _work(work, n_seqs, n_splits)
     _check(lib().mll_attn_decode_tma(_ptr(q), _ptr(qkv), ctypes.c_int(qkv.shape[1] if qkv is not None else 0),
                                      _ptr(cos), _ptr(sin), ctypes.c_int(int(interleaved)), ctypes.c_int(int(write_kv)),
                                      _ptr(k_cache), _ptr(v_cache), ctypes.c_longlong(k_cache.shape[0]), _ptr(seq_slot),
                                      _ptr(seq_ctx), _ptr(block_table), _ptr(scratch), _ptr(out), ctypes.c_int(n_seqs),
-                                     ctypes.c_int(n_heads), ctypes.c_int(n_kv_heads), ctypes.c_int(head_dim),
+                                     ctypes.c_int(n_heads), ctypes.c_int(n_kv_heads), ctypes.c_int(head_dim), ctypes.c_int(v_head_dim),
                                      ctypes.c_int(block_table.shape[1]), ctypes.c_int(n_splits), ctypes.c_int(window),
                                      ctypes.c_float(scale), _ptr(counters if n_splits > 1 else None),
                                      ctypes.c_int(int(USE_CLUSTER_MERGE)), _ptr(order), _ptr(work),
@@ -930,7 +943,7 @@ def _tma_decode(q, qkv, cos, sin, interleaved, write_kv, k_cache, v_cache, seq_s
 _cluster_capacity = {}
 
 
-def attention_decode_cluster_capacity(dtype: torch.dtype, head_dim: int, fused: bool):
+def attention_decode_cluster_capacity(dtype: torch.dtype, head_dim: int, fused: bool, v_head_dim: int = 0):
     """capacity[s], s = 0 .. 16: how many clusters of s blocks of the TMA decode kernel the device holds at once
     (0: no such cluster), or None when that kernel or its cluster merge is not what runs for this dtype and
     head size.  A launch with more clusters than that runs in two waves; measured on B200 at 8 kv heads of
@@ -939,10 +952,12 @@ def attention_decode_cluster_capacity(dtype: torch.dtype, head_dim: int, fused: 
     if not (USE_TMA_DECODE and USE_TENSOR_CORE_DECODE and USE_CLUSTER_MERGE and dtype == torch.bfloat16
             and lib().mll_attn_decode_tma_supported(dtype_code(dtype), head_dim)):
         return None
-    key = (head_dim, bool(fused))
+    v_head_dim = v_head_dim or head_dim
+    key = (head_dim, v_head_dim, bool(fused))
     if key not in _cluster_capacity:
         _cluster_capacity[key] = (0, 0) + tuple(
-            int(lib().mll_attn_decode_tma_resident_clusters(ctypes.c_int(head_dim), ctypes.c_int(int(fused)), ctypes.c_int(s)))
+            int(lib().mll_attn_decode_tma_resident_clusters(ctypes.c_int(head_dim), ctypes.c_int(v_head_dim),
+                                                            ctypes.c_int(int(fused)), ctypes.c_int(s)))
             for s in range(2, 17))
     return _cluster_capacity[key]
 
@@ -1008,16 +1023,19 @@ def attention_decode_fused(qkv, cos, sin, interleaved: bool, write_kv: bool, k_c
 PREFILL_TILE = 64  # query rows per entry of the work list that `attention_prefill` takes
 
 
-def attention_prefill_takes_chunks(dtype: torch.dtype, head_dim: int) -> bool:
-    """Whether `attention_prefill` would run the kernel that knows the chunk mask (bfloat16, heads of 64 or 128)."""
+def attention_prefill_takes_chunks(dtype: torch.dtype, head_dim: int, v_head_dim: int = 0) -> bool:
+    """Whether `attention_prefill` would run the kernel that knows the chunk mask and value heads of another size
+    (bfloat16, heads of 64 or 128)."""
     return bool(USE_TENSOR_CORE_PREFILL and USE_TCGEN05_PREFILL and dtype in _DTYPE_CODE
-                and lib().mll_attn_prefill_tc5_supported(dtype_code(dtype), head_dim))
+                and lib().mll_attn_prefill_tc5_supported(dtype_code(dtype), head_dim)
+                and lib().mll_attn_prefill_tc5_supported(dtype_code(dtype), v_head_dim or head_dim))
 
 
 def attention_prefill(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_qlen, tile_seq, tile_row0,
                       block_table, out, n_tiles: int, n_heads: int, n_kv_heads: int, head_dim: int,
                       window: int, scale: float, wide_tiles=None, chunk: int = 0, sink: bool = False,
-                      sink_values: Optional[torch.Tensor] = None, keep_first: int = 0, softcap: float = 0.0) -> None:
+                      sink_values: Optional[torch.Tensor] = None, keep_first: int = 0, softcap: float = 0.0,
+                      v_head_dim: int = 0) -> None:
     """Tiles of up to 64 query tokens of sequences with unequal lengths over the paged cache.
     `wide_tiles`: (sequence, first row) int32 lists of the same rows in tiles of 128, which the tcgen05 kernel
     works on; without them it walks the 64-row list and every other block finds nothing to do.
@@ -1025,8 +1043,9 @@ def attention_prefill(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_ql
     only if j // chunk == i // chunk.  `sink` (the same kernel only): one more term exp(0) in the softmax's denominator,
     or exp(sink_values[head]) with `sink_values` (float32 [Hq], not scaled).  `keep_first` (with a window) and
     `softcap` (the same kernel only): keys below `keep_first` stay visible; a score s becomes softcap * tanh(s / softcap)
-    after the scale."""
-    _check_attention(q, k_cache, v_cache, out, n_heads, n_kv_heads, head_dim)
+    after the scale.  `v_head_dim` (0: head_dim; the same kernel only): the values' head size."""
+    v_head_dim = v_head_dim or head_dim
+    _check_attention(q, k_cache, v_cache, out, n_heads, n_kv_heads, head_dim, v_head_dim)
     _check_sink_values(sink_values, n_heads)
     sink = bool(sink or sink_values is not None)
     for name, t in (("seq_slot", seq_slot), ("seq_ctx", seq_ctx), ("seq_qstart", seq_qstart),
@@ -1036,7 +1055,8 @@ def attention_prefill(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_ql
     if tile_seq.shape[0] < n_tiles or tile_row0.shape[0] < n_tiles:
         raise KernelError("attention prefill: tile lists shorter than the tile count")
     if (USE_TENSOR_CORE_PREFILL and USE_TCGEN05_PREFILL
-            and lib().mll_attn_prefill_tc5_supported(dtype_code(q.dtype), head_dim)):
+            and lib().mll_attn_prefill_tc5_supported(dtype_code(q.dtype), head_dim)
+            and lib().mll_attn_prefill_tc5_supported(dtype_code(q.dtype), v_head_dim)):
         if wide_tiles is not None:
             tile_seq, tile_row0 = wide_tiles
             _need(tile_seq, "attention wide tile_seq", torch.int32, 1)
@@ -1049,13 +1069,15 @@ def attention_prefill(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_ql
                                           _ptr(block_table), _ptr(out), ctypes.c_int(q.shape[0]),
                                           ctypes.c_longlong(k_cache.shape[0]), ctypes.c_int(n_tiles),
                                           ctypes.c_int(n_heads), ctypes.c_int(n_kv_heads), ctypes.c_int(head_dim),
+                                          ctypes.c_int(v_head_dim),
                                           ctypes.c_int(block_table.shape[1]), ctypes.c_int(window), ctypes.c_int(chunk),
                                           ctypes.c_float(scale), ctypes.c_int(int(sink)), _ptr(sink_values),
                                           ctypes.c_int(keep_first), ctypes.c_float(softcap), _stream()),
                "attention_prefill (tcgen05)")
         return
-    if chunk or sink or keep_first or softcap:
-        raise KernelError("attention prefill: only the tcgen05 kernel masks by chunks, has a sink, keeps first tokens or caps scores")
+    if chunk or sink or keep_first or softcap or v_head_dim != head_dim:
+        raise KernelError("attention prefill: only the tcgen05 kernel masks by chunks, has a sink, keeps first tokens, "
+                          "caps scores or has values of another size")
     if USE_TENSOR_CORE_PREFILL and lib().mll_attn_prefill_mma_supported(dtype_code(q.dtype), head_dim):
         _check(lib().mll_attn_prefill_mma(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(seq_slot), _ptr(seq_ctx),
                                           _ptr(seq_qstart), _ptr(seq_qlen), _ptr(tile_seq), _ptr(tile_row0),

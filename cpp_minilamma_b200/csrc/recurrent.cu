@@ -403,8 +403,9 @@ __device__ __forceinline__ void cp_async4(float* smem, const float* gmem) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(s), "l"(gmem));
 }
 
-// grid (column tiles, H, sequences).  Lane layout inside a warp: lane = r * (32 / R) + c; lane (r, c) holds rows
-// r * ROWS .. r * ROWS + ROWS - 1 of column c of the warp's columns.  Rows past d are padding: their k and q
+// grid (column tiles, H, sequences).  Lane layout inside a warp: lane = r * (32 / R) + c; lane (r, c) holds, of
+// column c of the warp's columns, rows 4 r .. 4 r + 3 of every run of 4 R rows, so that the R lanes of a column read a run
+// of q, k or g as R consecutive 16-byte words: one pass over the banks (with ROWS consecutive rows a lane it took four).  Rows past d are padding: their k and q
 // are staged as 0, so their S stays 0 and adds nothing.  The tokens' q, k, g, v and beta arrive in shared memory
 // `tok_stage` tokens at a time through a two-stage ring of asynchronous copies, so that the next tokens load
 // while these are worked on and the chain from token to token is arithmetic only.
@@ -436,7 +437,7 @@ __global__ void __launch_bounds__(THREADS) state_scan_kernel(ScanArgs a) {
   float s[ROWS];
 #pragma unroll
   for (int i = 0; i < ROWS; ++i) {
-    const int row = r * ROWS + i;
+    const int row = (i >> 2) * (4 * R) + r * 4 + (i & 3);
     s[i] = (live && row < d) ? S[(size_t)row * dv + col] : 0.f;
   }
   const int TS = a.tok_stage;
@@ -521,12 +522,12 @@ __global__ void __launch_bounds__(THREADS) state_scan_kernel(ScanArgs a) {
         if constexpr (SCALAR_DELTA) {
           // rows of k and q as 16-byte words; k's are read again for the write rather than held (a lane with 64 rows has
           // no registers left for them)
-          const float4* q4 = reinterpret_cast<const float4*>(q_s + tj * DP + r * ROWS);
-          const float4* k4 = reinterpret_cast<const float4*>(k_s + tj * DP + r * ROWS);
+          const float4* q4 = reinterpret_cast<const float4*>(q_s + tj * DP) + r;
+          const float4* k4 = reinterpret_cast<const float4*>(k_s + tj * DP) + r;
           float sk[4] = {0.f, 0.f, 0.f, 0.f}, sq[4] = {0.f, 0.f, 0.f, 0.f}, kq[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
           for (int i = 0; i < ROWS / 4; ++i) {
-            const float4 kw = k4[i], qw = q4[i];
+            const float4 kw = k4[i * R], qw = q4[i * R];
             sk[0] = fmaf(s[4 * i], kw.x, sk[0]); sk[1] = fmaf(s[4 * i + 1], kw.y, sk[1]);
             sk[2] = fmaf(s[4 * i + 2], kw.z, sk[2]); sk[3] = fmaf(s[4 * i + 3], kw.w, sk[3]);
             sq[0] = fmaf(s[4 * i], qw.x, sq[0]); sq[1] = fmaf(s[4 * i + 1], qw.y, sq[1]);
@@ -546,7 +547,7 @@ __global__ void __launch_bounds__(THREADS) state_scan_kernel(ScanArgs a) {
           u = b_s[tj] * fmaf(-gt, dk, u);
 #pragma unroll
           for (int i = 0; i < ROWS / 4; ++i) {
-            const float4 kw = k4[i];
+            const float4 kw = k4[i * R];
             s[4 * i] = fmaf(kw.x, u, gt * s[4 * i]); s[4 * i + 1] = fmaf(kw.y, u, gt * s[4 * i + 1]);
             s[4 * i + 2] = fmaf(kw.z, u, gt * s[4 * i + 2]); s[4 * i + 3] = fmaf(kw.w, u, gt * s[4 * i + 3]);
           }
@@ -557,9 +558,9 @@ __global__ void __launch_bounds__(THREADS) state_scan_kernel(ScanArgs a) {
         float qv[ROWS], kv[ROWS], gv[CHANNEL ? ROWS : 1];
 #pragma unroll
         for (int i = 0; i < ROWS; i += 4) {
-          *reinterpret_cast<float4*>(qv + i) = *reinterpret_cast<const float4*>(q_s + tj * DP + r * ROWS + i);
-          *reinterpret_cast<float4*>(kv + i) = *reinterpret_cast<const float4*>(k_s + tj * DP + r * ROWS + i);
-          if (CHANNEL) *reinterpret_cast<float4*>(gv + i) = *reinterpret_cast<const float4*>(g_s + tj * DP + r * ROWS + i);
+          *reinterpret_cast<float4*>(qv + i) = *reinterpret_cast<const float4*>(q_s + tj * DP + i * R + r * 4);
+          *reinterpret_cast<float4*>(kv + i) = *reinterpret_cast<const float4*>(k_s + tj * DP + i * R + r * 4);
+          if (CHANNEL) *reinterpret_cast<float4*>(gv + i) = *reinterpret_cast<const float4*>(g_s + tj * DP + i * R + r * 4);
         }
         if (DELTA) {
           float p4[4] = {0.f, 0.f, 0.f, 0.f};  // four sums side by side: the chain of additions is a quarter as long
@@ -598,7 +599,7 @@ __global__ void __launch_bounds__(THREADS) state_scan_kernel(ScanArgs a) {
   if (live) {
 #pragma unroll
     for (int i = 0; i < ROWS; ++i) {
-      const int row = r * ROWS + i;
+      const int row = (i >> 2) * (4 * R) + r * 4 + (i & 3);
       if (row < d) S[(size_t)row * dv + col] = s[i];
     }
   }

@@ -265,20 +265,43 @@ class ChunkedAttention(Mixer):
             K.conv_state_update(qkv, cache.state["conv"], step.seq_slot, step.seq_qstart, step.seq_qlen, step.n_seqs,
                                 self.channels, self.taps, bias=self.qkv_bias)
 
+    def _decode_items(self) -> int:
+        return self.n_kv_heads * -(-(self.n_heads // self.n_kv_heads) // 16)  # the TMA-fed kernel's blocks per sequence
+
+    def _decode_splits(self, n_seqs: int) -> int:
+        """Splits along every context of a single-token step, where a block per (sequence, kv head) would leave
+        multiprocessors idle: the most whose clusters are all resident at once, a function of the batch size alone, so
+        that a captured step keeps its launch.  (A sequence uses as many of them as its own length pays for.)"""
+        capacity = K.attention_decode_cluster_capacity(self.ctx.act_dtype, self.d, False, self.dv)
+        if capacity is None or not K.attention_decode_takes_window_extras(self.ctx.act_dtype, self.dv):
+            return 1
+        reach = self.window or self.chunk or self.ctx.max_positions
+        pages = min(16, -(-reach // K.PAGE) + (1 if self.window else 0))
+        blocks = n_seqs * self._decode_items()
+        fit = [s for s in range(2, pages + 1) if blocks <= capacity[s]]
+        return fit[-1] if fit else 1
+
     def _attend(self, step, q, cache, out) -> None:
         act = self.ctx.act_dtype
         learned = self.sink_values  # a sink with a score of its own per head, or None
         extra = {"keep_first": self.keep_first, "softcap": self.softcap}
         plain = not self.keep_first and not self.softcap  # what the Llama attention's kernels know
-        if ((plain or K.attention_decode_takes_window_extras(act, self.d)) and step.all_decode and self.d == self.dv
+        if ((plain or K.attention_decode_takes_window_extras(act, self.d)) and step.all_decode
+                and (self.d == self.dv or K.attention_decode_takes_value_size(act, self.d, self.dv))
                 and self.d % 16 == 0 and 16 <= self.d <= 256
                 and not (self.chunk and self.window) and act == torch.bfloat16
                 and (not self.sink or K.USE_TENSOR_CORE_DECODE)):
-            # single tokens, keys and values of one head size: the Llama attention's decode kernels (TMA-fed or
-            # mma.sync), which take the chunk as the key range's start; one block per (sequence, kv head)
-            K.attention_decode(q, cache.k, cache.v, step.seq_slot, step.seq_ctx, cache.block_table, None, out,
-                               step.n_seqs, self.n_heads, self.n_kv_heads, self.d, 1, self.window, self.scale,
-                               chunk=self.chunk, sink=self.sink, sink_values=learned, **extra)
+            # single tokens, keys and values of one head size or of two that the TMA-fed kernel takes: the Llama
+            # attention's decode kernels (TMA-fed or mma.sync), which take the chunk as the key range's start
+            splits, scratch, counters = self._decode_splits(step.n_seqs), None, None
+            if splits > 1:
+                scratch = step.ws.buffer("attn.scratch", (K.attention_decode_scratch_floats(
+                    step.n_seqs, self.n_heads, self.dv, splits),), torch.float32)
+                counters = step.ws.zeros("attn.counters", (step.n_seqs * self._decode_items(),), torch.int32)
+            K.attention_decode(q, cache.k, cache.v, step.seq_slot, step.seq_ctx, cache.block_table, scratch, out,
+                               step.n_seqs, self.n_heads, self.n_kv_heads, self.d, splits, self.window, self.scale,
+                               counters=counters, chunk=self.chunk, sink=self.sink, sink_values=learned,
+                               v_head_dim=self.dv, **extra)
             return
         if step.all_decode and self._tensor_cores():
             # single tokens that the kernels above do not take (a sink, values of another size): the tensor-core
@@ -293,14 +316,14 @@ class ChunkedAttention(Mixer):
                                     sink_values=learned, **extra)
             return
         tiles = step.meta.get(self.step_metadata_key()) if not step.all_decode else None
-        if tiles and self.d == self.dv and K.attention_prefill_takes_chunks(act, self.d):
-            # keys and values of one head size that the Llama attention's tcgen05 prompt kernel takes: that kernel,
-            # which knows the chunk mask too
+        if tiles and K.attention_prefill_takes_chunks(act, self.d, self.dv):
+            # head sizes that the Llama attention's tcgen05 prompt kernel takes: that kernel, which knows the chunk mask
+            # and values of another size too
             K.attention_prefill(q, cache.k, cache.v, step.seq_slot, step.seq_ctx, step.seq_qstart, step.seq_qlen,
                                 tiles["tile_seq"], tiles["tile_row0"], cache.block_table, out,
                                 tiles["tile_seq"].shape[0], self.n_heads, self.n_kv_heads, self.d, self.window,
                                 self.scale, wide_tiles=(tiles["wide_seq"], tiles["wide_row0"]), chunk=self.chunk,
-                                sink=self.sink, sink_values=learned, **extra)
+                                sink=self.sink, sink_values=learned, v_head_dim=self.dv, **extra)
             return
         if tiles and self._tensor_cores():
             K.local_attention_tiles(q, cache.k, cache.v, step.seq_slot, step.seq_ctx, step.seq_qstart, step.seq_qlen,
