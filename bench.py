@@ -690,10 +690,13 @@ def gopitar_rooflines(size, tokens, batch, context, peaks):
         out["gopitar", kind, "conv_attention_prepare"] = ("hbm", n * 2 * qkv + (n * 4 * qkv if kind == "decode" else 0))
         out["gopitar", kind, "lightning_prepare"] = ("hbm", n * R * 3 * e * (2 + 4))
         out["gopitar", kind, "state_scan (retention)"] = ("hbm", n * R * 4 * e * 4 + seqs * R * e * e * 8)
+        # the runs' matrices are not counted: what the recurrence must move is the same
+        out["gopitar", kind, "state_chunks (head decay)"] = out["gopitar", kind, "state_scan (retention)"]
         out["gopitar", kind, "row_norm_gate"] = ("hbm", n * R * e * (4 + 2 + 2))
         conv = n * H * 3 * e * 2 * 3 * 4 if kind == "decode" else 0  # the convolution's state, in and out
         out["gopitar", kind, "delta_prepare"] = ("hbm", n * H * 3 * e * (2 + 4) + conv)
         out["gopitar", kind, "state_scan (delta rule, head decay)"] = ("hbm", n * H * 4 * e * 4 + seqs * H * e * e * 8)
+        out["gopitar", kind, "state_chunks (delta rule)"] = out["gopitar", kind, "state_scan (delta rule, head decay)"]
         out["gopitar", kind, "head_norm_gate"] = ("hbm", n * H * e * (4 + 2 + 2))
         out["gopitar", kind, "heads_gate"] = ("hbm", n * H * dv * 4)
         for model in ("gopitar", "kupirax"):
@@ -773,6 +776,7 @@ def design_rooflines(size, tokens, batch, context, peaks):
         delta_io = n * H * (3 * d + 2 * dv + 1) * 4
         ret_state, delta_state = seqs * Hr * dr * dvr * 8, seqs * H * d * dv * 8
         out["kupirax", kind, "state_scan (retention)"] = ("hbm", ret_io + ret_state)
+        out["kupirax", kind, "state_chunks (head decay)"] = ("hbm", ret_io + ret_state)
         out["kupirax", kind, "state_scan (delta rule)"] = ("hbm", delta_io + delta_state)
         out["kupirax", kind, "retention_prepare"] = ("hbm", n * Hr * (2 * dr + 2 * dvr) * 2 + n * Hr * (2 * dr + dvr) * 4)
         out["kupirax", kind, "delta_prepare"] = ("hbm", n * (H * (2 * d + dv) * 2 + H * d * 4) + n * H * (3 * d + dv + 1) * 4)

@@ -25,7 +25,7 @@ SOURCES = ["elementwise.cu", "norm.cu", "rope_cache.cu", "attention.cu", "sampli
            "linear_small.cu", "linear_tma.cu", "linear_tc5.cu", "attention_mma.cu", "attention_mma_odd.cu",
            "attention_mma_prefill.cu", "attention_tc5.cu", "attention_decode_tma.cu", "device_error.cu",
            "attention_local.cu", "attention_local_mma.cu", "recurrent.cu", "latent.cu", "moe.cu", "moe_mma.cu",
-           "attention_mix.cu", "attention_mix_mma.cu", "rglru.cu"]
+           "attention_mix.cu", "attention_mix_mma.cu", "rglru.cu", "state_chunk.cu"]
 HEADERS = ["common.cuh", "no_alloc.h", "tensor_map.h", "attention_decode.cuh", "attention_mma.cuh", "device_error.h", "moe.cuh",
            "attention_mix.cuh"]
 LIB_NAME = "libmll_kernels.so"

@@ -16,6 +16,7 @@ from .build import KernelBuildError, load_library
 
 ABI_VERSION = 35
 MAX_TOP_K = 1024
+STATE_RUN = 32  # tokens a run of `state_chunks`
 
 
 class KernelError(RuntimeError):
@@ -41,6 +42,8 @@ def lib() -> ctypes.CDLL:
             raise KernelBuildError(
                 f"kernel library reports ABI {handle.mll_abi_version()}, the package expects {ABI_VERSION}; "
                 "remove csrc/_build and rebuild")
+        if handle.mll_state_chunk_tokens() != STATE_RUN:
+            raise KernelBuildError(f"kernel library built for runs of {handle.mll_state_chunk_tokens()} tokens, not {STATE_RUN}")
         if handle.mll_page() != PAGE:
             raise KernelBuildError(f"kernel library built for pages of {handle.mll_page()} positions, the cache uses {PAGE}")
         _lib = handle
@@ -1473,6 +1476,58 @@ def state_scan(q, k, v, g, beta, head_decay, state, out, seq_slot, seq_qstart, s
         _stream()),
         "state_scan (delta rule, head decay)" if scalar_delta else "state_scan (delta rule)" if delta else ("state_scan (channel decay)" if channel else
                                                  ("state_scan (token decay)" if per_token else "state_scan (retention)")))
+
+
+USE_STATE_CHUNKS = True  # tests switch it off to reach the token-by-token scan in prompt steps
+
+
+def state_chunks_supported(d: int, dv: int) -> bool:
+    return USE_STATE_CHUNKS and bool(lib().mll_state_chunks_supported(d, dv))
+
+
+def state_chunks_scratch(n_runs: int, n_heads: int, d: int, dv: int, delta: bool) -> int:
+    """Floats of scratch memory that `state_chunks` wants."""
+    lib().mll_state_chunks_scratch.restype = ctypes.c_longlong
+    return int(lib().mll_state_chunks_scratch(n_runs, n_heads, d, dv, int(delta)))
+
+
+def state_chunks(q, k, v, state, out, scratch, run_seq, run_row0, seq_run0, seq_slot, seq_qstart, seq_qlen, n_seqs: int,
+                 n_heads: int, n_kv_heads: int, d: int, dv: int, head_decay: Optional[torch.Tensor] = None,
+                 token_decay: Optional[torch.Tensor] = None, beta: Optional[torch.Tensor] = None) -> None:
+    """As `state_scan` for one decay per head (`head_decay` [H]) or per token and head (`token_decay` [T, H]; with `beta` the
+    delta rule), a run of up to STATE_RUN tokens at a time: run_seq, run_row0 (int32 [runs]) list every
+    sequence's runs one after another, seq_run0 (int32 [sequences]) its first.  Decays lie in [0, 1]."""
+    n = q.shape[0]
+    for name, t, width in (("q", q, n_kv_heads * d), ("k", k, n_kv_heads * d), ("v", v, n_heads * dv),
+                           ("out", out, n_heads * dv), ("token decay", token_decay, n_heads), ("beta", beta, n_heads)):
+        if t is None:
+            continue
+        _need(t, f"state chunks {name}", torch.float32, 2)
+        if tuple(t.shape) != (n, width):
+            raise KernelError(f"state chunks: {name} {tuple(t.shape)}, expected {(n, width)}")
+    if (head_decay is None) == (token_decay is None) or (beta is not None and token_decay is None):
+        raise KernelError("state chunks: one decay per head or one per token and head; the delta rule goes with the latter")
+    if head_decay is not None:
+        _need(head_decay, "state chunks decay", torch.float32, 1)
+        if head_decay.shape[0] != n_heads:
+            raise KernelError("state chunks: one decay per head is needed")
+    _need(state, "state chunks state", torch.float32, 4)
+    if tuple(state.shape[1:]) != (n_heads, d, dv):
+        raise KernelError(f"state chunks: state {tuple(state.shape)} for {n_heads} heads of {d} x {dv}")
+    for name, t in (("run_seq", run_seq), ("run_row0", run_row0), ("seq_run0", seq_run0)):
+        _need(t, f"state chunks {name}", torch.int32, 1)
+    n_runs = run_seq.shape[0]
+    if run_row0.shape[0] != n_runs or seq_run0.shape[0] < n_seqs:
+        raise KernelError("state chunks: the lists of runs differ in length")
+    _need(scratch, "state chunks scratch", torch.float32)
+    if scratch.numel() < state_chunks_scratch(n_runs, n_heads, d, dv, beta is not None):
+        raise KernelError("state chunks: scratch too small")
+    _check(lib().mll_state_chunks(
+        _ptr(q), _ptr(k), _ptr(v), _ptr(beta), _ptr(token_decay), _ptr(head_decay), _ptr(state), _ptr(out), _ptr(scratch),
+        _ptr(run_seq), _ptr(run_row0), _ptr(seq_run0), _ptr(seq_slot), _ptr(seq_qstart), _ptr(seq_qlen), ctypes.c_int(n_runs),
+        ctypes.c_int(n_seqs), ctypes.c_int(n_heads), ctypes.c_int(n_kv_heads), ctypes.c_int(d), ctypes.c_int(dv), _stream()),
+        "state_chunks (delta rule)" if beta is not None else
+        ("state_chunks (token decay)" if token_decay is not None else "state_chunks (head decay)"), kernels=2 if beta is not None else 4)
 
 
 def ssd_prepare(proj, conv_w, conv_b, conv_state, a_log, dt_bias, tok_seq, seq_slot, seq_qstart, q, k, u, xs, decay,

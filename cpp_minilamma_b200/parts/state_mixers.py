@@ -27,6 +27,9 @@ write, and normalise o by its root mean square (per head, or a row at once) befo
                      o + D_h x, times silu(z), normalised in a few equal parts of the row, times a weight, then W_o;
                      the last taps - 1 convolution inputs of a sequence are state too
 
+Where the decay is one number per head - fixed or per token - prompts take the recurrence a run of tokens at a time
+(`_recur`); decays per key channel and single tokens take it token by token.
+
 What enters the recurrence is float32 (decays, step sizes, gates, unit vectors, the state); the projections are
 products in the run's dtype.  Sizes, decays, tap counts and eps are parameters.
 """
@@ -51,11 +54,55 @@ def _pad_rows(matrix: torch.Tensor, multiple: int = 8) -> torch.Tensor:
     return torch.cat([matrix, torch.zeros((spare, matrix.shape[1]), dtype=matrix.dtype, device=matrix.device)], dim=0)
 
 
+RUNS = ("state_mixers.runs",)  # key of the step's lists of runs, shared by all layers
+CHUNK_FROM = 8                 # tokens a sequence (on average) from which a step takes its recurrences a run at a time
+
+
+def _run_lists(shape):
+    """The index arrays of a prompt step's recurrences taken a run of tokens at a time: (sequence, first row among its new
+    tokens) of every run, and every sequence's first run.  Steps of single tokens need no list."""
+    if shape.all_decode:
+        return {}
+    lists = {"run_seq": [], "run_row0": [], "seq_run0": []}
+    for i, n in enumerate(shape.lens):
+        lists["seq_run0"].append(len(lists["run_seq"]))
+        for row0 in range(0, n, K.STATE_RUN):
+            lists["run_seq"].append(i)
+            lists["run_row0"].append(row0)
+    return lists
+
+
+def _recur(step, q, k, v, state, o, H: int, G: int, d: int, dv: int, head_decay=None, token_decay=None, beta=None,
+           runs: bool = True) -> None:
+    """The recurrence with one decay per head over the step's tokens: a run of tokens at a time in prompt steps, token by
+    token otherwise (and where `runs` is off: a decay outside [0, 1] has no logarithm to work with)."""
+    lists = step.meta.get(RUNS) if runs and not step.all_decode else None
+    if lists and step.n_tokens >= CHUNK_FROM * step.n_seqs and K.state_chunks_supported(d, dv):
+        scratch = step.ws.buffer("state.runs", (K.state_chunks_scratch(lists["run_seq"].shape[0], H, d, dv, beta is not None),),
+                                 torch.float32)
+        K.state_chunks(q, k, v, state, o, scratch, lists["run_seq"], lists["run_row0"], lists["seq_run0"], step.seq_slot,
+                       step.seq_qstart, step.seq_qlen, step.n_seqs, H, G, d, dv, head_decay=head_decay,
+                       token_decay=token_decay, beta=beta)
+        return
+    K.state_scan(q, k, v, None, beta, head_decay, state, o, step.seq_slot, step.seq_qstart, step.seq_qlen, step.n_seqs, H, G,
+                 d, dv, token_decay=token_decay)
+
+
+class _RecursInRuns(Mixer):
+    """A state mixer whose prompt steps want the lists of runs."""
+
+    def step_metadata_key(self):
+        return RUNS
+
+    def prepare_step(self, shape):
+        return _run_lists(shape)
+
+
 def _same_dtype(mats):
     return [m.float() for m in mats] if len({m.dtype for m in mats}) > 1 else list(mats)
 
 
-class Retention(Mixer):
+class Retention(_RecursInRuns):
     """params: n_heads, head_dim, v_head_dim, decay (one per head), eps (of the head norm),
     position (PartSpec of a rotary encoding over `rotary_dims` dimensions, or None), rotary_dims,
     names {"q","k","v","g","o"}: tensor names."""
@@ -78,6 +125,7 @@ class Retention(Mixer):
             raise ValueError(f"retention: {self.rot} rotated dimensions of a head of {self.d}")
         self.position = shared_position_encoding(params["position"], ctx) if self.rot else None
         self.decay_t = torch.tensor(self.decay, dtype=torch.float32, device=ctx.device)
+        self.in_runs = all(0.0 <= x <= 1.0 for x in self.decay)
         self.proj: Optional[Linear] = None
         self.o: Optional[Linear] = None
 
@@ -111,8 +159,7 @@ class Retention(Mixer):
                             bool(self.position.interleaved) if self.position is not None else False,
                             1.0 / math.sqrt(d))
         o = ws.buffer("mix.o", (T, H * dv), torch.float32)
-        K.state_scan(q, k, v, None, None, self.decay_t, cache.state["S"], o, step.seq_slot, step.seq_qstart,
-                     step.seq_qlen, step.n_seqs, H, H, d, dv)
+        _recur(step, q, k, v, cache.state["S"], o, H, H, d, dv, head_decay=self.decay_t, runs=self.in_runs)
         gated = ws.buffer("mix.gated", (T, H * dv), self.ctx.act_dtype)
         K.head_norm_gate(o, None, proj, gated, H, dv, self.eps, K.GATE_SILU, gate_col=H * (2 * d + dv))
         return self.o.forward(step, gated, "o")
@@ -214,7 +261,7 @@ class GatedDeltaRule(Mixer):
         return self.o.forward(step, gated, "o")
 
 
-class HeadDecayDeltaRule(Mixer):
+class HeadDecayDeltaRule(_RecursInRuns):
     """params: n_heads, n_kv_heads (q and k heads; value head h reads q/k head h // (n_heads / n_kv_heads)), head_dim,
     v_head_dim, conv (taps), eps (of the head norm), unit_eps (inside the root of the unit length), out_name (workspace name
     of the result, default "o"), names: tensor names for "q", "k", "v" (their convolution taps are "<name>.conv"), "b", "a",
@@ -296,14 +343,13 @@ class HeadDecayDeltaRule(Mixer):
             K.conv_state_update(proj, cache.state["conv"], step.seq_slot, step.seq_qstart, step.seq_qlen, step.n_seqs,
                                 self.channels, self.taps)
         o = ws.buffer("mix.o", (T, H * dv), torch.float32)
-        K.state_scan(q, k, v, None, beta, None, cache.state["S"], o, step.seq_slot, step.seq_qstart, step.seq_qlen,
-                     step.n_seqs, H, G, d, dv, token_decay=decay)
+        _recur(step, q, k, v, cache.state["S"], o, H, G, d, dv, token_decay=decay, beta=beta)
         gated = ws.buffer("mix.gated", (T, H * dv), self.ctx.act_dtype)
         K.head_norm_gate(o, self.norm_w, proj, gated, H, dv, self.eps, K.GATE_SILU, gate_col=self.gate_col)
         return self.o.forward(step, gated, self.out_name, into=into)
 
 
-class LightningAttention(Mixer):
+class LightningAttention(_RecursInRuns):
     """params: n_heads, head_dim, v_head_dim, decay (one per head), eps (of the norm over the row of all heads), out_name
     (workspace name of the result, default "o"), names: tensor names for "q", "k", "v", "g", "norm", "o"."""
 
@@ -323,6 +369,7 @@ class LightningAttention(Mixer):
         if len(self.decay) != self.n_heads:
             raise ValueError(f"lightning attention: {len(self.decay)} decays for {self.n_heads} heads")
         self.decay_t = torch.tensor(self.decay, dtype=torch.float32, device=ctx.device)
+        self.in_runs = all(0.0 <= x <= 1.0 for x in self.decay)
         self.proj: Optional[Linear] = None
         self.o: Optional[Linear] = None
 
@@ -354,8 +401,7 @@ class LightningAttention(Mixer):
         v = ws.buffer("lightning.v", (T, H * dv), torch.float32)
         K.retention_prepare(proj, None, None, step.tok_pos, q, k, v, H, d, dv, 0, False, 1.0, silu=True)
         o = ws.buffer("lightning.o", (T, H * dv), torch.float32)
-        K.state_scan(q, k, v, None, None, self.decay_t, cache.state["S"], o, step.seq_slot, step.seq_qstart,
-                     step.seq_qlen, step.n_seqs, H, H, d, dv)
+        _recur(step, q, k, v, cache.state["S"], o, H, H, d, dv, head_decay=self.decay_t, runs=self.in_runs)
         gated = ws.buffer("lightning.gated", (T, H * dv), self.ctx.act_dtype)
         K.row_norm_gate(o, self.norm_w, proj, gated, self.eps, K.GATE_SIGMOID, gate_col=H * (2 * d + dv))
         return self.o.forward(step, gated, self.out_name)
@@ -437,7 +483,7 @@ class GatedLinearAttention(Mixer):
         return self.o.forward(step, gated, self.out_name)
 
 
-class StateSpace(Mixer):
+class StateSpace(_RecursInRuns):
     """params: n_heads, n_groups (heads of one group share B and C), v_head_dim (columns of x per head), state (rows of
     the state per head: the size of B and C), conv (taps), norm_groups (equal parts of the row that are normalised
     each by itself), eps (of that norm), out_name (workspace name of the result, default "o"),
@@ -511,8 +557,7 @@ class StateSpace(Mixer):
         K.conv_state_update(proj, cache.state["conv"], step.seq_slot, step.seq_qstart, step.seq_qlen, step.n_seqs,
                             self.channels, self.taps, first_column=self.inner)
         o = ws.buffer("ssd.o", (T, self.inner), torch.float32)
-        K.state_scan(q, k, u, None, None, None, cache.state["S"], o, step.seq_slot, step.seq_qstart, step.seq_qlen,
-                     step.n_seqs, H, G, d, dv, token_decay=decay)
+        _recur(step, q, k, u, cache.state["S"], o, H, G, d, dv, token_decay=decay)
         gated = ws.buffer("ssd.gated", (T, self.inner), self.ctx.act_dtype)
         K.gated_group_norm(o, xs, self.skip, proj, self.norm_w, gated, dv, self.parts, self.eps)
         return self.o.forward(step, gated, self.out_name)

@@ -462,6 +462,15 @@ def test_attention_inputs_behind_a_convolution(dtype, H, G, d, dv, rot, taps, in
         assert (state[slots[s]].cpu().double() - u[total[s] - (taps - 1):]).abs().max().item() <= 2e-6 * scale if taps > 1 else True
 
 
+def _in_runs(q, k, v, state, out, st, lens, H, G, d, dv, **decays):
+    from cpp_minilamma_b200.csrc import kernels as K
+    runs = [(s, r) for s, n in enumerate(lens) for r in range(0, n, K.STATE_RUN)]
+    first = [next(i for i, (s, _) in enumerate(runs) if s == which) for which in range(len(lens))]
+    scratch = torch.full((K.state_chunks_scratch(len(runs), H, d, dv, "beta" in decays),), float("nan"), device=DEV)
+    K.state_chunks(q, k, v, state, out, scratch, _ints([s for s, _ in runs]), _ints([r for _, r in runs]), _ints(first),
+                   st.seq_slot, st.seq_qstart, st.seq_qlen, len(lens), H, G, d, dv, **decays)
+
+
 def _delta_reference(q, k, v, g, beta, S, share):
     """float64, one sequence: q, k [T, G, d], v [T, H, dv], g, beta [T, H], S [H, d, dv] -> (o, S)."""
     out = []
@@ -480,10 +489,14 @@ def _delta_reference(q, k, v, g, beta, S, share):
     (1, 1, 256, 48, [40, 40]), (3, 1, 7, 9, [20, 60]), (2, 1, 300, 20, [18]), (8, 4, 64, 128, [1] * 80), (8, 8, 128, 128, [1] * 40),
     (16, 16, 32, 128, [1] * 20), (2, 1, 96, 80, [100, 32])])
 @pytest.mark.parametrize("strong", [False, True])
-def test_delta_rule_with_a_decay_per_head(H, G, d, dv, lens, strong):
-    """The recurrence in every layout its sizes and token counts select, twice in a row (the state handed on), against
-    float64; keys that repeat (the correction is then as large as the value), decays from 1 down to none at all."""
+@pytest.mark.parametrize("runs", [False, True])
+def test_delta_rule_with_a_decay_per_head(H, G, d, dv, lens, strong, runs):
+    """The recurrence in every layout its sizes and token counts select, and a run of tokens at a time, twice in a row (the
+    state handed on), against float64; keys that repeat (the correction is then as large as the value), decays from 1 down
+    to none at all."""
     from cpp_minilamma_b200.csrc import kernels as K
+    if runs and not K.state_chunks_supported(d, dv):
+        pytest.skip("sizes of the token-by-token scan")
     gen = torch.Generator(device="cpu").manual_seed(d + dv + len(lens))
     n_seqs, share = len(lens), torch.arange(H) // (H // G)
     state = torch.randn((n_seqs + 1, H, d, dv), generator=gen).to(DEV)
@@ -503,8 +516,11 @@ def test_delta_rule_with_a_decay_per_head(H, G, d, dv, lens, strong):
         st = make_step_state(DEV, slots, [0] * n_seqs, lens)
         out = torch.full((T, H * dv), float("nan"), device=DEV)
         flat = lambda x: x.reshape(T, -1).contiguous().to(DEV)
-        K.state_scan(flat(q), flat(k), flat(v), None, flat(beta), None, state, out, st.seq_slot, st.seq_qstart, st.seq_qlen,
-                     n_seqs, H, G, d, dv, token_decay=flat(g))
+        if runs:
+            _in_runs(flat(q), flat(k), flat(v), state, out, st, lens, H, G, d, dv, token_decay=flat(g), beta=flat(beta))
+        else:
+            K.state_scan(flat(q), flat(k), flat(v), None, flat(beta), None, state, out, st.seq_slot, st.seq_qstart, st.seq_qlen,
+                         n_seqs, H, G, d, dv, token_decay=flat(g))
         at = 0
         for s, n in zip(slots, lens):
             rows = slice(at, at + n)
@@ -521,9 +537,13 @@ def test_delta_rule_with_a_decay_per_head(H, G, d, dv, lens, strong):
 
 @pytest.mark.parametrize("H,d,dv,lens", [(2, 64, 64, [70, 1, 33]), (3, 32, 128, [300]), (8, 128, 128, [257, 3]), (1, 16, 16, [64]), (2, 12, 20, [90]),
                                          (2, 128, 32, [65, 63, 128]), (3, 5, 7, [40, 2]), (4, 64, 128, [1] * 90), (2, 256, 48, [40])])
-def test_recurrence_with_a_fixed_decay(H, d, dv, lens):
-    """One decay per head, from 0 (only the current token) to 1, in every layout, twice in a row, against float64."""
+@pytest.mark.parametrize("form", ["scan", "runs", "runs, decays per token"])
+def test_recurrence_with_a_fixed_decay(H, d, dv, lens, form):
+    """One decay per head, from 0 (only the current token) to 1, in every layout and a run of tokens at a time, twice in a
+    row, against float64."""
     from cpp_minilamma_b200.csrc import kernels as K
+    if form != "scan" and not K.state_chunks_supported(d, dv):
+        pytest.skip("sizes of the token-by-token scan")
     gen = torch.Generator(device="cpu").manual_seed(d + dv + len(lens))
     n_seqs, T = len(lens), sum(lens)
     decay = torch.tensor(([0.999, 0.3, 1.0, 0.97, 0.0, 0.6, 1e-8, 0.9999])[:H])
@@ -534,8 +554,13 @@ def test_recurrence_with_a_fixed_decay(H, d, dv, lens):
         st = make_step_state(DEV, list(range(n_seqs)), [0] * n_seqs, lens)
         out = torch.full((T, H * dv), float("nan"), device=DEV)
         flat = lambda x: x.reshape(T, -1).contiguous().to(DEV)
-        K.state_scan(flat(q), flat(k), flat(v), None, None, decay.to(DEV), state, out, st.seq_slot, st.seq_qstart, st.seq_qlen,
-                     n_seqs, H, H, d, dv)
+        if form == "scan":
+            K.state_scan(flat(q), flat(k), flat(v), None, None, decay.to(DEV), state, out, st.seq_slot, st.seq_qstart, st.seq_qlen,
+                         n_seqs, H, H, d, dv)
+        elif form == "runs":
+            _in_runs(flat(q), flat(k), flat(v), state, out, st, lens, H, H, d, dv, head_decay=decay.to(DEV))
+        else:
+            _in_runs(flat(q), flat(k), flat(v), state, out, st, lens, H, H, d, dv, token_decay=decay.expand(T, H).contiguous().to(DEV))
         at = 0
         for s, n in enumerate(lens):
             for t in range(at, at + n):
