@@ -447,36 +447,47 @@ __global__ void __launch_bounds__(128, 2) state_chunk_scan_kernel(ChunkArgs a) {
   const int run0 = a.seq_run0[seq];
   const size_t tok_base = (size_t)a.seq_qstart[seq];
 
-  auto load_products = [&](int c) {  // Q and W of run c
-    float* q_s = sm + L::Q + (c & 1) * L::ROWS;
-    float* w_s = sm + L::W + (c & 1) * L::ROWS;
-    const size_t at = ((size_t)(run0 + c) * H + h) * CH;
-    const int n = min(CH, len - c * CH);
-#pragma unroll
-    for (int i = tid; i < CH * WORDS; i += 128) {
-      const int r = i / WORDS, wd = i % WORDS;
-      const bool col = wd * 4 < d, in = r < n && col;
-      ch_copy16(q_s + i * 4, in ? a.q + ((tok_base + c * CH + r) * G + kvh) * d + wd * 4 : a.q, in);
-      ch_copy16(w_s + i * 4, col ? a.w + (at + r) * d + wd * 4 : a.w, col);
+  // A thread copies one word of every (128 / WORDS)-th row: its place in the first of them, in each matrix
+  constexpr int STEP = 128 / WORDS;
+  const int load_row = tid / WORDS, load_word = (tid % WORDS) * 4;
+  const bool load_col = load_word < d;
+  const size_t qk_ld = (size_t)G * d;
+  const float* q_at = a.q + (tok_base + load_row) * qk_ld + (size_t)kvh * d + load_word;
+  const float* k_at = a.k + (tok_base + load_row) * qk_ld + (size_t)kvh * d + load_word;
+  const float* w_at = a.w + (((size_t)run0 * H + h) * CH + load_row) * d + load_word;
+  const float* p_at = a.p + ((size_t)run0 * H + h) * CH * CH + tid * 4;
+  const float* u_at = a.u + (((size_t)run0 * H + h) * CH + (tid >> 2)) * dv + col0 + (tid & 3) * 4;
+  const float* f_at = a.factors + ((size_t)run0 * H + h) * CH_FACTORS + tid * 4;
+  auto load_products = [&](int c) {  // Q and W of run c, which follow those of run c - 1
+    float* q_s = sm + L::Q + (c & 1) * L::ROWS + tid * 4;
+    float* w_s = sm + L::W + (c & 1) * L::ROWS + tid * 4;
+    const int rows = load_col ? len - c * CH - load_row : 0;
+#pragma unroll 2
+    for (int j = 0; j < CH / STEP; ++j) {
+      const bool in = j * STEP < rows;
+      ch_copy16(q_s + j * 512, in ? q_at + j * STEP * qk_ld : a.q, in);
+      ch_copy16(w_s + j * 512, load_col ? w_at + (size_t)j * STEP * d : a.w, load_col);
     }
+    q_at += CH * qk_ld;
+    w_at += (size_t)H * CH * d;
   };
-  auto load_writes = [&](int c) {  // K, P, U and the factors of run c
-    const size_t at = (size_t)(run0 + c) * H + h;
-    const int n = min(CH, len - c * CH);
-#pragma unroll
-    for (int i = tid; i < CH * WORDS; i += 128) {
-      const int r = i / WORDS, wd = i % WORDS;
-      const bool in = r < n && wd * 4 < d;
-      ch_copy16(sm + L::K + i * 4, in ? a.k + ((tok_base + c * CH + r) * G + kvh) * d + wd * 4 : a.k, in);
+  auto load_writes = [&](int c) {  // K, P, U and the factors of run c, likewise
+    float* k_s = sm + L::K + tid * 4;
+    const int rows = load_col ? len - c * CH - load_row : 0;
+#pragma unroll 2
+    for (int j = 0; j < CH / STEP; ++j) {
+      const bool in = j * STEP < rows;
+      ch_copy16(k_s + j * 512, in ? k_at + j * STEP * qk_ld : a.k, in);
     }
-#pragma unroll
-    for (int i = tid; i < CH * CH / 4; i += 128) ch_copy16(sm + L::P + i * 4, a.p + at * CH * CH + i * 4, true);
-    {
-      const int r = tid >> 2, wd = tid & 3;
-      const bool in = col0 + wd * 4 < dv;
-      ch_copy16(sm + L::U + r * LD + wd * 4, in ? a.u + (at * CH + r) * dv + col0 + wd * 4 : a.u, in);
-    }
-    if (tid < CH_FACTORS / 4) ch_copy16(sm + L::F + tid * 4, a.factors + at * CH_FACTORS + tid * 4, true);
+    ch_copy16(sm + L::P + tid * 4, p_at, true);
+    ch_copy16(sm + L::P + tid * 4 + 512, p_at + 512, true);
+    const bool in = col0 + (tid & 3) * 4 < dv;
+    ch_copy16(sm + L::U + (tid >> 2) * LD + (tid & 3) * 4, in ? u_at : a.u, in);
+    if (tid < CH_FACTORS / 4) ch_copy16(sm + L::F + tid * 4, f_at, true);
+    k_at += CH * qk_ld;
+    p_at += (size_t)H * CH * CH;
+    u_at += (size_t)H * CH * dv;
+    f_at += (size_t)H * CH_FACTORS;
   };
 
   // this thread's piece of the state: rows dg RS .. + RS - 1, columns 4 sc .. 4 sc + 3
@@ -508,7 +519,8 @@ __global__ void __launch_bounds__(128, 2) state_chunk_scan_kernel(ChunkArgs a) {
     for (int i = 0; i < 4; ++i)
 #pragma unroll
       for (int j = 0; j < 4; ++j) acc[i][j] = corr[i][j] = 0.f;
-#pragma unroll
+    // rolled loops: the whole of a run's work unrolled is more than the instruction caches hold
+#pragma unroll 2
     for (int step = 0; step < WORDS / 4; ++step) {
       const int wd = kg + 4 * step;
       float4 m[4];
@@ -535,7 +547,7 @@ __global__ void __launch_bounds__(128, 2) state_chunk_scan_kernel(ChunkArgs a) {
 #pragma unroll
       for (int j = 0; j < 4; ++j) acc[i][j] *= grown;
     }
-#pragma unroll
+#pragma unroll 1
     for (int step = 0; step < CH / 16; ++step) {
       const int wd = kg + 4 * step;
       float4 m[4];

@@ -4,9 +4,10 @@ alone.
 Every test makes its own small configuration and weights (`tiny_gopitar`).  float32 runs must agree with the oracle to
 2e-4 of the largest logit (at least 2e-4 absolute): with the test weights a window one token off, a lost state, a tap or a
 bias forgotten moves logits by percents.  bfloat16 runs are compared with the same unrounded oracle, so their bound is that
-of rounding noise: mean error at most 0.5 % of the largest logit, and at most one row in fifty (or one) with an error above
+of rounding noise: mean error at most 0.5 % of the largest logit, and at most one row in twenty with an error above
 3 % of it - keys of a few dimensions scaled to unit length make single rows ill-conditioned: perturbing the oracle's own
-matrices by 2^-9 moves such a row by several percents.  The sharp test is float32."""
+matrices by 2^-8 moves up to one row in twelve that far in a model with heads of one dimension.  The sharp test is
+float32."""
 import json
 import os
 import subprocess
@@ -60,7 +61,7 @@ def close(got, ref, dtype, what):
         assert err.max() <= 2e-4 * scale, f"{what}: err {err.max():.3e} of {scale:.2f}, first at row {row}"
         return
     rows = err.max(axis=-1).reshape(-1) > 3e-2 * scale
-    assert rows.sum() <= max(1, len(rows) // 50) and err.mean() <= 5e-3 * scale, \
+    assert rows.sum() <= max(1, len(rows) // 20) and err.mean() <= 5e-3 * scale, \
         f"{what}: max {err.max():.3e} mean {err.mean():.3e} of {scale:.2f}, {rows.sum()} rows over, worst row {row}"
 
 
