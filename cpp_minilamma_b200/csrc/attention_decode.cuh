@@ -46,7 +46,15 @@ struct DecodeMmaArgs {
   // walked in front of the window's).  softcap > 0: a score s becomes softcap * tanh(s / softcap) after the scale.
   int keep_first;
   float softcap;
+  // the TMA-fed kernel only; optional [B, gate_ld]: head h's output times sigmoid(gate[b, h])
+  const __nv_bfloat16* gate;
+  int gate_ld;
 };
+
+// The factor on the output of query head `head` of sequence b.
+__device__ __forceinline__ float decode_gate(const DecodeMmaArgs& a, int b, int head) {
+  return a.gate ? 1.f / (1.f + expf(-__bfloat162float(a.gate[(size_t)b * a.gate_ld + head]))) : 1.f;
+}
 
 __device__ __forceinline__ float2 unpack_bf162(unsigned r) {
   return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r));
@@ -154,7 +162,7 @@ __device__ __forceinline__ void merge_decode_splits(const DecodeMmaArgs& a, int 
     }
     for (; sp < S; ++sp) acc0 = fmaf(__ldcg(po + (size_t)sp * D), w_s[row * S + sp], acc0);
     const float l = l_s[row];
-    a.out[head * D + col] = __float2bfloat16_rn(l > 0.f ? ((acc0 + acc1) + (acc2 + acc3)) / l : 0.f);
+    a.out[head * D + col] = __float2bfloat16_rn(l > 0.f ? ((acc0 + acc1) + (acc2 + acc3)) / l * decode_gate(a, b, h0 + row) : 0.f);
   }
 }
 

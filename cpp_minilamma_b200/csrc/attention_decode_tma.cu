@@ -509,7 +509,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
           l = fmaf(*cluster.map_shared_rank(merged_l + row, sp), w, l);
           v = fmaf(*cluster.map_shared_rank(merged + (size_t)row * DV + col, sp), w, v);
         }
-        a.out[((size_t)b * a.n_heads + h0 + row) * DV + col] = __float2bfloat16_rn(l > 0.f ? v / l : 0.f);
+        a.out[((size_t)b * a.n_heads + h0 + row) * DV + col] = __float2bfloat16_rn(l > 0.f ? v / l * decode_gate(a, b, h0 + row) : 0.f);
       }
     }
     cluster.sync();  // nobody leaves while another block may still read its shared memory
@@ -521,7 +521,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
     const size_t head = (size_t)b * a.n_heads + h0 + row;
     if (n_eff == 1) {
       const float l = merged_l[row];
-      a.out[head * DV + col] = __float2bfloat16_rn(l > 0.f ? merged[(size_t)row * DV + col] / l : 0.f);
+      a.out[head * DV + col] = __float2bfloat16_rn(l > 0.f ? merged[(size_t)row * DV + col] / l * decode_gate(a, b, h0 + row) : 0.f);
     } else {
       a.part_o[(head * a.n_splits + split) * DV + col] = merged[(size_t)row * DV + col];
       if (col == 0) {
@@ -654,14 +654,16 @@ MLL_API int mll_attn_decode_tma_resident_clusters(int head_dim, int v_head_dim, 
 // permutation of 0 .. n_seqs - 1; the blocks of sequence seq_order[0] start first (give the longest first).
 // work: optional list of work_pairs (sequence, split) entries (attention_decode.cuh) that replaces the grid over
 // sequences and splits, so that sequences of one launch have different numbers of splits; n_splits is then the
-// most any sequence has, and no cluster is formed.
+// most any sequence has, and no cluster is formed.  gate: optional bfloat16 [n_seqs, gate_ld], head h's output times
+// sigmoid(gate[b, h]).
 MLL_API int mll_attn_decode_tma(const void* q, const void* qkv, int qkv_ld, const float* cos_table,
                                 const float* sin_table, int interleaved, int write_kv, void* k_cache, void* v_cache,
                                 long long n_pages, const int* seq_slot, const int* seq_ctx, const int* block_table,
                                 float* scratch, void* out, int n_seqs, int n_heads, int n_kv_heads, int head_dim,
                                 int v_head_dim, int max_blocks, int n_splits, int window, float scale, int* counters,
                                 int cluster_merge, const int* seq_order, const int* work, int work_pairs, int sink,
-                                const float* sink_values, int keep_first, float softcap, cudaStream_t stream) {
+                                const float* sink_values, int keep_first, float softcap, const void* gate, int gate_ld,
+                                cudaStream_t stream) {
   MLL_REQUIRE(mll_attn_decode_tma_supported(MLL_BF16, head_dim) && mll_attn_decode_tma_supported(MLL_BF16, v_head_dim) &&
                   (qkv == nullptr || head_dim == v_head_dim),
               "attention decode (tma): head sizes %d / %d", head_dim, v_head_dim);
@@ -696,6 +698,8 @@ MLL_API int mll_attn_decode_tma(const void* q, const void* qkv, int qkv_ld, cons
               "attention decode (tma): kept first tokens need a window; no negative cap");
   a.keep_first = keep_first;
   a.softcap = softcap;
+  a.gate = (const __nv_bfloat16*)gate;
+  a.gate_ld = gate_ld;
   const int rows = work != nullptr ? work_pairs : n_seqs;  // the grid's second index
   if (head_dim != v_head_dim)
     return head_dim == 64 ? mll::launch_decode_tma<64, 128, false>(kmap, vmap, a, rows, cluster_merge, stream)

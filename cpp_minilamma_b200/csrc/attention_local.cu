@@ -282,60 +282,50 @@ __global__ void __launch_bounds__(256) conv_prepare_kernel(ConvPrepArgs a) {
   }
 }
 
-// V channels on their way through the convolution: taps and last inputs of this thread's channels in registers
+// The convolution's value y [V] at row t of channels c .. c + V - 1 in a step's first rows of a sequence (or any row: the
+// inputs before the step come from the sequence's state), inputs one by one
 template <typename T, int V, int TAPS>
-struct ConvWalk {
-  float w[V * TAPS], b[V], past[TAPS > 1 ? TAPS - 1 : 1][V];  // past[i]: the input i + 1 tokens ago
-
-  __device__ __forceinline__ void begin(const ConvPrepArgs& a, int c) {
-    load_floats<float, V * TAPS>(a.conv_w + (size_t)c * TAPS, w);
+__device__ __forceinline__ void conv_row(const ConvPrepArgs& a, int t, int local, const float* state, int C, int c,
+                                         const float* w, const float* b, float* y, float* advance) {
+  float past[TAPS][V];  // past[i]: the input i tokens ago
 #pragma unroll
-    for (int j = 0; j < V; ++j) b[j] = a.bias ? a.bias[c + j] : 0.f;
-  }
-  __device__ __forceinline__ void fetch(const ConvPrepArgs& a, int t, int c, float* x) const {
-    load_floats<T, V>((const T*)a.qkv + (size_t)t * a.ld + c, x);
+  for (int i = 0; i < TAPS; ++i) {
+    if (i <= local) {
+      load_floats<T, V>((const T*)a.qkv + (size_t)(t - i) * a.ld + c, past[i]);
 #pragma unroll
-    for (int j = 0; j < V; ++j) x[j] += b[j];
-  }
-  // the inputs before row t, the local-th of its sequence in this step
-  __device__ __forceinline__ void look_back(const ConvPrepArgs& a, int t, int local, const float* state, int C, int c) {
-#pragma unroll
-    for (int i = 0; i < TAPS - 1; ++i) {
-      if (i < local) fetch(a, t - i - 1, c, past[i]);
-      else load_floats<float, V>(state + (size_t)(local - i - 1 + TAPS - 1) * C + c, past[i]);
+      for (int j = 0; j < V; ++j) past[i][j] += b[j];
+    } else {
+      load_floats<float, V>(state + (size_t)(local - i + TAPS - 1) * C + c, past[i]);
     }
   }
-  // y = the convolution's value at row t; the row becomes the newest of the last inputs
-  __device__ __forceinline__ void next(const ConvPrepArgs& a, int t, int c, float* y, float* advance, int C) {
-    float x[V];
-    fetch(a, t, c, x);
 #pragma unroll
-    for (int j = 0; j < V; ++j) {
-      y[j] = w[j * TAPS + TAPS - 1] * x[j];
+  for (int j = 0; j < V; ++j) {
+    y[j] = w[j * TAPS + TAPS - 1] * past[0][j];
 #pragma unroll
-      for (int i = 0; i < TAPS - 1; ++i) y[j] = fmaf(w[j * TAPS + TAPS - 2 - i], past[i][j], y[j]);
-    }
-    if constexpr (TAPS > 1) {
-      if (advance) {
-#pragma unroll
-        for (int i = 0; i < TAPS - 1; ++i)
-          store_floats<float, V>(advance + (size_t)(TAPS - 2 - i) * C + c, i == 0 ? x : past[i - 1]);
-      }
-#pragma unroll
-      for (int i = TAPS - 2; i > 0; --i)
-#pragma unroll
-        for (int j = 0; j < V; ++j) past[i][j] = past[i - 1][j];
-#pragma unroll
-      for (int j = 0; j < V; ++j) past[0][j] = x[j];
-    }
+    for (int i = 1; i < TAPS; ++i) y[j] = fmaf(w[j * TAPS + TAPS - 1 - i], past[i][j], y[j]);
   }
-};
+  if (advance) {  // one token a sequence: the state moves on by this input
+#pragma unroll
+    for (int i = 0; i < TAPS - 1; ++i) store_floats<float, V>(advance + (size_t)(TAPS - 2 - i) * C + c, past[i]);
+  }
+}
 
 // grid (ceil(tokens / TB), ceil(units / 256)), 256 threads; a unit is a word of V channels, or the two words that the
-// rotation (pairs half a rotated part apart) turns together
+// rotation (pairs half a rotated part apart) turns together.  A thread walks TB rows with its channels' taps in registers;
+// the rows' words (and those of the TAPS - 1 rows before) are all fetched before the first is used.
 template <typename T, int TAPS, int TB>
 __global__ void __launch_bounds__(256) conv_prepare_walk_kernel(ConvPrepArgs a, int n_tokens) {
   constexpr int V = 4;
+  __shared__ int local_s[TB], slot_s[TB], pos_s[TB], page_s[TB];
+  const int t0 = blockIdx.x * TB;
+  if (threadIdx.x < TB && t0 + threadIdx.x < n_tokens) {
+    const int t = t0 + threadIdx.x, seq = a.tok_seq[t], slot = a.seq_slot[seq], pos = a.tok_pos[t];
+    local_s[threadIdx.x] = t - a.seq_qstart[seq];
+    slot_s[threadIdx.x] = slot;
+    pos_s[threadIdx.x] = pos;
+    page_s[threadIdx.x] = a.block_table[(size_t)slot * a.max_blocks + pos / MLL_PAGE];
+  }
+  __syncthreads();
   const int u = blockIdx.y * 256 + threadIdx.x;
   const int H = a.n_heads, G = a.n_kv_heads, d = a.d, dv = a.dv;
   const int hw = a.rot / (2 * V), nu = d / V - hw, vw = dv / V;
@@ -357,42 +347,65 @@ __global__ void __launch_bounds__(256) conv_prepare_walk_kernel(ConvPrepArgs a, 
     c = head * d + e;
   }
   const int far = hw * V;  // distance to the partner
-  ConvWalk<T, V, TAPS> one, two;
-  one.begin(a, c);
-  if (pair) two.begin(a, c + far);
-  const int t0 = blockIdx.x * TB, t1 = min(n_tokens, t0 + TB);
-  for (int t = t0; t < t1; ++t) {
-    const int seq = a.tok_seq[t], local = t - a.seq_qstart[seq], slot = a.seq_slot[seq], pos = a.tok_pos[t];
-    if (TAPS > 1 && (t == t0 || local == 0)) {
-      const float* state = a.conv_state + (size_t)slot * (TAPS - 1) * C;
-      one.look_back(a, t, local, state, C, c);
-      if (pair) two.look_back(a, t, local, state, C, c + far);
+  const int cols[2] = {c, c + far};
+  float w[2][V * TAPS], b[2][V];
+  constexpr int ROWS = TB + TAPS - 1;
+  RawWord<T, V> raw[2][TB > 1 ? ROWS : 1];
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    if (k == 1 && !pair) break;
+    load_floats<float, V * TAPS>(a.conv_w + (size_t)cols[k] * TAPS, w[k]);
+#pragma unroll
+    for (int j = 0; j < V; ++j) b[k][j] = a.bias ? a.bias[cols[k] + j] : 0.f;
+    if constexpr (TB > 1) {
+#pragma unroll
+      for (int i = 0; i < ROWS; ++i)  // rows outside the step: any row of it, whose word is not used
+        raw[k][i].fetch((const T*)a.qkv + (size_t)min(max(t0 + i - (TAPS - 1), 0), n_tokens - 1) * a.ld + cols[k]);
     }
-    float* advance = a.advance ? a.advance + (size_t)slot * (TAPS - 1) * C : nullptr;
-    float x[V], y[V];
-    one.next(a, t, c, x, advance, C);
+  }
+#pragma unroll
+  for (int r = 0; r < TB; ++r) {
+    const int t = t0 + r;
+    if (t >= n_tokens) break;
+    const int local = local_s[r], slot = slot_s[r], pos = pos_s[r];
+    float y[2][V];
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      if (k == 1 && !pair) break;
+      if (TB == 1 || local < TAPS - 1) {
+        const size_t own = (size_t)slot * (TAPS - 1) * C;
+        conv_row<T, V, TAPS>(a, t, local, a.conv_state + own, C, cols[k], w[k], b[k], y[k], a.advance ? a.advance + own : nullptr);
+      } else {
+#pragma unroll
+        for (int j = 0; j < V; ++j) {
+          y[k][j] = 0.f;
+#pragma unroll
+          for (int i = 0; i < TAPS; ++i)
+            y[k][j] = fmaf(w[k][j * TAPS + TAPS - 1 - i], raw[k][TB > 1 ? r + TAPS - 1 - i : 0][j] + b[k][j], y[k][j]);
+        }
+      }
+    }
     if (pair) {
-      two.next(a, t, c + far, y, advance, C);
       float co[V], si[V];
       load_floats<float, V>(a.cos_table + (size_t)pos * (a.rot >> 1) + e, co);
       load_floats<float, V>(a.sin_table + (size_t)pos * (a.rot >> 1) + e, si);
 #pragma unroll
       for (int j = 0; j < V; ++j) {
-        const float p = x[j], q = y[j];
-        x[j] = p * co[j] - q * si[j];
-        y[j] = q * co[j] + p * si[j];
+        const float p = y[0][j], q = y[1][j];
+        y[0][j] = p * co[j] - q * si[j];
+        y[1][j] = q * co[j] + p * si[j];
       }
     }
     T* dst;
     if (!is_v && head < H) {
       dst = (T*)a.q_out + (size_t)t * H * d + c;
     } else {
-      const int page = a.block_table[(size_t)slot * a.max_blocks + pos / MLL_PAGE], in_page = pos % MLL_PAGE;
+      const int page = page_s[r], in_page = pos % MLL_PAGE;
       dst = is_v ? (T*)a.v_cache + (((size_t)page * G + head) * MLL_PAGE + in_page) * dv + e
                  : (T*)a.k_cache + (((size_t)page * G + (head - H)) * MLL_PAGE + in_page) * d + e;
     }
-    store_floats<T, V>(dst, x);
-    if (pair) store_floats<T, V>(dst + far, y);
+    store_floats<T, V>(dst, y[0]);
+    if (pair) store_floats<T, V>(dst + far, y[1]);
   }
 }
 

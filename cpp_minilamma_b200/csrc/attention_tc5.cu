@@ -76,6 +76,14 @@ struct PrefillTc5Args {
   int keep_first;            // with a window: keys at positions below this stay visible
   float scale_over_cap;      // scale / cap, and cap / scale: a raw score s becomes (cap / scale) tanh(s scale / cap),
   float cap_over_scale;      // which the scale then turns into cap * tanh(..); both 0 without a cap
+  static constexpr bool GATED = false;
+};
+// The same for heads with a gate each.  A type of its own: the kernel without gates then compiles to what it was (the two
+// more parameters alone moved its register allocation: 63 -> 67 us for 2,048 tokens of 32 heads of 128).
+struct PrefillTc5GatedArgs : PrefillTc5Args {
+  static constexpr bool GATED = true;
+  const __nv_bfloat16* gate;  // [T, gate_ld]: head h's output times sigmoid(gate[t, h])
+  int gate_ld;
 };
 
 __device__ __forceinline__ unsigned a_smem(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
@@ -311,10 +319,10 @@ struct PrefillTc5Smem {
   static_assert(AB_COUNT * 8 + 16 <= 512, "the barriers must fit behind the tiles");
 };
 
-template <int D, int DV>
+template <int D, int DV, typename Args>
 __global__ void __launch_bounds__(PrefillTc5Smem<D, DV>::THREADS, 2)
 attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant__ CUtensorMap kmap,
-                        const __grid_constant__ CUtensorMap vmap, PrefillTc5Args a) {
+                        const __grid_constant__ CUtensorMap vmap, Args a) {
   using L = PrefillTc5Smem<D, DV>;
   constexpr int DB = D / 64, VB = DV / 64;  // 64-column boxes per row of Q and K, and of V
   constexpr int KS = L::KV_STAGES, SB = L::S_BUFS;
@@ -571,14 +579,19 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_c
       __syncwarp();  // one arrival a warp: 128 arrivals on one barrier are 128 shared-memory atomics in a row
       if (lane == 0) a_mbar_arrive(bar(L::AB_P_READY, sb));
     }
-    // the output row: O / l
+    // the output row: O / l, times the head's gate where there is one (its number is fetched before the last wait)
+    float gate_z = 0.f;
+    if constexpr (Args::GATED) {
+      if (r < rows) gate_z = __bfloat162float(a.gate[((size_t)qstart + row0 + r) * a.gate_ld + h]);
+    }
     wait(bar(L::AB_PV_DONE, (n_pages - 1) % SB), ((n_pages - 1) / SB) & 1);
     a_fence_after();
     {
       // tcgen05.ld is a warp-wide instruction: every thread of the warp reads its lane, and only the
       // threads that own a row of the sequence store
       const bool store = !*abort_flag && r < rows;
-      const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      const float inv_l = l_run > 0.f ? 1.f / l_run : 0.f;
+      const float inv = Args::GATED ? inv_l / (1.f + expf(-gate_z)) : inv_l;
       __nv_bfloat16* dst = a.out + ((size_t)qstart + row0 + (store ? r : 0)) * a.n_heads * DV + (size_t)h * DV;
 #pragma unroll
       for (int c = 0; c < DV; c += 32) {
@@ -610,12 +623,12 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_c
   }
 }
 
-template <int D, int DV>
-int launch_prefill_tc5(const CUtensorMap& qmap, const CUtensorMap& kmap, const CUtensorMap& vmap,
-                       const PrefillTc5Args& a, int n_tiles, cudaStream_t stream) {
+template <int D, int DV, typename Args>
+int launch_prefill_tc5_as(const CUtensorMap& qmap, const CUtensorMap& kmap, const CUtensorMap& vmap,
+                          const Args& a, int n_tiles, cudaStream_t stream) {
   using L = PrefillTc5Smem<D, DV>;
   const size_t smem = L::BYTES;
-  auto kernel = attn_prefill_tc5_kernel<D, DV>;
+  auto kernel = attn_prefill_tc5_kernel<D, DV, Args>;
   cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (err != cudaSuccess) {
     mll_set_error("attention prefill (tcgen05): cannot reserve %zu bytes of shared memory: %s", smem,
@@ -625,6 +638,13 @@ int launch_prefill_tc5(const CUtensorMap& qmap, const CUtensorMap& kmap, const C
   MLL_LAUNCH((kernel), dim3((unsigned)(n_tiles * a.n_heads)), L::THREADS, smem, stream, qmap, kmap, vmap, a);
   MLL_LAUNCH_CHECK();
   return 0;
+}
+
+template <int D, int DV>
+int launch_prefill_tc5(const CUtensorMap& qmap, const CUtensorMap& kmap, const CUtensorMap& vmap,
+                       const PrefillTc5GatedArgs& a, int n_tiles, cudaStream_t stream) {
+  return a.gate ? launch_prefill_tc5_as<D, DV, PrefillTc5GatedArgs>(qmap, kmap, vmap, a, n_tiles, stream)
+                : launch_prefill_tc5_as<D, DV, PrefillTc5Args>(qmap, kmap, vmap, a, n_tiles, stream);
 }
 
 }  // namespace mll
@@ -645,14 +665,16 @@ MLL_API int mll_attn_prefill_tc5_supported(int dtype, int head_dim) {
 }
 
 // Same contract as mll_attn_prefill (bfloat16, head_dim and v_head_dim 64 or 128; value pages and out rows have
-// v_head_dim columns a head); n_tokens is the number of
+// v_head_dim columns a head); gate: optional bfloat16 [n_tokens, gate_ld], head h's output times
+// sigmoid(gate[t, h]); n_tokens is the number of
 // rows of q and out, n_pages the number of pages of k_cache and v_cache.
 MLL_API int mll_attn_prefill_tc5(const void* q, const void* k_cache, const void* v_cache, const int* seq_slot,
                                  const int* seq_ctx, const int* seq_qstart, const int* seq_qlen, const int* tile_seq,
                                  const int* tile_row0, const int* block_table, void* out, int n_tokens,
                                  long long n_pages, int n_tiles, int n_heads, int n_kv_heads, int head_dim,
                                  int v_head_dim, int max_blocks, int window, int chunk, float scale, int sink,
-                                 const float* sink_values, int keep_first, float softcap, cudaStream_t stream) {
+                                 const float* sink_values, int keep_first, float softcap, const void* gate, int gate_ld,
+                                 cudaStream_t stream) {
   MLL_REQUIRE(mll_attn_prefill_tc5_supported(MLL_BF16, head_dim) && mll_attn_prefill_tc5_supported(MLL_BF16, v_head_dim),
               "attention prefill (tcgen05): head sizes %d / %d", head_dim, v_head_dim);
   MLL_REQUIRE(n_heads > 0 && n_kv_heads > 0 && n_heads % n_kv_heads == 0, "attention prefill (tcgen05): bad head counts");
@@ -670,10 +692,10 @@ MLL_API int mll_attn_prefill_tc5(const void* q, const void* k_cache, const void*
   if (mll::tensor_map_bf16(q, n_tokens, (long long)n_heads * head_dim, mll::A_ROWS, &qmap) != 0) return -1;
   if (mll::tensor_map_bf16(k_cache, n_pages * n_kv_heads * MLL_PAGE, head_dim, MLL_PAGE, &kmap) != 0) return -1;
   if (mll::tensor_map_bf16(v_cache, n_pages * n_kv_heads * MLL_PAGE, v_head_dim, MLL_PAGE, &vmap) != 0) return -1;
-  mll::PrefillTc5Args a{seq_slot, seq_ctx, seq_qstart, seq_qlen, tile_seq, tile_row0, block_table,
+  mll::PrefillTc5GatedArgs a{{seq_slot, seq_ctx, seq_qstart, seq_qlen, tile_seq, tile_row0, block_table,
                         (__nv_bfloat16*)out, n_heads, n_kv_heads, max_blocks, window, chunk, scale * 1.4426950408889634f,
                         (sink || sink_values) ? 1 : 0, sink_values, keep_first, softcap > 0.f ? scale / softcap : 0.f,
-                        softcap > 0.f ? softcap / scale : 0.f};
+                        softcap > 0.f ? softcap / scale : 0.f}, (const __nv_bfloat16*)gate, gate_ld};
   if (head_dim == 64 && v_head_dim == 64) return mll::launch_prefill_tc5<64, 64>(qmap, kmap, vmap, a, n_tiles, stream);
   if (head_dim == 64) return mll::launch_prefill_tc5<64, 128>(qmap, kmap, vmap, a, n_tiles, stream);
   if (v_head_dim == 64) return mll::launch_prefill_tc5<128, 64>(qmap, kmap, vmap, a, n_tiles, stream);

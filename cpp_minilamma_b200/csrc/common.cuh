@@ -181,6 +181,32 @@ __device__ __forceinline__ void store_floats(T* p, const float* v) {
   }
 }
 
+// V neighbouring values as they lie in memory, fetched through the read-only path (nothing writes them while the kernel
+// runs): a run of such words can be on its way before the first is used, whatever the kernel stores in between
+template <typename T, int V>
+struct RawWord {
+  static constexpr int REGS = V * (int)sizeof(T) / 4;
+  unsigned r[REGS];
+  __device__ __forceinline__ void fetch(const T* p) {
+    if constexpr (REGS % 4 == 0) {
+#pragma unroll
+      for (int i = 0; i < REGS; i += 4) {
+        const uint4 v = __ldg(reinterpret_cast<const uint4*>(p) + i / 4);
+        r[i] = v.x; r[i + 1] = v.y; r[i + 2] = v.z; r[i + 3] = v.w;
+      }
+    } else if constexpr (REGS == 2) {
+      const uint2 v = __ldg(reinterpret_cast<const uint2*>(p));
+      r[0] = v.x; r[1] = v.y;
+    } else {
+      r[0] = __ldg(reinterpret_cast<const unsigned*>(p));
+    }
+  }
+  __device__ __forceinline__ float operator[](int i) const {
+    if constexpr (sizeof(T) == 4) return __uint_as_float(r[i]);
+    else return __uint_as_float(i & 1 ? r[i >> 1] & 0xffff0000u : r[i >> 1] << 16);  // bfloat16 is float32's upper half
+  }
+};
+
 // 16-byte asynchronous copy global -> shared (both 16-byte aligned)
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
   unsigned s = (unsigned)__cvta_generic_to_shared(smem);

@@ -814,10 +814,11 @@ def attention_decode(q, k_cache, v_cache, seq_slot, seq_ctx, block_table, scratc
                      scale: float, counters: Optional[torch.Tensor] = None, order: Optional[torch.Tensor] = None,
                      work: Optional[torch.Tensor] = None, chunk: int = 0, sink: bool = False,
                      sink_values: Optional[torch.Tensor] = None, keep_first: int = 0, softcap: float = 0.0,
-                     v_head_dim: int = 0) -> None:
+                     v_head_dim: int = 0, gate=None) -> None:
     """One query token per sequence (q row i belongs to sequence i) over the paged cache.
     `v_head_dim` (0: head_dim): the values' head size, where it differs from the keys' (the TMA-fed kernel only; ask
-    `attention_decode_takes_value_size` first).
+    `attention_decode_takes_value_size` first).  `gate` = (rows [B, ld], first column), the same kernel only: head h's output
+    times sigmoid(rows[b, first column + h]).
     `keep_first` (with a window) and `softcap`: the TMA-fed kernel only (ask `attention_decode_takes_window_extras`
     first) - keys below `keep_first` stay visible; a score s becomes softcap * tanh(s / softcap) after the scale.
     `sink` (bfloat16 tensor-core kernels only): one more term exp(0) in the softmax's denominator, or
@@ -854,10 +855,11 @@ def attention_decode(q, k_cache, v_cache, seq_slot, seq_ctx, block_table, scratc
                                                 block_table, scratch, out, n_seqs, n_heads, n_kv_heads, head_dim,
                                                 n_splits, window, scale, counters, _order(order, n_seqs), work,
                                                 sink=sink, sink_values=sink_values, keep_first=keep_first, softcap=softcap,
-                                                v_head_dim=v_head_dim):
+                                                v_head_dim=v_head_dim, gate=gate):
         return
-    if keep_first or softcap or v_head_dim != head_dim:
-        raise KernelError("attention decode: only the TMA-fed kernel keeps first tokens, caps scores or has values of another size")
+    if keep_first or softcap or v_head_dim != head_dim or gate is not None:
+        raise KernelError("attention decode: only the TMA-fed kernel keeps first tokens, caps scores, "
+                          "gates its output or has values of another size")
     if work is not None:
         raise KernelError("attention decode: a work list was given, but the kernel that takes one does not run here")
     if USE_TENSOR_CORE_DECODE and lib().mll_attn_decode_mma_supported(code, head_dim):
@@ -882,6 +884,17 @@ def attention_decode(q, k_cache, v_cache, seq_slot, seq_ctx, block_table, scratc
                                  ctypes.c_int(head_dim), ctypes.c_int(block_table.shape[1]),
                                  ctypes.c_int(n_splits), ctypes.c_int(window), ctypes.c_float(scale),
                                  _stream()), "attention_decode", kernels=2 if n_splits > 1 else 1)
+
+
+def _head_gate(gate, rows: int, n_heads: int):
+    """(pointer, row stride) of a gate per head, (rows [T, ld] bfloat16, first column) or None."""
+    if gate is None:
+        return _ptr(None), ctypes.c_int(0)
+    t, col = gate
+    _need(t, "attention gate", torch.bfloat16, 2)
+    if t.shape[0] < rows or not 0 <= col <= t.shape[1] - n_heads:
+        raise KernelError("attention: the gate's columns lie outside its rows")
+    return ctypes.c_void_p(t.data_ptr() + col * t.element_size()), ctypes.c_int(t.shape[1])
 
 
 USE_FUSED_DECODE = True  # off: rotary encoding and cache write stay a kernel of their own in decode steps
@@ -918,7 +931,7 @@ def _work(work, n_seqs: int, n_splits: int):
 def _tma_decode(q, qkv, cos, sin, interleaved, write_kv, k_cache, v_cache, seq_slot, seq_ctx, block_table, scratch, out,
                 n_seqs, n_heads, n_kv_heads, head_dim, n_splits, window, scale, counters, order=None, work=None,
                 sink: bool = False, sink_values: Optional[torch.Tensor] = None, keep_first: int = 0,
-                softcap: float = 0.0, v_head_dim: int = 0) -> bool:
+                softcap: float = 0.0, v_head_dim: int = 0, gate=None) -> bool:
     """Runs the TMA-fed decode kernel when it takes the problem (bfloat16, head_dim 64/128, arrival
     counters whenever the context is split); returns whether it did."""
     if not (USE_TMA_DECODE and USE_TENSOR_CORE_DECODE and lib().mll_attn_decode_tma_supported(dtype_code(out.dtype), head_dim)):
@@ -936,7 +949,8 @@ def _tma_decode(q, qkv, cos, sin, interleaved, write_kv, k_cache, v_cache, seq_s
                                      ctypes.c_float(scale), _ptr(counters if n_splits > 1 else None),
                                      ctypes.c_int(int(USE_CLUSTER_MERGE)), _ptr(order), _ptr(work),
                                      ctypes.c_int(work.shape[0] if work is not None else 0), ctypes.c_int(int(sink)),
-                                     _ptr(sink_values), ctypes.c_int(keep_first), ctypes.c_float(softcap), _stream()),
+                                     _ptr(sink_values), ctypes.c_int(keep_first), ctypes.c_float(softcap),
+                                     *_head_gate(gate, n_seqs, n_heads), _stream()),
            "attention_decode (TMA, work list)" if work is not None
            else "attention_decode (TMA, cluster merge)" if USE_CLUSTER_MERGE and 2 <= n_splits <= 16
            else "attention_decode (TMA)")
@@ -1038,7 +1052,7 @@ def attention_prefill(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_ql
                       block_table, out, n_tiles: int, n_heads: int, n_kv_heads: int, head_dim: int,
                       window: int, scale: float, wide_tiles=None, chunk: int = 0, sink: bool = False,
                       sink_values: Optional[torch.Tensor] = None, keep_first: int = 0, softcap: float = 0.0,
-                      v_head_dim: int = 0) -> None:
+                      v_head_dim: int = 0, gate=None) -> None:
     """Tiles of up to 64 query tokens of sequences with unequal lengths over the paged cache.
     `wide_tiles`: (sequence, first row) int32 lists of the same rows in tiles of 128, which the tcgen05 kernel
     works on; without them it walks the 64-row list and every other block finds nothing to do.
@@ -1046,7 +1060,8 @@ def attention_prefill(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_ql
     only if j // chunk == i // chunk.  `sink` (the same kernel only): one more term exp(0) in the softmax's denominator,
     or exp(sink_values[head]) with `sink_values` (float32 [Hq], not scaled).  `keep_first` (with a window) and
     `softcap` (the same kernel only): keys below `keep_first` stay visible; a score s becomes softcap * tanh(s / softcap)
-    after the scale.  `v_head_dim` (0: head_dim; the same kernel only): the values' head size."""
+    after the scale.  `v_head_dim` (0: head_dim; the same kernel only): the values' head size.  `gate` = (rows [T, ld], first
+    column), the same kernel only: head h's output times sigmoid(rows[t, first column + h])."""
     v_head_dim = v_head_dim or head_dim
     _check_attention(q, k_cache, v_cache, out, n_heads, n_kv_heads, head_dim, v_head_dim)
     _check_sink_values(sink_values, n_heads)
@@ -1075,12 +1090,13 @@ def attention_prefill(q, k_cache, v_cache, seq_slot, seq_ctx, seq_qstart, seq_ql
                                           ctypes.c_int(v_head_dim),
                                           ctypes.c_int(block_table.shape[1]), ctypes.c_int(window), ctypes.c_int(chunk),
                                           ctypes.c_float(scale), ctypes.c_int(int(sink)), _ptr(sink_values),
-                                          ctypes.c_int(keep_first), ctypes.c_float(softcap), _stream()),
+                                          ctypes.c_int(keep_first), ctypes.c_float(softcap),
+                                          *_head_gate(gate, q.shape[0], n_heads), _stream()),
                "attention_prefill (tcgen05)")
         return
-    if chunk or sink or keep_first or softcap or v_head_dim != head_dim:
+    if chunk or sink or keep_first or softcap or v_head_dim != head_dim or gate is not None:
         raise KernelError("attention prefill: only the tcgen05 kernel masks by chunks, has a sink, keeps first tokens, "
-                          "caps scores or has values of another size")
+                          "caps scores, gates its output or has values of another size")
     if USE_TENSOR_CORE_PREFILL and lib().mll_attn_prefill_mma_supported(dtype_code(q.dtype), head_dim):
         _check(lib().mll_attn_prefill_mma(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(seq_slot), _ptr(seq_ctx),
                                           _ptr(seq_qstart), _ptr(seq_qlen), _ptr(tile_seq), _ptr(tile_row0),

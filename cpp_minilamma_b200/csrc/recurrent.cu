@@ -190,8 +190,8 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(DeltaPrepArgs a, int
 }
 
 // The same for up to four taps and heads that 32 lanes of V neighbouring channels hold: a warp owns one head (a q head, a
-// k head or a value head) and walks TB consecutive rows, with the taps and the last inputs of its channels in registers,
-// so that a row is read once and the taps once per TB rows.  grid (ceil(tokens / TB), ceil((2 G + H) / 4)), 128 threads.
+// k head or a value head) and walks TB consecutive rows with the taps and the last inputs of its channels in registers, so
+// that a row is read once and the taps once per TB rows.  grid (ceil(tokens / TB), ceil((2 G + H) / 4)), 128 threads.
 template <typename T, int V, int TAPS, int TB>
 __global__ void __launch_bounds__(128) delta_prepare_walk_kernel(DeltaPrepArgs a, int n_tokens) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -204,43 +204,64 @@ __global__ void __launch_bounds__(128) delta_prepare_walk_kernel(DeltaPrepArgs a
   const int c = (is_v ? 2 * nqk + (unit - 2 * G) * dv : unit * d) + lane * V;  // this lane's first channel
   const bool live = lane * V < width;
   const T* proj = (const T*)a.proj;
-  float w[V * TAPS], past[TAPS > 1 ? TAPS - 1 : 1][V];  // past[i]: the input i + 1 tokens ago
+  float w[V * TAPS], past[TAPS][V];  // past[i]: the input i tokens ago
 #pragma unroll
   for (int i = 0; i < V * TAPS; ++i) w[i] = 0.f;
-  if (live) load_floats<float, V * TAPS>(a.conv_w + (size_t)c * TAPS, w);
+#pragma unroll
+  for (int i = 0; i < TAPS; ++i)
+#pragma unroll
+    for (int j = 0; j < V; ++j) past[i][j] = 0.f;
+  const int t0 = blockIdx.x * TB, n_rows = min(TB, n_tokens - t0);
+  RawWord<T, V> row;  // fetched a row ahead
+  if (live) {
+    row.fetch(proj + (size_t)t0 * a.ld + c);
+    load_floats<float, V * TAPS>(a.conv_w + (size_t)c * TAPS, w);
+  }
+  // what the rows need one by one, looked up by a lane a row: their places, and a value head's beta and decay
+  int my_local = 0, my_slot = 0;
+  if (lane < n_rows) {
+    const int seq = a.tok_seq[t0 + lane];
+    my_local = t0 + lane - a.seq_qstart[seq];
+    my_slot = a.seq_slot[seq];
+  }
+  if (is_v && !a.rate && lane < 2 * TB) {
+    const int r = lane % TB, h = unit - 2 * G;
+    if (r < n_rows) {
+      const size_t t = (size_t)t0 + r;
+      const float z = to_float(proj[t * a.ld + C + (lane < TB ? 0 : H) + h]);
+      if (lane < TB) a.beta[t * H + h] = sigmoid_f(z);
+      else a.g[t * H + h] = expf(-expf(a.a_log[h]) * softplus_f(z + a.dt_bias[h]));
+    }
+  }
   const float f0 = is_q ? rsqrtf((float)d) : 1.f;
-  const int t0 = blockIdx.x * TB, t1 = min(n_tokens, t0 + TB);
-  for (int t = t0; t < t1; ++t) {
-    const int seq = a.tok_seq[t], local = t - a.seq_qstart[seq];
-    if (t == t0 || local == 0) {  // this warp's first row, or another sequence's: fetch the inputs before it
-      const float* state = a.conv_state + (size_t)a.seq_slot[seq] * (TAPS - 1) * C;
+  for (int r = 0; r < n_rows; ++r) {  // the same bound for the whole warp
+    const int t = t0 + r;
+    const int local = __shfl_sync(0xffffffffu, my_local, r), slot = __shfl_sync(0xffffffffu, my_slot, r);
+    if ((r == 0 || local == 0) && live) {  // this warp's first row, or another sequence's: fetch the inputs before it
+      const float* state = a.conv_state + (size_t)slot * (TAPS - 1) * C;
 #pragma unroll
-      for (int i = 0; i < TAPS - 1; ++i) {
-        if (live) {
-          if (i < local) load_floats<T, V>(proj + (size_t)(t - i - 1) * a.ld + c, past[i]);
-          else load_floats<float, V>(state + (size_t)(local - i - 1 + TAPS - 1) * C + c, past[i]);
-        } else {
-#pragma unroll
-          for (int j = 0; j < V; ++j) past[i][j] = 0.f;
-        }
+      for (int i = 1; i < TAPS; ++i) {
+        if (i <= local) load_floats<T, V>(proj + (size_t)(t - i) * a.ld + c, past[i]);
+        else load_floats<float, V>(state + (size_t)(local - i + TAPS - 1) * C + c, past[i]);
       }
     }
-    float x[V], y[V];
+    if (live) {
 #pragma unroll
-    for (int j = 0; j < V; ++j) x[j] = 0.f;
-    if (live) load_floats<T, V>(proj + (size_t)t * a.ld + c, x);
-    float ss = 0.f;
+      for (int j = 0; j < V; ++j) past[0][j] = row[j];
+      if (r + 1 < n_rows) row.fetch(proj + (size_t)(t + 1) * a.ld + c);
+    }
+    float y[V], ss = 0.f;
 #pragma unroll
     for (int j = 0; j < V; ++j) {
-      float z = w[j * TAPS + TAPS - 1] * x[j];
+      float z = w[j * TAPS + TAPS - 1] * past[0][j];
 #pragma unroll
-      for (int i = 0; i < TAPS - 1; ++i) z = fmaf(w[j * TAPS + TAPS - 2 - i], past[i][j], z);
+      for (int i = 1; i < TAPS; ++i) z = fmaf(w[j * TAPS + TAPS - 1 - i], past[i][j], z);
       y[j] = silu_f(z);
       ss = fmaf(y[j], y[j], ss);
     }
     if (is_v) {
       if (live) store_floats<float, V>(a.v + ((size_t)t * H + (unit - 2 * G)) * dv + lane * V, y);
-      delta_scalars(a, proj + (size_t)t * a.ld, (size_t)t, unit - 2 * G, C, lane);
+      if (a.rate) delta_scalars(a, proj + (size_t)t * a.ld, (size_t)t, unit - 2 * G, C, lane);
     } else {
       const float f = f0 / sqrtf(warp_sum(ss) + a.unit_eps);
 #pragma unroll
@@ -248,19 +269,14 @@ __global__ void __launch_bounds__(128) delta_prepare_walk_kernel(DeltaPrepArgs a
       if (live) store_floats<float, V>((is_q ? a.q : a.k) + ((size_t)t * G + (is_q ? unit : unit - G)) * d + lane * V, y);
     }
     if (a.advance && live) {  // one token a sequence: the state moves on by this input
-      float* state = a.advance + (size_t)a.seq_slot[seq] * (TAPS - 1) * C;
+      float* state = a.advance + (size_t)slot * (TAPS - 1) * C;
 #pragma unroll
-      for (int i = 0; i < TAPS - 1; ++i)
-        store_floats<float, V>(state + (size_t)(TAPS - 2 - i) * C + c, i == 0 ? x : past[i - 1]);
+      for (int i = 0; i < TAPS - 1; ++i) store_floats<float, V>(state + (size_t)(TAPS - 2 - i) * C + c, past[i]);
     }
 #pragma unroll
-    for (int i = TAPS - 2; i > 0; --i)
+    for (int i = TAPS - 1; i > 0; --i)
 #pragma unroll
       for (int j = 0; j < V; ++j) past[i][j] = past[i - 1][j];
-    if constexpr (TAPS > 1) {
-#pragma unroll
-      for (int j = 0; j < V; ++j) past[0][j] = x[j];
-    }
   }
 }
 
@@ -682,6 +698,32 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(const float* __rest
   }
 }
 
+// The same for heads that 32 lanes of four neighbouring channels hold (dv a multiple of 4, at most 128, everything aligned):
+// four heads a block, as above, the head in registers between its sum and its scaling.
+template <typename T, typename GateT>
+__global__ void __launch_bounds__(128) head_norm_gate_vec_kernel(const float* __restrict__ o, const float* __restrict__ weight,
+                                                                 const GateT* __restrict__ gate, int gate_ld,
+                                                                 T* __restrict__ out, long long n_heads_all, int n_heads,
+                                                                 int dv, float eps, int act) {
+  const long long at = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);  // token * n_heads + head
+  const int e = (threadIdx.x & 31) * 4;
+  if (at >= n_heads_all) return;
+  const int h = (int)(at % n_heads);
+  const size_t t = (size_t)(at / n_heads);
+  const bool live = e < dv;
+  float x[4] = {0.f, 0.f, 0.f, 0.f}, z[4], w[4] = {1.f, 1.f, 1.f, 1.f};
+  if (live) {
+    load_floats<float, 4>(o + (size_t)at * dv + e, x);
+    load_floats<GateT, 4>(gate + t * gate_ld + (size_t)h * dv + e, z);
+    if (weight) load_floats<float, 4>(weight + e, w);
+  }
+  const float f = 1.f / sqrtf(warp_sum((x[0] * x[0] + x[1] * x[1]) + (x[2] * x[2] + x[3] * x[3])) / (float)dv + eps);
+  if (!live) return;
+#pragma unroll
+  for (int j = 0; j < 4; ++j) x[j] = x[j] * f * w[j] * (act == 0 ? silu_f(z[j]) : sigmoid_f(z[j]));
+  store_floats<T, 4>(out + (size_t)at * dv + e, x);
+}
+
 // grid (tokens), 256 threads:   out[t, :] = o / sqrt(mean over the whole row(o^2) + eps) * weight * act(gate[t, :])
 template <typename T, typename GateT, bool VEC>
 __global__ void __launch_bounds__(256) row_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ weight,
@@ -1044,6 +1086,22 @@ MLL_API int mll_head_norm_gate(const float* o, const float* weight, const void* 
   MLL_REQUIRE(n_tokens >= 0 && n_heads > 0 && dv > 0 && gate_ld >= n_heads * dv, "head norm gate: bad sizes");
   MLL_REQUIRE(act == 0 || act == 1, "head norm gate: unknown activation %d", act);
   if (n_tokens == 0) return 0;
+  if (dv % 4 == 0 && dv <= 128 && gate_ld % 4 == 0 && ((uintptr_t)o | (uintptr_t)weight | (uintptr_t)out) % 16 == 0 &&
+      (uintptr_t)gate % (gate_dtype == MLL_F32 ? 16 : 8) == 0) {
+    const long long all = (long long)n_tokens * n_heads;
+    MLL_REQUIRE((all + 3) / 4 <= 0x7fffffffLL, "head norm gate: too many heads for one launch");
+    const unsigned blocks = (unsigned)((all + 3) / 4);
+#define MLL_HNGV(T, GT)                                                                                          \
+  MLL_LAUNCH((mll::head_norm_gate_vec_kernel<T, GT>), blocks, 128, 0, stream, o, weight, (const GT*)gate, gate_ld, (T*)out, \
+             all, n_heads, dv, eps, act)
+    if (out_dtype == MLL_F32 && gate_dtype == MLL_F32) MLL_HNGV(float, float);
+    else if (out_dtype == MLL_BF16 && gate_dtype == MLL_BF16) MLL_HNGV(__nv_bfloat16, __nv_bfloat16);
+    else if (out_dtype == MLL_BF16 && gate_dtype == MLL_F32) MLL_HNGV(__nv_bfloat16, float);
+    else MLL_REQUIRE(false, "head norm gate: dtypes %d / %d", out_dtype, gate_dtype);
+#undef MLL_HNGV
+    MLL_LAUNCH_CHECK();
+    return 0;
+  }
   const dim3 grid(n_tokens, (n_heads + 3) / 4);
   MLL_REQUIRE(grid.y <= 65535, "head norm gate: too many heads for one launch");
 #define MLL_HNG(T, GT)                                                                                          \

@@ -246,10 +246,10 @@ class ChunkedAttention(Mixer):
                                       float(self.qk_norm["eps"]) if self.qk_norm else 0.0, q_temp=self.q_temp,
                                       v_from_k=self.v_from_k, write_kv=not self.kv_shared)
         out = step.ws.buffer("attn", (T, self.n_heads * self.dv), act)
-        self._attend(step, q, cache, out)
-        if self.gate:
-            gate_col = self.n_heads * self.d + (0 if self.kv_shared else
-                                                self.n_kv_heads * (self.d if self.v_from_k else self.d + self.dv))
+        gate_col = self.n_heads * self.d + (0 if self.kv_shared else
+                                            self.n_kv_heads * (self.d if self.v_from_k else self.d + self.dv))
+        gated = self._attend(step, q, cache, out, (qkv, gate_col) if self.gate == "head" else None)
+        if self.gate and not gated:
             K.heads_gate(out, qkv, gate_col, out, self.n_heads, self.dv, per_head=self.gate == "head")
         return self.o.forward(step, out, self.out_name)
 
@@ -281,7 +281,8 @@ class ChunkedAttention(Mixer):
         fit = [s for s in range(2, pages + 1) if blocks <= capacity[s]]
         return fit[-1] if fit else 1
 
-    def _attend(self, step, q, cache, out) -> None:
+    def _attend(self, step, q, cache, out, gate) -> bool:
+        """The heads' outputs; True when they are already multiplied by `gate` (rows, first column), one number per head."""
         act = self.ctx.act_dtype
         learned = self.sink_values  # a sink with a score of its own per head, or None
         extra = {"keep_first": self.keep_first, "softcap": self.softcap}
@@ -298,11 +299,12 @@ class ChunkedAttention(Mixer):
                 scratch = step.ws.buffer("attn.scratch", (K.attention_decode_scratch_floats(
                     step.n_seqs, self.n_heads, self.dv, splits),), torch.float32)
                 counters = step.ws.zeros("attn.counters", (step.n_seqs * self._decode_items(),), torch.int32)
+            gate = gate if K.attention_decode_takes_value_size(act, self.d, self.dv) else None
             K.attention_decode(q, cache.k, cache.v, step.seq_slot, step.seq_ctx, cache.block_table, scratch, out,
                                step.n_seqs, self.n_heads, self.n_kv_heads, self.d, splits, self.window, self.scale,
                                counters=counters, chunk=self.chunk, sink=self.sink, sink_values=learned,
-                               v_head_dim=self.dv, **extra)
-            return
+                               v_head_dim=self.dv, gate=gate, **extra)
+            return gate is not None
         if step.all_decode and self._tensor_cores():
             # single tokens that the kernels above do not take (a sink, values of another size): the tensor-core
             # prompt kernel with a kv head's query heads as the rows of its tile
@@ -314,7 +316,7 @@ class ChunkedAttention(Mixer):
                                     cache.block_table, out, step.n_seqs, self.n_heads, self.n_kv_heads, self.d, self.dv,
                                     self.chunk, self.window, self.scale, sink=self.sink, n_splits=splits, scratch=scratch,
                                     sink_values=learned, **extra)
-            return
+            return False
         tiles = step.meta.get(self.step_metadata_key()) if not step.all_decode else None
         if tiles and K.attention_prefill_takes_chunks(act, self.d, self.dv):
             # head sizes that the Llama attention's tcgen05 prompt kernel takes: that kernel, which knows the chunk mask
@@ -323,17 +325,18 @@ class ChunkedAttention(Mixer):
                                 tiles["tile_seq"], tiles["tile_row0"], cache.block_table, out,
                                 tiles["tile_seq"].shape[0], self.n_heads, self.n_kv_heads, self.d, self.window,
                                 self.scale, wide_tiles=(tiles["wide_seq"], tiles["wide_row0"]), chunk=self.chunk,
-                                sink=self.sink, sink_values=learned, v_head_dim=self.dv, **extra)
-            return
+                                sink=self.sink, sink_values=learned, v_head_dim=self.dv, gate=gate, **extra)
+            return gate is not None
         if tiles and self._tensor_cores():
             K.local_attention_tiles(q, cache.k, cache.v, step.seq_slot, step.seq_ctx, step.seq_qstart, step.seq_qlen,
                                     tiles["tile_seq"], tiles["tile_row0"], cache.block_table, out, self.n_heads,
                                     self.n_kv_heads, self.d, self.dv, self.chunk, self.window, self.scale,
                                     sink=self.sink, sink_values=learned, **extra)
-            return
+            return False
         K.local_attention(q, cache.k, cache.v, step.tok_pos, step.tok_seq, step.seq_slot, cache.block_table, out,
                           self.n_heads, self.n_kv_heads, self.d, self.dv, self.chunk, self.window, self.scale,
                           sink=self.sink, sink_values=learned, **extra)
+        return False
 
 
 register_part("mixer", "chunked_attention", ChunkedAttention)

@@ -337,7 +337,7 @@ def _attention_reference(q, keys, values, pos0, scale, window, group):
 def test_attention_with_values_of_another_size(H, G, d, dv, window):
     """The tcgen05 prompt kernel and the TMA-fed single-token kernel (one block a sequence, and the context in 2, 5 and 20
     splits) with values wider and narrower than keys.  The key just inside the last query's window and the one just outside
-    it stand out; a page that is not the sequence's, or rows past its end, hold no numbers."""
+    it stand out; both multiply every head by its gate; a page that is not the sequence's, or rows past its end, hold no numbers."""
     from cpp_minilamma_b200.csrc import kernels as K
     gen = torch.Generator(device="cpu").manual_seed(d * 1000 + H)
     starts, lens = [0, 70, 300, 0], [150, 131, 1, 3]
@@ -360,6 +360,9 @@ def test_attention_with_values_of_another_size(H, G, d, dv, window):
             parts.append(_attention_reference(q[rows].double().view(-1, H, d), _dense(k_cache, table, s, ctxs[s]),
                                               _dense(v_cache, table, s, ctxs[s]), starts[s], scale, w, group))
         refs[w] = torch.cat(parts).view(T, H * dv)
+    gate = torch.randn((T, H + 9), generator=gen).to(torch.bfloat16)  # a number per row and head, from the third column on
+    for w in refs:
+        refs[w] = (refs[w].view(T, H, dv) * torch.sigmoid(gate[:, 2:2 + H].double())[..., None]).reshape(T, H * dv)
     want = refs[window]
     tol = 1.5e-2 * max(1.0, want.abs().max().item())
     last = [sum(lens[:i + 1]) - 1 for i in range(4)]
@@ -373,7 +376,7 @@ def test_attention_with_values_of_another_size(H, G, d, dv, window):
     out = torch.zeros((T, H * dv), dtype=torch.bfloat16, device=DEV)
     assert K.attention_prefill_takes_chunks(torch.bfloat16, d, dv)
     K.attention_prefill(qd, kc, vc, state.seq_slot, state.seq_ctx, state.seq_qstart, state.seq_qlen, seqs, rows, table_dev, out,
-                        len(tiles), H, G, d, window, scale, wide_tiles=(seqs, rows), v_head_dim=dv)
+                        len(tiles), H, G, d, window, scale, wide_tiles=(seqs, rows), v_head_dim=dv, gate=(gate.to(DEV), 2))
     err = (out.cpu().double() - want).abs()
     assert err.max().item() <= tol, ("prompt", err.max().item(), tol, int(err.max(dim=1).values.argmax()))
     one = make_step_state(DEV, [0, 1, 2, 3], [c - 1 for c in ctxs], [1] * 4)
@@ -383,7 +386,7 @@ def test_attention_with_values_of_another_size(H, G, d, dv, window):
         scratch = torch.full((K.attention_decode_scratch_floats(4, H, dv, splits),), float("nan"), device=DEV)
         counters = torch.zeros((4 * G * -(-group // 16),), dtype=torch.int32, device=DEV)
         K.attention_decode(qd[last].contiguous(), kc, vc, one.seq_slot, one.seq_ctx, table_dev, scratch, out, 4, H, G, d, splits,
-                           window, scale, counters=counters, v_head_dim=dv)
+                           window, scale, counters=counters, v_head_dim=dv, gate=(gate[last].contiguous().to(DEV), 2))
         err = (out.cpu().double() - want[last]).abs().max().item()
         assert err <= tol, ("single tokens", splits, err, tol)
 
