@@ -664,12 +664,12 @@ def gopitar_config(size):
     R = s["ret_heads"]
     pair = {"type": "parallel", "mlp": mlp,
             "mixer": {"left": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": 64, "vdim": 128, "conv": 3, "scale": 0.125,
-                               "mask": {"size": 1024}, "rot": {"base": 10000.0, "dims": 32}},
+                               "mask": {"size": 1024}, "rot": {"base": 500000.0, "dims": 32}},
                       "right": {"heads": R, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-5 - 4 * i / R) for i in range(R)]},
-                      "left_scale": 0.8, "right_scale": 1.1}}
+                      "left_scale": 0.7, "right_scale": 0.9}}
     delta = {"type": "delta", "mlp": mlp, "mixer": {"heads": s["heads"], "kv_heads": s["heads"], "dim": 128, "vdim": 128, "conv": 4}}
     return ml.config_from_dict({"architecture": "Gopitar", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5},
-                                "embedding": {"scale": 12.0}, "logit_softcap": 30.0, "layers": [pair, pair, delta] * s["groups"],
+                                "embedding": {"scale": 2.0}, "logit_softcap": 50.0, "layers": [pair, pair, delta] * s["groups"],
                                 "torch_dtype": "bfloat16"})
 
 

@@ -24,7 +24,7 @@ def right(heads=2, dim=12, vdim=20, decay=(0.7, 0.995)):
     return {"heads": heads, "dim": dim, "vdim": vdim, "decay": list(decay)}
 
 
-def pair(l, r, scales=(0.8, 1.1)):
+def pair(l, r, scales=(0.9, 1.3)):
     return "parallel", {"left": l, "right": r, "left_scale": scales[0], "right_scale": scales[1]}
 
 
@@ -76,7 +76,7 @@ CONFIGS = {
     # sizes at which the bfloat16 run takes its tensor-core kernels, values wider and narrower than keys
     "tensor": lambda: config([
         layer(pair(left(heads=8, kv_heads=2, dim=64, vdim=128, conv=3, scale=0.12, size=90, rot=32, base=10000.0),
-                   right(2, 64, 64, (0.6, 0.999))), 128),
+                   right(2, 64, 64, (0.7, 0.998))), 128),
         layer(delta(heads=4, kv_heads=2, dim=64, vdim=64, conv=4), 96),
         layer(pair(left(heads=4, kv_heads=4, dim=128, vdim=64, conv=4, scale=0.1, size=70, rot=128, base=100.0),
                    right(3, 32, 128, (0.9, 0.98, 0.9999))), 64),
